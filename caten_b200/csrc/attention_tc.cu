@@ -81,8 +81,8 @@ __device__ __forceinline__ void st_split8(unsigned char *tile, int row_hi, int r
   *reinterpret_cast<uint4 *>(tile + sw128(row_lo, chunk)) = pack8_lo(a, b);
 }
 
-// 2^x by the special-function unit alone (what exp2f uses inside, without its scaling of results
-// below 2^-126, which flush to zero here: such probabilities do not register in a row sum >= 1/e^8)
+// 2^x by one PTX ex2.approx instruction; results below 2^-126 flush to zero (such probabilities do not
+// register in a row sum >= 1/e^8)
 __device__ __forceinline__ float ex2_approx(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
