@@ -15,13 +15,14 @@ LIB_PATH = os.environ.get("CATEN_B200_LIB") or os.path.join(HERE, "libcaten_b200
 
 OK, EINVAL, ECUDA, EUNSUPPORTED, EDEVICE = 0, 1, 2, 3, 4
 F32, F16, Q4_0, Q8_0 = 0, 1, 2, 8
+BF16 = 30
 Q4_1, Q5_0, Q5_1 = 3, 6, 7                                # kept packed, like Q4_0 and Q8_0
 Q2_K, Q3_K, Q4_K, Q5_K, Q6_K = 10, 11, 12, 13, 14        # expanded to fp32 at upload
 BLOCK_FORMATS = (Q4_0, Q8_0, Q4_1, Q5_0, Q5_1, Q2_K, Q3_K, Q4_K, Q5_K, Q6_K)
-ACT_NONE, ACT_GELU, ACT_RELU = 0, 1, 2
+ACT_NONE, ACT_GELU, ACT_RELU, ACT_RELU_GLU = 0, 1, 2, 3
 PREC_FP32, PREC_BF16, PREC_BF16X3 = 0, 1, 2
-K_EMBED, K_LAYERNORM, K_GEMV, K_GEMM, K_ATTN_DECODE, K_ATTN_PREFILL, K_ARGMAX, K_COUNT = 0, 1, 2, 3, 4, 5, 6, 8
-KERNEL_CLASSES = ["embed", "layernorm", "gemv", "gemm", "attn_decode", "attn_prefill", "argmax", "decode_step"]
+K_EMBED, K_LAYERNORM, K_GEMV, K_GEMM, K_ATTN_DECODE, K_ATTN_PREFILL, K_ARGMAX, K_COUNT = 0, 1, 2, 3, 4, 5, 6, 10
+KERNEL_CLASSES = ["embed", "layernorm", "gemv", "gemm", "attn_decode", "attn_prefill", "argmax", "decode_step", "wkv", "prep"]
 DIST_ID_BYTES = 128
 PRECISIONS = {"fp32": PREC_FP32, "bf16": PREC_BF16, "bf16x3": PREC_BF16X3}
 
@@ -48,6 +49,24 @@ class GPT2Desc(C.Structure):
         ("ln2_g", _PFP), ("ln2_b", _PFP), ("fc_b", _PFP), ("mproj_b", _PFP),
         ("attn_w", _PFP), ("proj_w", _PFP), ("fc_w", _PFP), ("mproj_w", _PFP),
     ]
+
+
+MIX_ATTENTION, MIX_WKV = 0, 1
+
+
+class LayerDesc(C.Structure):
+    """Mirror of ``caten_b200_layer_desc``."""
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "kv_heads", "vdim", "window", "rot_dims", "qk_norm", "gated")] + [
+        ("scale", C.c_float), ("group_rows", C.c_int32), ("low_rank", C.c_int32),
+        ("norm1", C.c_float), ("norm1b", C.c_float), ("norm2", C.c_float), ("norm2b", C.c_float)] + [
+        (n, _vp) for n in ("rot_freq", "mu", "w0", "u", "norm", "in_w", "out_w", "w2", "ff_in", "ff_out")]
+
+
+class DecoderDesc(C.Structure):
+    """Mirror of ``caten_b200_decoder_desc``."""
+    _fields_ = [(n, C.c_int32) for n in ("n_layers", "width", "vocab", "max_seq_len", "batch", "precision", "max_rows", "max_portion",
+                                         "loop_start", "loop_stop", "loop_times")] + [
+        ("eps", C.c_float), ("final_gain", C.c_float), ("embed", _vp), ("head", _vp), ("loop_in", _vp), ("layers", C.POINTER(LayerDesc))]
 
 
 EXPR_MAX_DIMS, EXPR_MAX_OPERANDS, EXPR_MAX_CODE, EXPR_MAX_CONSTS = 6, 8, 96, 16
@@ -117,6 +136,16 @@ SIGNATURES = {
     "caten_b200_gpt2_logits": (_vp, [_vp]),
     "caten_b200_gpt2_kv": (C.c_int, [_vp, C.c_int, _PFP, _PFP]),
     "caten_b200_gpt2_launch_count": (_i64, [_vp]),
+    "caten_b200_decoder_create": (C.c_int, [_vp, C.POINTER(DecoderDesc), _PFP]),
+    "caten_b200_decoder_destroy": (C.c_int, [_vp]),
+    "caten_b200_decoder_step": (C.c_int, [_vp, _vp, _i64, _i64, _vp, _i64, _vp, _vp]),
+    "caten_b200_decoder_step_device": (C.c_int, [_vp, _vp, _i64, _i64, _vp]),
+    "caten_b200_decoder_decode": (C.c_int, [_vp, _vp, _i64, _i64, _vp]),
+    "caten_b200_decoder_logits": (_vp, [_vp]),
+    "caten_b200_decoder_runs": (_i64, [_vp]),
+    "caten_b200_decoder_capture": (C.c_int, [_vp, _vp]),
+    "caten_b200_decoder_cache_nbytes": (_i64, [_vp]),
+    "caten_b200_decoder_launch_count": (_i64, [_vp]),
     "caten_b200_dist_unique_id": (C.c_int, [_vp]),
     "caten_b200_dist_init": (C.c_int, [_vp, C.c_int, C.c_int, _vp]),
     "caten_b200_dist_finalize": (C.c_int, [_vp]),

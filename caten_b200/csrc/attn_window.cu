@@ -1,0 +1,561 @@
+// Grouped-query softmax attention with an optional sliding window: query i sees the keys j with
+// 0 <= i - j < window.  The cache of a sequence is a ring of `cap` positions (slot = position % cap),
+// so a windowed layer keeps window + one prompt portion whatever the sequence's length.
+//
+//   q, k   rotated on their first 2 * rot_pairs dims (interleaved pairs, angle = position * freq),
+//          then divided by their root mean square over the head (optional)
+//   out    softmax(q . k * scale) . v, times sigmoid(gate) per head (optional)
+//
+// Keys are cached rotated and normalised; everything here is fp32.
+#include "attn_window.cuh"
+
+namespace cb {
+
+namespace {
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+// One warp, one head of up to 256 dims: lane holds the pairs lane, lane + 32, ...
+struct HeadPairs {
+  float2 p[4];
+};
+__device__ __forceinline__ void rotate_pairs(HeadPairs &h, const float *__restrict__ freq, int rot_pairs, int pos, int lane) {
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int i = lane + 32 * j;
+    if (i < rot_pairs) {
+      float sn, cs;
+      sincosf((float)pos * freq[i], &sn, &cs);
+      const float u = h.p[j].x, v = h.p[j].y;
+      h.p[j].x = u * cs - v * sn;
+      h.p[j].y = v * cs + u * sn;
+    }
+  }
+}
+__device__ __forceinline__ float pairs_inv_rms(const HeadPairs &h, int D, float eps) {
+  float ss = 0.0f;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) ss += h.p[j].x * h.p[j].x + h.p[j].y * h.p[j].y;  // padding is zero
+  return 1.0f / sqrtf(warp_sum(ss) / (float)D + eps);
+}
+
+}  // namespace
+
+// ---------------------------------------------------------------------------------------------
+// Multi-token step: one CTA per row, one warp per head.
+// ---------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a) {
+  pdl_enter();
+  const int64_t r = blockIdx.x;
+  const int b = (int)(r / a.s), pos = a.n + (int)(r % a.s);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float *row = a.qkv + r * a.ld;
+  const int64_t slot = pos % a.cap;
+  for (int hd = warp; hd < a.H + 2 * a.G; hd += 8) {
+    const bool is_q = hd < a.H, is_k = !is_q && hd < a.H + a.G;
+    const int g = is_q ? 0 : (is_k ? hd - a.H : hd - a.H - a.G);
+    float *src = row + (is_q ? a.q_off + (int64_t)hd * a.Dp : is_k ? a.k_off + (int64_t)g * a.Dp : a.v_off + (int64_t)g * a.Ep);
+    const int np = (is_q || is_k ? a.Dp : a.Ep) / 2;
+    HeadPairs h;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = lane + 32 * j;
+      h.p[j] = i < np ? reinterpret_cast<const float2 *>(src)[i] : make_float2(0.f, 0.f);
+    }
+    float mul = 1.0f;
+    float *dst = src;
+    if (is_q || is_k) {
+      rotate_pairs(h, a.freq, a.rot_pairs, pos, lane);
+      if (a.qk_norm) mul = pairs_inv_rms(h, a.D, a.eps);
+    }
+    if (is_q) mul *= a.scale;
+    else if (is_k) dst = a.kc + (((int64_t)b * a.G + g) * a.cap + slot) * a.Dp;
+    else dst = a.vc + (((int64_t)b * a.G + g) * a.cap + slot) * a.Ep;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = lane + 32 * j;
+      if (i < np) reinterpret_cast<float2 *>(dst)[i] = make_float2(h.p[j].x * mul, h.p[j].y * mul);
+    }
+  }
+}
+
+int launch_attn_prep(caten_b200_ctx *ctx, const AttnArgs &a) {
+  const int64_t rows = (int64_t)a.B * a.s;
+  if (rows <= 0) return 0;
+  if (rows > 0x7fffffff || a.Dp > 256 || a.Ep > 256) return fail(ctx, CATEN_B200_EUNSUPPORTED, "attention: head size above 256");
+  launch_k(ctx, attn_prep_kernel, dim3((unsigned)rows), dim3(256), 0, a);
+  CB_LAUNCH_CHECK(ctx, "attn_prep_kernel");
+  return 0;
+}
+
+// ---------------------------------------------------------------------------------------------
+// Multi-token step on the CUDA cores, any head size up to 256: 32 queries of one head per CTA, keys
+// in blocks of 32, running maximum and sum.  Thread (ty, tx) of a 16 x 16 grid owns the scores of
+// queries 2 ty, 2 ty + 1 with keys tx, tx + 16, and of the same queries the value columns
+// 4 tx + 64 j .. + 3.
+// ---------------------------------------------------------------------------------------------
+constexpr int AW_T = 32;
+
+__global__ void __launch_bounds__(256) attn_window_simt_kernel(const AttnArgs a) {
+  extern __shared__ __align__(16) float sm[];
+  pdl_enter();
+  const int ldk = a.Dp + 4, ldv = a.Ep + 4;
+  float *Qs = sm, *Ks = Qs + AW_T * ldk, *Vs = Ks + AW_T * ldk, *Ps = Vs + AW_T * ldv;
+  const int q0 = blockIdx.x * AW_T, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
+  const int tx = tid & 15, ty = tid >> 4;
+  const int g = h / (a.H / a.G), t = a.n + a.s;
+  const float *kb = a.kc + ((int64_t)b * a.G + g) * a.cap * a.Dp;
+  const float *vb = a.vc + ((int64_t)b * a.G + g) * a.cap * a.Ep;
+  const int d4 = a.Dp / 4, e4 = a.Ep / 4;
+  for (int e = tid; e < AW_T * d4; e += 256) {
+    const int i = e / d4, c = e % d4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (q0 + i < a.s) v = reinterpret_cast<const float4 *>(a.qkv + ((int64_t)b * a.s + q0 + i) * a.ld + a.q_off + (int64_t)h * a.Dp)[c];
+    *reinterpret_cast<float4 *>(Qs + i * ldk + 4 * c) = v;
+  }
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  float4 o[2][4];
+#pragma unroll
+  for (int q = 0; q < 2; ++q)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[q][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+  const int W = a.window > 0 ? a.window : 0x3fffffff;
+  const int first = a.n + q0 - W + 1;
+  const int jbeg = first > 0 ? first / AW_T * AW_T : 0;
+  const int jend = min(t, a.n + q0 + AW_T);
+  for (int j0 = jbeg; j0 < jend; j0 += AW_T) {
+    __syncthreads();
+    for (int e = tid; e < AW_T * d4; e += 256) {
+      const int i = e / d4, c = e % d4;
+      *reinterpret_cast<float4 *>(Ks + i * ldk + 4 * c) =
+          j0 + i < t ? reinterpret_cast<const float4 *>(kb + (int64_t)((j0 + i) % a.cap) * a.Dp)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    for (int e = tid; e < AW_T * e4; e += 256) {
+      const int i = e / e4, c = e % e4;
+      *reinterpret_cast<float4 *>(Vs + i * ldv + 4 * c) =
+          j0 + i < t ? reinterpret_cast<const float4 *>(vb + (int64_t)((j0 + i) % a.cap) * a.Ep)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    __syncthreads();
+    float sc[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
+    for (int c = 0; c < d4; ++c) {
+      const float4 qa = *reinterpret_cast<const float4 *>(Qs + (2 * ty) * ldk + 4 * c), qb = *reinterpret_cast<const float4 *>(Qs + (2 * ty + 1) * ldk + 4 * c);
+      const float4 ka = *reinterpret_cast<const float4 *>(Ks + tx * ldk + 4 * c), kc2 = *reinterpret_cast<const float4 *>(Ks + (tx + 16) * ldk + 4 * c);
+      sc[0][0] = fmaf(qa.x, ka.x, fmaf(qa.y, ka.y, fmaf(qa.z, ka.z, fmaf(qa.w, ka.w, sc[0][0]))));
+      sc[0][1] = fmaf(qa.x, kc2.x, fmaf(qa.y, kc2.y, fmaf(qa.z, kc2.z, fmaf(qa.w, kc2.w, sc[0][1]))));
+      sc[1][0] = fmaf(qb.x, ka.x, fmaf(qb.y, ka.y, fmaf(qb.z, ka.z, fmaf(qb.w, ka.w, sc[1][0]))));
+      sc[1][1] = fmaf(qb.x, kc2.x, fmaf(qb.y, kc2.y, fmaf(qb.z, kc2.z, fmaf(qb.w, kc2.w, sc[1][1]))));
+    }
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      const int i = a.n + q0 + 2 * ty + q;  // the query's position
+      float mx = -INFINITY;
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int j = j0 + tx + 16 * e;
+        if (j > i || i - j >= W) sc[q][e] = -INFINITY;
+        mx = fmaxf(mx, sc[q][e]);
+      }
+#pragma unroll
+      for (int w = 8; w > 0; w >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, w));
+      const float mn = fmaxf(m[q], mx), mu = mn == -INFINITY ? 0.0f : mn;  // nothing visible yet: keep the differences defined
+      const float corr = exp2f((m[q] - mu) * kLog2e);
+      float rs = 0.0f;
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float p = exp2f((sc[q][e] - mu) * kLog2e);
+        Ps[(2 * ty + q) * (AW_T + 1) + tx + 16 * e] = p;
+        rs += p;
+      }
+#pragma unroll
+      for (int w = 8; w > 0; w >>= 1) rs += __shfl_xor_sync(0xffffffffu, rs, w);
+      l[q] = l[q] * corr + rs;
+      m[q] = mn;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) { o[q][j].x *= corr; o[q][j].y *= corr; o[q][j].z *= corr; o[q][j].w *= corr; }
+    }
+    __syncthreads();
+    for (int k = 0; k < AW_T; ++k) {
+      const float p0 = Ps[(2 * ty) * (AW_T + 1) + k], p1 = Ps[(2 * ty + 1) * (AW_T + 1) + k];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        if (4 * tx + 64 * j < a.Ep) {
+          const float4 v = *reinterpret_cast<const float4 *>(Vs + k * ldv + 4 * tx + 64 * j);
+          o[0][j].x = fmaf(p0, v.x, o[0][j].x); o[0][j].y = fmaf(p0, v.y, o[0][j].y);
+          o[0][j].z = fmaf(p0, v.z, o[0][j].z); o[0][j].w = fmaf(p0, v.w, o[0][j].w);
+          o[1][j].x = fmaf(p1, v.x, o[1][j].x); o[1][j].y = fmaf(p1, v.y, o[1][j].y);
+          o[1][j].z = fmaf(p1, v.z, o[1][j].z); o[1][j].w = fmaf(p1, v.w, o[1][j].w);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int q = 0; q < 2; ++q) {
+    const int qi = q0 + 2 * ty + q;
+    if (qi >= a.s) continue;
+    const int64_t r = (int64_t)b * a.s + qi;
+    float inv = 1.0f / l[q];
+    if (a.gate_off >= 0) inv *= sigmoidf(a.qkv[r * a.ld + a.gate_off + h]);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int c = 4 * tx + 64 * j;
+      if (c >= a.Ep) continue;
+      const float4 v = make_float4(o[q][j].x * inv, o[q][j].y * inv, o[q][j].z * inv, o[q][j].w * inv);
+      const int64_t at = r * a.out_ld + (int64_t)h * a.Ep + c;
+      if (a.bf.hi) {
+        *reinterpret_cast<uint2 *>(a.bf.hi + at) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+        if (a.bf.lo) *reinterpret_cast<uint2 *>(a.bf.lo + at) = make_uint2(pack_bf16(bf16_lo(v.x), bf16_lo(v.y)), pack_bf16(bf16_lo(v.z), bf16_lo(v.w)));
+      } else {
+        *reinterpret_cast<float4 *>(a.out + at) = v;
+      }
+    }
+  }
+}
+
+static int check_attn(caten_b200_ctx *ctx, const AttnArgs &a) {
+  if (a.H <= 0 || a.G <= 0 || a.H % a.G || a.D <= 0 || a.E <= 0 || a.Dp % 16 || a.Ep % 16 || a.D > a.Dp || a.E > a.Ep || a.cap <= 0 || a.n < 0)
+    return fail(ctx, CATEN_B200_EINVAL, "attention: bad shape");
+  if (a.Dp > 256 || a.Ep > 256) return fail(ctx, CATEN_B200_EUNSUPPORTED, "attention: head size above 256");
+  if (a.H > 65535 || a.B > 65535) return fail(ctx, CATEN_B200_EUNSUPPORTED, "attention: B or H > 65535");
+  return 0;
+}
+
+int launch_attn_window_prefill(caten_b200_ctx *ctx, const AttnArgs &a, int tensor_cores) {
+  if (a.B <= 0 || a.s <= 0) return 0;
+  if (int rc = check_attn(ctx, a)) return rc;
+  // every key the step's queries may see is still in the ring
+  const int64_t span = a.window > 0 && (int64_t)a.window - 1 < a.n ? (int64_t)a.window - 1 + a.s : (int64_t)a.n + a.s;
+  if (span > a.cap) return fail(ctx, CATEN_B200_EINVAL, "attention: %lld live positions in a ring of %lld", (long long)span, (long long)a.cap);
+  if (tensor_cores && a.Dp <= 128 && a.Ep <= 128) return launch_attention_tc_ex(ctx, a, 1.0f);
+  const size_t smem = ((size_t)2 * AW_T * (a.Dp + 4) + (size_t)AW_T * (a.Ep + 4) + (size_t)AW_T * (AW_T + 1)) * sizeof(float);
+  CB_CUDA(ctx, cudaFuncSetAttribute(attn_window_simt_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  launch_k(ctx, attn_window_simt_kernel, dim3((unsigned)((a.s + AW_T - 1) / AW_T), (unsigned)a.H, (unsigned)a.B), dim3(256), smem, a);
+  CB_LAUNCH_CHECK(ctx, "attn_window_simt_kernel");
+  return 0;
+}
+
+// ---------------------------------------------------------------------------------------------
+// Single-token step.  One CTA serves HPC query heads of one key/value head of one sequence, so a K / V
+// row is read once for all of them; with few sequences a thread-block cluster splits the keys and its
+// CTAs combine their (maximum, sum, output) through distributed shared memory.
+//   prologue  the step's q, k, v (from the projection or its split-K partial tiles), rotated and
+//             normalised by one warp each; the k / v row is appended to the ring
+//   scores    KL lanes x NV float4 per K row; the HPC x U dot products of a lane group are reduced
+//             together (each exchange halves the values a lane carries)
+//   softmax   two passes over the CTA's scores in shared memory
+//   output    P.V, summed over the row groups, rescaled over the cluster, gated
+// ---------------------------------------------------------------------------------------------
+constexpr int AD_THREADS = 256;
+
+template <int R>
+__device__ __forceinline__ float group_reduce(float *v, int lane, int lanes) {
+  int step = lanes >> 1;
+#pragma unroll
+  for (int r = R; r > 1; r >>= 1, step >>= 1) {
+    const bool up = (lane & step) != 0;
+#pragma unroll
+    for (int i = 0; i < r / 2; ++i) {
+      const float give = up ? v[i] : v[i + r / 2], keep = up ? v[i + r / 2] : v[i];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, step);
+    }
+  }
+  for (; step > 0; step >>= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], step);
+  return v[0];
+}
+
+template <int KL, int NV, int HPC>
+__global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const AttnArgs a, const int S, const int per_max) {
+  constexpr int GROUPS = AD_THREADS / KL;       // rows in flight per load
+  constexpr int U = HPC == 1 ? 8 : 4;           // loads in flight per lane
+  constexpr int R = U * HPC;                    // dot products reduced together (<= KL)
+  static_assert(R <= KL, "one value per lane after the exchanges");
+  constexpr int TPH = AD_THREADS / HPC;         // threads per head in the softmax
+  extern __shared__ __align__(16) float sm[];
+  const int Dp = a.Dp, Ep = a.Ep;
+  float *q = sm;                                // [HPC][Dp]
+  float *kn = q + HPC * Dp;                     // the step's key
+  float *vn = kn + Dp;                          // and value
+  float *gate = vn + Ep;                        // [4]
+  float *ml = gate + 4;                         // [HPC] max, [HPC] sum (read by the other CTAs of the cluster): 8
+  float *red = ml + 8;                          // 8
+  float *ol = red + 8;                          // [HPC][Ep] this CTA's output
+  float *part = ol + HPC * Ep;                  // [GROUPS][HPC][Ep]
+  float *sc = part + GROUPS * HPC * Ep;         // [HPC][per_max]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int h0 = blockIdx.x * HPC, b = blockIdx.y, rank = blockIdx.z;
+  const int rep = a.H / a.G, g = h0 / rep;
+  float *kb = a.kc + ((int64_t)b * a.G + g) * a.cap * Dp;
+  float *vb = a.vc + ((int64_t)b * a.G + g) * a.cap * Ep;
+  pdl_enter();
+  const int n = a.d_n ? *a.d_n : a.n;
+  const int t0 = a.window > 0 && n - a.window + 1 > 0 ? n - a.window + 1 : 0;
+  const int count = n + 1 - t0, per = (count + S - 1) / S;
+  const int jb = t0 + min(rank * per, count), je = t0 + min((rank + 1) * per, count);  // this CTA's keys
+
+  if (warp < HPC + 2) {
+    const bool is_q = warp < HPC, is_k = warp == HPC;
+    const int64_t off = is_q ? a.q_off + (int64_t)(h0 + warp) * Dp : is_k ? a.k_off + (int64_t)g * Dp : a.v_off + (int64_t)g * Ep;
+    const int np = (is_q || is_k ? Dp : Ep) / 2;
+    HeadPairs h;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = lane + 32 * j;
+      h.p[j] = make_float2(0.f, 0.f);
+      if (i < np) {
+        if (a.pin.splits > 0) h.p[j] = make_float2(partin_load1(a.pin, b, (int)off + 2 * i), partin_load1(a.pin, b, (int)off + 2 * i + 1));
+        else h.p[j] = reinterpret_cast<const float2 *>(a.qkv + (int64_t)b * a.ld + off)[i];
+      }
+    }
+    float mul = 1.0f;
+    if (is_q || is_k) {
+      rotate_pairs(h, a.freq, a.rot_pairs, n, lane);
+      if (a.qk_norm) mul = pairs_inv_rms(h, a.D, a.eps);
+    }
+    if (is_q) mul *= a.scale;
+    float *dst = is_q ? q + warp * Dp : is_k ? kn : vn;
+    float *row = is_k ? kb + (int64_t)(n % a.cap) * Dp : vb + (int64_t)(n % a.cap) * Ep;
+    const bool append = !is_q && rank == 0 && h0 % rep == 0;  // one CTA per key/value head
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = lane + 32 * j;
+      if (i < np) {
+        const float2 v = make_float2(h.p[j].x * mul, h.p[j].y * mul);
+        reinterpret_cast<float2 *>(dst)[i] = v;
+        if (append) reinterpret_cast<float2 *>(row)[i] = v;
+      }
+    }
+  } else if (warp == 7 && lane < HPC && a.gate_off >= 0) {
+    const int col = (int)a.gate_off + h0 + lane;
+    gate[lane] = sigmoidf(a.pin.splits > 0 ? partin_load1(a.pin, b, col) : a.qkv[(int64_t)b * a.ld + col]);
+  }
+  __syncthreads();
+
+  const int gi = tid / KL, gl = tid % KL;
+  const int cap = (int)a.cap, slot0 = jb % cap - jb;  // slot of key j: j + slot0, less cap past the ring's end
+  auto slot_of = [&](int j) { const int s = j + slot0; return (int64_t)(s >= cap ? s - cap : s); };
+  float4 q4[HPC][NV];
+#pragma unroll
+  for (int h = 0; h < HPC; ++h)
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+      const int c = gl + KL * v;
+      q4[h][v] = 4 * c < Dp ? reinterpret_cast<const float4 *>(q + h * Dp)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  for (int j0 = jb; j0 < je; j0 += GROUPS * U) {
+    float4 k4[U][NV];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int j = j0 + u * GROUPS + gi;
+#pragma unroll
+      for (int v = 0; v < NV; ++v) {
+        const int c = gl + KL * v;
+        k4[u][v] = j < je && j < n && 4 * c < Dp ? __ldcs(reinterpret_cast<const float4 *>(kb + slot_of(j) * Dp) + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j == n && j < je && 4 * c < Dp) k4[u][v] = reinterpret_cast<const float4 *>(kn)[c];  // the step's own key
+      }
+    }
+    float d[R];
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+      for (int h = 0; h < HPC; ++h) {
+        float x = 0.0f;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) x = fmaf(q4[h][v].x, k4[u][v].x, fmaf(q4[h][v].y, k4[u][v].y, fmaf(q4[h][v].z, k4[u][v].z, fmaf(q4[h][v].w, k4[u][v].w, x))));
+        d[u * HPC + h] = x;
+      }
+    const float x = group_reduce<R>(d, gl, KL);
+    if (gl % (KL / R) == 0) {
+      const int idx = gl / (KL / R), u = idx / HPC, h = idx % HPC, j = j0 + u * GROUPS + gi;
+      if (j < je) sc[h * per_max + j - jb] = x;
+    }
+  }
+  __syncthreads();
+  {
+    const int h = tid / TPH, i0 = tid % TPH, cnt = je - jb;
+    float *s = sc + h * per_max;
+    float m = -INFINITY;
+    for (int i = i0; i < cnt; i += TPH) m = fmaxf(m, s[i]);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+    if (lane == 0) red[warp] = m;
+    __syncthreads();
+    m = red[h * (8 / HPC)];
+#pragma unroll
+    for (int w = 1; w < 8 / HPC; ++w) m = fmaxf(m, red[h * (8 / HPC) + w]);
+    float ss = 0.0f;
+    for (int i = i0; i < cnt; i += TPH) {
+      const float e = exp2f((s[i] - m) * kLog2e);
+      s[i] = e;
+      ss += e;
+    }
+    ss = warp_sum(ss);
+    __syncthreads();
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    if (i0 == 0) {
+      ss = 0.0f;
+#pragma unroll
+      for (int w = 0; w < 8 / HPC; ++w) ss += red[h * (8 / HPC) + w];
+      ml[h] = m;
+      ml[4 + h] = ss;
+    }
+  }
+  {
+    float4 acc[HPC][NV];
+#pragma unroll
+    for (int h = 0; h < HPC; ++h)
+#pragma unroll
+      for (int v = 0; v < NV; ++v) acc[h][v] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int j0 = jb; j0 < je; j0 += GROUPS * U) {
+      float4 v4[U][NV];
+      float p[U][HPC];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int j = j0 + u * GROUPS + gi;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+          const int c = gl + KL * v;
+          v4[u][v] = j < je && j < n && 4 * c < Ep ? __ldcs(reinterpret_cast<const float4 *>(vb + slot_of(j) * Ep) + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+          if (j == n && j < je && 4 * c < Ep) v4[u][v] = reinterpret_cast<const float4 *>(vn)[c];
+        }
+#pragma unroll
+        for (int h = 0; h < HPC; ++h) p[u][h] = j < je ? sc[h * per_max + j - jb] : 0.0f;
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+#pragma unroll
+        for (int h = 0; h < HPC; ++h)
+#pragma unroll
+          for (int v = 0; v < NV; ++v) {
+            acc[h][v].x = fmaf(p[u][h], v4[u][v].x, acc[h][v].x);
+            acc[h][v].y = fmaf(p[u][h], v4[u][v].y, acc[h][v].y);
+            acc[h][v].z = fmaf(p[u][h], v4[u][v].z, acc[h][v].z);
+            acc[h][v].w = fmaf(p[u][h], v4[u][v].w, acc[h][v].w);
+          }
+    }
+#pragma unroll
+    for (int h = 0; h < HPC; ++h)
+#pragma unroll
+      for (int v = 0; v < NV; ++v) {
+        const int c = gl + KL * v;
+        if (4 * c < Ep) reinterpret_cast<float4 *>(part + (gi * HPC + h) * Ep)[c] = acc[h][v];
+      }
+  }
+  __syncthreads();
+  for (int i = tid; i < HPC * Ep; i += AD_THREADS) {
+    float o = 0.0f;
+#pragma unroll
+    for (int w = 0; w < GROUPS; ++w) o += part[w * HPC * Ep + i];
+    ol[i] = o;
+  }
+  auto finish = [&](int i, float o, float l) {
+    const int h = i / Ep;
+    o = o / l;
+    if (a.gate_off >= 0) o *= gate[h];
+    const int64_t at = (int64_t)b * a.out_ld + (int64_t)(h0 + h) * Ep + (i - h * Ep);
+    if (a.bf.hi) {
+      const __nv_bfloat16 hh = __float2bfloat16_rn(o);
+      a.bf.hi[at] = hh;
+      if (a.bf.lo) a.bf.lo[at] = __float2bfloat16_rn(o - __bfloat162float(hh));
+    } else {
+      a.out[at] = o;
+    }
+  };
+  if (S == 1) {
+    __syncthreads();
+    for (int i = tid; i < HPC * Ep; i += AD_THREADS) finish(i, ol[i], ml[4 + i / Ep]);
+    return;
+  }
+  // combine over the cluster; both barriers are reached by every thread of every CTA
+  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+  const uint32_t ml0 = (uint32_t)__cvta_generic_to_shared(ml), ol0 = (uint32_t)__cvta_generic_to_shared(ol);
+  auto remote = [&](uint32_t local, int z) {
+    uint32_t addr;
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(addr) : "r"(local), "r"(z));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
+    return v;
+  };
+  for (int i = rank + S * tid; i < HPC * Ep; i += S * AD_THREADS) {
+    const uint32_t h4 = 4u * (uint32_t)(i / Ep);
+    float m = -INFINITY;
+    for (int z = 0; z < S; ++z) m = fmaxf(m, remote(ml0 + h4, z));
+    float l = 0.0f, o = 0.0f;
+    for (int z = 0; z < S; ++z) {  // fixed order
+      const float f = exp2f((remote(ml0 + h4, z) - m) * kLog2e);  // a CTA without keys has maximum -inf and adds nothing
+      l = fmaf(f, remote(ml0 + 16u + h4, z), l);
+      o = fmaf(f, remote(ol0 + 4u * (uint32_t)i, z), o);
+    }
+    finish(i, o, l);
+  }
+  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+
+template <int KL, int NV, int HPC>
+static int launch_decode_t(caten_b200_ctx *ctx, const AttnArgs &a, int S, int per_max, size_t smem) {
+  if (smem > 48 * 1024) CB_CUDA(ctx, cudaFuncSetAttribute(attn_window_decode_kernel<KL, NV, HPC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3((unsigned)(a.H / HPC), (unsigned)a.B, (unsigned)S);
+  cfg.blockDim = dim3(AD_THREADS);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = ctx->stream;
+  cudaLaunchAttribute at[2];
+  int na = 0;
+  if (take_pdl(ctx)) {
+    at[na].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[na].val.programmaticStreamSerializationAllowed = 1;
+    ++na;
+  }
+  if (S > 1) {
+    at[na].id = cudaLaunchAttributeClusterDimension;
+    at[na].val.clusterDim.x = 1;
+    at[na].val.clusterDim.y = 1;
+    at[na].val.clusterDim.z = (unsigned)S;
+    ++na;
+  }
+  cfg.attrs = at;
+  cfg.numAttrs = na;
+  CB_CUDA(ctx, cudaLaunchKernelEx(&cfg, attn_window_decode_kernel<KL, NV, HPC>, a, S, per_max));
+  CB_LAUNCH_CHECK(ctx, "attn_window_decode_kernel");
+  return 0;
+}
+
+int launch_attn_window_decode(caten_b200_ctx *ctx, const AttnArgs &a) {
+  if (a.B <= 0) return 0;
+  if (a.s != 1) return fail(ctx, CATEN_B200_EINVAL, "attention: the decode kernel takes one token per sequence");
+  if (int rc = check_attn(ctx, a)) return rc;
+  // the most keys a query may see (with a device-side position: what the cache allows)
+  int64_t keys = a.d_n ? a.cap : (int64_t)a.n + 1;
+  if (a.window > 0 && a.window < keys) keys = a.window;
+  if (keys > a.cap) return fail(ctx, CATEN_B200_EINVAL, "attention: %lld live positions in a ring of %lld", (long long)keys, (long long)a.cap);
+  const int rep = a.H / a.G;
+  int hpc = rep % 4 == 0 ? 4 : rep % 2 == 0 ? 2 : 1;
+  const int wide = a.Dp > a.Ep ? a.Dp : a.Ep;
+  if (wide > 128 && hpc == 4) hpc = 2;  // registers
+  // few sequences: split the keys over the CTAs of a cluster (8 = portable size), at least 32 keys each
+  auto ctas = [&](int h, int s) { return (int64_t)a.B * (a.H / h) * s; };
+  int S = 1;
+  while (S < 8 && ctas(hpc, S) < ctx->sm_count && keys / (2 * S) >= 32) S *= 2;
+  while (hpc > 1 && ctas(hpc, S) * 2 <= ctx->sm_count) hpc /= 2;
+  const int kl = wide <= 64 ? 16 : 32, nv = wide <= 128 ? 1 : 2, groups = AD_THREADS / kl;
+  size_t smem = 0;
+  int64_t per_max = 0;
+  for (;;) {
+    per_max = (keys + S - 1) / S;
+    smem = ((size_t)hpc * a.Dp + a.Dp + a.Ep + 20 + (size_t)hpc * a.Ep * (1 + groups) + (size_t)hpc * per_max) * sizeof(float);
+    if (smem <= 200 * 1024) break;
+    if (S < 8) S *= 2;
+    else if (hpc > 1) hpc /= 2;
+    else return fail(ctx, CATEN_B200_EUNSUPPORTED, "attention: context too long for the decode kernel");
+  }
+#define AD_CASE(KL, NV)                                                                                    \
+  (hpc == 4 ? launch_decode_t<KL, NV, 4>(ctx, a, S, (int)per_max, smem)                                    \
+   : hpc == 2 ? launch_decode_t<KL, NV, 2>(ctx, a, S, (int)per_max, smem) : launch_decode_t<KL, NV, 1>(ctx, a, S, (int)per_max, smem))
+  if (kl == 16) return AD_CASE(16, 1);
+  if (nv == 1) return AD_CASE(32, 1);
+  return AD_CASE(32, 2);
+#undef AD_CASE
+}
+
+}  // namespace cb

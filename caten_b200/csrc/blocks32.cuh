@@ -64,6 +64,14 @@ __device__ __forceinline__ void load_w8(const void *qs, const __half *d, const _
     const __half *h = reinterpret_cast<const __half *>(&v);
 #pragma unroll
     for (int e = 0; e < 8; ++e) o[e] = __half2float(h[e]);
+  } else if (WT == CATEN_B200_BF16) {
+    const uint4 v = *reinterpret_cast<const uint4 *>((const uint16_t *)qs + row * K + (int64_t)kb * 32 + part * 8);
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      o[2 * e] = __uint_as_float(w[e] << 16);
+      o[2 * e + 1] = __uint_as_float(w[e] & 0xFFFF0000u);
+    }
   } else if (WT == CATEN_B200_Q8_0) {
     const int64_t bi = row * nkb + kb;
     const uint2 v = *reinterpret_cast<const uint2 *>((const int8_t *)qs + bi * 32 + part * 8);

@@ -10,6 +10,7 @@
 
 #include "common.cuh"
 #include "blocks32.cuh"
+#include "step_loop.cuh"
 
 namespace cb {
 
@@ -53,28 +54,23 @@ static int check_status(caten_b200_ctx *ctx) {
   return 0;
 }
 
-// Brackets one kernel-class call with events when that class is being profiled.
-struct ProfScope {
-  caten_b200_ctx *ctx;
-  cudaEvent_t b = nullptr;
-  ProfScope(caten_b200_ctx *c, int klass) : ctx(c) {
-    if (!(ctx->prof_mask & (1u << klass))) return;
-    cudaEvent_t a;
-    auto get = [&]() {
-      cudaEvent_t e;
-      if (!ctx->prof_pool.empty()) { e = ctx->prof_pool.back(); ctx->prof_pool.pop_back(); }
-      else cudaEventCreate(&e);
-      return e;
-    };
-    a = get();
-    b = get();
-    cudaEventRecord(a, ctx->stream);
-    ctx->prof.push_back({klass, a, b});
-  }
-  ~ProfScope() {
-    if (b) cudaEventRecord(b, ctx->stream);
-  }
-};
+ProfScope::ProfScope(caten_b200_ctx *c, int klass) : ctx(c) {
+  if (!(ctx->prof_mask & (1u << klass))) return;
+  cudaEvent_t a;
+  auto get = [&]() {
+    cudaEvent_t e;
+    if (!ctx->prof_pool.empty()) { e = ctx->prof_pool.back(); ctx->prof_pool.pop_back(); }
+    else cudaEventCreate(&e);
+    return e;
+  };
+  a = get();
+  b = get();
+  cudaEventRecord(a, ctx->stream);
+  ctx->prof.push_back({klass, a, b});
+}
+ProfScope::~ProfScope() {
+  if (b) cudaEventRecord(b, ctx->stream);
+}
 
 }  // namespace cb
 
@@ -271,7 +267,7 @@ int64_t caten_b200_weight_nbytes(int type, int64_t rows, int64_t cols) {
   const int64_t n = rows * cols;
   switch (type) {
     case CATEN_B200_F32: return n * 4;
-    case CATEN_B200_F16: return n * 2;
+    case CATEN_B200_F16: case CATEN_B200_BF16: return n * 2;
     case CATEN_B200_Q4_0: case CATEN_B200_Q4_1: case CATEN_B200_Q5_0: case CATEN_B200_Q5_1: case CATEN_B200_Q8_0:
       return cols % 32 ? -1 : n / 32 * cb::type_block_bytes(type);
   }
@@ -286,7 +282,7 @@ int caten_b200_weight_upload_device(caten_b200_ctx *ctx, int type, const void *d
   if (!d_blocks || rows <= 0 || cols <= 0) return fail(ctx, CATEN_B200_EINVAL, "weight_upload: NULL data or empty shape %lldx%lld", (long long)rows, (long long)cols);
   const int64_t nbytes = caten_b200_weight_nbytes(type, rows, cols);
   if (nbytes < 0)
-    return fail(ctx, CATEN_B200_EUNSUPPORTED, "weight_upload: ggml type %d with cols=%lld (types: F32=0 F16=1 Q4_0=2 Q4_1=3 Q5_0=6 Q5_1=7 Q8_0=8 Q2_K=10 Q3_K=11 Q4_K=12 Q5_K=13 Q6_K=14; cols a multiple of the block size)", type, (long long)cols);
+    return fail(ctx, CATEN_B200_EUNSUPPORTED, "weight_upload: ggml type %d with cols=%lld (types: F32=0 F16=1 Q4_0=2 Q4_1=3 Q5_0=6 Q5_1=7 Q8_0=8 Q2_K=10 Q3_K=11 Q4_K=12 Q5_K=13 Q6_K=14 BF16=30; cols a multiple of the block size)", type, (long long)cols);
   caten_b200_weight *w = new (std::nothrow) caten_b200_weight();
   if (!w) return fail(ctx, CATEN_B200_ECUDA, "out of host memory");
   w->type = type; w->rows = rows; w->cols = cols; w->ctx = ctx;
@@ -297,7 +293,7 @@ int caten_b200_weight_upload_device(caten_b200_ctx *ctx, int type, const void *d
     w->device_bytes = rows * cols * (int64_t)sizeof(float);
     if ((e = cudaMalloc(&w->qs, (size_t)(rows * cols) * sizeof(float))) != cudaSuccess) { delete w; return cuda_fail(ctx, e, "cudaMalloc(weight)"); }
     if (int rc = launch_dequant_extra(ctx, type, (const uint8_t *)d_blocks, rows * cols, (float *)w->qs)) { cudaFree(w->qs); delete w; return rc; }
-  } else if (type == CATEN_B200_F32 || type == CATEN_B200_F16) {
+  } else if (type == CATEN_B200_F32 || type == CATEN_B200_F16 || type == CATEN_B200_BF16) {
     w->device_bytes = nbytes;
     if ((e = cudaMalloc(&w->qs, (size_t)nbytes)) != cudaSuccess) { delete w; return cuda_fail(ctx, e, "cudaMalloc(weight)"); }
     if ((e = cudaMemcpyAsync(w->qs, d_blocks, (size_t)nbytes, cudaMemcpyDeviceToDevice, ctx->stream)) != cudaSuccess) {
@@ -337,7 +333,7 @@ int caten_b200_weight_upload(caten_b200_ctx *ctx, int type, const void *h_blocks
   if (!h_blocks || rows <= 0 || cols <= 0) return fail(ctx, CATEN_B200_EINVAL, "weight_upload: NULL data or empty shape %lldx%lld", (long long)rows, (long long)cols);
   const int64_t nbytes = caten_b200_weight_nbytes(type, rows, cols);
   if (nbytes < 0)
-    return fail(ctx, CATEN_B200_EUNSUPPORTED, "weight_upload: ggml type %d with cols=%lld (types: F32=0 F16=1 Q4_0=2 Q4_1=3 Q5_0=6 Q5_1=7 Q8_0=8 Q2_K=10 Q3_K=11 Q4_K=12 Q5_K=13 Q6_K=14; cols a multiple of the block size)", type, (long long)cols);
+    return fail(ctx, CATEN_B200_EUNSUPPORTED, "weight_upload: ggml type %d with cols=%lld (types: F32=0 F16=1 Q4_0=2 Q4_1=3 Q5_0=6 Q5_1=7 Q8_0=8 Q2_K=10 Q3_K=11 Q4_K=12 Q5_K=13 Q6_K=14 BF16=30; cols a multiple of the block size)", type, (long long)cols);
   // file / host bytes -> pinned bounce buffers -> a staging area on the device (kept by the context and reused by
   // the next upload: work on the stream is ordered, so the re-layout kernel has read it before it is overwritten)
   if (int rc = scratch_reserve(ctx, &ctx->upload_stage, (size_t)nbytes)) return rc;
@@ -374,6 +370,12 @@ int caten_b200_weight_dequant(caten_b200_ctx *ctx, const caten_b200_weight *w, f
 // kernels
 // ------------------------------------------------------------------------------------------------
 static bool aligned16(const void *p) { return ((uintptr_t)p & 15) == 0; }
+static int check_glu(caten_b200_ctx *ctx, const char *who, const caten_b200_weight *w, int act, const void *residual) {
+  if (act != CATEN_B200_ACT_RELU_GLU) return 0;
+  if (residual || w->rows % 2 || (w->type != CATEN_B200_F32 && w->type != CATEN_B200_F16 && w->type != CATEN_B200_BF16))
+    return fail(ctx, CATEN_B200_EUNSUPPORTED, "%s: the gated activation takes a dense weight with an even number of rows and no residual", who);
+  return 0;
+}
 
 int caten_b200_linear(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *d_x, const float *d_bias,
                       const float *d_residual, int act, float *d_y, int64_t M, int precision) {
@@ -381,13 +383,15 @@ int caten_b200_linear(caten_b200_ctx *ctx, const caten_b200_weight *w, const flo
   if (!w || !d_x || !d_y) return fail(ctx, CATEN_B200_EINVAL, "linear: NULL argument");
   if (M < 0) return fail(ctx, CATEN_B200_EINVAL, "linear: M < 0");
   if (M == 0) return 0;
-  if (act < 0 || act > 2) return fail(ctx, CATEN_B200_EINVAL, "linear: unknown activation %d", act);
+  if (act < 0 || act > CATEN_B200_ACT_RELU_GLU) return fail(ctx, CATEN_B200_EINVAL, "linear: unknown activation %d", act);
+  if (int rc = check_glu(ctx, "linear", w, act, d_residual)) return rc;
+  const int64_t ny = act == CATEN_B200_ACT_RELU_GLU ? w->rows / 2 : w->rows;
   if (!aligned16(d_x) || !aligned16(d_y)) return fail(ctx, CATEN_B200_EINVAL, "linear: x and y must be 16-byte aligned");
   ProfScope prof(ctx, M <= 4 ? CATEN_B200_K_GEMV : CATEN_B200_K_GEMM);
   if (M <= 4) {
     for (int64_t m = 0; m < M; ++m)
-      if (int rc = launch_gemv(ctx, w, d_x + m * w->cols, d_bias, d_residual ? d_residual + m * w->rows : nullptr, act,
-                               d_y + m * w->rows))
+      if (int rc = launch_gemv(ctx, w, d_x + m * w->cols, d_bias, d_residual ? d_residual + m * ny : nullptr, act,
+                               d_y + m * ny))
         return rc;
     return 0;
   }
@@ -405,13 +409,15 @@ int caten_b200_linear_noalloc(caten_b200_ctx *ctx, const caten_b200_weight *w, c
   if (!w || !d_x || !d_y) return fail(ctx, CATEN_B200_EINVAL, "linear_noalloc: NULL argument");
   if (M < 0) return fail(ctx, CATEN_B200_EINVAL, "linear_noalloc: M < 0");
   if (M == 0) return 0;
-  if (act < 0 || act > 2) return fail(ctx, CATEN_B200_EINVAL, "linear_noalloc: unknown activation %d", act);
+  if (act < 0 || act > CATEN_B200_ACT_RELU_GLU) return fail(ctx, CATEN_B200_EINVAL, "linear_noalloc: unknown activation %d", act);
+  if (int rc = check_glu(ctx, "linear_noalloc", w, act, d_residual)) return rc;
+  const int64_t ny = act == CATEN_B200_ACT_RELU_GLU ? w->rows / 2 : w->rows;
   if (!aligned16(d_x) || !aligned16(d_y)) return fail(ctx, CATEN_B200_EINVAL, "linear_noalloc: x and y must be 16-byte aligned");
   ProfScope prof(ctx, M <= 4 ? CATEN_B200_K_GEMV : CATEN_B200_K_GEMM);
   if (M <= 4) {  // the dequant-GEMV uses no scratch memory
     for (int64_t m = 0; m < M; ++m)
-      if (int rc = launch_gemv(ctx, w, d_x + m * w->cols, d_bias, d_residual ? d_residual + m * w->rows : nullptr, act,
-                               d_y + m * w->rows))
+      if (int rc = launch_gemv(ctx, w, d_x + m * w->cols, d_bias, d_residual ? d_residual + m * ny : nullptr, act,
+                               d_y + m * ny))
         return rc;
     return 0;
   }
@@ -502,6 +508,27 @@ int caten_b200_eval_expr(caten_b200_ctx *ctx, const caten_b200_expr *e) {
 // ------------------------------------------------------------------------------------------------
 // whole model
 // ------------------------------------------------------------------------------------------------
+namespace cb {
+
+int model_linear(caten_b200_ctx *ctx, int prec, const caten_b200_weight *w, const float *x, BfOut xbf, const float *bias, const float *res,
+                 int act, float *y, BfOut ybf, int64_t M, PartIn *defer, LinGroups grp) {
+  if (defer) *defer = PartIn();
+  if (M <= 0) return 0;
+  if (int rc = check_glu(ctx, "linear", w, act, res)) return rc;
+  const int64_t ny = act == CATEN_B200_ACT_RELU_GLU ? w->rows / 2 : w->rows;
+  ProfScope prof(ctx, M <= 4 ? CATEN_B200_K_GEMV : CATEN_B200_K_GEMM);
+  if (M <= 4) {
+    for (int64_t m = 0; m < M; ++m)
+      if (int rc = launch_gemv(ctx, w, x + m * w->cols, bias, res ? res + m * ny : nullptr, act, y + m * ny, grp)) return rc;
+    return 0;
+  }
+  if (prec == CATEN_B200_PREC_FP32) return launch_gemm_simt(ctx, w, x, bias, res, act, y, M, grp);
+  const int nsplit = prec == CATEN_B200_PREC_BF16X3 ? 3 : 1;
+  return launch_gemm_tc_ex(ctx, w, xbf.hi ? nullptr : x, xbf.hi, nsplit == 3 ? xbf.lo : nullptr, bias, res, act, y, ybf, M, nsplit, defer, grp);
+}
+
+}  // namespace cb
+
 struct caten_b200_gpt2 {
   caten_b200_ctx *ctx = nullptr;
   caten_b200_gpt2_desc desc;
@@ -516,17 +543,12 @@ struct caten_b200_gpt2 {
   cb::BfOut xn_bf, att_bf, ff_bf, last_bf;
   void *bf_arena = nullptr;
   float *ids_f32 = nullptr;  // staging for host ids [B * T]
-  int64_t *out_ids = nullptr;
   float *h_ids_pinned = nullptr;
   int64_t *h_out_pinned = nullptr;
   int64_t launches0 = 0;
   // decode replayed from a CUDA graph: position and ids live on the device
-  int *d_pos = nullptr, *h_pos_pinned = nullptr;
-  int64_t *ids_io = nullptr;   // [B] input ids of the next step
-  int64_t *ids_hist = nullptr; // [T, B] row n = ids produced by the step that started at position n
-  cudaGraphExec_t graph = nullptr;
-  void *graph_xbf = nullptr, *graph_wtmp = nullptr;  // scratch pointers baked into the graph
-  int64_t launches_per_step = 0;
+  cb::StepLoop loop;
+  int *h_pos_pinned = nullptr;
   // 1..4 sequences: the whole single-token step is one kernel (decode_small.cu); CATEN_B200_PERSISTENT=0 keeps
   // the kernel-per-operation path
   cb::DecodeSmall *ds = nullptr;
@@ -534,17 +556,9 @@ struct caten_b200_gpt2 {
   bool defer_reduce = true;  // CATEN_B200_DEFER_REDUCE=0 keeps a reduction kernel behind every split-K linear
 };
 
-// Linear inside the model: with a tensor-core precision and more than 4 rows the input arrives
-// already split into bf16 (hi, lo) from its producer and the output can be requested the same way.
 static int model_linear(caten_b200_gpt2 *m, const caten_b200_weight *w, const float *x, cb::BfOut xbf, const float *bias,
                         const float *res, int act, float *y, cb::BfOut ybf, int64_t M, cb::PartIn *defer = nullptr) {
-  if (defer) *defer = cb::PartIn();
-  caten_b200_ctx *ctx = m->ctx;
-  const int prec = m->desc.precision;
-  if (prec == CATEN_B200_PREC_FP32 || M <= 4) return caten_b200_linear(ctx, w, x, bias, res, act, y, M, prec);
-  ProfScope prof(ctx, CATEN_B200_K_GEMM);
-  const int nsplit = prec == CATEN_B200_PREC_BF16X3 ? 3 : 1;
-  return launch_gemm_tc_ex(ctx, w, nullptr, xbf.hi, nsplit == 3 ? xbf.lo : nullptr, bias, res, act, y, ybf, M, nsplit, defer);
+  return cb::model_linear(m->ctx, m->desc.precision, w, x, xbf, bias, res, act, y, ybf, M, defer);
 }
 
 extern "C" {
@@ -613,10 +627,7 @@ int caten_b200_gpt2_create(caten_b200_ctx *ctx, const caten_b200_gpt2_desc *dsc,
     }
   }
   if (!rc) rc = alloc(&m->ids_f32, B * T);
-  if (!rc) rc = caten_b200_malloc(ctx, (size_t)B * sizeof(int64_t), (void **)&m->out_ids);
-  if (!rc) rc = caten_b200_malloc(ctx, (size_t)B * sizeof(int64_t), (void **)&m->ids_io);
-  if (!rc) rc = caten_b200_malloc(ctx, (size_t)B * T * sizeof(int64_t), (void **)&m->ids_hist);
-  if (!rc) rc = caten_b200_malloc(ctx, sizeof(int), (void **)&m->d_pos);
+  if (!rc) rc = cb::step_loop_alloc(ctx, &m->loop, B, T);
   if (!rc && cudaMallocHost(&m->h_pos_pinned, sizeof(int)) != cudaSuccess) rc = fail(ctx, CATEN_B200_ECUDA, "cudaMallocHost(pos)");
   if (!rc && cudaMallocHost(&m->h_ids_pinned, (size_t)B * T * sizeof(float)) != cudaSuccess) rc = fail(ctx, CATEN_B200_ECUDA, "cudaMallocHost(ids)");
   if (!rc && cudaMallocHost(&m->h_out_pinned, (size_t)B * sizeof(int64_t)) != cudaSuccess) rc = fail(ctx, CATEN_B200_ECUDA, "cudaMallocHost(out ids)");
@@ -624,8 +635,8 @@ int caten_b200_gpt2_create(caten_b200_ctx *ctx, const caten_b200_gpt2_desc *dsc,
   if (const char *e = getenv("CATEN_B200_PERSISTENT")) persistent = atoi(e) != 0;
   if (!rc && persistent && cb::decode_small_supported(m->desc, m->attn_w.data(), m->proj_w.data(), m->fc_w.data(), m->mproj_w.data())) {
     const std::vector<const float *> vecs[8] = {m->ln1_g, m->ln1_b, m->attn_b, m->proj_b, m->ln2_g, m->ln2_b, m->fc_b, m->mproj_b};
-    rc = cb::decode_small_create(ctx, m->desc, m->attn_w, m->proj_w, m->fc_w, m->mproj_w, vecs, m->kc, m->vc, m->ids_io, m->out_ids,
-                                 m->ids_hist, m->d_pos, m->logits, &m->ds);
+    rc = cb::decode_small_create(ctx, m->desc, m->attn_w, m->proj_w, m->fc_w, m->mproj_w, vecs, m->kc, m->vc, m->loop.ids_io, m->loop.out_ids,
+                                 m->loop.hist, m->loop.d_pos, m->logits, &m->ds);
     m->ds_failures_seen = ctx->device_failures;
   }
   if (rc) { caten_b200_gpt2_destroy(m); return rc; }
@@ -643,13 +654,9 @@ int caten_b200_gpt2_destroy(caten_b200_gpt2 *m) {
   for (float *p : m->vc) if (p) cudaFree(p);
   float *bufs[] = {m->h, m->h2, m->xn, m->qkv, m->att, m->ff, m->last, m->logits, m->ids_f32};
   for (float *p : bufs) if (p) cudaFree(p);
-  if (m->graph) cudaGraphExecDestroy(m->graph);
+  cb::step_loop_free(&m->loop);
   cb::decode_small_destroy(m->ds);
   if (m->bf_arena) cudaFree(m->bf_arena);
-  if (m->out_ids) cudaFree(m->out_ids);
-  if (m->ids_io) cudaFree(m->ids_io);
-  if (m->ids_hist) cudaFree(m->ids_hist);
-  if (m->d_pos) cudaFree(m->d_pos);
   if (m->h_pos_pinned) cudaFreeHost(m->h_pos_pinned);
   if (m->h_ids_pinned) cudaFreeHost(m->h_ids_pinned);
   if (m->h_out_pinned) cudaFreeHost(m->h_out_pinned);
@@ -720,10 +727,10 @@ int caten_b200_gpt2_step_device(caten_b200_gpt2 *m, const float *d_ids_f32, cons
   const int64_t B = c.batch;
   if (s == 1 && m->ds) {
     // single-token step of a few sequences: the one-kernel path, fed from the device-side state
-    if (int rc = launch_begin_steps(ctx, d_ids_f32, d_ids_i64, m->ids_io, m->d_pos, n, B)) return rc;
+    if (int rc = launch_begin_steps(ctx, d_ids_f32, d_ids_i64, m->loop.ids_io, m->loop.d_pos, n, B)) return rc;
     if (int rc = decode_step_device_pos(m, n)) return rc;
-    if (d_out_ids != m->out_ids)
-      CB_CUDA(ctx, cudaMemcpyAsync(d_out_ids, m->out_ids, (size_t)B * sizeof(int64_t), cudaMemcpyDeviceToDevice, ctx->stream));
+    if (d_out_ids != m->loop.out_ids)
+      CB_CUDA(ctx, cudaMemcpyAsync(d_out_ids, m->loop.out_ids, (size_t)B * sizeof(int64_t), cudaMemcpyDeviceToDevice, ctx->stream));
     return 0;
   }
   int64_t per = m->max_rows / s;
@@ -755,12 +762,12 @@ int caten_b200_gpt2_step(caten_b200_gpt2 *m, const float *h_ids_f32, int64_t s, 
     // into the device-side state first); the result is the same as the kernel-by-kernel path
     if (n < 0 || n + 1 > m->desc.max_seq_len)
       return fail(ctx, CATEN_B200_EINVAL, "gpt2_step: s=1 n=%lld outside the cache (max_seq_len=%d)", (long long)n, m->desc.max_seq_len);
-    if (int rc = launch_begin_steps(ctx, m->ids_f32, nullptr, m->ids_io, m->d_pos, n, B)) return rc;
+    if (int rc = launch_begin_steps(ctx, m->ids_f32, nullptr, m->loop.ids_io, m->loop.d_pos, n, B)) return rc;
     if (int rc = decode_run(m, n, 1)) return rc;
-  } else if (int rc = caten_b200_gpt2_step_device(m, m->ids_f32, nullptr, s, n, m->out_ids)) {
+  } else if (int rc = caten_b200_gpt2_step_device(m, m->ids_f32, nullptr, s, n, m->loop.out_ids)) {
     return rc;
   }
-  CB_CUDA(ctx, cudaMemcpyAsync(m->h_out_pinned, m->out_ids, (size_t)B * sizeof(int64_t), cudaMemcpyDeviceToHost, ctx->stream));
+  CB_CUDA(ctx, cudaMemcpyAsync(m->h_out_pinned, m->loop.out_ids, (size_t)B * sizeof(int64_t), cudaMemcpyDeviceToHost, ctx->stream));
   if (int rc = caten_b200_sync(ctx)) return rc;
   memcpy(h_out_ids, m->h_out_pinned, (size_t)B * sizeof(int64_t));
   return 0;
@@ -779,53 +786,17 @@ static int decode_step_device_pos(caten_b200_gpt2 *m, int64_t n_host) {
     ProfScope prof(ctx, CATEN_B200_K_DECODE_STEP);
     return cb::decode_small_launch(ctx, m->ds);
   }
-  if (int rc = run_chunk(m, nullptr, m->ids_io, 0, c.batch, 1, n_host, m->d_pos)) return rc;
+  if (int rc = run_chunk(m, nullptr, m->loop.ids_io, 0, c.batch, 1, n_host, m->loop.d_pos)) return rc;
   if (int rc = model_linear(m, c.lm_head, m->last, m->last_bf, nullptr, nullptr, CATEN_B200_ACT_NONE, m->logits, cb::BfOut(), c.batch)) return rc;
-  if (int rc = launch_argmax(ctx, m->logits, c.batch, c.vocab, m->out_ids)) return rc;
-  return launch_finish_step(ctx, m->out_ids, m->ids_io, m->ids_hist, m->d_pos, c.batch);
+  if (int rc = launch_argmax(ctx, m->logits, c.batch, c.vocab, m->loop.out_ids)) return rc;
+  return launch_finish_step(ctx, m->loop.out_ids, m->loop.ids_io, m->loop.hist, m->loop.d_pos, c.batch);
 }
 
-// Runs `steps` single-token steps from the device-side state (ids_io, d_pos already loaded).
-// The launch sequence of a step is captured into a CUDA graph the first time and replayed.
+// Runs `steps` single-token steps from the device-side state.
 static int decode_run(caten_b200_gpt2 *m, int64_t n, int64_t steps) {
-  caten_b200_ctx *ctx = m->ctx;
-  const int64_t T = m->desc.max_seq_len;
-  int64_t done = 0;
   // event brackets cannot be placed inside a graph; a step that is one kernel already gains nothing from one
-  const bool use_graph = ctx->prof_mask == 0 && !m->ds;
-  if (use_graph && m->graph && (m->graph_xbf != ctx->xbf.ptr || m->graph_wtmp != ctx->wtmp.ptr)) {
-    cudaGraphExecDestroy(m->graph);  // scratch was re-allocated since the capture: its pointers are stale
-    m->graph = nullptr;
-  }
-  if (use_graph && !m->graph) {
-    // the first step runs eagerly: it sizes the scratch buffers and sets kernel attributes, which
-    // must not happen during capture
-    if (int rc = decode_step_device_pos(m, n)) return rc;
-    done = 1;
-    cudaGraph_t g = nullptr;
-    CB_CUDA(ctx, cudaStreamBeginCapture(ctx->stream, cudaStreamCaptureModeThreadLocal));
-    const int64_t before = ctx->launches;
-    const int rc = decode_step_device_pos(m, n + 1 < T ? n + 1 : T - 1);  // host-side position only feeds argument checks
-    const cudaError_t e = cudaStreamEndCapture(ctx->stream, &g);
-    m->launches_per_step = ctx->launches - before;
-    ctx->launches = before;  // captured, not launched
-    if (rc) { if (g) cudaGraphDestroy(g); return rc; }
-    if (e != cudaSuccess) return cuda_fail(ctx, e, "cudaStreamEndCapture");
-    const cudaError_t e2 = cudaGraphInstantiate(&m->graph, g, 0);
-    cudaGraphDestroy(g);
-    if (e2 != cudaSuccess) { m->graph = nullptr; return cuda_fail(ctx, e2, "cudaGraphInstantiate"); }
-    m->graph_xbf = ctx->xbf.ptr;
-    m->graph_wtmp = ctx->wtmp.ptr;
-  }
-  for (; done < steps; ++done) {
-    if (use_graph && m->graph) {
-      CB_CUDA(ctx, cudaGraphLaunch(m->graph, ctx->stream));
-      ctx->launches += m->launches_per_step;
-    } else if (int rc = decode_step_device_pos(m, n + done)) {
-      return rc;
-    }
-  }
-  return 0;
+  const bool use_graph = m->ctx->prof_mask == 0 && !m->ds;
+  return cb::step_loop_run(m->ctx, &m->loop, n, steps, m->desc.max_seq_len, use_graph, [m](int64_t pos) { return decode_step_device_pos(m, pos); });
 }
 
 int caten_b200_gpt2_decode(caten_b200_gpt2 *m, const int64_t *d_first_ids, int64_t n, int64_t steps, int64_t *d_out_ids) {
@@ -838,10 +809,10 @@ int caten_b200_gpt2_decode(caten_b200_gpt2 *m, const int64_t *d_first_ids, int64
   if (steps < 0 || n < 0 || n + steps > c.max_seq_len)
     return fail(ctx, CATEN_B200_EINVAL, "gpt2_decode: positions [%lld, %lld) outside the cache (max_seq_len=%d)", (long long)n, (long long)(n + steps), c.max_seq_len);
   if (steps == 0) return 0;
-  if (int rc = launch_begin_steps(ctx, nullptr, d_first_ids, m->ids_io, m->d_pos, n, B)) return rc;
+  if (int rc = launch_begin_steps(ctx, nullptr, d_first_ids, m->loop.ids_io, m->loop.d_pos, n, B)) return rc;
   if (int rc = decode_run(m, n, steps)) return rc;
   if (d_out_ids)
-    CB_CUDA(ctx, cudaMemcpyAsync(d_out_ids, m->ids_hist + n * B, (size_t)(steps * B) * sizeof(int64_t), cudaMemcpyDeviceToDevice, ctx->stream));
+    CB_CUDA(ctx, cudaMemcpyAsync(d_out_ids, m->loop.hist + n * B, (size_t)(steps * B) * sizeof(int64_t), cudaMemcpyDeviceToDevice, ctx->stream));
   return 0;
 }
 

@@ -78,6 +78,13 @@ __device__ __forceinline__ float partin_load1(const PartIn &p, long long m, int 
 }
 #endif
 
+// How a linear's input is laid out when groups of its output rows read different inputs: output rows
+// [g * group_rows, (g + 1) * group_rows) are multiplied with input plane g, which starts g * xplane rows after
+// plane 0 (same row stride).  group_rows = 0: one input.  group_rows is a multiple of 128.
+struct LinGroups {
+  int64_t group_rows = 0, xplane = 0;
+};
+
 struct Scratch {
   void *ptr = nullptr;
   size_t bytes = 0;
@@ -187,16 +194,16 @@ int launch_attention(caten_b200_ctx *ctx, const float *qkv, float *kc, float *vc
 int launch_attention_tc(caten_b200_ctx *ctx, const float *qkv, const float *kc, const float *vc, float *out, int64_t B,
                         int64_t s, int64_t n, int64_t H, int64_t T, cb::BfOut bf);
 int launch_gemv(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x, const float *bias,
-                const float *res, int act, float *y);
+                const float *res, int act, float *y, LinGroups grp = LinGroups());
 int launch_gemm_simt(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x, const float *bias,
-                     const float *res, int act, float *y, int64_t M);
+                     const float *res, int act, float *y, int64_t M, LinGroups grp = LinGroups());
 int launch_gemm_tc(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x, const float *bias,
                    const float *res, int act, float *y, int64_t M, int nsplit);
 // x given as fp32 (split by a pre-pass) or, when xhi is set, already as bf16 hi/lo; output as fp32 y
 // or, when ybf.hi is set, as bf16 hi/lo for the next GEMM
 int launch_gemm_tc_ex(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x, const __nv_bfloat16 *xhi,
                       const __nv_bfloat16 *xlo, const float *bias, const float *res, int act, float *y, cb::BfOut ybf,
-                      int64_t M, int nsplit, cb::PartIn *defer = nullptr);
+                      int64_t M, int nsplit, cb::PartIn *defer = nullptr, LinGroups grp = LinGroups());
 // `defer`: when the launch is split-K with no activation, skip the reduction kernel and describe the
 // partial tiles in *defer instead (bias and residual are then the consumer's job); otherwise
 // defer->splits stays 0 and y is complete
@@ -218,7 +225,12 @@ constexpr int WT_F32_T = 100;  // pseudo weight type: fp32 operand given as [K, 
 // many-row GEMM with both operands from shared memory (gemm_dense.cu)
 bool gemm_dense_applies(const caten_b200_ctx *ctx, int64_t M, int64_t N, int64_t K);
 int launch_gemm_dense(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *x, const __nv_bfloat16 *xhi, const __nv_bfloat16 *xlo,
-                      const float *bias, const float *res, int act, float *y, BfOut ybf, int64_t M, int64_t N, int64_t K, int nsplit);
+                      const float *bias, const float *res, int act, float *y, BfOut ybf, int64_t M, int64_t N, int64_t K, int nsplit,
+                      LinGroups grp = LinGroups());
+// the Linear of a model: GEMV for up to 4 rows, otherwise the GEMM of `prec`; with a tensor-core precision the input is
+// xbf when it is set (written by its producer), and the output can be requested the same way (ybf)
+int model_linear(caten_b200_ctx *ctx, int prec, const caten_b200_weight *w, const float *x, BfOut xbf, const float *bias, const float *res,
+                 int act, float *y, BfOut ybf, int64_t M, PartIn *defer = nullptr, LinGroups grp = LinGroups());
 
 // Whether the next launch may be a programmatic dependent launch; clears the pending-upload mark.
 inline bool take_pdl(caten_b200_ctx *ctx) {
@@ -260,6 +272,14 @@ inline cudaError_t launch_k(caten_b200_ctx *ctx, void (*kernel)(KArgs...), dim3 
   return cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
 }
 
+// Brackets one kernel-class call with events when that class is being profiled.
+struct ProfScope {
+  caten_b200_ctx *ctx;
+  cudaEvent_t b = nullptr;
+  ProfScope(caten_b200_ctx *c, int klass);
+  ~ProfScope();
+};
+
 // ---- device helpers ----
 
 // Blocks until the kernels this launch depends on have completed and their writes are visible
@@ -290,6 +310,9 @@ __device__ __forceinline__ float gelu_ref(float x) {
   const float r = 1.0f + th;
   return l * r;
 }
+
+// the gated activation of CATEN_B200_ACT_RELU_GLU
+__device__ __forceinline__ float relu_glu(float gate, float up) { return (gate > 0.0f ? gate : 0.0f) * up; }
 
 __device__ __forceinline__ float apply_act(float v, int act) {
   if (act == CATEN_B200_ACT_GELU) return gelu_ref(v);

@@ -36,6 +36,7 @@ struct GdArgs {
   int act, M, N, K;
   int tiles_f, tiles;         // feature tiles per row tile; all tiles
   int stages;
+  int group_rows, xplane;     // output rows [g * group_rows, ..) read input plane g, `xplane` rows after the one before it
   uint32_t idesc;
 };
 
@@ -125,6 +126,17 @@ __device__ __forceinline__ void gd_store_block(const GdArgs &a, const float *stg
     if (!o_ok || m >= a.M) continue;
     const float4 acc = *reinterpret_cast<const float4 *>(stg + t * 32 + 4 * fg);
     float v[4] = {acc.x + bias4.x, acc.y + bias4.y, acc.z + bias4.z, acc.w + bias4.w};
+    if (ACT == CATEN_B200_ACT_RELU_GLU) {  // two (gate, up) pairs -> two outputs
+      const float g0 = relu_glu(v[0], v[1]), g1 = relu_glu(v[2], v[3]);
+      const int64_t at2 = m * (a.N / 2) + o0 / 2;
+      if (a.yhi) {
+        *reinterpret_cast<uint32_t *>(a.yhi + at2) = pack_bf16(g0, g1);
+        if (a.ylo) *reinterpret_cast<uint32_t *>(a.ylo + at2) = pack_bf16(bf16_lo(g0), bf16_lo(g1));
+      } else {
+        *reinterpret_cast<float2 *>(a.y + at2) = make_float2(g0, g1);
+      }
+      continue;
+    }
     const int64_t at = m * a.N + o0;
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
@@ -238,6 +250,7 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
       bool ok = true;
       for (int tile = blockIdx.x; tile < a.tiles && ok; tile += gridDim.x) {
         const int f0 = (tile % a.tiles_f) * GD_BM, m0 = (tile / a.tiles_f) * GD_BN;
+        const int y0 = m0 + (f0 / a.group_rows) * a.xplane;
         for (int kc = 0; kc < num_k; ++kc) {
           if (!mbar_wait(empty(s), ph ^ 1u, abort_flag)) {
             if (!*abort_flag) { *abort_flag = 1; atomicCAS(a.status, 0, DEV_WAIT_TIMEOUT); a.status[1] = 11; a.status[2] = tile; }
@@ -247,8 +260,8 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
           mbar_expect_tx(full(s), STAGE_BYTES);
           tma_load_2d(st_whi(s), &tw_hi, full(s), kc * BK, f0);
           if (NSPLIT == 3) tma_load_2d(st_wlo(s), &tw_lo, full(s), kc * BK, f0);
-          tma_load_2d(st_xhi(s), &tx_hi, full(s), kc * BK, m0);
-          if (NSPLIT == 3) tma_load_2d(st_xlo(s), &tx_lo, full(s), kc * BK, m0);
+          tma_load_2d(st_xhi(s), &tx_hi, full(s), kc * BK, y0);
+          if (NSPLIT == 3) tma_load_2d(st_xlo(s), &tx_lo, full(s), kc * BK, y0);
           ++issued;
           if (++s == S) { s = 0; ph ^= 1u; }
         }
@@ -334,6 +347,7 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
         __syncwarp();
         const int m_first = m0 + half * (GD_BN / 2) + c;
         if (a.act == CATEN_B200_ACT_GELU) gd_store_block<CATEN_B200_ACT_GELU>(a, stg, lane, bias4, o0, o_ok, m_first);
+        else if (a.act == CATEN_B200_ACT_RELU_GLU) gd_store_block<CATEN_B200_ACT_RELU_GLU>(a, stg, lane, bias4, o0, o_ok, m_first);
         else if (a.act == CATEN_B200_ACT_RELU) gd_store_block<CATEN_B200_ACT_RELU>(a, stg, lane, bias4, o0, o_ok, m_first);
         else gd_store_block<CATEN_B200_ACT_NONE>(a, stg, lane, bias4, o0, o_ok, m_first);
       }
@@ -385,19 +399,24 @@ bool gemm_dense_applies(const caten_b200_ctx *ctx, int64_t M, int64_t N, int64_t
 
 // wt: a ggml type or WT_F32_T (then ws.qs is b[K, N] fp32).  x: fp32 [M, K], or its split bf16 copy when xhi is given.
 int launch_gemm_dense(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *x, const __nv_bfloat16 *xhi, const __nv_bfloat16 *xlo,
-                      const float *bias, const float *res, int act, float *y, BfOut ybf, int64_t M, int64_t N, int64_t K, int nsplit) {
+                      const float *bias, const float *res, int act, float *y, BfOut ybf, int64_t M, int64_t N, int64_t K, int nsplit,
+                      LinGroups grp) {
   if (!ctx->encode_tiled) return fail(ctx, CATEN_B200_ECUDA, "gemm_dense: cuTensorMapEncodeTiled is not available");
   if (K % GD_BK || M > 0x7fffffff || N > 0x7fffffff || K > 0x7fffffff) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemm_dense: shape %lldx%lldx%lld", (long long)M, (long long)N, (long long)K);
   if (nsplit != 1 && nsplit != 3) return fail(ctx, CATEN_B200_EINVAL, "gemm_dense: nsplit must be 1 or 3");
   const int parts = nsplit == 3 ? 2 : 1;
   // bf16 copy of the weights
+  const bool as_is = wt == CATEN_B200_BF16 && parts == 1;  // the weight is the operand: no copy
   const size_t wb = ((size_t)N * K * 2 + 1023) & ~(size_t)1023;
-  if (int rc = scratch_reserve(ctx, &ctx->wbf, wb * parts)) return rc;
+  if (!as_is)
+    if (int rc = scratch_reserve(ctx, &ctx->wbf, wb * parts)) return rc;
   __nv_bfloat16 *whi = (__nv_bfloat16 *)ctx->wbf.ptr, *wlo = parts == 2 ? (__nv_bfloat16 *)((uint8_t *)ctx->wbf.ptr + wb) : nullptr;
   int rc = 0;
-  switch (wt) {
+  if (as_is) whi = (__nv_bfloat16 *)ws.qs;
+  else switch (wt) {
     case CATEN_B200_F32: rc = launch_wsplit<CATEN_B200_F32>(ctx, ws, N, K, whi, wlo); break;
     case CATEN_B200_F16: rc = launch_wsplit<CATEN_B200_F16>(ctx, ws, N, K, whi, wlo); break;
+    case CATEN_B200_BF16: rc = launch_wsplit<CATEN_B200_BF16>(ctx, ws, N, K, whi, wlo); break;
     case CATEN_B200_Q4_0: rc = launch_wsplit<CATEN_B200_Q4_0>(ctx, ws, N, K, whi, wlo); break;
     case CATEN_B200_Q4_1: rc = launch_wsplit<CATEN_B200_Q4_1>(ctx, ws, N, K, whi, wlo); break;
     case CATEN_B200_Q5_0: rc = launch_wsplit<CATEN_B200_Q5_0>(ctx, ws, N, K, whi, wlo); break;
@@ -429,13 +448,15 @@ int launch_gemm_dense(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *
   const int bk = nsplit == 3 ? GdStage<3>::BK : GdStage<1>::BK;
   if ((rc = make_map(ctx, &twh, whi, N, K, GD_BM, bk))) return rc;
   if ((rc = make_map(ctx, &twl, wlo ? wlo : whi, N, K, GD_BM, bk))) return rc;
-  if ((rc = make_map(ctx, &txh, xhi, M, K, GD_BN, bk))) return rc;
-  if ((rc = make_map(ctx, &txl, nsplit == 3 ? xlo : xhi, M, K, GD_BN, bk))) return rc;
+  const int64_t xrows = grp.group_rows ? (N - 1) / grp.group_rows * grp.xplane + M : M;  // all planes of x
+  if ((rc = make_map(ctx, &txh, xhi, xrows, K, GD_BN, bk))) return rc;
+  if ((rc = make_map(ctx, &txl, nsplit == 3 ? xlo : xhi, xrows, K, GD_BN, bk))) return rc;
 
   GdArgs a;
   a.bias = bias; a.res = res; a.y = y; a.yhi = ybf.hi; a.ylo = ybf.lo; a.status = ctx->d_status;
   a.act = act; a.M = (int)M; a.N = (int)N; a.K = (int)K;
   a.tiles_f = (int)((N + GD_BM - 1) / GD_BM);
+  a.group_rows = grp.group_rows ? (int)grp.group_rows : a.tiles_f * GD_BM; a.xplane = (int)grp.xplane;
   const int64_t tiles = (int64_t)a.tiles_f * ((M + GD_BN - 1) / GD_BN);
   if (tiles > 0x7fffffff) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemm_dense: too many tiles");
   a.tiles = (int)tiles;

@@ -17,13 +17,14 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const void *__restrict__
                                                         const __half *__restrict__ mins, const uint32_t *__restrict__ qh5,
                                                         const float *__restrict__ x, const float *__restrict__ bias,
                                                         const float *res, float *y, int act, int64_t M, int64_t N,
-                                                        int64_t K, int64_t nkb) {
+                                                        int64_t K, int64_t nkb, int64_t group_rows, int64_t xplane) {
   __shared__ __align__(16) float Xs[SG_BK * SG_LD];  // [k][m]
   __shared__ __align__(16) float Ws[SG_BK * SG_LD];  // [k][n]
   pdl_enter();
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
   const int64_t m0 = (int64_t)blockIdx.y * SG_BM, n0 = (int64_t)blockIdx.x * SG_BN;
   const int lrow = tid & 63, part = tid >> 6;
+  x += (n0 / group_rows) * xplane * K;  // the input plane of this tile's output rows
   float acc[4][4];
 #pragma unroll
   for (int a = 0; a < 4; ++a)
@@ -69,6 +70,14 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const void *__restrict__
   for (int a = 0; a < 4; ++a) {
     const int64_t m = m0 + 4 * ty + a;
     if (m >= M) continue;
+    if (act == CATEN_B200_ACT_RELU_GLU) {
+#pragma unroll
+      for (int e = 0; e < 4; e += 2) {
+        const int64_t o = n0 + 4 * tx + e;
+        if (o < N) y[m * (N / 2) + o / 2] = relu_glu(acc[a][e] + (bias ? bias[o] : 0.0f), acc[a][e + 1] + (bias ? bias[o + 1] : 0.0f));
+      }
+      continue;
+    }
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int64_t o = n0 + 4 * tx + e;
@@ -84,23 +93,26 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const void *__restrict__
 
 template <int WT>
 static int launch_simt(caten_b200_ctx *ctx, const void *qs, const __half *d, const __half *mins, const uint32_t *qh5, const float *x,
-                       const float *bias, const float *res, int act, float *y, int64_t M, int64_t N, int64_t K) {
+                       const float *bias, const float *res, int act, float *y, int64_t M, int64_t N, int64_t K, LinGroups grp = LinGroups()) {
+  if (grp.group_rows % SG_BN) return fail(ctx, CATEN_B200_EINVAL, "gemm: input groups must be multiples of %d rows", SG_BN);
   if (K % 32) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemm: inner dimension %lld is not a multiple of 32", (long long)K);
   const int64_t gx = (N + SG_BN - 1) / SG_BN, gy = (M + SG_BM - 1) / SG_BM;
   if (gy > 65535) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemm: too many rows for one launch (%lld)", (long long)M);
-  launch_k(ctx, gemm_simt_kernel<WT>, dim3((unsigned)gx, (unsigned)gy), dim3(256), 0, qs, d, mins, qh5, x, bias, res, y, act, M, N, K, K / 32);
+  launch_k(ctx, gemm_simt_kernel<WT>, dim3((unsigned)gx, (unsigned)gy), dim3(256), 0, qs, d, mins, qh5, x, bias, res, y, act, M, N, K, K / 32,
+           grp.group_rows > 0 ? grp.group_rows : N + SG_BN, grp.xplane);
   CB_LAUNCH_CHECK(ctx, "gemm_simt_kernel");
   return 0;
 }
 
 int launch_gemm_simt(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x, const float *bias,
-                     const float *res, int act, float *y, int64_t M) {
+                     const float *res, int act, float *y, int64_t M, LinGroups grp) {
   if (M <= 0) return 0;
 #define SIMT_CASE(T) \
-  case T: return launch_simt<T>(ctx, w->qs, w->d, w->m, w->qh, x, bias, res, act, y, M, w->rows, w->cols)
+  case T: return launch_simt<T>(ctx, w->qs, w->d, w->m, w->qh, x, bias, res, act, y, M, w->rows, w->cols, grp)
   switch (w->type) {
     SIMT_CASE(CATEN_B200_F32);
     SIMT_CASE(CATEN_B200_F16);
+    SIMT_CASE(CATEN_B200_BF16);
     SIMT_CASE(CATEN_B200_Q8_0);
     SIMT_CASE(CATEN_B200_Q4_0);
     SIMT_CASE(CATEN_B200_Q4_1);

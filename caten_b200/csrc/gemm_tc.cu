@@ -54,6 +54,8 @@ struct TcArgs {
   int splits, cps;
   int cluster;  // 1: the `splits` CTAs of a tile form a thread-block cluster and reduce through distributed shared memory
   float *part;
+  // output rows [g * group_rows, (g + 1) * group_rows) read input plane g, `xplane` rows after the one before it
+  int group_rows, xplane;
   // when yhi is set the epilogue writes the result as split bf16 (operand of the next GEMM), not y
   __nv_bfloat16 *yhi, *ylo;
 };
@@ -259,6 +261,28 @@ template <> struct WRow<CATEN_B200_F16> {
   }
 };
 
+// bf16 rows are the operand already: the words go to tensor memory as they are (the low part is zero)
+template <> struct WRow<CATEN_B200_BF16> {
+  static constexpr int DEPTH = 3, GROUPS = 2;
+  uint32_t v[32];
+  __device__ __forceinline__ void load(const TcArgs &a, int64_t row, bool ok, int kc) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const uint4 q = ok ? __ldcs(reinterpret_cast<const uint4 *>((const uint16_t *)a.qs + row * a.K + (int64_t)kc * 64) + j) : make_uint4(0, 0, 0, 0);
+      v[4 * j] = q.x; v[4 * j + 1] = q.y; v[4 * j + 2] = q.z; v[4 * j + 3] = q.w;
+    }
+  }
+  template <int NSPLIT> __device__ __forceinline__ void store(uint32_t t_hi) const {
+    tmem_st16(t_hi, v);
+    tmem_st16(t_hi + 16, v + 16);
+    if (NSPLIT == 3) {
+      const uint32_t z[16] = {};
+      tmem_st16(t_hi + 32, z);
+      tmem_st16(t_hi + 48, z);
+    }
+  }
+};
+
 // fp32 rows: 64 floats per thread and chunk; two groups of four warps so that the registers fit
 template <> struct WRow<CATEN_B200_F32> {
   static constexpr int DEPTH = 1, GROUPS = 2;
@@ -291,6 +315,25 @@ template <> struct WRow<WT_F32_T> {
 
 template <int WT> constexpr int tc_threads() { return (WRow<WT>::GROUPS * 4 + 2) * 32; }
 
+// Two (gate, up) pairs of row m, features o .. o + 3 (o a multiple of 4), summed and gated: outputs o / 2 and o / 2 + 1.
+__device__ __forceinline__ void store_glu4(const float *r, const float *bias, int64_t o, int64_t N, int64_t m, float *y, __nv_bfloat16 *yhi,
+                                           __nv_bfloat16 *ylo) {
+#pragma unroll
+  for (int e = 0; e < 4; e += 2) {
+    if (o + e < N) {
+      const float v = relu_glu(bias ? r[e] + bias[o + e] : r[e], bias ? r[e + 1] + bias[o + e + 1] : r[e + 1]);
+      const int64_t at = m * (N / 2) + (o + e) / 2;
+      if (yhi) {
+        const __nv_bfloat16 h = __float2bfloat16_rn(v);
+        yhi[at] = h;
+        if (ylo) ylo[at] = __float2bfloat16_rn(v - __bfloat162float(h));
+      } else {
+        y[at] = v;
+      }
+    }
+  }
+}
+
 // Epilogue of one 16-column group held in registers: y[m, o] = act(acc + bias) + res.
 template <int ACT>
 __device__ __forceinline__ void epi_store16(const TcArgs &a, const uint32_t *r, float bias, int64_t o, int m_first) {
@@ -311,6 +354,28 @@ __device__ __forceinline__ void epi_store16(const TcArgs &a, const uint32_t *r, 
         if (a.ylo) a.ylo[at] = __float2bfloat16_rn(v - __bfloat162float(h));
       } else {
         yp[(int64_t)i * a.N] = v;
+      }
+    }
+  }
+}
+
+// Gated form: the lane pair (2j, 2j + 1) of the warp holds a (gate, up) feature pair; the whole warp calls it.
+__device__ __forceinline__ void epi_glu16(const TcArgs &a, const uint32_t *r, float bias, int64_t o, bool o_ok, int m_first) {
+  const int lim = a.M - m_first < 16 ? a.M - m_first : 16;
+  const int64_t n2 = a.N / 2;
+#pragma unroll
+  for (int i = 0; i < 16; ++i) {
+    const float mine = __uint_as_float(r[i]) + bias;
+    const float other = __shfl_xor_sync(0xffffffffu, mine, 1);
+    if (i < lim && o_ok && !(o & 1)) {
+      const float v = relu_glu(mine, other);
+      const int64_t at = ((int64_t)m_first + i) * n2 + (o >> 1);
+      if (a.yhi) {
+        const __nv_bfloat16 h = __float2bfloat16_rn(v);
+        a.yhi[at] = h;
+        if (a.ylo) a.ylo[at] = __float2bfloat16_rn(v - __bfloat162float(h));
+      } else {
+        a.y[at] = v;
       }
     }
   }
@@ -459,7 +524,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_hi, const __grid_constant_
           tmem_ld_wait();
         }
         if (a.splits == 1) {
-          if (o_ok && m0 + c < a.M) {
+          if (a.act == CATEN_B200_ACT_RELU_GLU) {
+            if (m0 + c < a.M) epi_glu16(a, r, bias, o, o_ok, m0 + c);
+          } else if (o_ok && m0 + c < a.M) {
             if (a.act == CATEN_B200_ACT_GELU) epi_store16<CATEN_B200_ACT_GELU>(a, r, bias, o, m0 + c);
             else if (a.act == CATEN_B200_ACT_RELU) epi_store16<CATEN_B200_ACT_RELU>(a, r, bias, o, m0 + c);
             else epi_store16<CATEN_B200_ACT_NONE>(a, r, bias, o, m0 + c);
@@ -489,14 +556,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_hi, const __grid_constant_
       pdl_wait();  // x is written by the preceding kernel
       int issued = 0, s = 0;
       uint32_t ph = 0;
+      const int y0 = m0 + (n0 / a.group_rows) * a.xplane;  // first row of the input plane this tile's output rows read
       for (int kc = 0; kc < num_k; ++kc) {
         if (!mbar_wait(empty(s), ph ^ 1u, abort_flag)) {
           if (!*abort_flag) { *abort_flag = 1; atomicCAS(a.status, 0, DEV_WAIT_TIMEOUT); a.status[1] = 3; a.status[2] = kc; }
           break;
         }
         mbar_expect_tx(full(s), stage_bytes);
-        tma_load_2d(smem_u32(stage_xhi(s)), &tm_hi, full(s), (kc0 + kc) * TC_BK, m0);
-        if (NSPLIT == 3) tma_load_2d(smem_u32(stage_xlo(s)), &tm_lo, full(s), (kc0 + kc) * TC_BK, m0);
+        tma_load_2d(smem_u32(stage_xhi(s)), &tm_hi, full(s), (kc0 + kc) * TC_BK, y0);
+        if (NSPLIT == 3) tma_load_2d(smem_u32(stage_xlo(s)), &tm_lo, full(s), (kc0 + kc) * TC_BK, y0);
         issued = kc + 1;
         if (++s == S) { s = 0; ph ^= 1u; }
       }
@@ -581,6 +649,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_hi, const __grid_constant_
           v.x += p.x; v.y += p.y; v.z += p.z; v.w += p.w;
         }
         const float r[4] = {v.x, v.y, v.z, v.w};
+        if (a.act == CATEN_B200_ACT_RELU_GLU) {
+          store_glu4(r, a.bias, (int64_t)n0 + r4, a.N, m, a.y, a.yhi, a.ylo);
+          continue;
+        }
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int64_t o = (int64_t)n0 + r4 + e;
@@ -643,6 +715,10 @@ __global__ void __launch_bounds__(256) splitk_reduce_kernel(const float *__restr
     v.x += a0.x; v.y += a0.y; v.z += a0.z; v.w += a0.w;
   }
   float r[4] = {v.x, v.y, v.z, v.w};
+  if (act == CATEN_B200_ACT_RELU_GLU) {
+    store_glu4(r, bias, o, N, m, y, yhi, ylo);
+    return;
+  }
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
     if (o + e < N) {
@@ -723,6 +799,7 @@ static int launch_tc(caten_b200_ctx *ctx, int wt, int nsplit, const CUtensorMap 
   switch (wt) {
     TC_CASE(CATEN_B200_F32);
     TC_CASE(CATEN_B200_F16);
+    TC_CASE(CATEN_B200_BF16);
     TC_CASE(CATEN_B200_Q4_0);
     TC_CASE(CATEN_B200_Q4_1);
     TC_CASE(CATEN_B200_Q5_0);
@@ -783,13 +860,15 @@ static WSrc wsrc_of(const caten_b200_weight *w) { return WSrc{w->qs, w->d, w->m,
 static int run_tc(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *x,
                   const float *bias, const float *res, int act, float *y, int64_t M, int64_t N, int64_t K, int nsplit,
                   const __nv_bfloat16 *xhi_pre = nullptr, const __nv_bfloat16 *xlo_pre = nullptr, BfOut ybf = BfOut(),
-                  PartIn *defer = nullptr) {
+                  PartIn *defer = nullptr, LinGroups grp = LinGroups()) {
   if (defer) *defer = PartIn();
+  if (grp.group_rows % TC_BM) return fail(ctx, CATEN_B200_EINVAL, "gemm_tc: input groups must be multiples of %d rows", TC_BM);
+  if (grp.group_rows && !xhi_pre) return fail(ctx, CATEN_B200_EINVAL, "gemm_tc: grouped inputs are given as bf16");
   if (M <= 0 || N <= 0) return 0;
   // thousands of rows (prefill): expand the weights once, both operands through TMA
   // (its epilogue moves 16 bytes at a time: bias, residual and outputs must be aligned for that)
   const uintptr_t align_bits = (uintptr_t)bias | (uintptr_t)res | (uintptr_t)y | (uintptr_t)ybf.hi | (uintptr_t)ybf.lo;
-  if (gemm_dense_applies(ctx, M, N, K) && !(align_bits & 15)) return launch_gemm_dense(ctx, wt, ws, x, xhi_pre, xlo_pre, bias, res, act, y, ybf, M, N, K, nsplit);
+  if (gemm_dense_applies(ctx, M, N, K) && !(align_bits & 15)) return launch_gemm_dense(ctx, wt, ws, x, xhi_pre, xlo_pre, bias, res, act, y, ybf, M, N, K, nsplit, grp);
   TcPlan p;
   // reduce inside a cluster: always (mode 1) or only when this launch needs its own epilogue (mode 2)
   const bool own_epilogue = !(defer && act == CATEN_B200_ACT_NONE && !ybf.hi && N % 4 == 0);
@@ -814,10 +893,12 @@ static int run_tc(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *x,
     CB_LAUNCH_CHECK(ctx, "split_bf16_kernel");
   }
   CUtensorMap mh, ml;
-  if (int rc = make_x_map(ctx, &mh, xhi, M, K, p.bnx)) return rc;
-  if (int rc = make_x_map(ctx, &ml, nsplit == 3 ? xlo : xhi, M, K, p.bnx)) return rc;
+  const int64_t xrows = grp.group_rows ? (N - 1) / grp.group_rows * grp.xplane + M : M;  // all planes of x
+  if (int rc = make_x_map(ctx, &mh, xhi, xrows, K, p.bnx)) return rc;
+  if (int rc = make_x_map(ctx, &ml, nsplit == 3 ? xlo : xhi, xrows, K, p.bnx)) return rc;
 
   TcArgs a;
+  a.group_rows = grp.group_rows ? (int)grp.group_rows : (int)(p.gx * TC_BM); a.xplane = (int)grp.xplane;
   a.qs = ws.qs; a.d = ws.d; a.m = ws.m; a.qh = ws.qh; a.bias = bias; a.res = res; a.y = y; a.status = ctx->d_status; a.act = act;
   a.yhi = ybf.hi; a.ylo = ybf.lo;
   a.M = (int)M; a.N = (int)N; a.K = (int)K; a.nkb = (int)ws.nkb; a.bnx = p.bnx;
@@ -902,6 +983,7 @@ int launch_gemm_tc_noalloc(caten_b200_ctx *ctx, const caten_b200_weight *w, cons
   if (int rc = make_x_map(ctx, &ml, nsplit == 3 ? xlo : xhi, M, K, p.bnx)) return rc;
 
   TcArgs a;
+  a.group_rows = (int)(p.gx * TC_BM); a.xplane = 0;
   a.qs = w->qs; a.d = w->d; a.m = w->m; a.qh = w->qh; a.bias = bias; a.res = res; a.y = y; a.status = ctx->d_status; a.act = act;
   a.yhi = nullptr; a.ylo = nullptr;
   a.M = (int)M; a.N = (int)N; a.K = (int)K; a.nkb = (int)w->nkb; a.bnx = p.bnx;
@@ -926,8 +1008,8 @@ int launch_gemm_tc(caten_b200_ctx *ctx, const caten_b200_weight *w, const float 
 
 int launch_gemm_tc_ex(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x, const __nv_bfloat16 *xhi,
                       const __nv_bfloat16 *xlo, const float *bias, const float *res, int act, float *y, BfOut ybf, int64_t M,
-                      int nsplit, PartIn *defer) {
-  return run_tc(ctx, w->type, wsrc_of(w), x, bias, res, act, y, M, w->rows, w->cols, nsplit, xhi, xlo, ybf, defer);
+                      int nsplit, PartIn *defer, LinGroups grp) {
+  return run_tc(ctx, w->type, wsrc_of(w), x, bias, res, act, y, M, w->rows, w->cols, nsplit, xhi, xlo, ybf, defer, grp);
 }
 
 int launch_relu_matmul_tc(caten_b200_ctx *ctx, const float *a, const float *b, float *c, int64_t M, int64_t K, int64_t N, int nsplit) {

@@ -117,7 +117,7 @@ __global__ void __launch_bounds__(GEMV_MAX_THREADS) gemv_blocked_kernel(GemvArgs
   }
 }
 
-// fp32 / fp16 weights: one warp per row, RI rows in flight, x in shared memory.
+// fp32 / fp16 / bf16 weights: one warp per row, RI rows in flight, x in shared memory.
 template <typename T> struct DenseLoad;
 template <> struct DenseLoad<float> {
   static constexpr int VEC = 4;
@@ -139,11 +139,34 @@ template <> struct DenseLoad<__half> {
   }
 };
 
+template <> struct DenseLoad<__nv_bfloat16> {
+  static constexpr int VEC = 8;
+  __device__ static __forceinline__ void load(const __nv_bfloat16 *p, float *o) {
+    const uint4 v = __ldcs(reinterpret_cast<const uint4 *>(p));
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      o[2 * i] = __uint_as_float(w[i] << 16);
+      o[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u);
+    }
+  }
+};
+
+// blockIdx.y = group of `group_rows` output rows with an input plane of its own (one group: N rows)
 template <typename T, int RI>
 __global__ void __launch_bounds__(256) gemv_dense_kernel(const T *__restrict__ W, const float *__restrict__ x,
                                                          const float *__restrict__ bias, const float *__restrict__ res,
-                                                         float *__restrict__ y, int act, int N, int K) {
+                                                         float *__restrict__ y, int act, int N, int K, int group_rows, int64_t xplane) {
   extern __shared__ float xs[];
+  {
+    const int64_t r0 = (int64_t)blockIdx.y * group_rows;
+    W += r0 * K;
+    x += (int64_t)blockIdx.y * xplane * K;
+    y += r0;
+    if (bias) bias += r0;
+    if (res) res += r0;
+    N = N - r0 < group_rows ? (int)(N - r0) : group_rows;
+  }
   // weights depend on no other kernel: the first tile of this warp's rows is loaded before the
   // wait for the producer of x
   pdl_launch_dependents();
@@ -204,6 +227,14 @@ __global__ void __launch_bounds__(256) gemv_dense_kernel(const T *__restrict__ W
         }
       }
     }
+    if (RI == 2 && act == CATEN_B200_ACT_RELU_GLU) {  // rows (base, base + 1) are a (gate, up) pair: base is even
+      float g = warp_sum(acc[0]), u = warp_sum(acc[RI - 1]);
+      if (lane == 0 && base < N) {
+        if (bias) { g = g + bias[base]; u = u + bias[base + 1]; }
+        y[base >> 1] = relu_glu(g, u);
+      }
+      continue;
+    }
 #pragma unroll
     for (int i = 0; i < RI; ++i) {
       float s = warp_sum(acc[i]);
@@ -234,10 +265,11 @@ static int launch_blocked(caten_b200_ctx *ctx, const GemvArgs &a) {
 }
 
 int launch_gemv(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x, const float *bias,
-                const float *res, int act, float *y) {
+                const float *res, int act, float *y, LinGroups grp) {
   if (w->rows > 0x7fffffff || w->cols > 0x7fffffff) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv: dimension too large");
   const int N = (int)w->rows, K = (int)w->cols;
   if (type_is_packed(w->type)) {
+    if (grp.group_rows || act == CATEN_B200_ACT_RELU_GLU) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv: input groups and the gated activation take dense weights");
     GemvArgs a;
     a.qs = w->qs; a.d = w->d; a.m = w->m; a.qh = w->qh; a.x = x; a.bias = bias; a.res = res; a.y = y; a.act = act; a.N = N;
     a.nkb = (int)w->nkb;
@@ -255,30 +287,31 @@ int launch_gemv(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x,
   }
   const size_t smem = (size_t)K * sizeof(float);
   if (smem > 160 * 1024) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv: cols=%d too wide", K);
-  // two rows per warp when that still gives every SM a CTA, else one row per warp (more CTAs)
-  const bool two = ((int64_t)N + 15) / 16 >= ctx->sm_count;
-  const int64_t groups = two ? ((int64_t)N + 15) / 16 : ((int64_t)N + 7) / 8;
-  int64_t grid = (int64_t)ctx->sm_count * 4;
+  const int ng = grp.group_rows > 0 ? (int)((N + grp.group_rows - 1) / grp.group_rows) : 1;
+  const int rows = grp.group_rows > 0 ? (int)grp.group_rows : N;  // per group
+  // two rows per warp when that still gives every SM a CTA (or the rows are pairs), else one row per warp (more CTAs)
+  const bool two = act == CATEN_B200_ACT_RELU_GLU || ((int64_t)rows + 15) / 16 * ng >= ctx->sm_count;
+  const int64_t groups = two ? ((int64_t)rows + 15) / 16 : ((int64_t)rows + 7) / 8;
+  int64_t grid = ((int64_t)ctx->sm_count * 4 + ng - 1) / ng;
   if (grid > groups) grid = groups;
-  if (w->type == CATEN_B200_F32) {
-    if (K % 4) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv f32: cols %% 4 != 0");
-    if (smem > 48 * 1024) {
-      cudaFuncSetAttribute(gemv_dense_kernel<float, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-      cudaFuncSetAttribute(gemv_dense_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    }
-    if (two) launch_k(ctx, gemv_dense_kernel<float, 2>, dim3((unsigned)grid), dim3(256), smem, (const float *)w->qs, x, bias, res, y, act, N, K);
-    else launch_k(ctx, gemv_dense_kernel<float, 1>, dim3((unsigned)grid), dim3(256), smem, (const float *)w->qs, x, bias, res, y, act, N, K);
-  } else if (w->type == CATEN_B200_F16) {
-    if (K % 8) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv f16: cols %% 8 != 0");
-    if (smem > 48 * 1024) {
-      cudaFuncSetAttribute(gemv_dense_kernel<__half, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-      cudaFuncSetAttribute(gemv_dense_kernel<__half, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    }
-    if (two) launch_k(ctx, gemv_dense_kernel<__half, 2>, dim3((unsigned)grid), dim3(256), smem, (const __half *)w->qs, x, bias, res, y, act, N, K);
-    else launch_k(ctx, gemv_dense_kernel<__half, 1>, dim3((unsigned)grid), dim3(256), smem, (const __half *)w->qs, x, bias, res, y, act, N, K);
-  } else {
-    return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv: weight type %d", w->type);
+#define GEMV_DENSE(T, CT)                                                                                                        \
+  do {                                                                                                                           \
+    if (K % DenseLoad<CT>::VEC) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv " T ": cols %% %d != 0", DenseLoad<CT>::VEC);    \
+    if (smem > 48 * 1024) {                                                                                                      \
+      cudaFuncSetAttribute(gemv_dense_kernel<CT, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                    \
+      cudaFuncSetAttribute(gemv_dense_kernel<CT, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                    \
+    }                                                                                                                            \
+    const dim3 g((unsigned)grid, (unsigned)ng);                                                                                  \
+    if (two) launch_k(ctx, gemv_dense_kernel<CT, 2>, g, dim3(256), smem, (const CT *)w->qs, x, bias, res, y, act, N, K, rows, grp.xplane); \
+    else launch_k(ctx, gemv_dense_kernel<CT, 1>, g, dim3(256), smem, (const CT *)w->qs, x, bias, res, y, act, N, K, rows, grp.xplane);     \
+  } while (0)
+  switch (w->type) {
+    case CATEN_B200_F32: GEMV_DENSE("f32", float); break;
+    case CATEN_B200_F16: GEMV_DENSE("f16", __half); break;
+    case CATEN_B200_BF16: GEMV_DENSE("bf16", __nv_bfloat16); break;
+    default: return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv: weight type %d", w->type);
   }
+#undef GEMV_DENSE
   CB_LAUNCH_CHECK(ctx, "gemv_dense_kernel");
   return 0;
 }

@@ -70,6 +70,8 @@ __global__ void dequant_kernel(int type, const void *__restrict__ qs, const __ha
     out[i] = ((const float *)qs)[i];
   } else if (type == CATEN_B200_F16) {
     out[i] = __half2float(((const __half *)qs)[i]);
+  } else if (type == CATEN_B200_BF16) {
+    out[i] = __bfloat162float(((const __nv_bfloat16 *)qs)[i]);
   } else if (type == CATEN_B200_Q8_0) {
     const int q = ((const int8_t *)qs)[blk * 32 + j];
     out[i] = (float)q * __half2float(d[blk]);

@@ -14,11 +14,12 @@ from typing import Optional
 import numpy as np
 
 from . import _lib as L
+from .model import Model, generate
 from .runtime import B200Buffer, B200Runtime, B200Weight
 from .synthetic import GPT2_SIZES, GPT2Params, Packed
 
 
-class GPT2:
+class GPT2(Model):
     def __init__(self, runtime: B200Runtime, params: GPT2Params, state_dict: dict, max_seq_len: int = 1024,
                  batch: int = 1, precision: str = "fp32", max_rows: int = 0, device_blobs: Optional[dict] = None):
         """``state_dict``: reference keys -> fp32 arrays, or :class:`Packed` for Linear weights.
@@ -27,6 +28,7 @@ class GPT2:
         this GPU (e.g. received through an NCCL broadcast); those entries of ``state_dict`` then
         only need ``ggml_type/rows/cols`` and are not read from the host."""
         self.rt, self.params, self.batch, self.max_seq_len = runtime, params, batch, max_seq_len
+        self.vocab_size = params.vocab_size
         self.precision = L.PRECISIONS[precision] if isinstance(precision, str) else int(precision)
         self._bufs, self._weights, self._keep = [], [], []
         self.weights = {}  # state-dict key -> B200Weight
@@ -106,53 +108,23 @@ class GPT2:
         self._h = h
         self._dev_ids = rt.open_buffer((2, batch), np.int64)  # ping-pong ids for device-resident decode
 
-    # -- one step from host ids: the call the reference's token loop makes --
-    def forward(self, x, s: Optional[int] = None, n: int = 0) -> np.ndarray:
-        """x: [batch, s] token ids (any numeric dtype; sent as float32 like gpt2.lisp:95).
-        Returns int64 [batch]: argmax of the logits at the last position."""
-        tok = np.ascontiguousarray(x, dtype=np.float32).reshape(self.batch, -1)
-        s = tok.shape[1] if s is None else int(s)
-        if s != tok.shape[1]:
-            raise ValueError("forward: s does not match x")
+    # -- entry points of caten_b200.model.Model --
+    def _step(self, tokens: np.ndarray, n: int) -> np.ndarray:
+        tok = np.ascontiguousarray(tokens, dtype=np.float32)   # ids go in as float32 like gpt2.lisp:95
         out = np.empty(self.batch, np.int64)
-        L.check(self.rt.ctx, self.rt.lib.caten_b200_gpt2_step(self._h, tok.ctypes.data, s, int(n), out.ctypes.data))
+        L.check(self.rt.ctx, self.rt.lib.caten_b200_gpt2_step(self._h, tok.ctypes.data, tok.shape[1], n, out.ctypes.data))
         return out
 
-    # -- device-resident variants (ids never leave HBM) --
-    def forward_device(self, ids: B200Buffer, s: int, n: int, out: B200Buffer) -> None:
+    def _step_device(self, ids: B200Buffer, s: int, n: int, out: B200Buffer) -> None:
         f32 = ids.ptr if ids.dtype == np.float32 else None
         i64 = ids.ptr if ids.dtype == np.int64 else None
-        L.check(self.rt.ctx, self.rt.lib.caten_b200_gpt2_step_device(self._h, f32, i64, int(s), int(n), out.ptr))
+        L.check(self.rt.ctx, self.rt.lib.caten_b200_gpt2_step_device(self._h, f32, i64, s, n, out.ptr))
 
-    def decode_device(self, first_ids: np.ndarray, start_pos: int, steps: int) -> np.ndarray:
-        """Greedy decode ``steps`` tokens with ids and position staying on the GPU (one C call; the
-        step is replayed from a CUDA graph); returns [batch, steps]."""
-        ids0 = self.rt.transfer_from_array(np.ascontiguousarray(first_ids, dtype=np.int64).reshape(self.batch))
-        hist = self.rt.open_buffer((steps, self.batch), np.int64)
-        self.decode_device_buffers(ids0, start_pos, steps, hist)
-        out = hist.numpy().T.copy()
-        hist.close()
-        ids0.close()
-        return out
+    def _decode(self, first_ids: B200Buffer, n: int, steps: int, out: Optional[B200Buffer]) -> None:
+        L.check(self.rt.ctx, self.rt.lib.caten_b200_gpt2_decode(self._h, first_ids.ptr, n, steps, out.ptr if out is not None else None))
 
-    def decode_device_buffers(self, first_ids: B200Buffer, start_pos: int, steps: int, out: Optional[B200Buffer] = None) -> None:
-        """Asynchronous form of :meth:`decode_device` on device buffers (``out``: [steps, batch] int64)."""
-        L.check(self.rt.ctx, self.rt.lib.caten_b200_gpt2_decode(self._h, first_ids.ptr, int(start_pos), int(steps),
-                                                                out.ptr if out is not None else None))
-
-    def logits(self) -> np.ndarray:
-        """[batch, vocab] fp32 logits of the last step."""
-        ptr = self.rt.lib.caten_b200_gpt2_logits(self._h)
-        return B200Buffer(self.rt, ptr, (self.batch, self.params.vocab_size), np.float32, owned=False).numpy()
-
-    def sample(self, uniform, temperature: float = 1.0, top_k: int = 0) -> np.ndarray:
-        """[batch] int64 ids drawn from the last step's logits (they stay on the device)."""
-        ptr = self.rt.lib.caten_b200_gpt2_logits(self._h)
-        lg = B200Buffer(self.rt, ptr, (self.batch, self.params.vocab_size), np.float32, owned=False)
-        ids = self.rt.sample(lg, uniform, temperature, top_k)
-        out = ids.numpy()
-        ids.close()
-        return out
+    def _logits_ptr(self) -> int:
+        return self.rt.lib.caten_b200_gpt2_logits(self._h)
 
     def kv_cache(self, layer: int):
         """(k, v) of one layer as numpy arrays [batch, heads, max_seq_len, 64]."""
@@ -195,23 +167,7 @@ def make_gpt2(model_type, state_dict: dict, runtime: Optional[B200Runtime] = Non
     return GPT2(rt, params, state_dict, max_seq_len=max_seq_len, batch=batch, precision=precision, **kw)
 
 
-def gpt2_generate(gpt2: GPT2, prompt_ids, max_length: int = 100, temperature: float = 0.0, top_k: int = 0, seed: int = 0) -> np.ndarray:
-    """`gpt2-generate` (apps/gpt2/gpt2.lisp:97-113) on token ids: the first call feeds the whole
-    prompt at start position 0, each later call one token; every call's argmax is appended.
-    Returns [batch, prompt_len + max_length] int64.  With ``temperature`` > 0 the next id is drawn
-    on the device from the step's logits instead (temperature / top-k sampling, seeded; beyond the
-    reference, whose loop is greedy)."""
-    tokens = np.ascontiguousarray(prompt_ids, dtype=np.int64).reshape(gpt2.batch, -1)
-    start_pos = 0
-    rng = np.random.Generator(np.random.PCG64(seed))
-    for _ in range(max_length):
-        in_tokens = tokens[:, start_pos:]
-        out = gpt2.forward(in_tokens, in_tokens.shape[1], start_pos)
-        if temperature > 0.0:
-            out = gpt2.sample(rng.random(gpt2.batch, dtype=np.float32), temperature, top_k)
-        start_pos = tokens.shape[1]
-        tokens = np.concatenate([tokens, out.reshape(-1, 1)], axis=1)
-    return tokens
+gpt2_generate = generate   # `gpt2-generate` (apps/gpt2/gpt2.lisp:97-113) without the tokenizer
 
 
 def make_gpt2_from_gguf(path: str, runtime: Optional[B200Runtime] = None, max_seq_len: Optional[int] = None, batch: int = 1,

@@ -37,7 +37,7 @@ enum {
   CATEN_B200_EDEVICE = 4      /* a kernel reported a failed internal check (e.g. a bounded wait ran out) */
 };
 
-/* ggml tensor type ids as stored in GGUF (external/gguf/tensor-info.lisp:3-34).  F32, F16, Q4_0
+/* ggml tensor type ids as stored in GGUF (external/gguf/tensor-info.lisp:3-34).  F32, F16, BF16, Q4_0
  * and Q8_0 weights stay in their file format on the device and the kernels unpack them; the other
  * block formats below (ids the reference lists but does not implement) are expanded to fp32 once
  * at upload, which is what the reference's loader does for every format it knows
@@ -45,12 +45,17 @@ enum {
 enum {
   CATEN_B200_F32 = 0, CATEN_B200_F16 = 1, CATEN_B200_Q4_0 = 2, CATEN_B200_Q8_0 = 8,
   CATEN_B200_Q4_1 = 3, CATEN_B200_Q5_0 = 6, CATEN_B200_Q5_1 = 7,
+  CATEN_B200_BF16 = 30,
   CATEN_B200_Q2_K = 10, CATEN_B200_Q3_K = 11, CATEN_B200_Q4_K = 12, CATEN_B200_Q5_K = 13, CATEN_B200_Q6_K = 14
 };
 
 /* epilogue applied by the Linear kernels after the bias: the scheduler fuses the activation
  * into the matmul kernel (source/test-suite/test-schedule.lisp:72-74). */
-enum { CATEN_B200_ACT_NONE = 0, CATEN_B200_ACT_GELU = 1, CATEN_B200_ACT_RELU = 2 };
+enum { CATEN_B200_ACT_NONE = 0, CATEN_B200_ACT_GELU = 1, CATEN_B200_ACT_RELU = 2,
+  /* gated: the weight's rows come in (gate, up) pairs, rows 2j and 2j + 1, and the linear has rows / 2
+   * outputs y[m, j] = max(gate, 0) * up.  Dense weights (F32, F16, BF16), an even number of rows, no
+   * residual. */
+  CATEN_B200_ACT_RELU_GLU = 3 };
 
 /* arithmetic of the Linear kernels when more than a few rows are multiplied at once:
  *   FP32    fp32 operands and accumulation on the CUDA cores (max-abs 1e-3 logit class)
@@ -278,6 +283,78 @@ int caten_b200_gpt2_kv(caten_b200_gpt2 *m, int layer, float **d_k, float **d_v);
 /* Number of kernel launches issued by this model's steps since creation. */
 int64_t caten_b200_gpt2_launch_count(caten_b200_gpt2 *m);
 
+/* ---- decoders described layer by layer ------------------------------------------------------------
+ * (No counterpart in the reference, whose only model graph is GPT-2's, external/llm/layers.lisp:54-90.)
+ * A decoder is a list of layers, each with a mixer and an optional feed-forward; a range of layers may
+ * run several times with the same weights (every pass has its own cache or state).  RMS norms with one
+ * scalar gain stand before and after every sublayer:
+ *   x += rms(mixer(rms(x) * norm1)) * norm1b;   x += rms(ff(rms(x) * norm2)) * norm2b
+ * Storage: heads are padded with zeros to a multiple of 16 (p16), rows of activations and the columns
+ * of weights to a multiple of 64 (p64); padded weight entries are zero.  wp = p64(width). */
+enum { CATEN_B200_MIX_ATTENTION = 0, CATEN_B200_MIX_WKV = 1 };
+typedef struct {
+  int32_t mixer;               /* CATEN_B200_MIX_* */
+  int32_t heads, dim;          /* query heads / heads of the recurrence and their size (<= 256) */
+  /* attention: grouped-query softmax attention in a sliding window (a query sees itself and the window - 1
+   * tokens before it; 0: every earlier token), q and k rotated on their first rot_dims dims (interleaved
+   * pairs, pair i by position * rot_freq[i]) and then, with qk_norm, divided by their root mean square;
+   * score = q . k * scale; with gated, head h's output times sigmoid(gate_h) */
+  int32_t kv_heads, vdim, window, rot_dims, qk_norm, gated;
+  float scale;
+  /* time mixing: rows of each of in_w's first four groups; stored rows of the decay's low-rank projection */
+  int32_t group_rows, low_rank;
+  /* gains of the norms */
+  float norm1, norm1b, norm2, norm2b;
+  /* device fp32 arrays (not owned) */
+  const float *rot_freq;       /* attention: [rot_dims / 2] */
+  const float *mu;             /* time mixing: [5, wp] token-shift weights of r, k, v, gate, decay */
+  const float *w0, *u, *norm;  /* time mixing: [p64(heads * p16(dim))] each; head h at h * p16(dim) */
+  /* attention: rows q [heads * p16(dim)], k, v [kv_heads * ...], gate [heads], padded to p64; cols wp.
+   * time mixing: groups r, k, v, gate of group_rows rows (a multiple of 128), then low_rank rows; cols wp. */
+  const caten_b200_weight *in_w;
+  const caten_b200_weight *out_w;   /* [wp, p64(heads * p16(vdim or dim))] */
+  const caten_b200_weight *w2;      /* time mixing, BF16: [p64(heads * p16(dim)), low_rank] */
+  const caten_b200_weight *ff_in;   /* (gate, up) row pairs [2 * p64(ff), wp]; NULL: no feed-forward */
+  const caten_b200_weight *ff_out;  /* [wp, p64(ff)] */
+} caten_b200_layer_desc;
+typedef struct {
+  int32_t n_layers, width, vocab, max_seq_len, batch, precision;
+  int32_t max_rows;            /* rows (sequences x tokens) processed at once; 0 = default */
+  int32_t max_portion;         /* tokens of a sequence processed at once; 0 = default.  A windowed layer's cache
+                                * holds window - 1 + max_portion positions, whatever max_seq_len is */
+  int32_t loop_start, loop_stop, loop_times;  /* layers [start, stop) run `times` times; stop <= start: no loop */
+  float eps;                   /* inside every root */
+  float final_gain;            /* gain of the norm before `head`, times the scale of the logits */
+  const caten_b200_weight *embed;    /* BF16 [vocab, wp] */
+  const caten_b200_weight *head;     /* [vocab, wp] */
+  const caten_b200_weight *loop_in;  /* x = loop_in . [x ; embedding output] before each pass: [wp, 2 wp]; NULL without a loop */
+  const caten_b200_layer_desc *layers;
+} caten_b200_decoder_desc;
+typedef struct caten_b200_decoder caten_b200_decoder;
+/* Allocates caches, states (zero) and the workspace.  Weights and arrays stay owned by the caller. */
+int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc *desc, caten_b200_decoder **m);
+int caten_b200_decoder_destroy(caten_b200_decoder *m);
+/* The next s tokens h_ids [B, s] (int64) of every sequence, at positions n ..; n = 0 starts new sequences
+ * (nothing earlier is kept), otherwise n is where the previous step ended.
+ * h_want [n_want]: ascending places in [0, s) whose logits are written to h_logits [B, n_want, vocab].
+ * h_out_ids [B]: argmax of the last position's logits.  Either may be NULL (n_want 0).  Synchronises. */
+int caten_b200_decoder_step(caten_b200_decoder *m, const int64_t *h_ids, int64_t s, int64_t n, const int64_t *h_want,
+                            int64_t n_want, float *h_logits, int64_t *h_out_ids);
+/* Same from device ids, without logits; d_out_ids [B] or NULL.  Asynchronous. */
+int caten_b200_decoder_step_device(caten_b200_decoder *m, const int64_t *d_ids, int64_t s, int64_t n, int64_t *d_out_ids);
+/* `steps` greedy single-token steps on the device, as caten_b200_gpt2_decode. */
+int caten_b200_decoder_decode(caten_b200_decoder *m, const int64_t *d_first_ids, int64_t n, int64_t steps, int64_t *d_out_ids);
+/* Device pointer to the [B, vocab] fp32 logits of the last position (of the last step that computed them). */
+const float *caten_b200_decoder_logits(caten_b200_decoder *m);
+/* Layer runs of a step: layers, each pass of a looped layer counting. */
+int64_t caten_b200_decoder_runs(caten_b200_decoder *m);
+/* Residual stream after every layer run of the following steps: h_buf [runs, B * s, width] fp32 in host memory,
+ * sized for the steps' s (which must fit one portion); NULL turns it off.  Slow (for checks). */
+int caten_b200_decoder_capture(caten_b200_decoder *m, float *h_buf);
+/* Bytes of device memory held by caches and states. */
+int64_t caten_b200_decoder_cache_nbytes(caten_b200_decoder *m);
+int64_t caten_b200_decoder_launch_count(caten_b200_decoder *m);
+
 /* ---- multi-GPU plane -------------------------------------------------------------------------------
  * No counterpart in the reference (multi-device execution is an item of its roadmap, Readme.md:181);
  * these entries let a host that cannot use torch.distributed (Common Lisp through CFFI) run the
@@ -368,7 +445,9 @@ enum {
   CATEN_B200_K_EMBED = 0, CATEN_B200_K_LAYERNORM = 1, CATEN_B200_K_GEMV = 2, CATEN_B200_K_GEMM = 3,
   CATEN_B200_K_ATTN_DECODE = 4, CATEN_B200_K_ATTN_PREFILL = 5, CATEN_B200_K_ARGMAX = 6,
   CATEN_B200_K_DECODE_STEP = 7,   /* the whole single-token step of 1..4 sequences, which is one kernel */
-  CATEN_B200_K_COUNT = 8
+  CATEN_B200_K_WKV = 8,           /* recurrence of a time-mixing layer */
+  CATEN_B200_K_PREP = 9,          /* rotation, q/k norm and cache append; token-shift mixes */
+  CATEN_B200_K_COUNT = 10
 };
 /* Starts timing the classes whose bit (1 << class) is set in class_mask. */
 int caten_b200_profile_begin(caten_b200_ctx *ctx, unsigned class_mask);
