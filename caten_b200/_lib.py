@@ -54,6 +54,18 @@ class GPT2Desc(C.Structure):
 MIX_ATTENTION, MIX_WKV = 0, 1
 
 
+class AttnDesc(C.Structure):
+    """Mirror of ``caten_b200_attn_desc``."""
+    _fields_ = [(n, C.c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "window", "rot_dims", "qk_norm", "gated")] + [
+        ("scale", C.c_float), ("eps", C.c_float), ("rot_freq", _vp)]
+
+
+class WkvDesc(C.Structure):
+    """Mirror of ``caten_b200_wkv_desc``."""
+    _fields_ = [(n, C.c_int32) for n in ("heads", "dim", "group_rows", "low_rank")] + [("eps", C.c_float)] + [
+        (n, _vp) for n in ("w0", "u", "norm", "w2")]
+
+
 class LayerDesc(C.Structure):
     """Mirror of ``caten_b200_layer_desc``."""
     _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "kv_heads", "vdim", "window", "rot_dims", "qk_norm", "gated")] + [
@@ -136,6 +148,8 @@ SIGNATURES = {
     "caten_b200_gpt2_logits": (_vp, [_vp]),
     "caten_b200_gpt2_kv": (C.c_int, [_vp, C.c_int, _PFP, _PFP]),
     "caten_b200_gpt2_launch_count": (_i64, [_vp]),
+    "caten_b200_attn_window": (C.c_int, [_vp, C.POINTER(AttnDesc), _vp, _i64, _vp, _vp, _i64, _vp, _i64, _i64, _i64, C.c_int]),
+    "caten_b200_wkv": (C.c_int, [_vp, C.POINTER(WkvDesc), _vp, _vp, _vp, _i64, _i64, _i64, C.c_int]),
     "caten_b200_decoder_create": (C.c_int, [_vp, C.POINTER(DecoderDesc), _PFP]),
     "caten_b200_decoder_destroy": (C.c_int, [_vp]),
     "caten_b200_decoder_step": (C.c_int, [_vp, _vp, _i64, _i64, _vp, _i64, _vp, _vp]),

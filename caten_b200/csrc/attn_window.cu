@@ -559,3 +559,35 @@ int launch_attn_window_decode(caten_b200_ctx *ctx, const AttnArgs &a) {
 }
 
 }  // namespace cb
+
+using namespace cb;
+
+extern "C" int caten_b200_attn_window(caten_b200_ctx *ctx, const caten_b200_attn_desc *c, float *d_qkv, int64_t ld, float *d_kcache,
+                                      float *d_vcache, int64_t cap, float *d_out, int64_t B, int64_t s, int64_t n, int precision) {
+  if (!ctx) return fail(nullptr, CATEN_B200_EINVAL, "attn_window: ctx is NULL");
+  cudaSetDevice(ctx->device);
+  if (!c || !d_qkv || !d_kcache || !d_vcache || !d_out) return fail(ctx, CATEN_B200_EINVAL, "attn_window: NULL argument");
+  if (B < 0 || s < 0 || n < 0 || cap <= 0 || cap % 64 || cap > 0x3fffffff || n + s > 0x3fffffff || c->heads <= 0 || c->kv_heads <= 0 || c->heads % c->kv_heads || c->dim <= 0 || c->vdim <= 0 ||
+      c->window < 0 || c->rot_dims < 0 || c->rot_dims % 2 || c->rot_dims > c->dim || (c->rot_dims && !c->rot_freq))
+    return fail(ctx, CATEN_B200_EINVAL, "attn_window: bad shape");
+  if (precision < CATEN_B200_PREC_FP32 || precision > CATEN_B200_PREC_BF16X3) return fail(ctx, CATEN_B200_EINVAL, "attn_window: unknown precision %d", precision);
+  AttnArgs a;
+  a.H = c->heads; a.G = c->kv_heads;
+  a.D = c->dim; a.Dp = (c->dim + 15) / 16 * 16; a.E = c->vdim; a.Ep = (c->vdim + 15) / 16 * 16;
+  a.qkv = d_qkv; a.ld = ld;
+  a.k_off = (int64_t)a.H * a.Dp; a.v_off = a.k_off + (int64_t)a.G * a.Dp;
+  a.gate_off = c->gated ? a.v_off + (int64_t)a.G * a.Ep : -1;
+  if (ld % 4 || ld < a.v_off + (int64_t)a.G * a.Ep + (c->gated ? a.H : 0)) return fail(ctx, CATEN_B200_EINVAL, "attn_window: ld=%lld", (long long)ld);
+  a.kc = d_kcache; a.vc = d_vcache; a.cap = cap;
+  a.out = d_out; a.out_ld = (int64_t)a.H * a.Ep;
+  a.B = (int)B; a.s = (int)s; a.n = (int)n;
+  a.window = c->window; a.rot_pairs = c->rot_dims / 2; a.freq = c->rot_freq; a.qk_norm = c->qk_norm; a.eps = c->eps; a.scale = c->scale;
+  if (B == 0 || s == 0) return 0;
+  ProfScope prof(ctx, s == 1 ? CATEN_B200_K_ATTN_DECODE : CATEN_B200_K_ATTN_PREFILL);
+  if (s == 1) return launch_attn_window_decode(ctx, a);
+  // checked before the append, which writes the ring
+  const int64_t live = c->window > 0 && c->window - 1 < n ? c->window - 1 + s : n + s;
+  if (live > cap) return fail(ctx, CATEN_B200_EINVAL, "attn_window: %lld live positions in a ring of %lld", (long long)live, (long long)cap);
+  if (int rc = launch_attn_prep(ctx, a)) return rc;
+  return launch_attn_window_prefill(ctx, a, precision != CATEN_B200_PREC_FP32);
+}

@@ -39,7 +39,7 @@ __global__ void __launch_bounds__(128) wkv_lowrank_kernel(const WkvArgs a, float
   const int64_t r = blockIdx.x;
   const float *src = a.y + r * a.ld + 4 * (int64_t)a.gr;
   for (int j = threadIdx.x; j < a.w1; j += 128) st_out(t, tb, r * a.w1 + j, tanhf(src[j]));
-  if ((int)(r % a.s) == a.s - 1) {
+  if (h && (int)(r % a.s) == a.s - 1) {
     const float4 *hr = reinterpret_cast<const float4 *>(h) + r * w4;
     float4 *st = reinterpret_cast<float4 *>(shift) + (r / a.s) * w4;
     for (int c = threadIdx.x; c < w4; c += 128) st[c] = hr[c];
@@ -329,3 +329,41 @@ int launch_wkv_decode(caten_b200_ctx *ctx, const WkvArgs &a) {
 }
 
 }  // namespace cb
+
+using namespace cb;
+
+extern "C" int caten_b200_wkv(caten_b200_ctx *ctx, const caten_b200_wkv_desc *c, const float *d_y, float *d_state, float *d_out, int64_t B,
+                              int64_t s, int64_t n, int precision) {
+  if (!ctx) return fail(nullptr, CATEN_B200_EINVAL, "wkv: ctx is NULL");
+  cudaSetDevice(ctx->device);
+  if (!c || !d_y || !d_state || !d_out || !c->w0 || !c->u || !c->norm || !c->w2) return fail(ctx, CATEN_B200_EINVAL, "wkv: NULL argument");
+  WkvArgs a;
+  a.H = c->heads; a.D = c->dim; a.Dp = (c->dim + 15) / 16 * 16;
+  const int64_t hd = ((int64_t)a.H * a.Dp + 63) / 64 * 64;
+  if (B < 0 || s < 0 || n < 0 || n + s > 0x7fffffff || c->heads <= 0 || c->dim <= 0 || c->group_rows % 4 || c->low_rank <= 0 || c->low_rank % 64 || c->w2->type != CATEN_B200_BF16 ||
+      c->w2->rows != hd || c->w2->cols != c->low_rank)
+    return fail(ctx, CATEN_B200_EINVAL, "wkv: bad shape");
+  if (precision < CATEN_B200_PREC_FP32 || precision > CATEN_B200_PREC_BF16X3) return fail(ctx, CATEN_B200_EINVAL, "wkv: unknown precision %d", precision);
+  if (B == 0 || s == 0) return 0;
+  a.y = d_y; a.gr = c->group_rows; a.w1 = c->low_rank; a.ld = 4ll * a.gr + a.w1;
+  a.w2 = (const __nv_bfloat16 *)c->w2->qs; a.w0 = c->w0; a.u = c->u; a.norm = c->norm; a.eps = c->eps;
+  a.state = d_state; a.out = d_out; a.out_ld = hd;
+  a.B = (int)B; a.s = (int)s; a.n = (int)n;
+  if (s == 1) {
+    ProfScope prof(ctx, CATEN_B200_K_WKV);
+    return launch_wkv_decode(ctx, a);
+  }
+  const int64_t R = B * s;
+  const size_t t_b = (size_t)(R * a.w1) * 4, d_b = (size_t)(R * hd) * 4;
+  auto al = [](size_t b) { return (b + 255) / 256 * 256; };
+  if (int rc = scratch_reserve(ctx, &ctx->wkv_tmp, al(t_b) + 2 * al(d_b) + al((size_t)hd * 4))) return rc;
+  uint8_t *base = (uint8_t *)ctx->wkv_tmp.ptr;
+  float *t = (float *)base, *d = (float *)(base + al(t_b)), *o = (float *)(base + al(t_b) + al(d_b)), *w0 = (float *)(base + al(t_b) + 2 * al(d_b));
+  CB_CUDA(ctx, cudaMemsetAsync(w0, 0, (size_t)hd * 4, ctx->stream));
+  CB_CUDA(ctx, cudaMemcpyAsync(w0, c->w0, (size_t)a.H * a.Dp * 4, cudaMemcpyDeviceToDevice, ctx->stream));
+  if (int rc = launch_wkv_lowrank(ctx, a, t, BfOut(), nullptr, nullptr, 0)) return rc;
+  if (int rc = model_linear(ctx, precision, c->w2, t, BfOut(), w0, nullptr, CATEN_B200_ACT_NONE, d, BfOut(), R)) return rc;
+  a.d = d; a.d_ld = hd; a.o = o; a.o_ld = hd;
+  ProfScope prof(ctx, CATEN_B200_K_WKV);
+  return launch_wkv_scan(ctx, a);
+}

@@ -240,6 +240,20 @@ class B200Runtime:
         L.check(self.ctx, self.lib.caten_b200_attention_ex(self.ctx, qkv.ptr, kcache.ptr, vcache.ptr, out.ptr, B, s, n, H, T, precision))
         return out
 
+    def attn_window(self, desc: L.AttnDesc, qkv: B200Buffer, kcache: B200Buffer, vcache: B200Buffer, B: int, s: int, n: int,
+                    precision: int = L.PREC_FP32) -> B200Buffer:
+        """Windowed grouped-query attention over ring caches [B, kv_heads, cap, head] (``caten_b200_attn_window``)."""
+        out = self.open_buffer((B * s, desc.heads * vcache.shape[3]), np.float32)
+        L.check(self.ctx, self.lib.caten_b200_attn_window(self.ctx, C.byref(desc), qkv.ptr, qkv.shape[-1], kcache.ptr, vcache.ptr, kcache.shape[2],
+                                                          out.ptr, B, s, n, precision))
+        return out
+
+    def wkv(self, desc: L.WkvDesc, y: B200Buffer, state: B200Buffer, B: int, s: int, n: int, precision: int = L.PREC_FP32) -> B200Buffer:
+        """Time mixing from its projections (``caten_b200_wkv``); ``state`` [B, heads, p16, p16] is carried."""
+        out = self.open_buffer((B * s, -(-desc.heads * state.shape[3] // 64) * 64), np.float32)
+        L.check(self.ctx, self.lib.caten_b200_wkv(self.ctx, C.byref(desc), y.ptr, state.ptr, out.ptr, B, s, n, precision))
+        return out
+
     def argmax(self, x: B200Buffer) -> B200Buffer:
         rows, V = x.shape
         out = self.open_buffer((rows,), np.int64)

@@ -20,7 +20,7 @@ def bf16_to_f32(bits: np.ndarray) -> np.ndarray:
 def f32_to_bf16(x: np.ndarray) -> np.ndarray:
     """Bit patterns (uint16) of finite fp32 values rounded to the nearest bf16, ties to even."""
     u = np.ascontiguousarray(x, np.float32).view(np.uint32)
-    return ((u + np.uint32(0x7FFF) + ((u >> np.uint32(16)) & np.uint32(1))) >> np.uint32(16)).astype(np.uint16)
+    return ((u + np.uint32(0x7FFF) + ((u >> np.uint32(16)) & np.uint32(1))) >> np.uint32(16)).astype(np.uint16).reshape(np.shape(x))
 
 
 class SafeTensors:

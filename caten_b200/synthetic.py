@@ -149,6 +149,67 @@ def synth_state_dict(p: GPT2Params, wtype: str = "f32", seed: int = 0, max_seq_l
     return sd
 
 
+def binusun_config(width: int, vocab: int, order: str, ff: int, heads: int, kv_heads: int, dim: int, vdim: int, window: int, wkv_heads: int, wkv_dim: int,
+                   rot_dims: int, rot_base: float = 10000.0, scaling: dict | None = None, scale: float | None = None, loop: tuple | None = None,
+                   eps: float = 1e-5, logit_scale: float = 1.0) -> dict:
+    """A Binusun configuration (the content of config.json).  ``order``: one letter per layer, "a" attention or "w"
+    time mixing; an upper-case letter adds a feed-forward of width ``ff``.  ``loop``: (start, stop, times)."""
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": window}, "scale": dim ** -0.5 if scale is None else scale,
+           "rot": {"base": rot_base, "dims": rot_dims, "scaling": scaling}}
+    mix = {"heads": wkv_heads, "dim": wkv_dim}
+    layers = [{"type": "attention" if c in "aA" else "wkv", "mixer": dict(att) if c in "aA" else dict(mix),
+               "mlp": {"kind": "dense", "ff": ff} if c.isupper() else None} for c in order]
+    return {"architecture": "Binusun", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": eps}, "logit_scale": logit_scale,
+            "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]} if loop else None}
+
+
+def synth_binusun(cfg: dict, seed: int = 0, low_rank: int = 16) -> dict:
+    """Random weights of a Binusun configuration: tensor name -> bf16 bit patterns (uint16).  Matrices ~ N(0, 1 / in),
+    so that projections of a normed row have unit scale; norm gains around 1; the decays spread over (0, 1)."""
+    from .safetensors import f32_to_bf16
+    rng = np.random.Generator(np.random.PCG64(seed))
+    width, vocab, t = cfg["width"], cfg["vocab"], {}
+
+    def mat(name, rows, cols):
+        t[name] = f32_to_bf16(rng.standard_normal((rows, cols), dtype=np.float32) * np.float32(cols ** -0.5))
+
+    def vec(name, shape, mean, std):
+        t[name] = f32_to_bf16(np.float32(mean) + rng.standard_normal(shape, dtype=np.float32) * np.float32(std))
+
+    t["embed"] = f32_to_bf16(rng.standard_normal((vocab, width), dtype=np.float32))
+    if cfg.get("loop"):
+        mat("loop.in", width, 2 * width)
+    for i, l in enumerate(cfg["layers"]):
+        pre, m = f"l{i}.", l["mixer"]
+        mix = pre + "mix."
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if l["mlp"] else ()):
+            vec(pre + n, (), 1.0, 0.1)
+        if l["type"] == "attention":
+            H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            for n, r in (("q", H * D), ("k", G * D), ("v", G * E), ("g", H)):
+                mat(mix + n, r, width)
+            mat(mix + "o", width, H * E)
+        else:
+            hd = m["heads"] * m["dim"]
+            for c in "rkvgw":
+                vec(mix + "mu." + c, (width,), 0.5, 0.25)
+            for c in "rkvg":
+                mat(mix + c, hd, width)
+            mat(mix + "w1", low_rank, width)
+            mat(mix + "w2", hd, low_rank)
+            vec(mix + "w0", (hd,), -2.0, 1.5)
+            vec(mix + "u", (m["heads"], m["dim"]), 0.0, 0.5)
+            vec(mix + "norm", (hd,), 1.0, 0.1)
+            mat(mix + "o", width, hd)
+        if l["mlp"]:
+            mat(pre + "mlp.gate", l["mlp"]["ff"], width)
+            mat(pre + "mlp.up", l["mlp"]["ff"], width)
+            mat(pre + "mlp.down", width, l["mlp"]["ff"])
+    vec("final.norm", (), 1.0, 0.1)
+    mat("head", vocab, width)
+    return t
+
+
 def synth_prompts(batch: int, length: int, vocab: int, seed: int = 0) -> np.ndarray:
     """[batch, length] int64 token ids uniform in [0, vocab)."""
     rng = np.random.Generator(np.random.PCG64(seed))

@@ -283,6 +283,37 @@ int caten_b200_gpt2_kv(caten_b200_gpt2 *m, int layer, float **d_k, float **d_v);
 /* Number of kernel launches issued by this model's steps since creation. */
 int64_t caten_b200_gpt2_launch_count(caten_b200_gpt2 *m);
 
+/* ---- attention with windows and grouped heads; time mixing ---------------------------------------
+ * The two mixers of the layer-by-layer decoders below, for a host that runs its own layer loop.  Storage
+ * rules as there: heads padded with zeros to a multiple of 16 floats (p16), fp32 activations. */
+typedef struct {
+  int32_t heads, kv_heads, dim, vdim;  /* query head h reads key/value head h / (heads / kv_heads); sizes <= 256 */
+  int32_t window;                      /* position i sees j with 0 <= i - j < window; 0: every j <= i */
+  int32_t rot_dims;                    /* even; interleaved pairs rotated by position * rot_freq[pair] */
+  int32_t qk_norm;                     /* 1: q and k divided by sqrt(mean(x^2) + eps) after the rotation */
+  int32_t gated;                       /* 1: head h's output times sigmoid(gate_h) */
+  float scale, eps;
+  const float *rot_freq;               /* device, [rot_dims / 2] */
+} caten_b200_attn_desc;
+/* s tokens per sequence at positions n ..: appends k and v to the ring caches (slot = position % cap) and writes
+ * softmax(q . k * scale) . v.  qkv [B * s, ld]: q heads, k heads, v heads, gate logits (q is overwritten with its rotated,
+ * normalised form when s > 1); caches [B, kv_heads, cap, p16(dim)] and [.., p16(vdim)], cap a multiple of 64 and at least
+ * min(window - 1, n) + s (without a window n + s); out [B * s, heads * p16(vdim)].  precision: CATEN_B200_PREC_*. */
+int caten_b200_attn_window(caten_b200_ctx *ctx, const caten_b200_attn_desc *desc, float *d_qkv, int64_t ld, float *d_kcache,
+                           float *d_vcache, int64_t cap, float *d_out, int64_t B, int64_t s, int64_t n, int precision);
+typedef struct {
+  int32_t heads, dim;                  /* state [dim, dim] per head, dim <= 256 */
+  int32_t group_rows, low_rank;        /* column layout of y; low_rank a multiple of 64 */
+  float eps;
+  const float *w0, *u, *norm;          /* device, [heads * p16(dim)] each */
+  const caten_b200_weight *w2;         /* BF16 [p64(heads * p16(dim)), low_rank] */
+} caten_b200_wkv_desc;
+/* y [B * s, 4 * group_rows + low_rank]: r, k, v, gate, and the decay's low-rank input.  Per head, from state [B, heads,
+ * p16(dim), p16(dim)] (read as zero when n = 0):  o = (S + diag(u) k v^T)^T r;  S = diag(w) S + k v^T;
+ * w = exp(-exp(w2 . tanh(low rank) + w0));  out [B * s, p64(heads * p16(dim))] = o / rms(o) * norm * silu(gate). */
+int caten_b200_wkv(caten_b200_ctx *ctx, const caten_b200_wkv_desc *desc, const float *d_y, float *d_state, float *d_out, int64_t B,
+                   int64_t s, int64_t n, int precision);
+
 /* ---- decoders described layer by layer ------------------------------------------------------------
  * (No counterpart in the reference, whose only model graph is GPT-2's, external/llm/layers.lisp:54-90.)
  * A decoder is a list of layers, each with a mixer and an optional feed-forward; a range of layers may
