@@ -8,6 +8,7 @@
 //
 // Keys are cached rotated and normalised; everything here is fp32.
 #include "attn_window.cuh"
+#include "tcgen05.cuh"
 
 namespace cb {
 
@@ -239,14 +240,27 @@ int launch_attn_window_prefill(caten_b200_ctx *ctx, const AttnArgs &a, int tenso
 // Single-token step.  One CTA serves HPC query heads of one key/value head of one sequence, so a K / V
 // row is read once for all of them; with few sequences a thread-block cluster splits the keys and its
 // CTAs combine their (maximum, sum, output) through distributed shared memory.
-//   prologue  the step's q, k, v (from the projection or its split-K partial tiles), rotated and
-//             normalised by one warp each; the k / v row is appended to the ring
-//   scores    KL lanes x NV float4 per K row; the HPC x U dot products of a lane group are reduced
-//             together (each exchange halves the values a lane carries)
-//   softmax   two passes over the CTA's scores in shared memory
-//   output    P.V, summed over the row groups, rescaled over the cluster, gated
+//   producer warp   streams the history in chunks of CH rows, all of K and then all of V, into a ring of
+//                   shared-memory stages (one bulk copy per chunk, two where it crosses the ring's end);
+//                   V arrives while the last scores and the softmax are computed
+//   prologue        the step's q, k, v (from the projection or its split-K partial tiles), rotated and
+//                   normalised by one warp each; the k / v row is appended to the cache
+//   scores          KL lanes x NV float4 per K row; the HPC x U dot products of a lane group are reduced
+//                   together (each exchange halves the values a lane carries)
+//   softmax         two passes over the CTA's scores in shared memory
+//   output          P.V, summed over the row groups, rescaled over the cluster, gated
+// Every mbarrier wait is bounded; when one runs out the CTA records it in the status word, leaves its
+// loops, waits for its copies in flight, takes part in the cluster barriers and writes no output.
 // ---------------------------------------------------------------------------------------------
-constexpr int AD_THREADS = 256;
+constexpr int AD_WORK = 256, AD_THREADS = AD_WORK + 32, AD_STAGES = 3;
+
+__device__ __forceinline__ void work_sync() { asm volatile("bar.sync 1, %0;" ::"n"(AD_WORK) : "memory"); }
+__device__ __forceinline__ void bulk_load(uint32_t dst, const void *src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
+}
+__device__ __forceinline__ void bulk_hint(const void *src, uint32_t bytes) {
+  asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(src), "r"(bytes) : "memory");
+}
 
 template <int R>
 __device__ __forceinline__ float group_reduce(float *v, int lane, int lanes) {
@@ -264,190 +278,281 @@ __device__ __forceinline__ float group_reduce(float *v, int lane, int lanes) {
   return v[0];
 }
 
+template <int KL, int NV> struct AdShape {
+  static constexpr int GROUPS = AD_WORK / KL;             // rows per load
+  static constexpr int U = NV == 2 ? 2 : 4;               // loads per lane and chunk
+  static constexpr int CH = GROUPS * U;                   // rows per chunk: 16 KB at the widest head of the class
+};
+
 template <int KL, int NV, int HPC>
-__global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const AttnArgs a, const int S, const int per_max) {
-  constexpr int GROUPS = AD_THREADS / KL;       // rows in flight per load
-  constexpr int U = HPC == 1 ? 8 : 4;           // loads in flight per lane
+__global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const AttnArgs a, const int S, const int per_max, const long long hint_bytes,
+                                                                        int *status) {
+  constexpr int GROUPS = AdShape<KL, NV>::GROUPS, U = AdShape<KL, NV>::U, CH = AdShape<KL, NV>::CH;
   constexpr int R = U * HPC;                    // dot products reduced together (<= KL)
   static_assert(R <= KL, "one value per lane after the exchanges");
-  constexpr int TPH = AD_THREADS / HPC;         // threads per head in the softmax
+  constexpr int TPH = AD_WORK / HPC;            // threads per head in the softmax
   extern __shared__ __align__(16) float sm[];
-  const int Dp = a.Dp, Ep = a.Ep;
-  float *q = sm;                                // [HPC][Dp]
+  const int Dp = a.Dp, Ep = a.Ep, wide = Dp > Ep ? Dp : Ep;
+  float *ring = sm;                             // [AD_STAGES][CH][wide]; afterwards the row groups' outputs [GROUPS][HPC][Ep]
+  float *q = ring + AD_STAGES * CH * wide;      // [HPC][Dp]
   float *kn = q + HPC * Dp;                     // the step's key
   float *vn = kn + Dp;                          // and value
   float *gate = vn + Ep;                        // [4]
   float *ml = gate + 4;                         // [HPC] max, [HPC] sum (read by the other CTAs of the cluster): 8
   float *red = ml + 8;                          // 8
   float *ol = red + 8;                          // [HPC][Ep] this CTA's output
-  float *part = ol + HPC * Ep;                  // [GROUPS][HPC][Ep]
-  float *sc = part + GROUPS * HPC * Ep;         // [HPC][per_max]
+  uint64_t *bars = reinterpret_cast<uint64_t *>(ol + HPC * Ep);  // full [AD_STAGES], empty [AD_STAGES]
+  volatile int *abort_flag = reinterpret_cast<volatile int *>(bars + 2 * AD_STAGES);  // [0] a wait ran out; [1] never set; 4 words
+  float *sc = reinterpret_cast<float *>(bars + 2 * AD_STAGES + 2);  // [per_max][HPC]
+  const uint32_t bar0 = smem_u32(bars);
+  auto full = [&](int s) { return bar0 + 8u * s; };
+  auto empty = [&](int s) { return bar0 + 8u * (AD_STAGES + s); };
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int h0 = blockIdx.x * HPC, b = blockIdx.y, rank = blockIdx.z;
-  const int rep = a.H / a.G, g = h0 / rep;
+  const int rep = a.H / a.G, g = h0 / rep, cap = (int)a.cap;
   float *kb = a.kc + ((int64_t)b * a.G + g) * a.cap * Dp;
   float *vb = a.vc + ((int64_t)b * a.G + g) * a.cap * Ep;
+  // this CTA's keys of the step at position n: [jb, je), of which [jb, hb) are history
+  auto range = [&](int n, int &jb, int &je) {
+    const int t0 = a.window > 0 && n - a.window + 1 > 0 ? n - a.window + 1 : 0;
+    const int count = n + 1 - t0, per = (count + S - 1) / S;
+    jb = t0 + min(rank * per, count);
+    je = t0 + min((rank + 1) * per, count);
+  };
+  if (tid == 0) {
+    for (int s = 0; s < AD_STAGES; ++s) {
+      mbar_init(full(s), 1);
+      mbar_init(empty(s), AD_WORK / 32);
+    }
+    abort_flag[0] = abort_flag[1] = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  // While the kernels before this one still run, the first CTAs ask for their history to be brought into L2 (see
+  // attn_decode_kernel: a hint, limited to what fits L2; a stale position only changes what is asked for).
+  if (warp == AD_WORK / 32) {
+    int jb, je, n = a.d_n ? *reinterpret_cast<const volatile int *>(a.d_n) : a.n;
+    n = n < 0 ? 0 : n > 0x3fffffff ? 0x3fffffff : n;
+    range(n, jb, je);
+    const int hb = min(je, n);
+    const long long bytes = (long long)(hb - jb) * (Dp + Ep) * 4;
+    const long long index = ((long long)b * gridDim.x + blockIdx.x) * S + rank;
+    if (hb > jb && hb - jb <= cap && (index + 1) * bytes <= hint_bytes) {
+      const int which = lane & 1, piece = lane >> 1, w = which ? Ep : Dp;   // 16 pieces each of K and V
+      const int rows = (hb - jb + 15) / 16, s0 = (jb + piece * rows) % cap, r = min(rows, hb - jb - piece * rows);
+      if (r > 0) bulk_hint((which ? vb : kb) + (int64_t)s0 * w, (uint32_t)(min(r, cap - s0) * w) * 4u);
+    }
+  }
+  __syncthreads();
   pdl_enter();
   const int n = a.d_n ? *a.d_n : a.n;
-  const int t0 = a.window > 0 && n - a.window + 1 > 0 ? n - a.window + 1 : 0;
-  const int count = n + 1 - t0, per = (count + S - 1) / S;
-  const int jb = t0 + min(rank * per, count), je = t0 + min((rank + 1) * per, count);  // this CTA's keys
+  int jb, je;
+  range(n, jb, je);
+  const int hb = min(je, n), hist = hb - jb, nc = (hist + CH - 1) / CH;
+  const bool own_new = je == n + 1 && je > jb;   // the step's own key is in this CTA's range
+  const int cnt = hist + (own_new ? 1 : 0);
 
-  if (warp < HPC + 2) {
-    const bool is_q = warp < HPC, is_k = warp == HPC;
-    const int64_t off = is_q ? a.q_off + (int64_t)(h0 + warp) * Dp : is_k ? a.k_off + (int64_t)g * Dp : a.v_off + (int64_t)g * Ep;
-    const int np = (is_q || is_k ? Dp : Ep) / 2;
-    HeadPairs h;
+  if (warp == AD_WORK / 32) {
+    if (lane == 0) {
+      int issued = 0;
+      for (int i = 0; i < 2 * nc; ++i) {
+        const int s = i % AD_STAGES;
+        if (i >= AD_STAGES && !mbar_wait(empty(s), (uint32_t)(i / AD_STAGES - 1) & 1u, abort_flag)) {
+          if (!*abort_flag) { *abort_flag = 1; atomicCAS(status, 0, DEV_WAIT_TIMEOUT); status[1] = 20; }
+          break;
+        }
+        const bool isv = i >= nc;
+        const int c = isv ? i - nc : i, w = isv ? Ep : Dp;
+        const int rows = min(CH, hist - c * CH), s0 = (jb + c * CH) % cap, r0 = min(rows, cap - s0);
+        const float *base = isv ? vb : kb;
+        const uint32_t dst = smem_u32(ring + s * CH * wide);
+        mbar_expect_tx(full(s), (uint32_t)(rows * w) * 4u);
+        bulk_load(dst, base + (int64_t)s0 * w, (uint32_t)(r0 * w) * 4u, full(s));
+        if (r0 < rows) bulk_load(dst + (uint32_t)(r0 * w) * 4u, base, (uint32_t)((rows - r0) * w) * 4u, full(s));
+        issued = i + 1;
+      }
+      if (*abort_flag)  // copies in flight land before the CTA's shared memory is released
+        for (int i = issued > AD_STAGES ? issued - AD_STAGES : 0; i < issued; ++i) mbar_wait(full(i % AD_STAGES), (uint32_t)(i / AD_STAGES) & 1u, abort_flag + 1);
+    }
+    __syncwarp();
+  } else {
+    if (warp < HPC + 2) {
+      const bool is_q = warp < HPC, is_k = warp == HPC;
+      const int64_t off = is_q ? a.q_off + (int64_t)(h0 + warp) * Dp : is_k ? a.k_off + (int64_t)g * Dp : a.v_off + (int64_t)g * Ep;
+      const int np = (is_q || is_k ? Dp : Ep) / 2;
+      HeadPairs h;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int i = lane + 32 * j;
-      h.p[j] = make_float2(0.f, 0.f);
-      if (i < np) {
-        if (a.pin.splits > 0) h.p[j] = make_float2(partin_load1(a.pin, b, (int)off + 2 * i), partin_load1(a.pin, b, (int)off + 2 * i + 1));
-        else h.p[j] = reinterpret_cast<const float2 *>(a.qkv + (int64_t)b * a.ld + off)[i];
+      for (int j = 0; j < 4; ++j) {
+        const int i = lane + 32 * j;
+        h.p[j] = make_float2(0.f, 0.f);
+        if (i < np) {
+          if (a.pin.splits > 0) h.p[j] = make_float2(partin_load1(a.pin, b, (int)off + 2 * i), partin_load1(a.pin, b, (int)off + 2 * i + 1));
+          else h.p[j] = reinterpret_cast<const float2 *>(a.qkv + (int64_t)b * a.ld + off)[i];
+        }
+      }
+      float mul = 1.0f;
+      if (is_q || is_k) {
+        rotate_pairs(h, a.freq, a.rot_pairs, n, lane);
+        if (a.qk_norm) mul = pairs_inv_rms(h, a.D, a.eps);
+      }
+      if (is_q) mul *= a.scale;
+      float *dst = is_q ? q + warp * Dp : is_k ? kn : vn;
+      float *row = is_k ? kb + (int64_t)(n % cap) * Dp : vb + (int64_t)(n % cap) * Ep;
+      const bool append = !is_q && rank == 0 && h0 % rep == 0;  // one CTA per key/value head
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int i = lane + 32 * j;
+        if (i < np) {
+          const float2 v = make_float2(h.p[j].x * mul, h.p[j].y * mul);
+          reinterpret_cast<float2 *>(dst)[i] = v;
+          if (append) reinterpret_cast<float2 *>(row)[i] = v;
+        }
+      }
+    } else if (warp == 7 && lane < HPC && a.gate_off >= 0) {
+      const int col = (int)a.gate_off + h0 + lane;
+      gate[lane] = sigmoidf(a.pin.splits > 0 ? partin_load1(a.pin, b, col) : a.qkv[(int64_t)b * a.ld + col]);
+    }
+    work_sync();
+    const int gi = tid / KL, gl = tid % KL;
+    if (own_new && warp < HPC) {
+      float x = 0.0f;
+      for (int i = lane; i < Dp; i += 32) x = fmaf(q[warp * Dp + i], kn[i], x);
+      x = warp_sum(x);
+      if (lane == 0) sc[hist * HPC + warp] = x;
+    }
+    bool ok = true;
+    {
+      float4 q4[HPC][NV];
+#pragma unroll
+      for (int h = 0; h < HPC; ++h)
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+          const int c = gl + KL * v;
+          q4[h][v] = 4 * c < Dp ? reinterpret_cast<const float4 *>(q + h * Dp)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+      for (int i = 0; i < nc && ok; ++i) {
+        const int s = i % AD_STAGES;
+        ok = __all_sync(0xffffffffu, mbar_wait(full(s), (uint32_t)(i / AD_STAGES) & 1u, abort_flag));
+        if (!ok) break;
+        const float *st = ring + s * CH * wide;
+        float d[R];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int row = u * GROUPS + gi;
+          float4 k4[NV];
+#pragma unroll
+          for (int v = 0; v < NV; ++v) {
+            const int c = gl + KL * v;
+            k4[v] = i * CH + row < hist && 4 * c < Dp ? reinterpret_cast<const float4 *>(st + row * Dp)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+          }
+#pragma unroll
+          for (int h = 0; h < HPC; ++h) {
+            float x = 0.0f;
+#pragma unroll
+            for (int v = 0; v < NV; ++v) x = fmaf(q4[h][v].x, k4[v].x, fmaf(q4[h][v].y, k4[v].y, fmaf(q4[h][v].z, k4[v].z, fmaf(q4[h][v].w, k4[v].w, x))));
+            d[u * HPC + h] = x;
+          }
+        }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(empty(s));
+        const float x = group_reduce<R>(d, gl, KL);
+        if (gl % (KL / R) == 0) {
+          const int idx = gl / (KL / R), row = i * CH + (idx / HPC) * GROUPS + gi;
+          if (row < hist) sc[row * HPC + idx % HPC] = x;
+        }
       }
     }
-    float mul = 1.0f;
-    if (is_q || is_k) {
-      rotate_pairs(h, a.freq, a.rot_pairs, n, lane);
-      if (a.qk_norm) mul = pairs_inv_rms(h, a.D, a.eps);
-    }
-    if (is_q) mul *= a.scale;
-    float *dst = is_q ? q + warp * Dp : is_k ? kn : vn;
-    float *row = is_k ? kb + (int64_t)(n % a.cap) * Dp : vb + (int64_t)(n % a.cap) * Ep;
-    const bool append = !is_q && rank == 0 && h0 % rep == 0;  // one CTA per key/value head
+    if (!ok && lane == 0 && !*abort_flag) { *abort_flag = 1; atomicCAS(status, 0, DEV_WAIT_TIMEOUT); status[1] = 21; }
+    work_sync();
+    {
+      const int h = tid / TPH, i0 = tid % TPH;
+      float m = -INFINITY;
+      for (int i = i0; i < cnt; i += TPH) m = fmaxf(m, sc[i * HPC + h]);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int i = lane + 32 * j;
-      if (i < np) {
-        const float2 v = make_float2(h.p[j].x * mul, h.p[j].y * mul);
-        reinterpret_cast<float2 *>(dst)[i] = v;
-        if (append) reinterpret_cast<float2 *>(row)[i] = v;
+      for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+      if (lane == 0) red[warp] = m;
+      work_sync();
+      m = red[h * (8 / HPC)];
+#pragma unroll
+      for (int w = 1; w < 8 / HPC; ++w) m = fmaxf(m, red[h * (8 / HPC) + w]);
+      float ss = 0.0f;
+      for (int i = i0; i < cnt; i += TPH) {
+        const float e = exp2f((sc[i * HPC + h] - m) * kLog2e);
+        sc[i * HPC + h] = e;
+        ss += e;
+      }
+      ss = warp_sum(ss);
+      work_sync();
+      if (lane == 0) red[warp] = ss;
+      work_sync();
+      if (i0 == 0) {
+        ss = 0.0f;
+#pragma unroll
+        for (int w = 0; w < 8 / HPC; ++w) ss += red[h * (8 / HPC) + w];
+        ml[h] = m;
+        ml[4 + h] = ss;
       }
     }
-  } else if (warp == 7 && lane < HPC && a.gate_off >= 0) {
-    const int col = (int)a.gate_off + h0 + lane;
-    gate[lane] = sigmoidf(a.pin.splits > 0 ? partin_load1(a.pin, b, col) : a.qkv[(int64_t)b * a.ld + col]);
-  }
-  __syncthreads();
-
-  const int gi = tid / KL, gl = tid % KL;
-  const int cap = (int)a.cap, slot0 = jb % cap - jb;  // slot of key j: j + slot0, less cap past the ring's end
-  auto slot_of = [&](int j) { const int s = j + slot0; return (int64_t)(s >= cap ? s - cap : s); };
-  float4 q4[HPC][NV];
-#pragma unroll
-  for (int h = 0; h < HPC; ++h)
-#pragma unroll
-    for (int v = 0; v < NV; ++v) {
-      const int c = gl + KL * v;
-      q4[h][v] = 4 * c < Dp ? reinterpret_cast<const float4 *>(q + h * Dp)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
-  for (int j0 = jb; j0 < je; j0 += GROUPS * U) {
-    float4 k4[U][NV];
-#pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int j = j0 + u * GROUPS + gi;
-#pragma unroll
-      for (int v = 0; v < NV; ++v) {
-        const int c = gl + KL * v;
-        k4[u][v] = j < je && j < n && 4 * c < Dp ? __ldcs(reinterpret_cast<const float4 *>(kb + slot_of(j) * Dp) + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-        if (j == n && j < je && 4 * c < Dp) k4[u][v] = reinterpret_cast<const float4 *>(kn)[c];  // the step's own key
-      }
-    }
-    float d[R];
-#pragma unroll
-    for (int u = 0; u < U; ++u)
-#pragma unroll
-      for (int h = 0; h < HPC; ++h) {
-        float x = 0.0f;
-#pragma unroll
-        for (int v = 0; v < NV; ++v) x = fmaf(q4[h][v].x, k4[u][v].x, fmaf(q4[h][v].y, k4[u][v].y, fmaf(q4[h][v].z, k4[u][v].z, fmaf(q4[h][v].w, k4[u][v].w, x))));
-        d[u * HPC + h] = x;
-      }
-    const float x = group_reduce<R>(d, gl, KL);
-    if (gl % (KL / R) == 0) {
-      const int idx = gl / (KL / R), u = idx / HPC, h = idx % HPC, j = j0 + u * GROUPS + gi;
-      if (j < je) sc[h * per_max + j - jb] = x;
-    }
-  }
-  __syncthreads();
-  {
-    const int h = tid / TPH, i0 = tid % TPH, cnt = je - jb;
-    float *s = sc + h * per_max;
-    float m = -INFINITY;
-    for (int i = i0; i < cnt; i += TPH) m = fmaxf(m, s[i]);
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-    if (lane == 0) red[warp] = m;
-    __syncthreads();
-    m = red[h * (8 / HPC)];
-#pragma unroll
-    for (int w = 1; w < 8 / HPC; ++w) m = fmaxf(m, red[h * (8 / HPC) + w]);
-    float ss = 0.0f;
-    for (int i = i0; i < cnt; i += TPH) {
-      const float e = exp2f((s[i] - m) * kLog2e);
-      s[i] = e;
-      ss += e;
-    }
-    ss = warp_sum(ss);
-    __syncthreads();
-    if (lane == 0) red[warp] = ss;
-    __syncthreads();
-    if (i0 == 0) {
-      ss = 0.0f;
-#pragma unroll
-      for (int w = 0; w < 8 / HPC; ++w) ss += red[h * (8 / HPC) + w];
-      ml[h] = m;
-      ml[4 + h] = ss;
-    }
-  }
-  {
     float4 acc[HPC][NV];
 #pragma unroll
     for (int h = 0; h < HPC; ++h)
 #pragma unroll
-      for (int v = 0; v < NV; ++v) acc[h][v] = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int j0 = jb; j0 < je; j0 += GROUPS * U) {
-      float4 v4[U][NV];
-      float p[U][HPC];
+      for (int v = 0; v < NV; ++v) {
+        const int c = gl + KL * v;
+        const float p = own_new && gi == 0 ? sc[hist * HPC + h] : 0.0f;
+        const float4 x = 4 * c < Ep ? reinterpret_cast<const float4 *>(vn)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+        acc[h][v] = make_float4(p * x.x, p * x.y, p * x.z, p * x.w);
+      }
+    for (int i = nc; i < 2 * nc && ok; ++i) {
+      const int s = i % AD_STAGES;
+      ok = __all_sync(0xffffffffu, mbar_wait(full(s), (uint32_t)(i / AD_STAGES) & 1u, abort_flag));
+      if (!ok) break;
+      const float *st = ring + s * CH * wide;
 #pragma unroll
       for (int u = 0; u < U; ++u) {
-        const int j = j0 + u * GROUPS + gi;
+        const int row = u * GROUPS + gi, key = (i - nc) * CH + row;
+        if (key < hist) {
+          float p[HPC];
+          if (HPC == 4) *reinterpret_cast<float4 *>(p) = *reinterpret_cast<const float4 *>(sc + key * HPC);
+          else
+#pragma unroll
+            for (int h = 0; h < HPC; ++h) p[h] = sc[key * HPC + h];
+#pragma unroll
+          for (int v = 0; v < NV; ++v) {
+            const int c = gl + KL * v;
+            const float4 x = 4 * c < Ep ? reinterpret_cast<const float4 *>(st + row * Ep)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int h = 0; h < HPC; ++h) {
+              acc[h][v].x = fmaf(p[h], x.x, acc[h][v].x);
+              acc[h][v].y = fmaf(p[h], x.y, acc[h][v].y);
+              acc[h][v].z = fmaf(p[h], x.z, acc[h][v].z);
+              acc[h][v].w = fmaf(p[h], x.w, acc[h][v].w);
+            }
+          }
+        }
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(empty(s));
+    }
+    if (!ok && lane == 0 && !*abort_flag) { *abort_flag = 1; atomicCAS(status, 0, DEV_WAIT_TIMEOUT); status[1] = 22; }
+    work_sync();  // every chunk has been consumed: the ring becomes the exchange buffer of the row groups
+    if (!*abort_flag) {
+      float *part = ring;
+#pragma unroll
+      for (int h = 0; h < HPC; ++h)
 #pragma unroll
         for (int v = 0; v < NV; ++v) {
           const int c = gl + KL * v;
-          v4[u][v] = j < je && j < n && 4 * c < Ep ? __ldcs(reinterpret_cast<const float4 *>(vb + slot_of(j) * Ep) + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-          if (j == n && j < je && 4 * c < Ep) v4[u][v] = reinterpret_cast<const float4 *>(vn)[c];
+          if (4 * c < Ep) reinterpret_cast<float4 *>(part + (gi * HPC + h) * Ep)[c] = acc[h][v];
         }
-#pragma unroll
-        for (int h = 0; h < HPC; ++h) p[u][h] = j < je ? sc[h * per_max + j - jb] : 0.0f;
-      }
-#pragma unroll
-      for (int u = 0; u < U; ++u)
-#pragma unroll
-        for (int h = 0; h < HPC; ++h)
-#pragma unroll
-          for (int v = 0; v < NV; ++v) {
-            acc[h][v].x = fmaf(p[u][h], v4[u][v].x, acc[h][v].x);
-            acc[h][v].y = fmaf(p[u][h], v4[u][v].y, acc[h][v].y);
-            acc[h][v].z = fmaf(p[u][h], v4[u][v].z, acc[h][v].z);
-            acc[h][v].w = fmaf(p[u][h], v4[u][v].w, acc[h][v].w);
-          }
     }
+    work_sync();
+    if (!*abort_flag)
+      for (int i = tid; i < HPC * Ep; i += AD_WORK) {
+        float o = 0.0f;
 #pragma unroll
-    for (int h = 0; h < HPC; ++h)
-#pragma unroll
-      for (int v = 0; v < NV; ++v) {
-        const int c = gl + KL * v;
-        if (4 * c < Ep) reinterpret_cast<float4 *>(part + (gi * HPC + h) * Ep)[c] = acc[h][v];
+        for (int w = 0; w < GROUPS; ++w) o += ring[w * HPC * Ep + i];
+        ol[i] = o;
       }
-  }
-  __syncthreads();
-  for (int i = tid; i < HPC * Ep; i += AD_THREADS) {
-    float o = 0.0f;
-#pragma unroll
-    for (int w = 0; w < GROUPS; ++w) o += part[w * HPC * Ep + i];
-    ol[i] = o;
   }
   auto finish = [&](int i, float o, float l) {
     const int h = i / Ep;
@@ -464,12 +569,13 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
   };
   if (S == 1) {
     __syncthreads();
-    for (int i = tid; i < HPC * Ep; i += AD_THREADS) finish(i, ol[i], ml[4 + i / Ep]);
+    if (!*abort_flag)
+      for (int i = tid; i < HPC * Ep; i += AD_THREADS) finish(i, ol[i], ml[4 + i / Ep]);
     return;
   }
   // combine over the cluster; both barriers are reached by every thread of every CTA
   asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-  const uint32_t ml0 = (uint32_t)__cvta_generic_to_shared(ml), ol0 = (uint32_t)__cvta_generic_to_shared(ol);
+  const uint32_t ml0 = smem_u32(ml), ol0 = smem_u32(ol);
   auto remote = [&](uint32_t local, int z) {
     uint32_t addr;
     float v;
@@ -477,18 +583,19 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
     asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
     return v;
   };
-  for (int i = rank + S * tid; i < HPC * Ep; i += S * AD_THREADS) {
-    const uint32_t h4 = 4u * (uint32_t)(i / Ep);
-    float m = -INFINITY;
-    for (int z = 0; z < S; ++z) m = fmaxf(m, remote(ml0 + h4, z));
-    float l = 0.0f, o = 0.0f;
-    for (int z = 0; z < S; ++z) {  // fixed order
-      const float f = exp2f((remote(ml0 + h4, z) - m) * kLog2e);  // a CTA without keys has maximum -inf and adds nothing
-      l = fmaf(f, remote(ml0 + 16u + h4, z), l);
-      o = fmaf(f, remote(ol0 + 4u * (uint32_t)i, z), o);
+  if (!*abort_flag)
+    for (int i = rank + S * tid; i < HPC * Ep; i += S * AD_THREADS) {
+      const uint32_t h4 = 4u * (uint32_t)(i / Ep);
+      float m = -INFINITY;
+      for (int z = 0; z < S; ++z) m = fmaxf(m, remote(ml0 + h4, z));
+      float l = 0.0f, o = 0.0f;
+      for (int z = 0; z < S; ++z) {  // fixed order
+        const float f = exp2f((remote(ml0 + h4, z) - m) * kLog2e);  // a CTA without keys has maximum -inf and adds nothing
+        l = fmaf(f, remote(ml0 + 16u + h4, z), l);
+        o = fmaf(f, remote(ol0 + 4u * (uint32_t)i, z), o);
+      }
+      finish(i, o, l);
     }
-    finish(i, o, l);
-  }
   asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 
@@ -516,7 +623,7 @@ static int launch_decode_t(caten_b200_ctx *ctx, const AttnArgs &a, int S, int pe
   }
   cfg.attrs = at;
   cfg.numAttrs = na;
-  CB_CUDA(ctx, cudaLaunchKernelEx(&cfg, attn_window_decode_kernel<KL, NV, HPC>, a, S, per_max));
+  CB_CUDA(ctx, cudaLaunchKernelEx(&cfg, attn_window_decode_kernel<KL, NV, HPC>, a, S, per_max, ctx->attn_prefetch_bytes, ctx->d_status));
   CB_LAUNCH_CHECK(ctx, "attn_window_decode_kernel");
   return 0;
 }
@@ -538,12 +645,15 @@ int launch_attn_window_decode(caten_b200_ctx *ctx, const AttnArgs &a) {
   int S = 1;
   while (S < 8 && ctas(hpc, S) < ctx->sm_count && keys / (2 * S) >= 32) S *= 2;
   while (hpc > 1 && ctas(hpc, S) * 2 <= ctx->sm_count) hpc /= 2;
-  const int kl = wide <= 64 ? 16 : 32, nv = wide <= 128 ? 1 : 2, groups = AD_THREADS / kl;
+  const int kl = wide <= 64 ? 16 : 32, nv = wide <= 128 ? 1 : 2;
+  const int ch = AD_WORK / kl * (nv == 2 ? 2 : 4);
   size_t smem = 0;
   int64_t per_max = 0;
   for (;;) {
     per_max = (keys + S - 1) / S;
-    smem = ((size_t)hpc * a.Dp + a.Dp + a.Ep + 20 + (size_t)hpc * a.Ep * (1 + groups) + (size_t)hpc * per_max) * sizeof(float);
+    // (the row groups' outputs, hpc / 4 of [ch][4][Ep] / U floats, fit the ring they reuse)
+    smem = ((size_t)AD_STAGES * ch * wide + (size_t)hpc * a.Dp + a.Dp + a.Ep + 20 + (size_t)hpc * a.Ep + (size_t)hpc * per_max) * sizeof(float) +
+           (2 * AD_STAGES + 2) * 8;
     if (smem <= 200 * 1024) break;
     if (S < 8) S *= 2;
     else if (hpc > 1) hpc /= 2;

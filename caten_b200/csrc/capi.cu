@@ -137,6 +137,7 @@ int caten_b200_destroy(caten_b200_ctx *ctx) {
   if (ctx->wtmp.ptr) cudaFree(ctx->wtmp.ptr);
   if (ctx->wbf.ptr) cudaFree(ctx->wbf.ptr);
   if (ctx->wkv_tmp.ptr) cudaFree(ctx->wkv_tmp.ptr);
+  if (ctx->wkv_chunks.ptr) cudaFree(ctx->wkv_chunks.ptr);
   if (ctx->upload_stage.ptr) cudaFree(ctx->upload_stage.ptr);
   for (int k = 0; k < 2; ++k) {
     if (ctx->pin[k]) cudaFreeHost(ctx->pin[k]);

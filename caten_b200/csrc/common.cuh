@@ -103,6 +103,7 @@ struct caten_b200_ctx {
   cb::Scratch xbf;           // bf16 copy (hi, lo) of the activation operand of the tensor-core GEMM
   cb::Scratch wtmp;          // split-K partial tiles of the tensor-core GEMM
   cb::Scratch wbf;           // bf16 copy (hi, lo) of the weight operand of the many-row GEMM
+  cb::Scratch wkv_chunks;    // per-chunk states of a time-mixing prompt
   cb::Scratch wkv_tmp;       // intermediates of a stand-alone time-mixing call
   cb::Scratch upload_stage;  // raw blocks of the weight being uploaded, before their re-layout
   void *pin[2] = {nullptr, nullptr};          // pinned bounce buffers for large copies from pageable host memory

@@ -4,8 +4,12 @@
 // then o is divided by its root mean square over the head, times a gain and silu(gate).
 // The state starts at zero with the sequence (position 0) and is carried from step to step.
 //
-// Multi-token steps walk the tokens in order (fp32, no reordering of the recurrence), which is
-// parallel over sequences, heads, value columns and keys: a thread keeps 4 KQ keys x CPT value
+// Prompts (heads up to 64) are computed in chunks of 64 tokens, all of them at once: within a chunk the
+// output is a causal matrix product and the state's contribution another, so only the chunk states form a
+// chain.  Everything stays fp32, and every decay factor is the exponential of a sum of non-positive
+// numbers (never a quotient of two cumulative products, which could underflow).
+//
+// Short multi-token steps, and wider heads, walk the tokens in order: a thread keeps 4 KQ keys x CPT value
 // columns of the state in registers, so a token costs three fused multiply-adds per element and one
 // exchange over the few lanes that share a column, which is off the chain from token to token.
 #include "wkv.cuh"
@@ -167,6 +171,322 @@ __global__ void __launch_bounds__(WS_THREADS) wkv_scan_kernel(const WkvArgs a, c
     }
 }
 
+// ---------------------------------------------------------------------------------------------
+// Chunked form.  With e = -log w, subchunks of 16 tokens, and for token t of subchunk a
+//   P_t = sum of e before t in a,  Q_t = sum of e after t in a,  tot_a = sum of e in a:
+//   out from earlier tokens s of subchunk b < a:  sum_i r_t k_s exp(-P_t - Q_s - tot_{b+1} - .. - tot_{a-1})
+//   out from earlier tokens of the same subchunk: the product of the decays in between, multiplied up
+//   out from the state before the chunk:          r_t exp(-P_t - tot_0 - .. - tot_{a-1}) . S
+//   the chunk's contribution to the state:        k_s exp(-Q_s - tot_{b+1} - .. - tot_3) v_s
+// wkv_chunk_kernel: the first two, the contribution U, and exp(-sum tot); leaves the scaled r in d.
+// wkv_states_kernel: walks the chunks, replacing U by the state before the chunk.
+// wkv_out_kernel: adds the state's part, then the head's norm and the gate.
+// ---------------------------------------------------------------------------------------------
+constexpr int WC_T = 64, WC_D = 64, WC_LD = 68, WC_THREADS = 256;   // tokens per chunk, head size, row pitch in shared memory
+constexpr size_t WC_SMEM = (size_t)(5 * WC_T * WC_LD + 2 * 4 * WC_D) * sizeof(float);
+
+__global__ void __launch_bounds__(WC_THREADS, 2) wkv_chunk_kernel(const WkvArgs a, float *__restrict__ U, float *__restrict__ decays) {
+  extern __shared__ __align__(16) float sm[];
+  float *rs = sm, *ks = rs + WC_T * WC_LD, *vs = ks + WC_T * WC_LD, *ws = vs + WC_T * WC_LD, *As = ws + WC_T * WC_LD;
+  float *tot = As + WC_T * WC_LD;   // [4][WC_D] sums of e per subchunk
+  float *g = tot + 4 * WC_D;        // [4][WC_D] exp(-tot)
+  const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, Dp = a.Dp;
+  const int t0 = c * WC_T, tn = min(WC_T, a.s - t0);
+  const int64_t row0 = (int64_t)b * a.s + t0;
+  pdl_enter();
+  // tokens past the end and channels past the head: r = k = v = 0 and no decay
+  for (int e = tid; e < 4 * WC_T * (WC_D / 4); e += WC_THREADS) {
+    const int which = e >> 10, t = (e >> 4) & 63, c4 = e & 15;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    const bool ok = t < tn && 4 * c4 < Dp;
+    if (ok) {
+      const float *src = which < 3 ? a.y + (row0 + t) * a.ld + (int64_t)which * a.gr + (int64_t)h * Dp : a.d + (row0 + t) * a.d_ld + (int64_t)h * Dp;
+      v = reinterpret_cast<const float4 *>(src)[c4];
+      if (which == 3) v = make_float4(expf(v.x), expf(v.y), expf(v.z), expf(v.w));
+    }
+    *reinterpret_cast<float4 *>((which == 0 ? rs : which == 1 ? ks : which == 2 ? vs : ws) + t * WC_LD + 4 * c4) = v;
+  }
+  __syncthreads();
+  const int sub = tid >> 6, ch = tid & 63;   // this thread's subchunk and channel in the element-wise passes
+  float ev[16];
+  {
+    float sum = 0.0f;
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      ev[j] = ws[(16 * sub + j) * WC_LD + ch];
+      sum += ev[j];
+      ws[(16 * sub + j) * WC_LD + ch] = expf(-ev[j]);
+    }
+    tot[sub * WC_D + ch] = sum;
+    g[sub * WC_D + ch] = expf(-sum);
+  }
+  __syncthreads();
+  // ---- same subchunk: four lanes per token s, 16 channels each ----
+  {
+    const int s = tid >> 2, qd = tid & 3, s16 = s & 15;
+    float q[16], acc = 0.0f;
+#pragma unroll
+    for (int m = 0; m < 4; ++m) {
+      const int i = 4 * (qd + 4 * m);
+      const float4 k4 = *reinterpret_cast<const float4 *>(ks + s * WC_LD + i), r4 = *reinterpret_cast<const float4 *>(rs + s * WC_LD + i);
+      float4 u4 = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < Dp) u4 = *reinterpret_cast<const float4 *>(a.u + (int64_t)h * Dp + i);
+      q[4 * m] = k4.x; q[4 * m + 1] = k4.y; q[4 * m + 2] = k4.z; q[4 * m + 3] = k4.w;
+      acc = fmaf(r4.x * u4.x, k4.x, fmaf(r4.y * u4.y, k4.y, fmaf(r4.z * u4.z, k4.z, fmaf(r4.w * u4.w, k4.w, acc))));
+    }
+    acc += __shfl_xor_sync(0xffffffffu, acc, 1);
+    acc += __shfl_xor_sync(0xffffffffu, acc, 2);
+    if (qd == 0) {
+      As[s * WC_LD + s] = acc;
+      for (int t = s - s16; t < s; ++t) As[t * WC_LD + s] = 0.0f;   // later tokens of the subchunk do not reach back
+    }
+    for (int dt = 1; dt < 16; ++dt) {
+      const bool on = s16 + dt < 16;
+      const int t = on ? s + dt : s;
+      acc = 0.0f;
+#pragma unroll
+      for (int m = 0; m < 4; ++m) {
+        const int i = 4 * (qd + 4 * m);
+        const float4 r4 = *reinterpret_cast<const float4 *>(rs + t * WC_LD + i), w4 = *reinterpret_cast<const float4 *>(ws + t * WC_LD + i);
+        acc = fmaf(r4.x, q[4 * m], fmaf(r4.y, q[4 * m + 1], fmaf(r4.z, q[4 * m + 2], fmaf(r4.w, q[4 * m + 3], acc))));
+        q[4 * m] *= w4.x; q[4 * m + 1] *= w4.y; q[4 * m + 2] *= w4.z; q[4 * m + 3] *= w4.w;
+      }
+      acc += __shfl_xor_sync(0xffffffffu, acc, 1);
+      acc += __shfl_xor_sync(0xffffffffu, acc, 2);
+      if (on && qd == 0) As[t * WC_LD + s] = acc;
+    }
+  }
+  __syncthreads();
+  // ---- r_t exp(-P_t), k_t exp(-Q_t) ----
+  {
+    float sum = 0.0f;
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      rs[(16 * sub + j) * WC_LD + ch] *= expf(-sum);
+      sum += ev[j];
+    }
+    sum = 0.0f;
+#pragma unroll
+    for (int j = 15; j >= 0; --j) {
+      ks[(16 * sub + j) * WC_LD + ch] *= expf(-sum);
+      sum += ev[j];
+    }
+  }
+  __syncthreads();
+  const int tx = tid & 15, ty = tid >> 4;
+  // ---- earlier subchunks: thread (ty, tx) owns (token ty of subchunk a, token tx of subchunk b) for all a > b ----
+  {
+    float a10 = 0.f, a21 = 0.f, a32 = 0.f, a20 = 0.f, a31 = 0.f, a30 = 0.f;
+#pragma unroll 4
+    for (int i = 0; i < WC_D; i += 4) {
+      const float4 g1 = *reinterpret_cast<const float4 *>(g + WC_D + i), g2 = *reinterpret_cast<const float4 *>(g + 2 * WC_D + i);
+      float4 r[4], k[3];
+#pragma unroll
+      for (int j = 1; j < 4; ++j) r[j] = *reinterpret_cast<const float4 *>(rs + (ty + 16 * j) * WC_LD + i);
+#pragma unroll
+      for (int j = 0; j < 3; ++j) k[j] = *reinterpret_cast<const float4 *>(ks + (tx + 16 * j) * WC_LD + i);
+#define WC_DOT(acc, R, K) acc = fmaf((R).x, (K).x, fmaf((R).y, (K).y, fmaf((R).z, (K).z, fmaf((R).w, (K).w, acc))))
+      WC_DOT(a10, r[1], k[0]);
+      WC_DOT(a21, r[2], k[1]);
+      WC_DOT(a32, r[3], k[2]);
+      k[0].x *= g1.x; k[0].y *= g1.y; k[0].z *= g1.z; k[0].w *= g1.w;
+      k[1].x *= g2.x; k[1].y *= g2.y; k[1].z *= g2.z; k[1].w *= g2.w;
+      WC_DOT(a20, r[2], k[0]);
+      WC_DOT(a31, r[3], k[1]);
+      k[0].x *= g2.x; k[0].y *= g2.y; k[0].z *= g2.z; k[0].w *= g2.w;
+      WC_DOT(a30, r[3], k[0]);
+#undef WC_DOT
+    }
+    As[(ty + 16) * WC_LD + tx] = a10;
+    As[(ty + 32) * WC_LD + tx] = a20;
+    As[(ty + 48) * WC_LD + tx] = a30;
+    As[(ty + 32) * WC_LD + tx + 16] = a21;
+    As[(ty + 48) * WC_LD + tx + 16] = a31;
+    As[(ty + 48) * WC_LD + tx + 32] = a32;
+  }
+  __syncthreads();
+  // ---- scale r for the state before the chunk (written over d) and k for the state after it ----
+  {
+    float fr = 1.0f, fk = 1.0f, all = 1.0f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float f = g[j * WC_D + ch];
+      if (j < sub) fr *= f;
+      if (j > sub) fk *= f;
+      all *= f;
+    }
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      const int t = 16 * sub + j;
+      ks[t * WC_LD + ch] *= fk;
+      if (t < tn && ch < Dp) a.d[(row0 + t) * a.d_ld + (int64_t)h * Dp + ch] = rs[t * WC_LD + ch] * fr;
+    }
+    if (sub == 0) decays[(((int64_t)b * a.H + h) * gridDim.x + c) * WC_D + ch] = all;
+  }
+  // ---- outputs from within the chunk: tokens ty + 16 j, columns 4 tx .. 4 tx + 3 ----
+  {
+    float4 o[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int sb = 0; sb < 4; ++sb) {
+#pragma unroll
+      for (int s4 = 0; s4 < 16; s4 += 4) {
+        const int s = 16 * sb + s4;
+        float4 v[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[e] = *reinterpret_cast<const float4 *>(vs + (s + e) * WC_LD + 4 * tx);
+#pragma unroll
+        for (int j = sb; j < 4; ++j) {
+          const float4 A = *reinterpret_cast<const float4 *>(As + (ty + 16 * j) * WC_LD + s);
+          o[j].x = fmaf(A.x, v[0].x, fmaf(A.y, v[1].x, fmaf(A.z, v[2].x, fmaf(A.w, v[3].x, o[j].x))));
+          o[j].y = fmaf(A.x, v[0].y, fmaf(A.y, v[1].y, fmaf(A.z, v[2].y, fmaf(A.w, v[3].y, o[j].y))));
+          o[j].z = fmaf(A.x, v[0].z, fmaf(A.y, v[1].z, fmaf(A.z, v[2].z, fmaf(A.w, v[3].z, o[j].z))));
+          o[j].w = fmaf(A.x, v[0].w, fmaf(A.y, v[1].w, fmaf(A.z, v[2].w, fmaf(A.w, v[3].w, o[j].w))));
+        }
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int t = ty + 16 * j;
+      if (t < tn && 4 * tx < Dp) *reinterpret_cast<float4 *>(a.o + (row0 + t) * a.o_ld + (int64_t)h * Dp + 4 * tx) = o[j];
+    }
+  }
+  __syncthreads();  // k is scaled
+  // ---- contribution to the state: keys 4 ty .. + 3, values 4 tx .. + 3 ----
+  {
+    float4 acc[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int s = 0; s < WC_T; ++s) {
+      const float4 k = *reinterpret_cast<const float4 *>(ks + s * WC_LD + 4 * ty), v = *reinterpret_cast<const float4 *>(vs + s * WC_LD + 4 * tx);
+      const float kk[4] = {k.x, k.y, k.z, k.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        acc[j].x = fmaf(kk[j], v.x, acc[j].x);
+        acc[j].y = fmaf(kk[j], v.y, acc[j].y);
+        acc[j].z = fmaf(kk[j], v.z, acc[j].z);
+        acc[j].w = fmaf(kk[j], v.w, acc[j].w);
+      }
+    }
+    float *dst = U + (((int64_t)b * a.H + h) * gridDim.x + c) * (WC_D * WC_D);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) *reinterpret_cast<float4 *>(dst + (4 * ty + j) * WC_D + 4 * tx) = acc[j];
+  }
+}
+
+// one thread per four values of a state row: U[c] <- S; S <- exp(-sum tot_c) S + U[c]
+__global__ void __launch_bounds__(256) wkv_states_kernel(const WkvArgs a, float *__restrict__ U, const float *__restrict__ decays, int chunks) {
+  pdl_enter();
+  const int h = blockIdx.y, b = blockIdx.z, Dp = a.Dp;
+  const int e = blockIdx.x * 256 + threadIdx.x, key = e >> 4, v4 = (e & 15) * 4;   // of WC_D x WC_D
+  const int64_t bh = (int64_t)b * a.H + h;
+  float4 *u = reinterpret_cast<float4 *>(U + bh * chunks * (WC_D * WC_D)) + e;
+  const float *w = decays + bh * chunks * WC_D + key;
+  float4 *st = reinterpret_cast<float4 *>(a.state + (bh * Dp + key) * Dp + v4);
+  const bool in = key < Dp && v4 < Dp;
+  float4 S = in && a.n > 0 ? *st : make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int c0 = 0; c0 < chunks; c0 += 4) {
+    float4 uc[4];
+    float wc[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (c0 + j < chunks) {
+        uc[j] = u[(int64_t)(c0 + j) * (WC_D * WC_D / 4)];
+        wc[j] = w[(int64_t)(c0 + j) * WC_D];
+      }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (c0 + j < chunks) {
+        u[(int64_t)(c0 + j) * (WC_D * WC_D / 4)] = S;
+        S.x = fmaf(wc[j], S.x, uc[j].x); S.y = fmaf(wc[j], S.y, uc[j].y); S.z = fmaf(wc[j], S.z, uc[j].z); S.w = fmaf(wc[j], S.w, uc[j].w);
+      }
+  }
+  if (in) *st = S;
+}
+
+__global__ void __launch_bounds__(WC_THREADS) wkv_out_kernel(const WkvArgs a, const float *__restrict__ U) {
+  __shared__ __align__(16) float rs[WC_T * WC_LD], S[WC_D * WC_LD];
+  const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, Dp = a.Dp;
+  const int t0 = c * WC_T, tn = min(WC_T, a.s - t0);
+  const int64_t row0 = (int64_t)b * a.s + t0;
+  pdl_enter();
+  const float4 *src = reinterpret_cast<const float4 *>(U + (((int64_t)b * a.H + h) * gridDim.x + c) * (WC_D * WC_D));
+  for (int e = tid; e < WC_T * 16; e += WC_THREADS) {
+    const int t = e >> 4, c4 = e & 15;
+    float4 r = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (t < tn && 4 * c4 < Dp) r = reinterpret_cast<const float4 *>(a.d + (row0 + t) * a.d_ld + (int64_t)h * Dp)[c4];
+    *reinterpret_cast<float4 *>(rs + t * WC_LD + 4 * c4) = r;
+    *reinterpret_cast<float4 *>(S + t * WC_LD + 4 * c4) = src[e];
+  }
+  __syncthreads();
+  const int tx = tid & 15, ty = tid >> 4;
+  float4 o[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int t = ty + 16 * j;
+    o[j] = t < tn && 4 * tx < Dp ? *reinterpret_cast<const float4 *>(a.o + (row0 + t) * a.o_ld + (int64_t)h * Dp + 4 * tx) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+#pragma unroll 4
+  for (int i = 0; i < WC_D; i += 4) {
+    float4 v[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] = *reinterpret_cast<const float4 *>(S + (i + e) * WC_LD + 4 * tx);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float4 r = *reinterpret_cast<const float4 *>(rs + (ty + 16 * j) * WC_LD + i);
+      o[j].x = fmaf(r.x, v[0].x, fmaf(r.y, v[1].x, fmaf(r.z, v[2].x, fmaf(r.w, v[3].x, o[j].x))));
+      o[j].y = fmaf(r.x, v[0].y, fmaf(r.y, v[1].y, fmaf(r.z, v[2].y, fmaf(r.w, v[3].y, o[j].y))));
+      o[j].z = fmaf(r.x, v[0].z, fmaf(r.y, v[1].z, fmaf(r.z, v[2].z, fmaf(r.w, v[3].z, o[j].z))));
+      o[j].w = fmaf(r.x, v[0].w, fmaf(r.y, v[1].w, fmaf(r.z, v[2].w, fmaf(r.w, v[3].w, o[j].w))));
+    }
+  }
+  const float4 nw = 4 * tx < Dp ? *reinterpret_cast<const float4 *>(a.norm + (int64_t)h * Dp + 4 * tx) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    float ss = (o[j].x * o[j].x + o[j].y * o[j].y) + (o[j].z * o[j].z + o[j].w * o[j].w);
+#pragma unroll
+    for (int m = 8; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+    const int t = ty + 16 * j;
+    if (t < tn && 4 * tx < Dp) {
+      const float inv = 1.0f / sqrtf(ss / (float)a.D + a.eps);
+      const float4 z = *reinterpret_cast<const float4 *>(a.y + (row0 + t) * a.ld + 3 * (int64_t)a.gr + (int64_t)h * Dp + 4 * tx);
+      const float4 v = make_float4(o[j].x * inv * nw.x * silu(z.x), o[j].y * inv * nw.y * silu(z.y), o[j].z * inv * nw.z * silu(z.z), o[j].w * inv * nw.w * silu(z.w));
+      const int64_t at = (row0 + t) * a.out_ld + (int64_t)h * Dp + 4 * tx;
+      if (a.bf.hi) {
+        *reinterpret_cast<uint2 *>(a.bf.hi + at) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+        if (a.bf.lo) *reinterpret_cast<uint2 *>(a.bf.lo + at) = make_uint2(pack_bf16(bf16_lo(v.x), bf16_lo(v.y)), pack_bf16(bf16_lo(v.z), bf16_lo(v.w)));
+      } else {
+        *reinterpret_cast<float4 *>(a.out + at) = v;
+      }
+    }
+  }
+}
+
+static int check_wkv(caten_b200_ctx *ctx, const WkvArgs &a) {
+  if (a.H <= 0 || a.D <= 0 || a.D > a.Dp || a.Dp % 16 || a.gr < a.H * a.Dp || a.n < 0) return fail(ctx, CATEN_B200_EINVAL, "wkv: bad shape");
+  if (a.Dp > 256) return fail(ctx, CATEN_B200_EUNSUPPORTED, "wkv: head size above 256");
+  if (a.H > 65535 || a.B > 65535) return fail(ctx, CATEN_B200_EUNSUPPORTED, "wkv: B or H > 65535");
+  return 0;
+}
+
+static int launch_chunked(caten_b200_ctx *ctx, const WkvArgs &a) {
+  const int chunks = (a.s + WC_T - 1) / WC_T;
+  const size_t n = (size_t)a.B * a.H * chunks;
+  if (int rc = scratch_reserve(ctx, &ctx->wkv_chunks, n * (WC_D * WC_D + WC_D) * sizeof(float))) return rc;
+  float *U = (float *)ctx->wkv_chunks.ptr, *decays = U + n * (WC_D * WC_D);
+  const dim3 grid((unsigned)chunks, (unsigned)a.H, (unsigned)a.B);
+  CB_CUDA(ctx, cudaFuncSetAttribute(wkv_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)WC_SMEM));
+  launch_k(ctx, wkv_chunk_kernel, grid, dim3(WC_THREADS), WC_SMEM, a, U, decays);
+  CB_LAUNCH_CHECK(ctx, "wkv_chunk_kernel");
+  launch_k(ctx, wkv_states_kernel, dim3(WC_D * WC_D / 4 / 256, (unsigned)a.H, (unsigned)a.B), dim3(256), 0, a, U, decays, chunks);
+  CB_LAUNCH_CHECK(ctx, "wkv_states_kernel");
+  launch_k(ctx, wkv_out_kernel, grid, dim3(WC_THREADS), 0, a, U);
+  CB_LAUNCH_CHECK(ctx, "wkv_out_kernel");
+  return 0;
+}
+
 // heads' norm and gate of one row: one warp per head
 __global__ void __launch_bounds__(256) wkv_gate_kernel(const WkvArgs a) {
   pdl_enter();
@@ -191,13 +511,6 @@ __global__ void __launch_bounds__(256) wkv_gate_kernel(const WkvArgs a) {
   }
 }
 
-static int check_wkv(caten_b200_ctx *ctx, const WkvArgs &a) {
-  if (a.H <= 0 || a.D <= 0 || a.D > a.Dp || a.Dp % 16 || a.gr < a.H * a.Dp || a.n < 0) return fail(ctx, CATEN_B200_EINVAL, "wkv: bad shape");
-  if (a.Dp > 256) return fail(ctx, CATEN_B200_EUNSUPPORTED, "wkv: head size above 256");
-  if (a.H > 65535 || a.B > 65535) return fail(ctx, CATEN_B200_EUNSUPPORTED, "wkv: B or H > 65535");
-  return 0;
-}
-
 template <int KQ, int CPT>
 static int launch_scan_t(caten_b200_ctx *ctx, const WkvArgs &a) {
   int KS = 1;
@@ -213,6 +526,7 @@ static int launch_scan_t(caten_b200_ctx *ctx, const WkvArgs &a) {
 int launch_wkv_scan(caten_b200_ctx *ctx, const WkvArgs &a) {
   if (a.B <= 0 || a.s <= 0) return 0;
   if (int rc = check_wkv(ctx, a)) return rc;
+  if (a.Dp <= WC_D && a.s >= 32) return launch_chunked(ctx, a);
   // few heads and sequences: fewer keys per thread, so that more warps share the work of a token
   const int64_t warps = (int64_t)a.B * a.H * ((a.Dp * a.Dp + 511) / 512);  // of 16 keys x 1 column per thread
   int rc;

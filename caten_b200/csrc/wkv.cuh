@@ -11,8 +11,9 @@ struct WkvArgs {
   PartIn pin;                       // single-token steps: the projections may still be split-K partial tiles
   int64_t ld = 0;
   int gr = 0, w1 = 0;
-  // multi-token steps: the decay's second projection, tanh(low rank) . W2 + w0 (one row of d_ld floats per token)
-  const float *d = nullptr;
+  // multi-token steps: the decay's second projection, tanh(low rank) . W2 + w0 (one row of d_ld floats per token;
+  // overwritten)
+  float *d = nullptr;
   int64_t d_ld = 0;
   // single-token steps form it themselves
   const __nv_bfloat16 *w2 = nullptr;  // [H * Dp, w1]
