@@ -3,6 +3,7 @@
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
                     [--workload xl-q4_0-b256|medium-q4_0-b64|small-q8_0-b1|small-f32-b1|xl-q4_0-b1]
                     [--precision bf16x3|bf16|fp32] [--scaling strong|weak]
+    python bench.py --compare binusun      # prefill and decode of Binusun layers beside GPT-2 at equal size
 
 A "step" is one KV-cached greedy decode step of the whole batch (one new token per sequence).
 Default workload: GPT-2 XL, Q4_0 weights, ONE batch of 256 sequences, 512-token prompts, 256 decoded
@@ -200,8 +201,148 @@ def oracle_parity(model, params, fsd, nb: int, precision: str, threads: int, pro
             "ids_equal_where_decisive": f"{ids_equal}/{ids_checked}"}
 
 
+# ------------------------------------------------------------------ --compare binusun
+# Layers of the sizes a real model would have, random weights, one GPU; GPT-2 with the same width, vocabulary and weight
+# format (bf16) and about the same number of weights read per token.
+COMPARE_SIZES = {
+    # width: (layer order, ff, heads, kv_heads, head size, window, heads and head size of the time mixing, loop, GPT-2 layers)
+    1024: dict(order="wAAwAAAAAAAA", ff=2816, heads=8, kv_heads=4, dim=128, window=1024, wkv=(16, 64), gpt2_layers=10),
+    2048: dict(order="wAAwAAAA", ff=5632, heads=16, kv_heads=4, dim=128, window=1024, wkv=(32, 64), gpt2_layers=6),
+}
+COMPARE_PREFILL = ((1, 2048), (8, 1024))     # (sequences, tokens)
+COMPARE_DECODE = (1, 16, 64, 256)            # sequences, at contexts of about 1 100 tokens
+
+
+def compare_rooflines(kind, model, mode, B, s, ctx, peaks):
+    """Algorithmic work of one step by kernel class -> seconds at the measured peaks.  ``kind``: dict of the sizes;
+    ``mode``: "prefill" (s tokens per sequence from position 0) or "decode" (one token at context ``ctx``)."""
+    hbm, tf = peaks
+    w, rows = kind["width"], B * (s if mode == "prefill" else 1)
+    t = {}
+    if mode == "prefill":
+        t["linears"] = max(2.0 * rows * kind["layer_weights"] / tf, 2.0 * kind["layer_weights"] / hbm)
+        # keys each query sees, summed over the tokens of a sequence
+        pairs = lambda win: sum(min(i + 1, win) if win else i + 1 for i in range(s))
+        t["attention"] = sum(4.0 * B * H * D * pairs(win) for H, G, D, win in kind["attn"]) / tf
+        t["norms"] = kind["norms"] * rows * w * kind["norm_bytes"][mode] / hbm
+        # r, k, v, gate, decay in; out
+        t["wkv"] = sum(rows * H * D * (5 * 4 + 2) for H, D in kind["wkv"]) / hbm
+    else:
+        t["linears"] = 2.0 * (kind["layer_weights"] + kind["head_weights"]) / hbm
+        t["attention"] = sum(8.0 * B * G * D * (min(ctx, win) if win else ctx) for H, G, D, win in kind["attn"]) / hbm
+        t["norms"] = kind["norms"] * rows * w * kind["norm_bytes"][mode] / hbm
+        t["wkv"] = sum(8.0 * B * H * D * D for H, D in kind["wkv"]) / hbm
+    return {k: v for k, v in t.items() if v}
+
+
+COMPARE_CLASSES = {"linears": ("gemm", "gemv"), "attention": ("attn_prefill", "attn_decode"), "norms": ("layernorm",), "wkv": ("wkv",), "prep": ("prep",)}
+
+
+def compare_binusun():
+    import torch
+    from caten_b200 import _lib as L_
+    from caten_b200 import synthetic as S
+    from caten_b200.binusun import Binusun, parse_config
+    from caten_b200.gpt2 import GPT2
+    from caten_b200.runtime import B200Runtime
+    from caten_b200.safetensors import f32_to_bf16
+    torch.cuda.set_device(0)
+    hbm, src = load_peaks()
+    burst, sustained = load_tensor_peak()
+    peaks = (hbm * 1e9, burst * 1e12)
+    rt = B200Runtime(0)
+    ext = torch.cuda.ExternalStream(rt.stream, device=torch.device("cuda", 0))
+    V = 32000
+
+    def ev():
+        e = torch.cuda.Event(enable_timing=True)
+        e.record(ext)
+        return e
+
+    rng = np.random.Generator(np.random.PCG64(0))
+    results = []
+    sampler = ClockSampler(0)
+    for width, z in COMPARE_SIZES.items():
+        cfg = S.binusun_config(width, V, z["order"], z["ff"], z["heads"], z["kv_heads"], z["dim"], z["dim"], z["window"], *z["wkv"], rot_dims=z["dim"] // 2)
+        tensors = S.synth_binusun(cfg, seed=0, low_rank=64)
+        attn = [l["mixer"] for l in cfg["layers"] if l["type"] == "attention"]
+        wkv = [l["mixer"] for l in cfg["layers"] if l["type"] == "wkv"]
+        n_layer = sum(v.size for k, v in tensors.items() if v.ndim == 2 and k[0] == "l")
+        bin_kind = dict(width=width, layer_weights=n_layer, head_weights=V * width, norms=sum(4 if l["mlp"] else 2 for l in cfg["layers"]) / 2,
+                        norm_bytes={"prefill": 14, "decode": 14},   # sublayer output and stream in, stream and bf16 operand out
+                        attn=[(m["heads"], m["kv_heads"], m["dim"], m["mask"]["size"]) for m in attn], wkv=[(m["heads"], m["dim"]) for m in wkv])
+        gp = S.GPT2Params(z["gpt2_layers"], width // 64, width, V)
+        gsd = S.synth_state_dict(gp, "f32", seed=0, max_seq_len=2304)
+        for k, v in gsd.items():
+            if v.ndim == 2 and not k.startswith("w"):
+                gsd[k] = S.Packed(L_.BF16, v.shape[0], v.shape[1], f32_to_bf16(v).view(np.uint8).reshape(-1))
+        gpt_kind = dict(width=width, layer_weights=12 * width * width * gp.n_layers, head_weights=V * width, norms=2 * gp.n_layers,
+                        norm_bytes={"prefill": 6, "decode": 14},    # prompts add the residual in the linear's epilogue
+                        attn=[(gp.n_heads, gp.n_heads, 64, 0)] * gp.n_layers, wkv=[])
+
+        def make(name, B, T):
+            if name == "binusun":
+                return Binusun(rt, parse_config(cfg), tensors, max_seq_len=T, batch=B, precision="bf16")
+            return GPT2(rt, gp, gsd, max_seq_len=T, batch=B, precision="bf16")
+
+        def classes(prof, steps, roof):
+            out = {}
+            for c, names in COMPARE_CLASSES.items():
+                ms = sum(prof[n][0] for n in names if n in prof) / steps
+                if ms:
+                    out[c] = {"us": round(ms * 1e3, 1), **({"frac_of_roofline": round(roof[c] * 1e3 / ms, 4)} if c in roof else {})}
+            return out
+
+        for mode, cases in (("prefill", COMPARE_PREFILL), ("decode", [(B, 1024) for B in COMPARE_DECODE])):
+            for B, s in cases:
+                row = {"width": width, "mode": mode, "sequences": B, "tokens" if mode == "prefill" else "context": s if mode == "prefill" else 1104}
+                for name, kind in (("binusun", bin_kind), ("gpt2", gpt_kind)):
+                    m = make(name, B, s if mode == "prefill" else 1200)
+                    ids = rt.transfer_from_array(rng.integers(0, V, (B, s), dtype=np.int64))
+                    out = rt.open_buffer((B,), np.int64)
+                    m.forward_device(ids, s, 0, out)
+                    roof = compare_rooflines(kind, m, mode, B, s, 1104, peaks)
+                    if mode == "prefill":
+                        for _ in range(3):
+                            m.forward_device(ids, s, 0, out)
+                        rt.sync()
+                        e0 = ev()
+                        for _ in range(5):
+                            m.forward_device(ids, s, 0, out)
+                        e1 = ev()
+                        rt.sync()
+                        ms, toks = e0.elapsed_time(e1) / 5, B * s
+                        rt.profile_begin()
+                        m.forward_device(ids, s, 0, out)
+                        prof = rt.profile_end()
+                        steps = 1
+                    else:
+                        m.decode_device_buffers(out, 1024, 40, None)     # captures the step's graph; warm-up
+                        rt.sync()
+                        e0 = ev()
+                        m.decode_device_buffers(out, 1064, 64, None)
+                        e1 = ev()
+                        rt.sync()
+                        ms, toks = e0.elapsed_time(e1) / 64, B
+                        rt.profile_begin()
+                        m.decode_device_buffers(out, 1128, 8, None)
+                        prof = rt.profile_end()
+                        steps = 8
+                    row[name] = {"ms": round(ms, 4), "tokens_per_s": round(toks / ms * 1e3), "weights_M": round((kind["layer_weights"] + kind["head_weights"]) / 1e6, 1),
+                                 "frac_of_roofline": round(sum(roof.values()) * 1e3 / ms, 4), "classes": classes(prof, steps, roof)}
+                    m.close(); ids.close(); out.close()
+                results.append(row)
+    clocks = sampler.stop()
+    rt.close()
+    print(json.dumps({"metric": "binusun_and_gpt2_layers", "data": "synthetic", "dtype": "bf16 weights and GEMM operands, fp32 otherwise", "n_gpus": 1,
+                      "peaks": {"hbm_gbs": hbm, "bf16_tflops": burst, "source": src},
+                      "timing": "CUDA events; decode steps replayed from a CUDA graph; classes from a separate pass with events around every launch (a few us each)",
+                      "l2": "weights and caches exceed L2 except where the batch is small", "clocks": clocks, "results": results}))
+
+
 def main():
     ap = argparse.ArgumentParser()
+    ap.add_argument("--compare", choices=["binusun"], default=None, help="prefill and decode throughput of a design's layers beside GPT-2 at equal size, instead of the benchmark")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=None)
     ap.add_argument("--warmup", type=int, default=3)
@@ -221,6 +362,8 @@ def main():
     ap.add_argument("--no-parity", action="store_true", help="skip the short oracle check of the benchmarked model")
     ap.add_argument("--no-extras", action="store_true", help="skip the prefill/GEMV/kernel-breakdown side measurements")
     args = ap.parse_args()
+    if args.compare:
+        return compare_binusun()
 
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))

@@ -585,15 +585,27 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
   };
   if (!*abort_flag)
     for (int i = rank + S * tid; i < HPC * Ep; i += S * AD_THREADS) {
+      // all CTAs' values are requested together: S <= 8 loads in flight instead of a chain of round trips
       const uint32_t h4 = 4u * (uint32_t)(i / Ep);
-      float m = -INFINITY;
-      for (int z = 0; z < S; ++z) m = fmaxf(m, remote(ml0 + h4, z));
-      float l = 0.0f, o = 0.0f;
-      for (int z = 0; z < S; ++z) {  // fixed order
-        const float f = exp2f((remote(ml0 + h4, z) - m) * kLog2e);  // a CTA without keys has maximum -inf and adds nothing
-        l = fmaf(f, remote(ml0 + 16u + h4, z), l);
-        o = fmaf(f, remote(ol0 + 4u * (uint32_t)i, z), o);
-      }
+      float mz[8], lz[8], oz[8];
+#pragma unroll
+      for (int z = 0; z < 8; ++z)
+        if (z < S) {
+          mz[z] = remote(ml0 + h4, z);
+          lz[z] = remote(ml0 + 16u + h4, z);
+          oz[z] = remote(ol0 + 4u * (uint32_t)i, z);
+        }
+      float m = -INFINITY, l = 0.0f, o = 0.0f;
+#pragma unroll
+      for (int z = 0; z < 8; ++z)
+        if (z < S) m = fmaxf(m, mz[z]);
+#pragma unroll
+      for (int z = 0; z < 8; ++z)
+        if (z < S) {  // fixed order
+          const float f = exp2f((mz[z] - m) * kLog2e);  // a CTA without keys has maximum -inf and adds nothing
+          l = fmaf(f, lz[z], l);
+          o = fmaf(f, oz[z], o);
+        }
       finish(i, o, l);
     }
   asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");

@@ -175,7 +175,8 @@ __global__ void __launch_bounds__(WS_THREADS) wkv_scan_kernel(const WkvArgs a, c
 // Chunked form.  With e = -log w, subchunks of 16 tokens, and for token t of subchunk a
 //   P_t = sum of e before t in a,  Q_t = sum of e after t in a,  tot_a = sum of e in a:
 //   out from earlier tokens s of subchunk b < a:  sum_i r_t k_s exp(-P_t - Q_s - tot_{b+1} - .. - tot_{a-1})
-//   out from earlier tokens of the same subchunk: the product of the decays in between, multiplied up
+//   out from earlier tokens of the same subchunk: the same with segments of 8, 4 and 2 tokens in place of
+//     subchunks (every pair of tokens is split by exactly one level's segment boundary)
 //   out from the state before the chunk:          r_t exp(-P_t - tot_0 - .. - tot_{a-1}) . S
 //   the chunk's contribution to the state:        k_s exp(-Q_s - tot_{b+1} - .. - tot_3) v_s
 // wkv_chunk_kernel: the first two, the contribution U, and exp(-sum tot); leaves the scaled r in d.
@@ -183,11 +184,44 @@ __global__ void __launch_bounds__(WS_THREADS) wkv_scan_kernel(const WkvArgs a, c
 // wkv_out_kernel: adds the state's part, then the head's norm and the gate.
 // ---------------------------------------------------------------------------------------------
 constexpr int WC_T = 64, WC_D = 64, WC_LD = 68, WC_THREADS = 256;   // tokens per chunk, head size, row pitch in shared memory
-constexpr size_t WC_SMEM = (size_t)(5 * WC_T * WC_LD + 2 * 4 * WC_D) * sizeof(float);
+constexpr size_t WC_SMEM = (size_t)(6 * WC_T * WC_LD + 2 * 4 * WC_D) * sizeof(float);
+
+__device__ __forceinline__ float exp_neg(float x) { return exp2f(-1.4426950408889634f * x); }
+
+__device__ __forceinline__ float dot_rows(const float *p, const float *q) {
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < WC_D; i += 4) {
+    const float4 x = *reinterpret_cast<const float4 *>(p + i), y = *reinterpret_cast<const float4 *>(q + i);
+    acc.x = fmaf(x.x, y.x, acc.x); acc.y = fmaf(x.y, y.y, acc.y); acc.z = fmaf(x.z, y.z, acc.z); acc.w = fmaf(x.w, y.w, acc.w);
+  }
+  return (acc.x + acc.y) + (acc.z + acc.w);
+}
+
+// One subchunk's channel at segment length 2 M: tokens of a segment's first half carry k decayed to its middle, those of
+// the second half r decayed from it (16 tokens, e in registers).
+template <int M>
+__device__ __forceinline__ void split_level(const float *ev, const float *r, const float *k, float *x) {
+#pragma unroll
+  for (int seg = 0; seg < 16; seg += 2 * M) {
+    float sum = 0.0f;
+#pragma unroll
+    for (int j = seg + M - 1; j >= seg; --j) {
+      x[j * WC_LD] = k[j * WC_LD] * exp_neg(sum);
+      sum += ev[j];
+    }
+    sum = 0.0f;
+#pragma unroll
+    for (int j = seg + M; j < seg + 2 * M; ++j) {
+      x[j * WC_LD] = r[j * WC_LD] * exp_neg(sum);
+      sum += ev[j];
+    }
+  }
+}
 
 __global__ void __launch_bounds__(WC_THREADS, 2) wkv_chunk_kernel(const WkvArgs a, float *__restrict__ U, float *__restrict__ decays) {
   extern __shared__ __align__(16) float sm[];
-  float *rs = sm, *ks = rs + WC_T * WC_LD, *vs = ks + WC_T * WC_LD, *ws = vs + WC_T * WC_LD, *As = ws + WC_T * WC_LD;
+  float *rs = sm, *ks = rs + WC_T * WC_LD, *vs = ks + WC_T * WC_LD, *ws = vs + WC_T * WC_LD, *xs = ws + WC_T * WC_LD, *As = xs + WC_T * WC_LD;
   float *tot = As + WC_T * WC_LD;   // [4][WC_D] sums of e per subchunk
   float *g = tot + 4 * WC_D;        // [4][WC_D] exp(-tot)
   const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, Dp = a.Dp;
@@ -208,6 +242,7 @@ __global__ void __launch_bounds__(WC_THREADS, 2) wkv_chunk_kernel(const WkvArgs 
   }
   __syncthreads();
   const int sub = tid >> 6, ch = tid & 63;   // this thread's subchunk and channel in the element-wise passes
+  const float *rc = rs + 16 * sub * WC_LD + ch, *kc = ks + 16 * sub * WC_LD + ch;
   float ev[16];
   {
     float sum = 0.0f;
@@ -215,60 +250,55 @@ __global__ void __launch_bounds__(WC_THREADS, 2) wkv_chunk_kernel(const WkvArgs 
     for (int j = 0; j < 16; ++j) {
       ev[j] = ws[(16 * sub + j) * WC_LD + ch];
       sum += ev[j];
-      ws[(16 * sub + j) * WC_LD + ch] = expf(-ev[j]);
     }
     tot[sub * WC_D + ch] = sum;
-    g[sub * WC_D + ch] = expf(-sum);
+    g[sub * WC_D + ch] = exp_neg(sum);
+    split_level<8>(ev, rc, kc, ws + 16 * sub * WC_LD + ch);   // (a thread's own elements of ws)
+    split_level<4>(ev, rc, kc, xs + 16 * sub * WC_LD + ch);
   }
   __syncthreads();
-  // ---- same subchunk: four lanes per token s, 16 channels each ----
+  // ---- same subchunk, one pair of tokens (t, s < t) per thread and level ----
   {
-    const int s = tid >> 2, qd = tid & 3, s16 = s & 15;
-    float q[16], acc = 0.0f;
-#pragma unroll
-    for (int m = 0; m < 4; ++m) {
-      const int i = 4 * (qd + 4 * m);
-      const float4 k4 = *reinterpret_cast<const float4 *>(ks + s * WC_LD + i), r4 = *reinterpret_cast<const float4 *>(rs + s * WC_LD + i);
-      float4 u4 = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (i < Dp) u4 = *reinterpret_cast<const float4 *>(a.u + (int64_t)h * Dp + i);
-      q[4 * m] = k4.x; q[4 * m + 1] = k4.y; q[4 * m + 2] = k4.z; q[4 * m + 3] = k4.w;
-      acc = fmaf(r4.x * u4.x, k4.x, fmaf(r4.y * u4.y, k4.y, fmaf(r4.z * u4.z, k4.z, fmaf(r4.w * u4.w, k4.w, acc))));
-    }
-    acc += __shfl_xor_sync(0xffffffffu, acc, 1);
-    acc += __shfl_xor_sync(0xffffffffu, acc, 2);
-    if (qd == 0) {
-      As[s * WC_LD + s] = acc;
-      for (int t = s - s16; t < s; ++t) As[t * WC_LD + s] = 0.0f;   // later tokens of the subchunk do not reach back
-    }
-    for (int dt = 1; dt < 16; ++dt) {
-      const bool on = s16 + dt < 16;
-      const int t = on ? s + dt : s;
-      acc = 0.0f;
-#pragma unroll
-      for (int m = 0; m < 4; ++m) {
-        const int i = 4 * (qd + 4 * m);
-        const float4 r4 = *reinterpret_cast<const float4 *>(rs + t * WC_LD + i), w4 = *reinterpret_cast<const float4 *>(ws + t * WC_LD + i);
-        acc = fmaf(r4.x, q[4 * m], fmaf(r4.y, q[4 * m + 1], fmaf(r4.z, q[4 * m + 2], fmaf(r4.w, q[4 * m + 3], acc))));
-        q[4 * m] *= w4.x; q[4 * m + 1] *= w4.y; q[4 * m + 2] *= w4.z; q[4 * m + 3] *= w4.w;
+    const int bl = tid >> 6, t8 = (tid >> 3) & 7, s8 = tid & 7;
+    As[(16 * bl + 8 + t8) * WC_LD + 16 * bl + s8] = dot_rows(ws + (16 * bl + 8 + t8) * WC_LD, ws + (16 * bl + s8) * WC_LD);
+    if (tid < 128) {
+      const int base = 8 * (tid >> 4), t = base + 4 + ((tid >> 2) & 3), s_ = base + (tid & 3);
+      As[t * WC_LD + s_] = dot_rows(xs + t * WC_LD, xs + s_ * WC_LD);
+    } else if (tid < 192) {   // the token itself, with the bonus
+      const int t = tid - 128;
+      float acc = 0.0f;
+#pragma unroll 4
+      for (int i = 0; i < Dp; i += 4) {
+        const float4 k4 = *reinterpret_cast<const float4 *>(ks + t * WC_LD + i), r4 = *reinterpret_cast<const float4 *>(rs + t * WC_LD + i);
+        const float4 u4 = *reinterpret_cast<const float4 *>(a.u + (int64_t)h * Dp + i);
+        acc = fmaf(r4.x * u4.x, k4.x, fmaf(r4.y * u4.y, k4.y, fmaf(r4.z * u4.z, k4.z, fmaf(r4.w * u4.w, k4.w, acc))));
       }
-      acc += __shfl_xor_sync(0xffffffffu, acc, 1);
-      acc += __shfl_xor_sync(0xffffffffu, acc, 2);
-      if (on && qd == 0) As[t * WC_LD + s] = acc;
+      As[t * WC_LD + t] = acc;
+      for (int s_ = t + 1; s_ < (t | 15) + 1; ++s_) As[t * WC_LD + s_] = 0.0f;   // later tokens of the subchunk do not reach back
+    } else if (tid < 224) {   // neighbours: nothing decays in between
+      const int s_ = 2 * (tid - 192);
+      As[(s_ + 1) * WC_LD + s_] = dot_rows(rs + (s_ + 1) * WC_LD, ks + s_ * WC_LD);
     }
   }
   __syncthreads();
+  split_level<2>(ev, rc, kc, ws + 16 * sub * WC_LD + ch);
+  __syncthreads();
+  if (tid < 64) {
+    const int base = 4 * (tid >> 2), t = base + 2 + ((tid >> 1) & 1), s_ = base + (tid & 1);
+    As[t * WC_LD + s_] = dot_rows(ws + t * WC_LD, ws + s_ * WC_LD);
+  }
   // ---- r_t exp(-P_t), k_t exp(-Q_t) ----
   {
     float sum = 0.0f;
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
-      rs[(16 * sub + j) * WC_LD + ch] *= expf(-sum);
+      rs[(16 * sub + j) * WC_LD + ch] *= exp_neg(sum);
       sum += ev[j];
     }
     sum = 0.0f;
 #pragma unroll
     for (int j = 15; j >= 0; --j) {
-      ks[(16 * sub + j) * WC_LD + ch] *= expf(-sum);
+      ks[(16 * sub + j) * WC_LD + ch] *= exp_neg(sum);
       sum += ev[j];
     }
   }
@@ -387,17 +417,17 @@ __global__ void __launch_bounds__(256) wkv_states_kernel(const WkvArgs a, float 
   float4 *st = reinterpret_cast<float4 *>(a.state + (bh * Dp + key) * Dp + v4);
   const bool in = key < Dp && v4 < Dp;
   float4 S = in && a.n > 0 ? *st : make_float4(0.f, 0.f, 0.f, 0.f);
-  for (int c0 = 0; c0 < chunks; c0 += 4) {
-    float4 uc[4];
-    float wc[4];
+  for (int c0 = 0; c0 < chunks; c0 += 8) {
+    float4 uc[8];
+    float wc[8];
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
+    for (int j = 0; j < 8; ++j)
       if (c0 + j < chunks) {
         uc[j] = u[(int64_t)(c0 + j) * (WC_D * WC_D / 4)];
         wc[j] = w[(int64_t)(c0 + j) * WC_D];
       }
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
+    for (int j = 0; j < 8; ++j)
       if (c0 + j < chunks) {
         u[(int64_t)(c0 + j) * (WC_D * WC_D / 4)] = S;
         S.x = fmaf(wc[j], S.x, uc[j].x); S.y = fmaf(wc[j], S.y, uc[j].y); S.z = fmaf(wc[j], S.z, uc[j].z); S.w = fmaf(wc[j], S.w, uc[j].w);
@@ -545,7 +575,7 @@ int launch_wkv_scan(caten_b200_ctx *ctx, const WkvArgs &a) {
 // ---------------------------------------------------------------------------------------------
 constexpr int WD_THREADS = 256, WD_U = 4;
 
-__global__ void __launch_bounds__(WD_THREADS) wkv_decode_kernel(const WkvArgs a) {
+__global__ void __launch_bounds__(WD_THREADS, 4) wkv_decode_kernel(const WkvArgs a) {
   extern __shared__ __align__(16) float sm[];
   const int Dp = a.Dp, h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   float *r = sm, *k = r + Dp, *v = k + Dp, *w = v + Dp, *g = w + Dp, *t = g + Dp, *red = t + a.w1, *part = red + 8;
@@ -553,17 +583,26 @@ __global__ void __launch_bounds__(WD_THREADS) wkv_decode_kernel(const WkvArgs a)
   const int vq = tid % d4, kr = tid / d4;
   const bool on = kr < RP;
   float4 *st = reinterpret_cast<float4 *>(a.state + ((int64_t)b * a.H + h) * Dp * Dp);
+  // parameters first (they depend on no other kernel): this thread's share of the decay's second projection, when two
+  // passes of one 16-byte piece cover it
+  const bool ahead = a.w1 == 64 && Dp <= WD_THREADS / 4;
+  uint4 wq[2];
+#pragma unroll
+  for (int p = 0; p < 2; ++p) {
+    const int c = (tid >> 3) + WD_THREADS / 8 * p;
+    wq[p] = ahead && c < Dp ? *reinterpret_cast<const uint4 *>(a.w2 + ((int64_t)h * Dp + c) * 64 + (tid & 7) * 8) : make_uint4(0u, 0u, 0u, 0u);
+  }
   pdl_enter();
-  const bool fresh = (a.d_n ? *a.d_n : a.n) == 0;
   float4 s[WD_U];
   auto load = [&](int base) {
 #pragma unroll
     for (int i = 0; i < WD_U; ++i) {
       const int key = base + kr + RP * i;
-      s[i] = on && key < Dp && !fresh ? st[(int64_t)key * d4 + vq] : make_float4(0.f, 0.f, 0.f, 0.f);
+      s[i] = on && key < Dp ? __ldcs(st + (int64_t)key * d4 + vq) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   };
-  load(0);
+  load(0);   // (discarded at position 0; waiting for the position first would put its latency before the state's)
+  const bool fresh = (a.d_n ? *a.d_n : a.n) == 0;
   auto proj = [&](int col) { return a.pin.splits > 0 ? partin_load1(a.pin, b, col) : a.y[(int64_t)b * a.ld + col]; };
   for (int i = tid; i < 4 * Dp; i += WD_THREADS) {
     const int which = i / Dp, c = i - which * Dp;
@@ -572,18 +611,23 @@ __global__ void __launch_bounds__(WD_THREADS) wkv_decode_kernel(const WkvArgs a)
   for (int j = tid; j < a.w1; j += WD_THREADS) t[j] = tanhf(proj(4 * a.gr + j));
   __syncthreads();
   // decay: eight lanes per channel, each 8 weights (16 bytes) at a time
-  for (int c = tid >> 3; c < Dp; c += WD_THREADS / 8) {
+  auto dot8 = [&](uint4 q, int j) {
+    const uint32_t qq[4] = {q.x, q.y, q.z, q.w};
+    float x = 0.0f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      x = fmaf(__uint_as_float(qq[e] << 16), t[j + 2 * e], x);
+      x = fmaf(__uint_as_float(qq[e] & 0xFFFF0000u), t[j + 2 * e + 1], x);
+    }
+    return x;
+  };
+  int pass = 0;
+  for (int c = tid >> 3; c < Dp; c += WD_THREADS / 8, ++pass) {
     const __nv_bfloat16 *wr = a.w2 + ((int64_t)h * Dp + c) * a.w1;
     float x = 0.0f;
-    for (int j = (tid & 7) * 8; j < a.w1; j += 64) {
-      const uint4 q = *reinterpret_cast<const uint4 *>(wr + j);
-      const uint32_t qq[4] = {q.x, q.y, q.z, q.w};
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        x = fmaf(__uint_as_float(qq[e] << 16), t[j + 2 * e], x);
-        x = fmaf(__uint_as_float(qq[e] & 0xFFFF0000u), t[j + 2 * e + 1], x);
-      }
-    }
+    if (ahead) x = dot8(pass ? wq[1] : wq[0], (tid & 7) * 8);
+    else
+      for (int j = (tid & 7) * 8; j < a.w1; j += 64) x += dot8(*reinterpret_cast<const uint4 *>(wr + j), j);
     x += __shfl_xor_sync(0xffffffffu, x, 4);
     x += __shfl_xor_sync(0xffffffffu, x, 2);
     x += __shfl_xor_sync(0xffffffffu, x, 1);
@@ -604,6 +648,7 @@ __global__ void __launch_bounds__(WD_THREADS) wkv_decode_kernel(const WkvArgs a)
 #pragma unroll
     for (int i = 0; i < WD_U; ++i) {
       const int key = base + kr + RP * i;
+      if (fresh) s[i] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (on && key < Dp) {
         const float rk = r[key], kk = k[key], wk = w[key];
         o.x = fmaf(rk, s[i].x, o.x); o.y = fmaf(rk, s[i].y, o.y); o.z = fmaf(rk, s[i].z, o.z); o.w = fmaf(rk, s[i].w, o.w);
