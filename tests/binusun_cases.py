@@ -10,7 +10,7 @@ SCALING = {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 256}
 # single key/value heads, windows from one token up, loops at the start, in the middle, over everything and none
 CASES = {
     "attention": (S.binusun_config(96, 131, "A", 80, 4, 2, 32, 32, 9, 1, 16, 32, scale=0.4), 8),
-    "wkv": (S.binusun_config(64, 100, "w", 64, 1, 1, 16, 16, 4, 2, 24, 16), 5),
+    "wkv": (S.binusun_config(64, 100, "w", 64, 1, 1, 16, 16, 4, 2, 24, 16), 200),
     "mixed": (S.binusun_config(160, 203, "wAaW", 96, 6, 2, 40, 24, 21, 3, 16, 12, rot_base=500.0, scaling=SCALING, loop=(1, 3, 2), logit_scale=1.5), 11),
     "loop_all": (S.binusun_config(72, 97, "Aw", 40, 3, 3, 20, 48, 33, 2, 40, 20, loop=(0, 2, 3), eps=1e-3), 16),
     "loop_once": (S.binusun_config(256, 64, "aWA", 192, 8, 1, 64, 64, 70, 2, 64, 64, scaling=SCALING, loop=(2, 3, 1), logit_scale=0.5), 70),
