@@ -35,6 +35,38 @@ __device__ __forceinline__ void rotate_pairs(HeadPairs &h, const float *__restri
     }
   }
 }
+// A head of row m whose linear left split-K partial tiles: every pair's partial values are requested together, two
+// splits at a time, and added in split order.
+__device__ __forceinline__ void load_pairs_pending(HeadPairs &h, const PartIn &pin, int m, int off, int np, int lane) {
+  const float *src[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int o = off + 2 * (lane + 32 * j);
+    const long long tile = (long long)(m / pin.bnx) * pin.tiles_x + (o >> 7);
+    src[j] = pin.part + (tile * pin.bnx + m % pin.bnx) * 128 + (o & 127);
+    h.p[j] = make_float2(0.f, 0.f);
+  }
+  for (int z = 0; z < pin.splits; z += 2) {
+    float2 t[2][4];
+#pragma unroll
+    for (int u = 0; u < 2; ++u)
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (lane + 32 * j < np && z + u < pin.splits) t[u][j] = __ldcs(reinterpret_cast<const float2 *>(src[j] + (long long)(z + u) * pin.zstride));
+#pragma unroll
+    for (int u = 0; u < 2; ++u)
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (lane + 32 * j < np && z + u < pin.splits) { h.p[j].x += t[u][j].x; h.p[j].y += t[u][j].y; }
+  }
+  if (pin.bias)
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (lane + 32 * j < np) {
+        h.p[j].x += pin.bias[off + 2 * (lane + 32 * j)];
+        h.p[j].y += pin.bias[off + 2 * (lane + 32 * j) + 1];
+      }
+}
 __device__ __forceinline__ float pairs_inv_rms(const HeadPairs &h, int D, float eps) {
   float ss = 0.0f;
 #pragma unroll
@@ -252,7 +284,7 @@ int launch_attn_window_prefill(caten_b200_ctx *ctx, const AttnArgs &a, int tenso
 // Every mbarrier wait is bounded; when one runs out the CTA records it in the status word, leaves its
 // loops, waits for its copies in flight, takes part in the cluster barriers and writes no output.
 // ---------------------------------------------------------------------------------------------
-constexpr int AD_WORK = 256, AD_THREADS = AD_WORK + 32, AD_STAGES = 3;
+constexpr int AD_WORK = 256, AD_THREADS = AD_WORK + 32, AD_MIN_STAGES = 3, AD_MAX_STAGES = 8;
 
 __device__ __forceinline__ void work_sync() { asm volatile("bar.sync 1, %0;" ::"n"(AD_WORK) : "memory"); }
 __device__ __forceinline__ void bulk_load(uint32_t dst, const void *src, uint32_t bytes, uint32_t bar) {
@@ -285,7 +317,7 @@ template <int KL, int NV> struct AdShape {
 };
 
 template <int KL, int NV, int HPC>
-__global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const AttnArgs a, const int S, const int per_max, const long long hint_bytes,
+__global__ void __launch_bounds__(AD_THREADS, NV == 1 ? 3 : 1) attn_window_decode_kernel(const AttnArgs a, const int S, const int stages, const int per_max, const long long hint_bytes,
                                                                         int *status) {
   constexpr int GROUPS = AdShape<KL, NV>::GROUPS, U = AdShape<KL, NV>::U, CH = AdShape<KL, NV>::CH;
   constexpr int R = U * HPC;                    // dot products reduced together (<= KL)
@@ -293,20 +325,20 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
   constexpr int TPH = AD_WORK / HPC;            // threads per head in the softmax
   extern __shared__ __align__(16) float sm[];
   const int Dp = a.Dp, Ep = a.Ep, wide = Dp > Ep ? Dp : Ep;
-  float *ring = sm;                             // [AD_STAGES][CH][wide]; afterwards the row groups' outputs [GROUPS][HPC][Ep]
-  float *q = ring + AD_STAGES * CH * wide;      // [HPC][Dp]
+  float *ring = sm;                             // [stages][CH][wide]; afterwards the row groups' outputs [GROUPS][HPC][Ep]
+  float *q = ring + stages * CH * wide;      // [HPC][Dp]
   float *kn = q + HPC * Dp;                     // the step's key
   float *vn = kn + Dp;                          // and value
   float *gate = vn + Ep;                        // [4]
   float *ml = gate + 4;                         // [HPC] max, [HPC] sum (read by the other CTAs of the cluster): 8
   float *red = ml + 8;                          // 8
   float *ol = red + 8;                          // [HPC][Ep] this CTA's output
-  uint64_t *bars = reinterpret_cast<uint64_t *>(ol + HPC * Ep);  // full [AD_STAGES], empty [AD_STAGES]
-  volatile int *abort_flag = reinterpret_cast<volatile int *>(bars + 2 * AD_STAGES);  // [0] a wait ran out; [1] never set; 4 words
-  float *sc = reinterpret_cast<float *>(bars + 2 * AD_STAGES + 2);  // [per_max][HPC]
+  uint64_t *bars = reinterpret_cast<uint64_t *>(ol + HPC * Ep);  // full, empty: [AD_MAX_STAGES] each
+  volatile int *abort_flag = reinterpret_cast<volatile int *>(bars + 2 * AD_MAX_STAGES);  // [0] a wait ran out; [1] never set; 4 words
+  float *sc = reinterpret_cast<float *>(bars + 2 * AD_MAX_STAGES + 2);  // [per_max][HPC]
   const uint32_t bar0 = smem_u32(bars);
   auto full = [&](int s) { return bar0 + 8u * s; };
-  auto empty = [&](int s) { return bar0 + 8u * (AD_STAGES + s); };
+  auto empty = [&](int s) { return bar0 + 8u * (AD_MAX_STAGES + s); };
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int h0 = blockIdx.x * HPC, b = blockIdx.y, rank = blockIdx.z;
   const int rep = a.H / a.G, g = h0 / rep, cap = (int)a.cap;
@@ -320,7 +352,7 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
     je = t0 + min((rank + 1) * per, count);
   };
   if (tid == 0) {
-    for (int s = 0; s < AD_STAGES; ++s) {
+    for (int s = 0; s < stages; ++s) {
       mbar_init(full(s), 1);
       mbar_init(empty(s), AD_WORK / 32);
     }
@@ -353,10 +385,10 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
 
   if (warp == AD_WORK / 32) {
     if (lane == 0) {
-      int issued = 0;
+      int issued = 0, s = 0;
+      uint32_t ph = 1;   // (a fresh barrier's previous phase counts as complete)
       for (int i = 0; i < 2 * nc; ++i) {
-        const int s = i % AD_STAGES;
-        if (i >= AD_STAGES && !mbar_wait(empty(s), (uint32_t)(i / AD_STAGES - 1) & 1u, abort_flag)) {
+        if (!mbar_wait(empty(s), ph, abort_flag)) {
           if (!*abort_flag) { *abort_flag = 1; atomicCAS(status, 0, DEV_WAIT_TIMEOUT); status[1] = 20; }
           break;
         }
@@ -369,9 +401,10 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
         bulk_load(dst, base + (int64_t)s0 * w, (uint32_t)(r0 * w) * 4u, full(s));
         if (r0 < rows) bulk_load(dst + (uint32_t)(r0 * w) * 4u, base, (uint32_t)((rows - r0) * w) * 4u, full(s));
         issued = i + 1;
+        if (++s == stages) { s = 0; ph ^= 1u; }
       }
       if (*abort_flag)  // copies in flight land before the CTA's shared memory is released
-        for (int i = issued > AD_STAGES ? issued - AD_STAGES : 0; i < issued; ++i) mbar_wait(full(i % AD_STAGES), (uint32_t)(i / AD_STAGES) & 1u, abort_flag + 1);
+        for (int i = issued > stages ? issued - stages : 0; i < issued; ++i) mbar_wait(full(i % stages), (uint32_t)(i / stages) & 1u, abort_flag + 1);
     }
     __syncwarp();
   } else {
@@ -380,13 +413,13 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
       const int64_t off = is_q ? a.q_off + (int64_t)(h0 + warp) * Dp : is_k ? a.k_off + (int64_t)g * Dp : a.v_off + (int64_t)g * Ep;
       const int np = (is_q || is_k ? Dp : Ep) / 2;
       HeadPairs h;
+      if (a.pin.splits > 0) {
+        load_pairs_pending(h, a.pin, b, (int)off, np, lane);
+      } else {
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int i = lane + 32 * j;
-        h.p[j] = make_float2(0.f, 0.f);
-        if (i < np) {
-          if (a.pin.splits > 0) h.p[j] = make_float2(partin_load1(a.pin, b, (int)off + 2 * i), partin_load1(a.pin, b, (int)off + 2 * i + 1));
-          else h.p[j] = reinterpret_cast<const float2 *>(a.qkv + (int64_t)b * a.ld + off)[i];
+        for (int j = 0; j < 4; ++j) {
+          const int i = lane + 32 * j;
+          h.p[j] = i < np ? reinterpret_cast<const float2 *>(a.qkv + (int64_t)b * a.ld + off)[i] : make_float2(0.f, 0.f);
         }
       }
       float mul = 1.0f;
@@ -420,6 +453,8 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
       if (lane == 0) sc[hist * HPC + warp] = x;
     }
     bool ok = true;
+    int s = 0;           // stage and phase of the chunk being consumed
+    uint32_t ph = 0;
     {
       float4 q4[HPC][NV];
 #pragma unroll
@@ -430,8 +465,7 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
           q4[h][v] = 4 * c < Dp ? reinterpret_cast<const float4 *>(q + h * Dp)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
         }
       for (int i = 0; i < nc && ok; ++i) {
-        const int s = i % AD_STAGES;
-        ok = __all_sync(0xffffffffu, mbar_wait(full(s), (uint32_t)(i / AD_STAGES) & 1u, abort_flag));
+        ok = __all_sync(0xffffffffu, mbar_wait(full(s), ph, abort_flag));
         if (!ok) break;
         const float *st = ring + s * CH * wide;
         float d[R];
@@ -454,6 +488,7 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
         }
         __syncwarp();
         if (lane == 0) mbar_arrive(empty(s));
+        if (++s == stages) { s = 0; ph ^= 1u; }
         const float x = group_reduce<R>(d, gl, KL);
         if (gl % (KL / R) == 0) {
           const int idx = gl / (KL / R), row = i * CH + (idx / HPC) * GROUPS + gi;
@@ -503,8 +538,7 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
         acc[h][v] = make_float4(p * x.x, p * x.y, p * x.z, p * x.w);
       }
     for (int i = nc; i < 2 * nc && ok; ++i) {
-      const int s = i % AD_STAGES;
-      ok = __all_sync(0xffffffffu, mbar_wait(full(s), (uint32_t)(i / AD_STAGES) & 1u, abort_flag));
+      ok = __all_sync(0xffffffffu, mbar_wait(full(s), ph, abort_flag));
       if (!ok) break;
       const float *st = ring + s * CH * wide;
 #pragma unroll
@@ -532,6 +566,7 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
       }
       __syncwarp();
       if (lane == 0) mbar_arrive(empty(s));
+      if (++s == stages) { s = 0; ph ^= 1u; }
     }
     if (!ok && lane == 0 && !*abort_flag) { *abort_flag = 1; atomicCAS(status, 0, DEV_WAIT_TIMEOUT); status[1] = 22; }
     work_sync();  // every chunk has been consumed: the ring becomes the exchange buffer of the row groups
@@ -612,7 +647,7 @@ __global__ void __launch_bounds__(AD_THREADS) attn_window_decode_kernel(const At
 }
 
 template <int KL, int NV, int HPC>
-static int launch_decode_t(caten_b200_ctx *ctx, const AttnArgs &a, int S, int per_max, size_t smem) {
+static int launch_decode_t(caten_b200_ctx *ctx, const AttnArgs &a, int S, int stages, int per_max, size_t smem) {
   if (smem > 48 * 1024) CB_CUDA(ctx, cudaFuncSetAttribute(attn_window_decode_kernel<KL, NV, HPC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3((unsigned)(a.H / HPC), (unsigned)a.B, (unsigned)S);
@@ -635,7 +670,7 @@ static int launch_decode_t(caten_b200_ctx *ctx, const AttnArgs &a, int S, int pe
   }
   cfg.attrs = at;
   cfg.numAttrs = na;
-  CB_CUDA(ctx, cudaLaunchKernelEx(&cfg, attn_window_decode_kernel<KL, NV, HPC>, a, S, per_max, ctx->attn_prefetch_bytes, ctx->d_status));
+  CB_CUDA(ctx, cudaLaunchKernelEx(&cfg, attn_window_decode_kernel<KL, NV, HPC>, a, S, stages, per_max, ctx->attn_prefetch_bytes, ctx->d_status));
   CB_LAUNCH_CHECK(ctx, "attn_window_decode_kernel");
   return 0;
 }
@@ -656,6 +691,8 @@ int launch_attn_window_decode(caten_b200_ctx *ctx, const AttnArgs &a) {
   auto ctas = [&](int h, int s) { return (int64_t)a.B * (a.H / h) * s; };
   int S = 1;
   while (S < 8 && ctas(hpc, S) < ctx->sm_count && keys / (2 * S) >= 32) S *= 2;
+  // a little more than one wave (3 CTAs per SM): halves even out the second
+  if (S == 1 && ctas(hpc, 1) > 3 * ctx->sm_count && ctas(hpc, 1) < 6 * ctx->sm_count && keys >= 256) S = 2;
   while (hpc > 1 && ctas(hpc, S) * 2 <= ctx->sm_count) hpc /= 2;
   const int kl = wide <= 64 ? 16 : 32, nv = wide <= 128 ? 1 : 2;
   const int ch = AD_WORK / kl * (nv == 2 ? 2 : 4);
@@ -664,16 +701,23 @@ int launch_attn_window_decode(caten_b200_ctx *ctx, const AttnArgs &a) {
   for (;;) {
     per_max = (keys + S - 1) / S;
     // (the row groups' outputs, hpc / 4 of [ch][4][Ep] / U floats, fit the ring they reuse)
-    smem = ((size_t)AD_STAGES * ch * wide + (size_t)hpc * a.Dp + a.Dp + a.Ep + 20 + (size_t)hpc * a.Ep + (size_t)hpc * per_max) * sizeof(float) +
-           (2 * AD_STAGES + 2) * 8;
+    smem = ((size_t)AD_MIN_STAGES * ch * wide + (size_t)hpc * a.Dp + a.Dp + a.Ep + 20 + (size_t)hpc * a.Ep + (size_t)hpc * per_max) * sizeof(float) +
+           (2 * AD_MAX_STAGES + 2) * 8;
     if (smem <= 200 * 1024) break;
     if (S < 8) S *= 2;
     else if (hpc > 1) hpc /= 2;
     else return fail(ctx, CATEN_B200_EUNSUPPORTED, "attention: context too long for the decode kernel");
   }
+  // a small grid leaves shared memory for a deeper ring: at most as many stages as there are chunks, and about 200 KB per SM
+  int stages = AD_MIN_STAGES;
+  // (a large cluster is placed inside one group of SMs: its CTAs share SMs even when the grid alone would not need to)
+  const size_t stage = (size_t)ch * wide * sizeof(float);
+  size_t per_sm = (size_t)((ctas(hpc, S) + ctx->sm_count - 1) / ctx->sm_count);
+  if (S >= 4 && per_sm < 2) per_sm = 2;
+  while (stages < AD_MAX_STAGES && stages < 2 * ((per_max + ch - 1) / ch) && (smem + stage) * per_sm <= 200 * 1024) { ++stages; smem += stage; }
 #define AD_CASE(KL, NV)                                                                                    \
-  (hpc == 4 ? launch_decode_t<KL, NV, 4>(ctx, a, S, (int)per_max, smem)                                    \
-   : hpc == 2 ? launch_decode_t<KL, NV, 2>(ctx, a, S, (int)per_max, smem) : launch_decode_t<KL, NV, 1>(ctx, a, S, (int)per_max, smem))
+  (hpc == 4 ? launch_decode_t<KL, NV, 4>(ctx, a, S, stages, (int)per_max, smem)                                    \
+   : hpc == 2 ? launch_decode_t<KL, NV, 2>(ctx, a, S, stages, (int)per_max, smem) : launch_decode_t<KL, NV, 1>(ctx, a, S, stages, (int)per_max, smem))
   if (kl == 16) return AD_CASE(16, 1);
   if (nv == 1) return AD_CASE(32, 1);
   return AD_CASE(32, 2);

@@ -573,9 +573,10 @@ int launch_wkv_scan(caten_b200_ctx *ctx, const WkvArgs &a) {
 // Single-token step: one CTA per (head, sequence) reads and writes the head's state once.  The first
 // state rows are requested before the decay is formed.
 // ---------------------------------------------------------------------------------------------
-constexpr int WD_THREADS = 256, WD_U = 4;
+constexpr int WD_THREADS = 128, WD_U = 8, WD_P = 4;   // WD_P: passes over the channels of a 64-wide head
 
-__global__ void __launch_bounds__(WD_THREADS, 4) wkv_decode_kernel(const WkvArgs a) {
+
+__global__ void __launch_bounds__(WD_THREADS, 6) wkv_decode_kernel(const WkvArgs a) {
   extern __shared__ __align__(16) float sm[];
   const int Dp = a.Dp, h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   float *r = sm, *k = r + Dp, *v = k + Dp, *w = v + Dp, *g = w + Dp, *t = g + Dp, *red = t + a.w1, *part = red + 8;
@@ -583,12 +584,12 @@ __global__ void __launch_bounds__(WD_THREADS, 4) wkv_decode_kernel(const WkvArgs
   const int vq = tid % d4, kr = tid / d4;
   const bool on = kr < RP;
   float4 *st = reinterpret_cast<float4 *>(a.state + ((int64_t)b * a.H + h) * Dp * Dp);
-  // parameters first (they depend on no other kernel): this thread's share of the decay's second projection, when two
+  // parameters first (they depend on no other kernel): this thread's share of the decay's second projection, when a few
   // passes of one 16-byte piece cover it
-  const bool ahead = a.w1 == 64 && Dp <= WD_THREADS / 4;
-  uint4 wq[2];
+  const bool ahead = a.w1 == 64 && Dp <= WD_THREADS / 8 * WD_P;
+  uint4 wq[WD_P];
 #pragma unroll
-  for (int p = 0; p < 2; ++p) {
+  for (int p = 0; p < WD_P; ++p) {
     const int c = (tid >> 3) + WD_THREADS / 8 * p;
     wq[p] = ahead && c < Dp ? *reinterpret_cast<const uint4 *>(a.w2 + ((int64_t)h * Dp + c) * 64 + (tid & 7) * 8) : make_uint4(0u, 0u, 0u, 0u);
   }
@@ -603,12 +604,16 @@ __global__ void __launch_bounds__(WD_THREADS, 4) wkv_decode_kernel(const WkvArgs
   };
   load(0);   // (discarded at position 0; waiting for the position first would put its latency before the state's)
   const bool fresh = (a.d_n ? *a.d_n : a.n) == 0;
-  auto proj = [&](int col) { return a.pin.splits > 0 ? partin_load1(a.pin, b, col) : a.y[(int64_t)b * a.ld + col]; };
-  for (int i = tid; i < 4 * Dp; i += WD_THREADS) {
-    const int which = i / Dp, c = i - which * Dp;
-    (which == 0 ? r : which == 1 ? k : which == 2 ? v : g)[c] = proj(which * a.gr + h * Dp + c);
+  // r, k, v, gate of this head and the low-rank input, four values per thread and request
+  const int items = 4 * d4 + a.w1 / 4;
+  for (int i = tid; i < items; i += WD_THREADS) {
+    const bool lr = i >= 4 * d4;
+    const int which = i / d4, c = lr ? 4 * (i - 4 * d4) : 4 * (i - which * d4);
+    const int col = lr ? 4 * a.gr + c : which * a.gr + h * Dp + c;
+    float4 p = a.pin.splits > 0 ? partin_load4(a.pin, b, col) : *reinterpret_cast<const float4 *>(a.y + (int64_t)b * a.ld + col);
+    if (lr) p = make_float4(tanhf(p.x), tanhf(p.y), tanhf(p.z), tanhf(p.w));
+    *reinterpret_cast<float4 *>((lr ? t : which == 0 ? r : which == 1 ? k : which == 2 ? v : g) + c) = p;
   }
-  for (int j = tid; j < a.w1; j += WD_THREADS) t[j] = tanhf(proj(4 * a.gr + j));
   __syncthreads();
   // decay: eight lanes per channel, each 8 weights (16 bytes) at a time
   auto dot8 = [&](uint4 q, int j) {
@@ -621,17 +626,25 @@ __global__ void __launch_bounds__(WD_THREADS, 4) wkv_decode_kernel(const WkvArgs
     }
     return x;
   };
-  int pass = 0;
-  for (int c = tid >> 3; c < Dp; c += WD_THREADS / 8, ++pass) {
-    const __nv_bfloat16 *wr = a.w2 + ((int64_t)h * Dp + c) * a.w1;
-    float x = 0.0f;
-    if (ahead) x = dot8(pass ? wq[1] : wq[0], (tid & 7) * 8);
-    else
-      for (int j = (tid & 7) * 8; j < a.w1; j += 64) x += dot8(*reinterpret_cast<const uint4 *>(wr + j), j);
+  auto channel = [&](int c, float x) {
     x += __shfl_xor_sync(0xffffffffu, x, 4);
     x += __shfl_xor_sync(0xffffffffu, x, 2);
     x += __shfl_xor_sync(0xffffffffu, x, 1);
     if ((tid & 7) == 0) w[c] = decay(x + a.w0[(int64_t)h * Dp + c]);
+  };
+  if (ahead) {
+#pragma unroll
+    for (int p = 0; p < WD_P; ++p) {
+      const int c = (tid >> 3) + WD_THREADS / 8 * p;
+      if (c < Dp) channel(c, dot8(wq[p], (tid & 7) * 8));   // (whole warps: Dp is a multiple of 4)
+    }
+  } else {
+    for (int c = tid >> 3; c < Dp; c += WD_THREADS / 8) {
+      const __nv_bfloat16 *wr = a.w2 + ((int64_t)h * Dp + c) * a.w1;
+      float x = 0.0f;
+      for (int j = (tid & 7) * 8; j < a.w1; j += 64) x += dot8(*reinterpret_cast<const uint4 *>(wr + j), j);
+      channel(c, x);
+    }
   }
   float x = 0.0f;
   for (int i = tid; i < Dp; i += WD_THREADS) x = fmaf(r[i] * a.u[(int64_t)h * Dp + i], k[i], x);
@@ -658,20 +671,29 @@ __global__ void __launch_bounds__(WD_THREADS, 4) wkv_decode_kernel(const WkvArgs
   }
   if (on) reinterpret_cast<float4 *>(part + kr * Dp)[vq] = o;
   __syncthreads();
-  float ov = 0.0f;
-  if (tid < Dp) {
-    for (int i = 0; i < RP; ++i) ov += part[i * Dp + tid];
-    ov = fmaf(v[tid], ruk, ov);
+  constexpr int OC = 256 / WD_THREADS;   // output columns per thread at the widest head
+  float ov[OC], ss = 0.0f;
+#pragma unroll
+  for (int p = 0; p < OC; ++p) {
+    const int c = tid + WD_THREADS * p;
+    ov[p] = 0.0f;
+    if (c < Dp) {
+      for (int i = 0; i < RP; ++i) ov[p] += part[i * Dp + c];
+      ov[p] = fmaf(v[c], ruk, ov[p]);
+    }
+    ss += ov[p] * ov[p];
   }
-  float ss = warp_sum(ov * ov);  // threads past the head hold zero
+  ss = warp_sum(ss);
   if (lane == 0) red[warp] = ss;
   __syncthreads();
   ss = red[0];
 #pragma unroll
   for (int i = 1; i < WD_THREADS / 32; ++i) ss += red[i];
-  if (tid < Dp) {
-    const float inv = 1.0f / sqrtf(ss / (float)a.D + a.eps);
-    st_out(a.out, a.bf, (int64_t)b * a.out_ld + (int64_t)h * Dp + tid, ov * inv * a.norm[(int64_t)h * Dp + tid] * silu(g[tid]));
+  const float inv = 1.0f / sqrtf(ss / (float)a.D + a.eps);
+#pragma unroll
+  for (int p = 0; p < OC; ++p) {
+    const int c = tid + WD_THREADS * p;
+    if (c < Dp) st_out(a.out, a.bf, (int64_t)b * a.out_ld + (int64_t)h * Dp + c, ov[p] * inv * a.norm[(int64_t)h * Dp + c] * silu(g[c]));
   }
 }
 
