@@ -1,7 +1,7 @@
 // Prefill attention (s > 1) on the 5th-generation tensor cores over an fp32 KV cache, for head sizes up
 // to 128 (NQ / NE = 64-wide blocks of the query/key / value head), grouped query heads, an optional
 // sliding window and a ring-buffered cache (attn_window.cuh).  GPT-2 (head dim 64, a cache
-// [B, H, T, 64] that never wraps, no window) is the case NQ = NE = 1.  Same semantics as the SIMT kernels in attention.cu
+// [B, H, T, 64] that never wraps, no window) is the PLAIN case of NQ = NE = 1.  Same semantics as the SIMT kernels in attention.cu
 // (external/llm/layers.lisp:3-5,19-51: S = (q.K^T) * 0.125 + causal mask; P = softmax(S) with
 // exp(x) = exp2(x * 1/ln2), two passes: row maximum first, then exp and sum; O = P.V), with both
 // contractions as bf16 hi/lo split products accumulated in fp32 (every operand x = x_hi + x_lo;
@@ -103,7 +103,9 @@ __device__ __forceinline__ float4 scale4(float4 v, float c) { return make_float4
 
 }  // namespace
 
-template <int NQ, int NE>
+// PLAIN: heads of exactly 64, no window, a cache that never wraps (GPT-2): the masks' lower ends, the ring arithmetic and
+// the zero-filled head columns compile away.
+template <int NQ, int NE, bool PLAIN>
 __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_kernel(const AttnArgs p, float qscale, int *status, uint32_t idesc_n64) {
   using Lay = AtLayout<NQ, NE>;
   constexpr uint32_t AT_OFF_Q = Lay::OFF_Q, AT_OFF_K = Lay::OFF_K, AT_OFF_V = Lay::OFF_V, AT_OFF_SK = Lay::OFF_SK, AT_OFF_SV = Lay::OFF_SV, AT_OFF_MISC = Lay::OFF_MISC;
@@ -138,12 +140,13 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
   const uint32_t tlane = tmem_base + ((uint32_t)(quad * 32) << 16);
   pdl_enter();
 
-  const int64_t head = (int64_t)b * p.G + h / (p.H / p.G);  // the key/value head this query head reads
-  const float *kb = p.kc + head * p.cap * p.Dp;
-  const float *vb = p.vc + head * p.cap * p.Ep;
-  const int W = p.window > 0 ? p.window : 0x3fffffff;
+  const int Dp = PLAIN ? 64 : p.Dp, Ep = PLAIN ? 64 : p.Ep;
+  const int64_t head = (int64_t)b * p.G + (PLAIN ? h : h / (p.H / p.G));  // the key/value head this query head reads
+  const float *kb = p.kc + head * p.cap * Dp;
+  const float *vb = p.vc + head * p.cap * Ep;
+  const int W = !PLAIN && p.window > 0 ? p.window : 0x3fffffff;
   const int kend = min(t, n + q0 + AT_Q);  // keys beyond the last query of this tile are masked
-  const int kfirst = n + q0 - W + 1;       // first key the tile's first query sees
+  const int kfirst = PLAIN ? 0 : n + q0 - W + 1;       // first key the tile's first query sees
   const int kbeg = kfirst > 0 ? kfirst / AT_K * AT_K : 0;
   const int nblk = (kend - kbeg + AT_K - 1) / AT_K;
   const int qi = min(q0 + r, s - 1);  // rows past the end of the step mask like the last row (their output is dropped)
@@ -152,7 +155,7 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
 
   const uint64_t dq = umma_desc(smem_u32(sm + AT_OFF_Q)), dk = umma_desc(smem_u32(sm + AT_OFF_K)), dv = umma_desc(smem_u32(sm + AT_OFF_V));
   const uint32_t idesc_pv = idesc_n64 | (1u << 16);  // B operand MN-major: V rows (keys) with the dims contiguous
-  const int ksteps = p.Dp / 16;
+  const int ksteps = Dp / 16;
   uint32_t ph = 0;
   int ok = 1;
 
@@ -160,13 +163,13 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
   // the end of the context and columns past the head are zero-filled
   auto prefetch = [&](const float *base, int j0, uint32_t stage_off, auto nb, int width) {
     constexpr int NB = decltype(nb)::value;
-    const int slot0 = (int)(j0 % p.cap);
+    const int slot0 = PLAIN ? j0 : (int)(j0 % p.cap);
 #pragma unroll
     for (int i = 0; i < 4 * NB; ++i) {
       const int piece = tid + 256 * i, row = piece / (16 * NB), c16 = piece % (16 * NB);
-      const bool okk = j0 + row < t && c16 * 4 < width;
+      const bool okk = j0 + row < t && (PLAIN || c16 * 4 < width);
       int slot = slot0 + row;
-      if (slot >= (int)p.cap) slot -= (int)p.cap;
+      if (!PLAIN && slot >= (int)p.cap) slot -= (int)p.cap;
       cp_async16(smem_u32(sm + stage_off + row * (NB * 256 + 16) + c16 * 16), base + (okk ? (int64_t)slot * width + c16 * 4 : 0), okk ? 16u : 0u);
     }
   };
@@ -186,20 +189,20 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
     ok = __syncthreads_and(ok);
   };
 
-  prefetch(kb, kbeg, AT_OFF_SK, IntC<NQ>(), p.Dp);
-  prefetch(vb, kbeg, AT_OFF_SV, IntC<NE>(), p.Ep);
+  prefetch(kb, kbeg, AT_OFF_SK, IntC<NQ>(), Dp);
+  prefetch(vb, kbeg, AT_OFF_SV, IntC<NE>(), Ep);
   cp_async_commit();
   // Q tiles: rows [0,128) hi, [128,256) lo per block; GPT-2's 1/8 score scale is folded in (a power of two: exact)
   {
     const bool okq = q0 + r < s;
-    const float4 *src = reinterpret_cast<const float4 *>(p.qkv + ((int64_t)b * s + (okq ? q0 + r : 0)) * p.ld + p.q_off + (int64_t)h * p.Dp);
+    const float4 *src = reinterpret_cast<const float4 *>(p.qkv + ((int64_t)b * s + (okq ? q0 + r : 0)) * p.ld + p.q_off + (int64_t)h * Dp);
 #pragma unroll
     for (int kb_ = 0; kb_ < NQ; ++kb_) {
       float4 v[8];
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const int c4 = 16 * kb_ + 8 * hf + i;
-        v[i] = okq && 4 * c4 < p.Dp ? scale4(src[c4], qscale) : make_float4(0.f, 0.f, 0.f, 0.f);
+        v[i] = okq && (PLAIN || 4 * c4 < Dp) ? scale4(src[c4], qscale) : make_float4(0.f, 0.f, 0.f, 0.f);
       }
 #pragma unroll
       for (int c = 0; c < 4; ++c) st_split8(sm + AT_OFF_Q + kb_ * 32768, r, 128 + r, 4 * hf + c, v[2 * c], v[2 * c + 1]);
@@ -278,8 +281,8 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
     }
     // the next step's rows start to arrive while the MMAs run (issued after them: the MMAs are the critical path)
     if (blk + 1 < nblk) {
-      prefetch(kb, j0 + AT_K, AT_OFF_SK, IntC<NQ>(), p.Dp);
-      prefetch(vb, j0 + AT_K, AT_OFF_SV, IntC<NE>(), p.Ep);
+      prefetch(kb, j0 + AT_K, AT_OFF_SK, IntC<NQ>(), Dp);
+      prefetch(vb, j0 + AT_K, AT_OFF_SV, IntC<NE>(), Ep);
       cp_async_commit();
     }
     wait_mma();
@@ -295,7 +298,7 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
       float mloc = -INFINITY;
 #pragma unroll
       for (int e = 0; e < 32; ++e)
-        if (e <= lim && e >= low) mloc = fmaxf(mloc, __uint_as_float(a[e]));
+        if (e <= lim && (PLAIN || e >= low)) mloc = fmaxf(mloc, __uint_as_float(a[e]));
       red[hf * 128 + r] = mloc;
       __syncthreads();
       const float mstep = fmaxf(red[r], red[128 + r]);
@@ -328,7 +331,7 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
 #pragma unroll
         for (int e = 0; e < 16; ++e) {
           const float val = __uint_as_float(a[16 * c + e]);
-          pr[e] = (16 * c + e <= lim && 16 * c + e >= low) ? ex2_approx((val - m) * kAtInvLn2) : 0.0f;
+          pr[e] = (16 * c + e <= lim && (PLAIN || 16 * c + e >= low)) ? ex2_approx((val - m) * kAtInvLn2) : 0.0f;
           lsum += pr[e];
         }
         uint32_t phi[8], plo[8];
@@ -375,7 +378,7 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
   if (ok) {
     float inv = 1.0f / (red[r] + red[128 + r]);
     const int64_t orow = (int64_t)b * s + q0 + r;
-    if (p.gate_off >= 0 && q0 + r < s) inv *= 1.0f / (1.0f + expf(-p.qkv[orow * p.ld + p.gate_off + h]));
+    if (!PLAIN && p.gate_off >= 0 && q0 + r < s) inv *= 1.0f / (1.0f + expf(-p.qkv[orow * p.ld + p.gate_off + h]));
 #pragma unroll
     for (int w = 0; w < NE; ++w) {
       uint32_t a[32];
@@ -387,10 +390,10 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
       for (int e = 0; e < 32; ++e) o[e] = __uint_as_float(a[e]) * inv;
       if (q0 + r < s) {
         const int c0 = 64 * w + 32 * hf;
-        const int64_t at = orow * p.out_ld + (int64_t)h * p.Ep + c0;
+        const int64_t at = orow * p.out_ld + (int64_t)h * Ep + c0;
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          if (c0 + 8 * i >= p.Ep) continue;
+          if (!PLAIN && c0 + 8 * i >= Ep) continue;
           const float *v = o + 8 * i;
           if (p.bf.hi) {
             *reinterpret_cast<uint4 *>(p.bf.hi + at + 8 * i) =
@@ -418,13 +421,13 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
   }
 }
 
-template <int NQ, int NE>
+template <int NQ, int NE, bool PLAIN = false>
 static int launch_at(caten_b200_ctx *ctx, const AttnArgs &a, float qscale) {
   const uint32_t base = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(AT_Q >> 4) << 24);  // fp32 accumulate, bf16 x bf16, M = 128
   const uint32_t idesc_n64 = base | ((uint32_t)(64 >> 3) << 17);
   constexpr size_t smem = AtLayout<NQ, NE>::SMEM;
-  CB_CUDA(ctx, cudaFuncSetAttribute(attn_prefill_tc_kernel<NQ, NE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  launch_k(ctx, attn_prefill_tc_kernel<NQ, NE>, dim3((unsigned)((a.s + AT_Q - 1) / AT_Q), (unsigned)a.H, (unsigned)a.B), dim3(256), smem, a, qscale,
+  CB_CUDA(ctx, cudaFuncSetAttribute(attn_prefill_tc_kernel<NQ, NE, PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  launch_k(ctx, attn_prefill_tc_kernel<NQ, NE, PLAIN>, dim3((unsigned)((a.s + AT_Q - 1) / AT_Q), (unsigned)a.H, (unsigned)a.B), dim3(256), smem, a, qscale,
            ctx->d_status, idesc_n64);
   CB_LAUNCH_CHECK(ctx, "attn_prefill_tc_kernel");
   return 0;
@@ -450,7 +453,7 @@ int launch_attention_tc(caten_b200_ctx *ctx, const float *qkv, const float *kc, 
   a.out = out; a.bf = bf; a.out_ld = H * 64;
   a.B = (int)B; a.s = (int)s; a.n = (int)n; a.H = a.G = (int)H;
   a.D = a.Dp = a.E = a.Ep = 64;
-  return launch_attention_tc_ex(ctx, a, 0.125f);
+  return launch_at<1, 1, true>(ctx, a, 0.125f);
 }
 
 }  // namespace cb
