@@ -19,7 +19,7 @@ BF16 = 30
 Q4_1, Q5_0, Q5_1 = 3, 6, 7                                # kept packed, like Q4_0 and Q8_0
 Q2_K, Q3_K, Q4_K, Q5_K, Q6_K = 10, 11, 12, 13, 14        # expanded to fp32 at upload
 BLOCK_FORMATS = (Q4_0, Q8_0, Q4_1, Q5_0, Q5_1, Q2_K, Q3_K, Q4_K, Q5_K, Q6_K)
-ACT_NONE, ACT_GELU, ACT_RELU, ACT_RELU_GLU = 0, 1, 2, 3
+ACT_NONE, ACT_GELU, ACT_RELU, ACT_RELU_GLU, ACT_SILU_GLU = 0, 1, 2, 3, 4
 PREC_FP32, PREC_BF16, PREC_BF16X3 = 0, 1, 2
 K_EMBED, K_LAYERNORM, K_GEMV, K_GEMM, K_ATTN_DECODE, K_ATTN_PREFILL, K_ARGMAX, K_COUNT = 0, 1, 2, 3, 4, 5, 6, 10
 KERNEL_CLASSES = ["embed", "layernorm", "gemv", "gemm", "attn_decode", "attn_prefill", "argmax", "decode_step", "wkv", "prep"]
@@ -51,7 +51,7 @@ class GPT2Desc(C.Structure):
     ]
 
 
-MIX_ATTENTION, MIX_WKV = 0, 1
+MIX_ATTENTION, MIX_WKV, MIX_LATENT, MIX_RETENTION = 0, 1, 2, 3
 
 
 class AttnDesc(C.Structure):
@@ -71,14 +71,16 @@ class LayerDesc(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "kv_heads", "vdim", "window", "rot_dims", "qk_norm", "gated")] + [
         ("scale", C.c_float), ("group_rows", C.c_int32), ("low_rank", C.c_int32),
         ("norm1", C.c_float), ("norm1b", C.c_float), ("norm2", C.c_float), ("norm2b", C.c_float)] + [
-        (n, _vp) for n in ("rot_freq", "mu", "w0", "u", "norm", "in_w", "out_w", "w2", "ff_in", "ff_out")]
+        (n, _vp) for n in ("rot_freq", "mu", "w0", "u", "norm", "in_w", "out_w", "w2", "ff_in", "ff_out")] + [
+        (n, C.c_int32) for n in ("kv_rank", "q_rank", "parallel", "ff_act", "experts", "top")] + [
+        (n, _vp) for n in ("norm1_w", "norm2_w", "q_norm", "kv_norm", "powers", "uq_w", "uk_w", "kv_w", "router")]
 
 
 class DecoderDesc(C.Structure):
     """Mirror of ``caten_b200_decoder_desc``."""
     _fields_ = [(n, C.c_int32) for n in ("n_layers", "width", "vocab", "max_seq_len", "batch", "precision", "max_rows", "max_portion",
                                          "loop_start", "loop_stop", "loop_times")] + [
-        ("eps", C.c_float), ("final_gain", C.c_float), ("embed", _vp), ("head", _vp), ("loop_in", _vp), ("layers", C.POINTER(LayerDesc))]
+        ("eps", C.c_float), ("final_gain", C.c_float), ("embed", _vp), ("head", _vp), ("loop_in", _vp), ("loop_step", _vp), ("final_norm", _vp), ("layers", C.POINTER(LayerDesc))]
 
 
 EXPR_MAX_DIMS, EXPR_MAX_OPERANDS, EXPR_MAX_CODE, EXPR_MAX_CONSTS = 6, 8, 96, 16

@@ -23,7 +23,7 @@ INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 OBJ_DIR = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libcaten_b200.so")
 SOURCES = ["capi.cu", "decode_small.cu", "kernels_misc.cu", "gemv.cu", "gemm_simt.cu", "gemm_tc.cu", "gemm_dense.cu", "attention.cu", "attention_tc.cu", "gguf.cu", "expr.cu", "dequant_extra.cu", "sample.cu", "dist.cu", "llama_ops.cu",
-           "stream_norm.cu", "attn_window.cu", "wkv.cu", "decoder.cu"]
+           "stream_norm.cu", "attn_window.cu", "wkv.cu", "latent.cu", "retention.cu", "moe.cu", "decoder.cu"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-fmad=false", "-Xcompiler", "-fPIC", "-Xptxas", "-v"]
 

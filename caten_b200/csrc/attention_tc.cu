@@ -142,8 +142,10 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
 
   const int Dp = PLAIN ? 64 : p.Dp, Ep = PLAIN ? 64 : p.Ep;
   const int64_t head = (int64_t)b * p.G + (PLAIN ? h : h / (p.H / p.G));  // the key/value head this query head reads
-  const float *kb = p.kc + head * p.cap * Dp;
-  const float *vb = p.vc + head * p.cap * Ep;
+  const int64_t kv_head = head - (int64_t)b * p.G;
+  const float *kb = PLAIN ? p.kc + head * p.cap * 64 : p.kc + b * p.k_seq + kv_head * p.k_head;
+  const float *vb = PLAIN ? p.vc + head * p.cap * 64 : p.vc + b * p.v_seq + kv_head * p.v_head;
+  const float *kx = !PLAIN && p.kx ? p.kx + b * p.cap * p.kx_ld - p.kx_from : nullptr;   // column c of the key, c >= kx_from
   const int W = !PLAIN && p.window > 0 ? p.window : 0x3fffffff;
   const int kend = min(t, n + q0 + AT_Q);  // keys beyond the last query of this tile are masked
   const int kfirst = PLAIN ? 0 : n + q0 - W + 1;       // first key the tile's first query sees
@@ -161,7 +163,7 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
 
   // copy the 64 rows [j0, j0+64) of one head's K or V history into a staging buffer; rows past
   // the end of the context and columns past the head are zero-filled
-  auto prefetch = [&](const float *base, int j0, uint32_t stage_off, auto nb, int width) {
+  auto prefetch = [&](const float *base, int64_t ld, int j0, uint32_t stage_off, auto nb, int width, bool key) {
     constexpr int NB = decltype(nb)::value;
     const int slot0 = PLAIN ? j0 : (int)(j0 % p.cap);
 #pragma unroll
@@ -170,7 +172,9 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
       const bool okk = j0 + row < t && (PLAIN || c16 * 4 < width);
       int slot = slot0 + row;
       if (!PLAIN && slot >= (int)p.cap) slot -= (int)p.cap;
-      cp_async16(smem_u32(sm + stage_off + row * (NB * 256 + 16) + c16 * 16), base + (okk ? (int64_t)slot * width + c16 * 4 : 0), okk ? 16u : 0u);
+      const float *src = base + (okk ? (int64_t)slot * (PLAIN ? 64 : ld) + c16 * 4 : 0);
+      if (!PLAIN && key && okk && c16 * 4 >= p.kx_from) src = kx + (int64_t)slot * p.kx_ld + c16 * 4;
+      cp_async16(smem_u32(sm + stage_off + row * (NB * 256 + 16) + c16 * 16), src, okk ? 16u : 0u);
     }
   };
   auto staged_row = [&](uint32_t row_off, int block, float4 *v) {  // this thread's 16 dims of its key row
@@ -189,8 +193,8 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
     ok = __syncthreads_and(ok);
   };
 
-  prefetch(kb, kbeg, AT_OFF_SK, IntC<NQ>(), Dp);
-  prefetch(vb, kbeg, AT_OFF_SV, IntC<NE>(), Ep);
+  prefetch(kb, p.k_ld, kbeg, AT_OFF_SK, IntC<NQ>(), Dp, true);
+  prefetch(vb, p.v_ld, kbeg, AT_OFF_SV, IntC<NE>(), Ep, false);
   cp_async_commit();
   // Q tiles: rows [0,128) hi, [128,256) lo per block; GPT-2's 1/8 score scale is folded in (a power of two: exact)
   {
@@ -281,8 +285,8 @@ __global__ void __launch_bounds__(256, AtLayout<NQ, NE>::CTAS) attn_prefill_tc_k
     }
     // the next step's rows start to arrive while the MMAs run (issued after them: the MMAs are the critical path)
     if (blk + 1 < nblk) {
-      prefetch(kb, j0 + AT_K, AT_OFF_SK, IntC<NQ>(), Dp);
-      prefetch(vb, j0 + AT_K, AT_OFF_SV, IntC<NE>(), Ep);
+      prefetch(kb, p.k_ld, j0 + AT_K, AT_OFF_SK, IntC<NQ>(), Dp, true);
+      prefetch(vb, p.v_ld, j0 + AT_K, AT_OFF_SV, IntC<NE>(), Ep, false);
       cp_async_commit();
     }
     wait_mma();
@@ -433,7 +437,9 @@ static int launch_at(caten_b200_ctx *ctx, const AttnArgs &a, float qscale) {
   return 0;
 }
 
-int launch_attention_tc_ex(caten_b200_ctx *ctx, const AttnArgs &a, float qscale) {
+int launch_attention_tc_ex(caten_b200_ctx *ctx, const AttnArgs &args, float qscale) {
+  AttnArgs a = args;
+  a.fill_strides();
   if (a.Dp > 128 || a.Ep > 128) return fail(ctx, CATEN_B200_EUNSUPPORTED, "attention_tc: head size above 128");
   const bool wq = a.Dp > 64, we = a.Ep > 64;
   if (wq && we) return launch_at<2, 2>(ctx, a, qscale);

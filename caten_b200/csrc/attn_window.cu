@@ -139,8 +139,9 @@ __global__ void __launch_bounds__(256) attn_window_simt_kernel(const AttnArgs a)
   const int q0 = blockIdx.x * AW_T, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
   const int tx = tid & 15, ty = tid >> 4;
   const int g = h / (a.H / a.G), t = a.n + a.s;
-  const float *kb = a.kc + ((int64_t)b * a.G + g) * a.cap * a.Dp;
-  const float *vb = a.vc + ((int64_t)b * a.G + g) * a.cap * a.Ep;
+  const float *kb = a.kc + b * a.k_seq + g * a.k_head;
+  const float *vb = a.vc + b * a.v_seq + g * a.v_head;
+  const float *kx = a.kx + (a.kx ? b * a.cap * a.kx_ld : 0);
   const int d4 = a.Dp / 4, e4 = a.Ep / 4;
   for (int e = tid; e < AW_T * d4; e += 256) {
     const int i = e / d4, c = e % d4;
@@ -162,13 +163,15 @@ __global__ void __launch_bounds__(256) attn_window_simt_kernel(const AttnArgs a)
     __syncthreads();
     for (int e = tid; e < AW_T * d4; e += 256) {
       const int i = e / d4, c = e % d4;
+      const int64_t slot = (j0 + i) % a.cap;
       *reinterpret_cast<float4 *>(Ks + i * ldk + 4 * c) =
-          j0 + i < t ? reinterpret_cast<const float4 *>(kb + (int64_t)((j0 + i) % a.cap) * a.Dp)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+          j0 + i >= t ? make_float4(0.f, 0.f, 0.f, 0.f)
+                      : *reinterpret_cast<const float4 *>(4 * c < a.kx_from ? kb + slot * a.k_ld + 4 * c : kx + slot * a.kx_ld + 4 * c - a.kx_from);
     }
     for (int e = tid; e < AW_T * e4; e += 256) {
       const int i = e / e4, c = e % e4;
       *reinterpret_cast<float4 *>(Vs + i * ldv + 4 * c) =
-          j0 + i < t ? reinterpret_cast<const float4 *>(vb + (int64_t)((j0 + i) % a.cap) * a.Ep)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+          j0 + i < t ? reinterpret_cast<const float4 *>(vb + (int64_t)((j0 + i) % a.cap) * a.v_ld)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     __syncthreads();
     float sc[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
@@ -254,7 +257,9 @@ static int check_attn(caten_b200_ctx *ctx, const AttnArgs &a) {
   return 0;
 }
 
-int launch_attn_window_prefill(caten_b200_ctx *ctx, const AttnArgs &a, int tensor_cores) {
+int launch_attn_window_prefill(caten_b200_ctx *ctx, const AttnArgs &args, int tensor_cores) {
+  AttnArgs a = args;
+  a.fill_strides();
   if (a.B <= 0 || a.s <= 0) return 0;
   if (int rc = check_attn(ctx, a)) return rc;
   // every key the step's queries may see is still in the ring

@@ -14,6 +14,12 @@ struct AttnArgs {
   // caches [B, G, cap, Dp] and [B, G, cap, Ep]; position p lives in slot p % cap
   float *kc = nullptr, *vc = nullptr;
   int64_t cap = 0;
+  // multi-token steps may find keys and values elsewhere: floats between positions, key/value heads and sequences (ld 0: the
+  // caches as above), and the key's columns from kx_from on in rows kx [B, cap, kx_ld] common to the heads
+  int64_t k_ld = 0, k_head = 0, k_seq = 0, v_ld = 0, v_head = 0, v_seq = 0;
+  const float *kx = nullptr;
+  int64_t kx_ld = 0;
+  int kx_from = 0;
   float *out = nullptr;             // [B * s, out_ld], head h at column h * Ep: fp32, or
   BfOut bf;                         // bf16
   int64_t out_ld = 0;
@@ -26,6 +32,12 @@ struct AttnArgs {
   const float *freq = nullptr;
   int qk_norm = 0;                  // q and k divided by their root mean square over D after the rotation
   float eps = 0.0f, scale = 1.0f;   // score = q . k * scale
+
+  void fill_strides() {
+    if (k_ld == 0) { k_ld = Dp; k_head = cap * Dp; k_seq = G * k_head; }
+    if (v_ld == 0) { v_ld = Ep; v_head = cap * Ep; v_seq = G * v_head; }
+    if (!kx) kx_from = Dp;
+  }
 };
 
 // Rotation and q/k norm of a multi-token step: q in place (times scale), k and v into the cache.

@@ -137,7 +137,7 @@ int caten_b200_destroy(caten_b200_ctx *ctx) {
   if (ctx->wtmp.ptr) cudaFree(ctx->wtmp.ptr);
   if (ctx->wbf.ptr) cudaFree(ctx->wbf.ptr);
   if (ctx->wkv_tmp.ptr) cudaFree(ctx->wkv_tmp.ptr);
-  if (ctx->wkv_chunks.ptr) cudaFree(ctx->wkv_chunks.ptr);
+  if (ctx->chunk_states.ptr) cudaFree(ctx->chunk_states.ptr);
   if (ctx->upload_stage.ptr) cudaFree(ctx->upload_stage.ptr);
   for (int k = 0; k < 2; ++k) {
     if (ctx->pin[k]) cudaFreeHost(ctx->pin[k]);
@@ -373,7 +373,7 @@ int caten_b200_weight_dequant(caten_b200_ctx *ctx, const caten_b200_weight *w, f
 // ------------------------------------------------------------------------------------------------
 static bool aligned16(const void *p) { return ((uintptr_t)p & 15) == 0; }
 static int check_glu(caten_b200_ctx *ctx, const char *who, const caten_b200_weight *w, int act, const void *residual) {
-  if (act != CATEN_B200_ACT_RELU_GLU) return 0;
+  if (!act_is_glu(act)) return 0;
   if (residual || w->rows % 2 || (w->type != CATEN_B200_F32 && w->type != CATEN_B200_F16 && w->type != CATEN_B200_BF16))
     return fail(ctx, CATEN_B200_EUNSUPPORTED, "%s: the gated activation takes a dense weight with an even number of rows and no residual", who);
   return 0;
@@ -385,9 +385,9 @@ int caten_b200_linear(caten_b200_ctx *ctx, const caten_b200_weight *w, const flo
   if (!w || !d_x || !d_y) return fail(ctx, CATEN_B200_EINVAL, "linear: NULL argument");
   if (M < 0) return fail(ctx, CATEN_B200_EINVAL, "linear: M < 0");
   if (M == 0) return 0;
-  if (act < 0 || act > CATEN_B200_ACT_RELU_GLU) return fail(ctx, CATEN_B200_EINVAL, "linear: unknown activation %d", act);
+  if (act < 0 || act > CATEN_B200_ACT_SILU_GLU) return fail(ctx, CATEN_B200_EINVAL, "linear: unknown activation %d", act);
   if (int rc = check_glu(ctx, "linear", w, act, d_residual)) return rc;
-  const int64_t ny = act == CATEN_B200_ACT_RELU_GLU ? w->rows / 2 : w->rows;
+  const int64_t ny = act_is_glu(act) ? w->rows / 2 : w->rows;
   if (!aligned16(d_x) || !aligned16(d_y)) return fail(ctx, CATEN_B200_EINVAL, "linear: x and y must be 16-byte aligned");
   ProfScope prof(ctx, M <= 4 ? CATEN_B200_K_GEMV : CATEN_B200_K_GEMM);
   if (M <= 4) {
@@ -411,9 +411,9 @@ int caten_b200_linear_noalloc(caten_b200_ctx *ctx, const caten_b200_weight *w, c
   if (!w || !d_x || !d_y) return fail(ctx, CATEN_B200_EINVAL, "linear_noalloc: NULL argument");
   if (M < 0) return fail(ctx, CATEN_B200_EINVAL, "linear_noalloc: M < 0");
   if (M == 0) return 0;
-  if (act < 0 || act > CATEN_B200_ACT_RELU_GLU) return fail(ctx, CATEN_B200_EINVAL, "linear_noalloc: unknown activation %d", act);
+  if (act < 0 || act > CATEN_B200_ACT_SILU_GLU) return fail(ctx, CATEN_B200_EINVAL, "linear_noalloc: unknown activation %d", act);
   if (int rc = check_glu(ctx, "linear_noalloc", w, act, d_residual)) return rc;
-  const int64_t ny = act == CATEN_B200_ACT_RELU_GLU ? w->rows / 2 : w->rows;
+  const int64_t ny = act_is_glu(act) ? w->rows / 2 : w->rows;
   if (!aligned16(d_x) || !aligned16(d_y)) return fail(ctx, CATEN_B200_EINVAL, "linear_noalloc: x and y must be 16-byte aligned");
   ProfScope prof(ctx, M <= 4 ? CATEN_B200_K_GEMV : CATEN_B200_K_GEMM);
   if (M <= 4) {  // the dequant-GEMV uses no scratch memory
@@ -517,7 +517,8 @@ int model_linear(caten_b200_ctx *ctx, int prec, const caten_b200_weight *w, cons
   if (defer) *defer = PartIn();
   if (M <= 0) return 0;
   if (int rc = check_glu(ctx, "linear", w, act, res)) return rc;
-  const int64_t ny = act == CATEN_B200_ACT_RELU_GLU ? w->rows / 2 : w->rows;
+  const int64_t ny = grp.ldy ? grp.ldy : act_is_glu(act) ? w->rows / 2 : w->rows;
+  if (res && !grp.plain_output()) return fail(ctx, CATEN_B200_EUNSUPPORTED, "linear: a residual needs the plain output layout");
   ProfScope prof(ctx, M <= 4 ? CATEN_B200_K_GEMV : CATEN_B200_K_GEMM);
   if (M <= 4) {
     for (int64_t m = 0; m < M; ++m)

@@ -80,9 +80,22 @@ __device__ __forceinline__ float partin_load1(const PartIn &p, long long m, int 
 
 // How a linear's input is laid out when groups of its output rows read different inputs: output rows
 // [g * group_rows, (g + 1) * group_rows) are multiplied with input plane g, which starts g * xplane rows after
-// plane 0 (same row stride).  group_rows = 0: one input.  group_rows is a multiple of 128.
+// plane 0 (same row stride).  group_rows = 0: one input.  group_rows is a multiple of 4.  And where the output goes:
+// rows of ldy columns (0: the outputs side by side, nothing between rows), group g's from column g * ygroup on (0:
+// group_rows).  A layout of its own is written by the linear itself, never left as partial tiles.
 struct LinGroups {
-  int64_t group_rows = 0, xplane = 0;
+  int64_t group_rows = 0, xplane = 0, ygroup = 0, ldy = 0;
+  bool plain_output() const { return ygroup == 0 && ldy == 0; }
+};
+
+// Mixture of experts: rows of the activations sorted by expert.  Expert e owns the sorted rows [offsets[e],
+// offsets[e + 1]) (device memory) and the weight's rows [e * rows / experts, (e + 1) * rows / experts).
+struct ExpertRows {
+  int experts = 0, top = 0;
+  int64_t pairs = 0;             // (token, expert) pairs = tokens * top
+  const int *offsets = nullptr;  // [experts + 1]
+  const int *src = nullptr;      // [pairs] token of a sorted row
+  const float *weight = nullptr; // [pairs] factor of a sorted row's products (NULL: 1), before the activation
 };
 
 struct Scratch {
@@ -103,7 +116,7 @@ struct caten_b200_ctx {
   cb::Scratch xbf;           // bf16 copy (hi, lo) of the activation operand of the tensor-core GEMM
   cb::Scratch wtmp;          // split-K partial tiles of the tensor-core GEMM
   cb::Scratch wbf;           // bf16 copy (hi, lo) of the weight operand of the many-row GEMM
-  cb::Scratch wkv_chunks;    // per-chunk states of a time-mixing prompt
+  cb::Scratch chunk_states;    // per-chunk states of a recurrent layer's prompt
   cb::Scratch wkv_tmp;       // intermediates of a stand-alone time-mixing call
   cb::Scratch upload_stage;  // raw blocks of the weight being uploaded, before their re-layout
   void *pin[2] = {nullptr, nullptr};          // pinned bounce buffers for large copies from pageable host memory
@@ -216,6 +229,15 @@ int launch_relu_matmul_simt(caten_b200_ctx *ctx, const float *a, const float *b,
 int launch_relu_matmul_tc(caten_b200_ctx *ctx, const float *a, const float *b, float *c, int64_t M, int64_t K,
                           int64_t N, int nsplit);
 
+// Linears of a mixture of experts (the rows of x belong to different experts):
+//   up to 4 tokens   pair p = token * top + choice, one row each: expert[p], input row p / xdiv, factor weight[p] (or NULL)
+int launch_gemv_experts(caten_b200_ctx *ctx, const caten_b200_weight *w, int64_t rows, const float *x, const int *expert, const float *weight,
+                        int64_t pairs, int xdiv, int act, float *y);
+//   fp32             sorted row r reads x row src[r] (src NULL: r)
+int launch_gemm_simt_experts(caten_b200_ctx *ctx, const caten_b200_weight *w, const ExpertRows &er, const float *x, const int *src, int act, float *y);
+//   tensor cores     x sorted, in bf16 (gemm_dense.cu); BF16 weights
+int launch_gemm_experts(caten_b200_ctx *ctx, const caten_b200_weight *w, const ExpertRows &er, BfOut x, int act, float *y, BfOut ybf, int nsplit);
+
 // where a weight operand lives
 struct WSrc {
   const void *qs;
@@ -313,8 +335,12 @@ __device__ __forceinline__ float gelu_ref(float x) {
   return l * r;
 }
 
-// the gated activation of CATEN_B200_ACT_RELU_GLU
-__device__ __forceinline__ float relu_glu(float gate, float up) { return (gate > 0.0f ? gate : 0.0f) * up; }
+__host__ __device__ constexpr bool act_is_glu(int act) { return act == CATEN_B200_ACT_RELU_GLU || act == CATEN_B200_ACT_SILU_GLU; }
+__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+// the gated activations
+__device__ __forceinline__ float glu(int act, float gate, float up) {
+  return (act == CATEN_B200_ACT_SILU_GLU ? silu(gate) : (gate > 0.0f ? gate : 0.0f)) * up;
+}
 
 __device__ __forceinline__ float apply_act(float v, int act) {
   if (act == CATEN_B200_ACT_GELU) return gelu_ref(v);

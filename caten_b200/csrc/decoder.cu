@@ -1,6 +1,8 @@
 // Decoders described layer by layer (caten_b200_decoder_desc): the layer loop, caches and states, and
 // the step entry points.  The kernels are those of the other models where they exist (linears,
-// arg-max, device-resident step loop) plus stream_norm.cu, attn_window.cu / attention_tc.cu and wkv.cu.
+// arg-max, device-resident step loop) plus stream_norm.cu, attn_window.cu / attention_tc.cu, latent.cu, wkv.cu,
+// retention.cu and moe.cu.
+#include <math.h>
 #include <stdlib.h>
 #include <string.h>
 
@@ -8,6 +10,9 @@
 #include <vector>
 
 #include "attn_window.cuh"
+#include "latent.cuh"
+#include "moe.cuh"
+#include "retention.cuh"
 #include "step_loop.cuh"
 #include "stream_norm.cuh"
 #include "wkv.cuh"
@@ -19,12 +24,17 @@ namespace {
 int64_t p16(int64_t n) { return (n + 15) / 16 * 16; }
 int64_t p64(int64_t n) { return (n + 63) / 64 * 64; }
 
+// A latent layer takes portions of up to this many tokens per sequence in the absorbed form (latent.cu)
+constexpr int LATENT_ABSORB = 4;
+
 struct Run {            // one execution of a layer in a step
   int layer = 0;
-  bool pass_start = false;   // loop_in comes right before it
+  bool pass_start = false;   // a pass of the loop starts right before it
+  int pass = 0;              // which one
   float *kc = nullptr, *vc = nullptr;        // attention: ring caches [B, G, cap, Dp / Ep]
   int64_t cap = 0;
-  float *state = nullptr, *shift = nullptr;  // time mixing: [B, H, Dp, Dp] and [B, wp]
+  float *state = nullptr, *shift = nullptr;  // time mixing: [B, H, Dp, Dp] and [B, wp]; retention: [B, H, Dp, Ep]
+  uint8_t *latents = nullptr;                // latent attention: [B, cap, p16(kv_rank) + p16(rot_dims)], bf16 or fp32
 };
 
 }  // namespace
@@ -44,6 +54,19 @@ struct caten_b200_decoder {
   float *tl = nullptr;    // fp32 operand of w2
   int64_t hp_rows = 0;    // fp32 operands feed the GEMV (up to 4 rows) and the exact GEMM
   BfOut hp_bf, act_bf, tl_bf, last_bf;
+  // latent attention
+  std::vector<caten_b200_weight> uv;   // per layer: the value rows of kv_w
+  int64_t abs_rows = 0, kv_rows = 0, part_floats = 0;
+  float *cq = nullptr, *q = nullptr;                        // query latent, queries
+  float *qn = nullptr, *qcat = nullptr, *olat = nullptr;    // absorbed form: [H][abs_rows][p64(dim)], [abs_rows, H, KC], [H][abs_rows][Kr]
+  float *part = nullptr, *ml = nullptr;                     // its key splits
+  float *lat = nullptr, *kr = nullptr, *kvx = nullptr;      // expanded form: latents, key parts, keys and values of kv_rows cached rows
+  BfOut cq_bf, qn_bf, qcat_bf, olat_bf, lat_bf;
+  float *ret_o = nullptr;                                   // retention: raw outputs of heads with values wider than 256
+  // mixture of experts
+  int *ex_id = nullptr, *ex_off = nullptr, *ex_src = nullptr, *ex_pos = nullptr;
+  float *ex_w = nullptr, *ex_ws = nullptr, *ea = nullptr, *ye = nullptr;   // ea: experts' activations; ye: their outputs [pairs, wp]
+  BfOut xs_bf, ea_bf;                                       // rows sorted by expert
   float *last = nullptr, *logits = nullptr;
   int *d_rows = nullptr;
   int64_t *ids = nullptr, *h_ids = nullptr, *h_out = nullptr;
@@ -71,9 +94,13 @@ static int dec_bf(Dec *m, BfOut *b, int64_t n) {
 
 static bool shape_is(const caten_b200_weight *w, int64_t rows, int64_t cols) { return w && w->rows == rows && w->cols == cols; }
 
+static bool bf16_is(const caten_b200_weight *w, int64_t rows, int64_t cols) { return shape_is(w, rows, cols) && w->type == CATEN_B200_BF16; }
+// columns of a layer's out_w that the mixer fills
+static int64_t mixer_cols(const caten_b200_layer_desc &c) { return p64(c.heads * p16(c.mixer == CATEN_B200_MIX_WKV ? c.dim : c.vdim)); }
+
 static int check_layer(caten_b200_ctx *ctx, int l, const caten_b200_layer_desc &c, int64_t wp) {
   const int64_t Dp = p16(c.dim);
-  if (c.heads <= 0 || c.dim <= 0 || c.dim > 256) return fail(ctx, CATEN_B200_EUNSUPPORTED, "decoder: layer %d: %d heads of %d (sizes 1..256)", l, c.heads, c.dim);
+  if (c.heads <= 0 || c.dim <= 0 || c.dim > (c.mixer == CATEN_B200_MIX_RETENTION ? 512 : 256)) return fail(ctx, CATEN_B200_EUNSUPPORTED, "decoder: layer %d: %d heads of %d (sizes 1..256)", l, c.heads, c.dim);
   int64_t out_cols = 0;
   if (c.mixer == CATEN_B200_MIX_ATTENTION) {
     if (c.kv_heads <= 0 || c.heads % c.kv_heads || c.vdim <= 0 || c.vdim > 256 || c.window < 0 || c.rot_dims < 0 || c.rot_dims % 2 || c.rot_dims > c.dim || (c.rot_dims && !c.rot_freq))
@@ -87,13 +114,51 @@ static int check_layer(caten_b200_ctx *ctx, int l, const caten_b200_layer_desc &
     if (!shape_is(c.in_w, 4ll * c.group_rows + c.low_rank, wp) || !shape_is(c.w2, p64(c.heads * Dp), c.low_rank) || c.w2->type != CATEN_B200_BF16)
       return fail(ctx, CATEN_B200_EINVAL, "decoder: layer %d: in_w or w2 has the wrong shape or type", l);
     out_cols = p64(c.heads * Dp);
+  } else if (c.mixer == CATEN_B200_MIX_LATENT) {
+    const int64_t Pp = p16(c.rot_dims), Ep = p16(c.vdim), H = c.heads;
+    if (c.vdim <= 0 || c.vdim > 256 || Dp + Pp > 256 || c.rot_dims < 0 || c.rot_dims % 2 || (c.rot_dims && !c.rot_freq) || c.kv_rank <= 0 || c.kv_rank > 1024 || c.q_rank <= 0 || c.q_rank > 8192 || !c.q_norm || !c.kv_norm)
+      return fail(ctx, CATEN_B200_EUNSUPPORTED, "decoder: layer %d: latent attention with heads of %d + %d / %d, latents of %d and %d", l, c.dim, c.rot_dims, c.vdim, c.q_rank, c.kv_rank);
+    if (!shape_is(c.in_w, p64(p64(c.q_rank) + p16(c.kv_rank) + Pp), wp) || !shape_is(c.uq_w, H * (Dp + Pp), p64(c.q_rank)) || !bf16_is(c.uk_w, H * p16(c.kv_rank), p64(c.dim)) ||
+        !bf16_is(c.kv_w, H * (Dp + Ep), p64(c.kv_rank)))
+      return fail(ctx, CATEN_B200_EINVAL, "decoder: layer %d: a latent attention weight has the wrong shape or type", l);
+    out_cols = p64(H * Ep);
+  } else if (c.mixer == CATEN_B200_MIX_RETENTION) {
+    if (c.vdim <= 0 || c.vdim > 1024 || c.rot_dims < 0 || c.rot_dims % 2 || c.rot_dims > c.dim || (c.rot_dims && !c.rot_freq) || !c.powers)
+      return fail(ctx, CATEN_B200_EUNSUPPORTED, "decoder: layer %d: retention with heads of %d x %d", l, c.dim, c.vdim);
+    if (!shape_is(c.in_w, p64(2ll * c.heads * (Dp + p16(c.vdim))), wp)) return fail(ctx, CATEN_B200_EINVAL, "decoder: layer %d: in_w has the wrong shape", l);
+    out_cols = p64(c.heads * p16(c.vdim));
   } else {
     return fail(ctx, CATEN_B200_EUNSUPPORTED, "decoder: layer %d: unknown mixer %d", l, c.mixer);
   }
+  if (c.parallel) {
+    if (c.mixer == CATEN_B200_MIX_WKV || !c.norm1_w || (c.ff_in && !c.norm2_w)) return fail(ctx, CATEN_B200_EUNSUPPORTED, "decoder: layer %d: no parallel form", l);
+    if (c.ff_in && !act_is_glu(c.ff_act)) return fail(ctx, CATEN_B200_EINVAL, "decoder: layer %d: unknown activation %d", l, c.ff_act);
+    const int64_t E = c.experts;
+    if (E > 0) {
+      if (E > 1024 || c.top < 1 || c.top > E || !bf16_is(c.router, p64(E), wp) || !c.ff_in || c.ff_in->rows % (128 * E) || !bf16_is(c.ff_in, c.ff_in->rows, wp) ||
+          !bf16_is(c.ff_out, E * wp, c.ff_in->rows / E / 2))
+        return fail(ctx, CATEN_B200_EINVAL, "decoder: layer %d: the experts' weights do not fit each other", l);
+    } else if (c.ff_in) {
+      if (c.ff_in->cols != wp || c.ff_in->rows % 128 || c.ff_out) return fail(ctx, CATEN_B200_EINVAL, "decoder: layer %d: the feed-forward weights do not fit each other", l);
+      out_cols += c.ff_in->rows / 2;
+    }
+    if (!shape_is(c.out_w, wp, out_cols)) return fail(ctx, CATEN_B200_EINVAL, "decoder: layer %d: out_w must be %lldx%lld", l, (long long)wp, (long long)out_cols);
+    return 0;
+  }
+  if (c.experts) return fail(ctx, CATEN_B200_EUNSUPPORTED, "decoder: layer %d: experts need a parallel layer", l);
   if (!shape_is(c.out_w, wp, out_cols)) return fail(ctx, CATEN_B200_EINVAL, "decoder: layer %d: out_w must be %lldx%lld", l, (long long)wp, (long long)out_cols);
   if (c.ff_in && (c.ff_in->cols != wp || c.ff_in->rows % 128 || !shape_is(c.ff_out, wp, c.ff_in->rows / 2)))
     return fail(ctx, CATEN_B200_EINVAL, "decoder: layer %d: the feed-forward weights do not fit each other", l);
   return 0;
+}
+
+static LatentArgs latent_args(const Dec *m, const caten_b200_layer_desc &c) {
+  LatentArgs a;
+  a.H = c.heads; a.D = c.dim; a.Dp = (int)p16(c.dim); a.P = c.rot_dims; a.Pp = (int)p16(c.rot_dims); a.E = c.vdim; a.Ep = (int)p16(c.vdim);
+  a.K = c.kv_rank; a.Kp = (int)p16(c.kv_rank); a.Kr = (int)p64(c.kv_rank); a.Q = c.q_rank; a.Qr = (int)p64(c.q_rank);
+  a.freq = c.rot_freq; a.q_norm = c.q_norm; a.kv_norm = c.kv_norm; a.eps = m->desc.eps; a.scale = c.scale;
+  a.cache_bf16 = m->desc.precision == CATEN_B200_PREC_BF16;
+  return a;
 }
 
 extern "C" {
@@ -110,7 +175,8 @@ int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc
   if (!shape_is(dsc->embed, V, wp) || dsc->embed->type != CATEN_B200_BF16 || !shape_is(dsc->head, V, wp))
     return fail(ctx, CATEN_B200_EINVAL, "decoder_create: embed (BF16) and head must be %lldx%lld", (long long)V, (long long)wp);
   const bool loops = dsc->loop_stop > dsc->loop_start;
-  if (loops && (dsc->loop_start < 0 || dsc->loop_stop > L || dsc->loop_times < 1 || !shape_is(dsc->loop_in, wp, 2 * wp)))
+  if (loops && (dsc->loop_start < 0 || dsc->loop_stop > L || dsc->loop_times < 1 || (!dsc->loop_in && !dsc->loop_step) || (dsc->loop_in && !shape_is(dsc->loop_in, wp, 2 * wp)) ||
+                (!dsc->loop_in && !dsc->layers[dsc->loop_start].parallel)))
     return fail(ctx, CATEN_B200_EINVAL, "decoder_create: bad loop");
   for (int l = 0; l < L; ++l)
     if (int rc = check_layer(ctx, l, dsc->layers[l], wp)) return rc;
@@ -122,11 +188,11 @@ int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc
   m->desc.layers = nullptr;
   m->wp = wp;
   m->any_loop = loops;
-  auto add_run = [&](int l, bool start) { Run r; r.layer = l; r.pass_start = start; m->runs.push_back(r); };
+  auto add_run = [&](int l, bool start, int pass = 0) { Run r; r.layer = l; r.pass_start = start; r.pass = pass; m->runs.push_back(r); };
   if (loops) {
     for (int l = 0; l < dsc->loop_start; ++l) add_run(l, false);
     for (int t = 0; t < dsc->loop_times; ++t)
-      for (int l = dsc->loop_start; l < dsc->loop_stop; ++l) add_run(l, l == dsc->loop_start);
+      for (int l = dsc->loop_start; l < dsc->loop_stop; ++l) add_run(l, l == dsc->loop_start, t);
     for (int l = dsc->loop_stop; l < L; ++l) add_run(l, false);
   } else {
     for (int l = 0; l < L; ++l) add_run(l, false);
@@ -146,6 +212,12 @@ int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc
   m->portion = portion;
   const int64_t R = max_rows;
   int64_t ny = 64, nd = 0, n_act = 64, low = 64;
+  int64_t l_cq = 0, l_q = 0, l_qn = 0, l_cat = 0, l_o = 0, l_c = 0, l_kr = 0, l_kv = 0, l_part = 0, ret_o = 0, experts = 0, top = 0, ex_ff = 0;   // floats per row
+  bool any_par = false;
+  m->kv_rows = T > max_rows ? T : max_rows;
+  m->abs_rows = max_rows < LATENT_ABSORB * B ? max_rows : LATENT_ABSORB * B;
+  auto most = [](int64_t *a, int64_t b) { if (b > *a) *a = b; };
+  m->uv.resize(L);
   for (const auto &c : m->layers) {
     if (c.in_w->rows > ny) ny = c.in_w->rows;
     if (c.out_w->cols > n_act) n_act = c.out_w->cols;
@@ -155,8 +227,24 @@ int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc
       if (c.w2->rows > nd) nd = c.w2->rows;
       if (c.low_rank > low) low = c.low_rank;
     }
+    if (c.parallel) any_par = true;
+    if (c.mixer == CATEN_B200_MIX_LATENT) {
+      const int64_t H = c.heads, Dp = p16(c.dim), Pp = p16(c.rot_dims), Kp = p16(c.kv_rank), Kr = p64(c.kv_rank);
+      most(&l_cq, p64(c.q_rank)); most(&l_q, H * (Dp + Pp)); most(&l_qn, H * p64(c.dim)); most(&l_cat, H * (Kp + Pp)); most(&l_o, H * Kr);
+      most(&l_c, Kr); most(&l_kr, Pp > 0 ? Pp : 16); most(&l_kv, c.kv_w->rows);
+      LatentArgs a = latent_args(m, c);
+      a.B = (int)B; a.cap = p64(T);
+      most(&l_part, latent_splits(ctx, a, B, a.cap) * B * H * Kr);
+      most(&l_part, 4 * B * H * Kr);
+      caten_b200_weight &uv = m->uv[(size_t)(&c - m->layers.data())];
+      uv = *c.kv_w;
+      uv.rows = H * p16(c.vdim);
+      uv.qs = (uint16_t *)uv.qs + H * Dp * uv.cols;
+    }
+    if (c.mixer == CATEN_B200_MIX_RETENTION && p16(c.vdim) > 256) most(&ret_o, c.heads * p16(c.vdim));
+    if (c.experts) { most(&ny, c.router->rows); most(&experts, c.experts); most(&top, c.top); most(&ex_ff, c.ff_out->cols); }
   }
-  m->planes = m->any_wkv ? 5 : loops ? 2 : 1;
+  m->planes = m->any_wkv ? 5 : loops || any_par ? 2 : 1;
   const bool exact = dsc->precision == CATEN_B200_PREC_FP32;
   m->hp_rows = exact ? R : 4;
   m->cap_rows = B > 64 ? B : 64;
@@ -173,6 +261,13 @@ int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc
       rc = dec_floats(m, &r.kc, B * c.kv_heads * r.cap * Dp);
       if (!rc) rc = dec_floats(m, &r.vc, B * c.kv_heads * r.cap * Ep);
       bytes = B * c.kv_heads * r.cap * (Dp + Ep) * 4;
+    } else if (c.mixer == CATEN_B200_MIX_LATENT) {
+      r.cap = p64(T);
+      bytes = B * r.cap * (p16(c.kv_rank) + p16(c.rot_dims)) * (dsc->precision == CATEN_B200_PREC_BF16 ? 2 : 4);
+      rc = dec_alloc(m, (void **)&r.latents, (size_t)bytes);
+    } else if (c.mixer == CATEN_B200_MIX_RETENTION) {
+      bytes = B * c.heads * Dp * p16(c.vdim) * 4;
+      rc = dec_floats(m, &r.state, bytes / 4);
     } else {
       rc = dec_floats(m, &r.state, B * c.heads * Dp * Dp);
       if (!rc) rc = dec_floats(m, &r.shift, B * wp);
@@ -194,6 +289,39 @@ int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc
     if (!rc) rc = dec_floats(m, &m->o, R * nd);
     if (!rc) rc = dec_floats(m, &m->tl, m->hp_rows * low);
     if (!rc) rc = dec_bf(m, &m->tl_bf, R * low);
+  }
+  if (!rc && l_q) {
+    const int64_t A = m->abs_rows, small = A < m->hp_rows ? A : m->hp_rows;   // rows of fp32 operands
+    rc = dec_floats(m, &m->cq, m->hp_rows * l_cq);
+    if (!rc) rc = dec_bf(m, &m->cq_bf, R * l_cq);
+    if (!rc) rc = dec_floats(m, &m->q, R * l_q);
+    if (!rc) rc = dec_floats(m, &m->qn, A * l_qn);
+    if (!rc) rc = dec_bf(m, &m->qn_bf, A * l_qn);
+    if (!rc) rc = dec_floats(m, &m->qcat, small * l_cat);
+    if (!rc) rc = dec_bf(m, &m->qcat_bf, A * l_cat);
+    if (!rc) rc = dec_floats(m, &m->olat, A * l_o);
+    if (!rc) rc = dec_bf(m, &m->olat_bf, A * l_o);
+    m->part_floats = l_part;
+    if (!rc) rc = dec_floats(m, &m->part, l_part);
+    if (!rc) rc = dec_floats(m, &m->ml, l_part / 16);
+    if (!rc) rc = dec_floats(m, &m->lat, (exact ? m->kv_rows : 4) * l_c);
+    if (!rc) rc = dec_bf(m, &m->lat_bf, m->kv_rows * l_c);
+    if (!rc) rc = dec_floats(m, &m->kr, m->kv_rows * l_kr);
+    if (!rc) rc = dec_floats(m, &m->kvx, m->kv_rows * l_kv);
+  }
+  if (!rc && ret_o) rc = dec_floats(m, &m->ret_o, R * ret_o);
+  if (!rc && experts) {
+    const int64_t P = R * top;
+    rc = dec_alloc(m, (void **)&m->ex_id, (size_t)P * sizeof(int));
+    if (!rc) rc = dec_alloc(m, (void **)&m->ex_off, (size_t)(experts + 1) * sizeof(int));
+    if (!rc) rc = dec_alloc(m, (void **)&m->ex_src, (size_t)P * sizeof(int));
+    if (!rc) rc = dec_alloc(m, (void **)&m->ex_pos, (size_t)P * sizeof(int));
+    if (!rc) rc = dec_floats(m, &m->ex_w, P);
+    if (!rc) rc = dec_floats(m, &m->ex_ws, P);
+    if (!rc) rc = dec_floats(m, &m->ea, m->hp_rows * top * ex_ff);
+    if (!rc) rc = dec_bf(m, &m->ea_bf, P * ex_ff);
+    if (!rc) rc = dec_bf(m, &m->xs_bf, P * wp);
+    if (!rc) rc = dec_floats(m, &m->ye, P * wp);
   }
   if (!rc) rc = dec_floats(m, &m->last, m->cap_rows * wp);
   if (!rc) rc = dec_bf(m, &m->last_bf, m->cap_rows * wp);
@@ -237,6 +365,9 @@ struct Pending {
   int in = SN_EMBED;
   PartIn pin;
   float post = 1.0f;
+  const float *ye = nullptr;   // SN_SUM: outputs of experts
+  const int *pos = nullptr;
+  int top = 0;
 };
 
 class StepRunner {
@@ -251,12 +382,17 @@ class StepRunner {
   int layers() {
     for (size_t i = 0; i < m_->runs.size(); ++i) {
       const Run &r = m_->runs[i];
-      if (r.pass_start) {
+      size_t finished = i;
+      if (r.pass_start && m_->desc.loop_in) {
         if (int rc = boundary(SN_CONCAT, 0.0f, i)) return rc;
         if (int rc = linear(m_->desc.loop_in, m_->hp, m_->hp_bf, nullptr, m_->y2, none_, defer_ ? &pend_.pin : nullptr)) return rc;
         pend_.in = SN_COPY;
+        finished = 0;
+      } else if (r.pass_start && m_->capture && i > 0) {   // the stream as the layer before left it
+        if (int rc = boundary(SN_NONE, 0.0f, i)) return rc;
+        finished = 0;
       }
-      if (int rc = layer(r, r.pass_start ? 0 : i)) return rc;
+      if (int rc = layer(r, finished)) return rc;
     }
     if (m_->capture) {
       if (int rc = boundary(SN_NONE, 0.0f, m_->runs.size())) return rc;
@@ -270,6 +406,7 @@ class StepRunner {
   int final_norm(int64_t at, int64_t count, int64_t stride, const int *rows) {
     StreamArgs a = stream();
     a.pre = m_->desc.final_gain;
+    a.w1 = m_->desc.final_norm;
     a.x_out = nullptr;  // other rows may still be wanted: the pending stage stays
     a.rows = rows;
     a.src_stride = stride;
@@ -277,7 +414,7 @@ class StepRunner {
     if (prec_ != CATEN_B200_PREC_FP32) a.hb = offset(m_->last_bf, at * m_->wp);
     if (head_rows_small_) a.hb = BfOut();
     ProfScope prof(ctx_, CATEN_B200_K_LAYERNORM);
-    return launch_stream_norm(ctx_, pend_.in, SN_NORM, a, count);
+    return launch_stream_norm(ctx_, pend_.in, a.w1 ? SN_NORM2 : SN_NORM, a, count);
   }
   // Forms the pending stream rows now: the split-K tiles they are made of live in scratch that the next linear reuses.
   int materialise() { return pend_.in == SN_KEEP ? 0 : boundary(SN_NONE, 0.0f, 0); }
@@ -295,6 +432,7 @@ class StepRunner {
   StreamArgs stream() const {
     StreamArgs a;
     a.y = m_->y2; a.pin = pend_.pin; a.post = pend_.post;
+    a.ye = pend_.ye; a.pos = pend_.pos; a.top = pend_.top;
     a.x = m_->x; a.x_out = m_->x; a.x0 = m_->x0;
     a.table = (const __nv_bfloat16 *)m_->desc.embed->qs;
     a.ids = p_.ids; a.ids_ld = p_.ids_ld; a.vocab = m_->desc.vocab; a.s = (int)p_.s;
@@ -306,9 +444,12 @@ class StepRunner {
   }
 
   // Ends the previous sublayer and prepares the next operation's input; afterwards the stream is x.
-  int boundary(int out, float pre, size_t finished_runs, const caten_b200_layer_desc *shift_layer = nullptr, const Run *shift_run = nullptr, float *to_fp32 = nullptr) {
+  int boundary(int out, float pre, size_t finished_runs, const caten_b200_layer_desc *shift_layer = nullptr, const Run *shift_run = nullptr, float *to_fp32 = nullptr,
+               const caten_b200_layer_desc *parallel = nullptr, const Run *pass = nullptr) {
     StreamArgs a = stream();
     a.pre = pre;
+    if (parallel) { a.w1 = parallel->norm1_w; a.w2 = parallel->ff_in ? parallel->norm2_w : nullptr; }
+    if (pass) { a.step = m_->desc.loop_step + (int64_t)pass->pass * m_->wp; a.add_x0 = pass->pass > 0; }
     if (to_fp32) { a.h = to_fp32; a.hb = BfOut(); }
     if (out == SN_SHIFT) { a.mu = shift_layer->mu; a.shift = shift_run->shift + p_.b0 * m_->wp; }
     {
@@ -327,7 +468,8 @@ class StepRunner {
 
   int layer(const Run &r, size_t finished_runs) {
     const caten_b200_layer_desc &c = m_->layers[r.layer];
-    if (int rc = c.mixer == CATEN_B200_MIX_ATTENTION ? attention(r, c, finished_runs) : wkv(r, c, finished_runs)) return rc;
+    if (int rc = mixer(r, c, finished_runs)) return rc;
+    if (c.parallel) return finish_parallel(c);
     if (int rc = linear(c.out_w, m_->act, m_->act_bf, nullptr, m_->y2, none_, defer_ ? &pend_.pin : nullptr)) return rc;
     pend_.in = SN_ADD;
     pend_.post = c.norm1b;
@@ -340,8 +482,151 @@ class StepRunner {
     return 0;
   }
 
+  int mixer(const Run &r, const caten_b200_layer_desc &c, size_t finished_runs) {
+    switch (c.mixer) {
+      case CATEN_B200_MIX_ATTENTION: return attention(r, c, finished_runs);
+      case CATEN_B200_MIX_LATENT: return latent(r, c, finished_runs);
+      case CATEN_B200_MIX_RETENTION: return retention(r, c, finished_runs);
+      default: return wkv(r, c, finished_runs);
+    }
+  }
+
+  // The norm before a mixer; a parallel layer's feed-forward gets its own beside it (plane 1).
+  int enter(const Run &r, const caten_b200_layer_desc &c, size_t finished_runs) {
+    if (!c.parallel) return boundary(SN_NORM, c.norm1, finished_runs);
+    return boundary(SN_NORM2, 0.0f, finished_runs, nullptr, nullptr, nullptr, &c, r.pass_start && !m_->desc.loop_in ? &r : nullptr);
+  }
+
+  // The feed-forward beside the mixer, and one linear over both outputs.
+  int finish_parallel(const caten_b200_layer_desc &c) {
+    const float *h2 = m_->hp + plane_ * m_->wp;
+    const BfOut h2_bf = offset(m_->hp_bf, plane_ * m_->wp);
+    Pending next;
+    next.in = SN_SUM;
+    if (c.experts) {
+      if (int rc = experts(c, h2, h2_bf, &next)) return rc;
+    } else if (c.ff_in) {
+      LinGroups to;
+      to.ldy = c.out_w->cols;
+      const int64_t col = mixer_cols(c);
+      if (int rc = linear(c.ff_in, h2, h2_bf, nullptr, m_->act + col, offset(bf(m_->act_bf), col), nullptr, c.ff_act, to)) return rc;
+    }
+    if (int rc = linear(c.out_w, m_->act, m_->act_bf, nullptr, m_->y2, none_, defer_ ? &next.pin : nullptr)) return rc;
+    pend_ = next;
+    return 0;
+  }
+
+  int experts(const caten_b200_layer_desc &c, const float *h2, BfOut h2_bf, Pending *next) {
+    RouteArgs a;
+    if (int rc = linear(c.router, h2, h2_bf, nullptr, m_->y, none_, defer_ ? &a.pin : nullptr)) return rc;
+    const bool sorted = R_ > 4;
+    const int64_t rows_in = c.ff_in->rows / c.experts, pairs = R_ * c.top;
+    a.z = m_->y; a.ld = c.router->rows; a.rows = (int)R_; a.experts = c.experts; a.top = c.top;
+    a.expert = m_->ex_id; a.weight = m_->ex_w; a.offsets = m_->ex_off; a.src = m_->ex_src; a.sorted_weight = m_->ex_ws; a.pos = m_->ex_pos;
+    {
+      ProfScope prof(ctx_, CATEN_B200_K_PREP);
+      if (int rc = launch_moe_route(ctx_, a, sorted)) return rc;
+      if (fused_)
+        if (int rc = launch_moe_gather(ctx_, h2_bf, m_->ex_src, pairs, m_->wp, m_->xs_bf)) return rc;
+    }
+    next->ye = m_->ye;
+    next->top = c.top;
+    next->pos = sorted ? m_->ex_pos : nullptr;
+    ProfScope prof(ctx_, sorted ? CATEN_B200_K_GEMM : CATEN_B200_K_GEMV);
+    if (!sorted) {
+      if (int rc = launch_gemv_experts(ctx_, c.ff_in, rows_in, h2, m_->ex_id, m_->ex_w, pairs, c.top, c.ff_act, m_->ea)) return rc;
+      return launch_gemv_experts(ctx_, c.ff_out, m_->wp, m_->ea, m_->ex_id, nullptr, pairs, 1, CATEN_B200_ACT_NONE, m_->ye);
+    }
+    ExpertRows er;
+    er.experts = c.experts; er.top = c.top; er.pairs = pairs; er.offsets = m_->ex_off; er.src = m_->ex_src;
+    ExpertRows in = er;
+    in.weight = m_->ex_ws;
+    if (!fused_) {
+      if (int rc = launch_gemm_simt_experts(ctx_, c.ff_in, in, h2, m_->ex_src, c.ff_act, m_->ea)) return rc;
+      return launch_gemm_simt_experts(ctx_, c.ff_out, er, m_->ea, nullptr, CATEN_B200_ACT_NONE, m_->ye);
+    }
+    const int nsplit = prec_ == CATEN_B200_PREC_BF16X3 ? 3 : 1;
+    if (int rc = launch_gemm_experts(ctx_, c.ff_in, in, m_->xs_bf, c.ff_act, nullptr, m_->ea_bf, nsplit)) return rc;
+    return launch_gemm_experts(ctx_, c.ff_out, er, m_->ea_bf, CATEN_B200_ACT_NONE, m_->ye, none_, nsplit);
+  }
+
+  int latent(const Run &r, const caten_b200_layer_desc &c, size_t finished_runs) {
+    if (int rc = enter(r, c, finished_runs)) return rc;
+    LatentArgs a = latent_args(m_, c);
+    PartIn pin;
+    if (int rc = linear(c.in_w, m_->hp, m_->hp_bf, nullptr, m_->y, none_, defer_ ? &pin : nullptr)) return rc;
+    a.cap = r.cap;
+    a.cache = r.latents + p_.b0 * r.cap * a.KC() * (a.cache_bf16 ? 2 : 4);
+    a.B = (int)p_.nb; a.s = (int)p_.s; a.n = (int)p_.n; a.d_n = p_.d_n;
+    { ProfScope prof(ctx_, CATEN_B200_K_PREP); if (int rc = launch_latent_prep(ctx_, a, m_->y, pin, c.in_w->rows, m_->cq, bf(m_->cq_bf))) return rc; }
+    const bool absorbed = p_.s <= LATENT_ABSORB;
+    pin = PartIn();
+    if (int rc = linear(c.uq_w, m_->cq, m_->cq_bf, nullptr, m_->q, none_, defer_ && absorbed ? &pin : nullptr)) return rc;
+    const int64_t ldq = c.uq_w->rows;
+    if (absorbed) {
+      { ProfScope prof(ctx_, CATEN_B200_K_PREP);
+        if (int rc = launch_latent_q_absorbed(ctx_, a, m_->q, pin, ldq, m_->abs_rows, m_->qn, bf(m_->qn_bf), m_->qcat, bf(m_->qcat_bf))) return rc; }
+      LinGroups up;
+      up.group_rows = a.Kp; up.xplane = m_->abs_rows; up.ygroup = a.KC(); up.ldy = (int64_t)a.H * a.KC();
+      if (int rc = linear(c.uk_w, m_->qn, m_->qn_bf, nullptr, m_->qcat, bf(m_->qcat_bf), nullptr, CATEN_B200_ACT_NONE, up)) return rc;
+      LatentAbsorbed x;
+      x.qcat = m_->qcat; x.qcat_bf = bf(m_->qcat_bf); x.o = m_->olat; x.o_bf = bf(m_->olat_bf); x.plane = m_->abs_rows; x.part = m_->part; x.ml = m_->ml;
+      x.splits = latent_splits(ctx_, a, R_, p_.d_n ? a.cap : p_.n + p_.s);
+      while (x.splits > 1 && x.splits * R_ * a.H * a.Kr > m_->part_floats) --x.splits;
+      { ProfScope prof(ctx_, CATEN_B200_K_ATTN_DECODE); if (int rc = launch_latent_absorbed(ctx_, a, x)) return rc; }
+      LinGroups down;
+      down.group_rows = a.Ep; down.xplane = m_->abs_rows; down.ygroup = a.Ep; down.ldy = c.out_w->cols;
+      return linear(&m_->uv[r.layer], m_->olat, m_->olat_bf, nullptr, m_->act, bf(m_->act_bf), nullptr, CATEN_B200_ACT_NONE, down);
+    }
+    { ProfScope prof(ctx_, CATEN_B200_K_PREP); if (int rc = launch_latent_q_expanded(ctx_, a, m_->q, ldq)) return rc; }
+    // keys and values of every cached token, for as many sequences at a time as the buffer takes
+    const int64_t t = p_.n + p_.s, per = m_->kv_rows / t < 1 ? 1 : m_->kv_rows / t;
+    for (int64_t b = 0; b < p_.nb; b += per) {
+      const int64_t nb = p_.nb - b < per ? p_.nb - b : per, rows = nb * t;
+      const bool small = prec_ == CATEN_B200_PREC_FP32 || rows <= 4;
+      { ProfScope prof(ctx_, CATEN_B200_K_PREP); if (int rc = launch_latent_gather(ctx_, a, (int)b, (int)nb, (int)t, m_->lat, small ? BfOut() : m_->lat_bf, m_->kr)) return rc; }
+      if (int rc = model_linear(ctx_, prec_, c.kv_w, m_->lat, small ? BfOut() : m_->lat_bf, nullptr, nullptr, CATEN_B200_ACT_NONE, m_->kvx, none_, rows)) return rc;
+      AttnArgs x;
+      x.H = x.G = a.H;
+      x.D = a.D + a.P; x.Dp = a.Dq(); x.E = a.E; x.Ep = a.Ep;
+      x.qkv = m_->q + b * p_.s * ldq; x.ld = ldq;
+      x.kc = m_->kvx; x.vc = m_->kvx + (int64_t)a.H * a.Dp;
+      x.cap = t;
+      x.k_ld = x.v_ld = c.kv_w->rows; x.k_head = a.Dp; x.v_head = a.Ep; x.k_seq = x.v_seq = t * x.k_ld;
+      x.kx = a.Pp ? m_->kr : nullptr; x.kx_ld = a.Pp; x.kx_from = a.Dp;
+      x.out_ld = c.out_w->cols;
+      x.out = m_->act + b * p_.s * x.out_ld;
+      x.bf = offset(bf(m_->act_bf), b * p_.s * x.out_ld);
+      x.B = (int)nb; x.s = (int)p_.s; x.n = (int)p_.n;
+      ProfScope prof(ctx_, CATEN_B200_K_ATTN_PREFILL);
+      if (int rc = launch_attn_window_prefill(ctx_, x, prec_ != CATEN_B200_PREC_FP32 && ctx_->attn_tc)) return rc;
+    }
+    return 0;
+  }
+
+  int retention(const Run &r, const caten_b200_layer_desc &c, size_t finished_runs) {
+    if (int rc = enter(r, c, finished_runs)) return rc;
+    RetentionArgs a;
+    if (int rc = linear(c.in_w, m_->hp, m_->hp_bf, nullptr, m_->y, none_, defer_ && p_.s == 1 ? &a.pin : nullptr)) return rc;
+    a.H = c.heads; a.D = c.dim; a.Dp = (int)p16(c.dim); a.E = c.vdim; a.Ep = (int)p16(c.vdim);
+    a.y = m_->y; a.ld = c.in_w->rows;
+    a.k_off = a.H * a.Dp; a.v_off = 2 * a.k_off; a.g_off = a.v_off + a.H * a.Ep;
+    a.freq = c.rot_freq; a.rot_pairs = c.rot_dims / 2; a.kscale = (float)(1.0 / sqrt((double)c.dim)); a.powers = c.powers; a.eps = m_->desc.eps;
+    a.state = r.state + p_.b0 * a.H * a.Dp * a.Ep;
+    a.out = m_->act; a.bf = bf(m_->act_bf); a.out_ld = c.out_w->cols;
+    a.o = m_->ret_o;
+    a.B = (int)p_.nb; a.s = (int)p_.s; a.n = (int)p_.n; a.d_n = p_.d_n;
+    if (p_.s == 1) {
+      ProfScope prof(ctx_, CATEN_B200_K_WKV);
+      return launch_retention_decode(ctx_, a);
+    }
+    { ProfScope prof(ctx_, CATEN_B200_K_PREP); if (int rc = launch_retention_prep(ctx_, a)) return rc; }
+    ProfScope prof(ctx_, CATEN_B200_K_WKV);
+    return launch_retention_chunks(ctx_, a);
+  }
+
   int attention(const Run &r, const caten_b200_layer_desc &c, size_t finished_runs) {
-    if (int rc = boundary(SN_NORM, c.norm1, finished_runs)) return rc;
+    if (int rc = enter(r, c, finished_runs)) return rc;
     AttnArgs a;
     if (int rc = linear(c.in_w, m_->hp, m_->hp_bf, nullptr, m_->y, none_, defer_ && p_.s == 1 ? &a.pin : nullptr)) return rc;
     a.H = c.heads; a.G = c.kv_heads;

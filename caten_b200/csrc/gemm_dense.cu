@@ -11,6 +11,11 @@
 //               activation and the residual, store — while the next tile's MMAs run
 // Tile = 128 output features (TMEM lanes) x 256 rows (TMEM columns); a stage holds 64 k (bf16) or 32 k (split bf16).
 // Split-bf16 (NSPLIT = 3) issues W_hi.x_hi + W_lo.x_hi + W_hi.x_lo per k-step, as the decode GEMM.
+// EXPERTS (mixture of experts): the rows of x are sorted by expert; expert e's rows [offsets[e], offsets[e + 1]), read on
+// the device, are multiplied with its own rows of W.  The tile list is formed from the offsets in every CTA; a row tile
+// may reach into the next expert's rows, whose products are not stored.  The row tile is as narrow as the experts' rows
+// are few (bn), so that a decode step reads each weight once beside little else.  Products are scaled by the row's weight
+// before the activation.
 // Every mbarrier wait is bounded: when one runs out the role records it in the status word,
 // every role leaves its loop, copies in flight are awaited, tensor memory is freed.
 #include "blocks32.cuh"
@@ -36,9 +41,46 @@ struct GdArgs {
   int act, M, N, K;
   int tiles_f, tiles;         // feature tiles per row tile; all tiles
   int stages;
-  int group_rows, xplane;     // output rows [g * group_rows, ..) read input plane g, `xplane` rows after the one before it
+  // output rows [g * group_rows, ..) read input plane g, `xplane` rows after the one before it, and go to columns
+  // [g * ygroup, ..) of rows of ldy; a group has tiles_per_group feature tiles, the last one possibly partial
+  int group_rows, xplane, ygroup, ldy, tiles_per_group;
   uint32_t idesc;
+  int bn;                     // EXPERTS: activation rows per tile (GD_BN otherwise)
+  ExpertRows er;
 };
+
+constexpr int GD_MAX_EXPERTS = 1024;
+
+// One output tile: features [f0, f_end), activation rows [m0, m_end), first row of its x tile
+struct GdTile {
+  int f0, f_end, m0, m_end, x0, shift;
+};
+template <bool EXPERTS>
+__device__ __forceinline__ GdTile gd_tile(const GdArgs &a, int tile, const int *first) {
+  GdTile t;
+  if (EXPERTS) {   // first[e] = index of expert e's first tile
+    int lo = 0, hi = a.er.experts;   // the last e with first[e] <= tile (an expert without rows has no tiles)
+    while (hi - lo > 1) {
+      const int mid = (lo + hi) >> 1;
+      if (first[mid] <= tile) lo = mid; else hi = mid;
+    }
+    const int i = tile - first[lo];
+    t.f0 = lo * a.group_rows + (i % a.tiles_f) * GD_BM;
+    t.f_end = (lo + 1) * a.group_rows;
+    t.m0 = t.x0 = a.er.offsets[lo] + (i / a.tiles_f) * a.bn;
+    t.m_end = a.er.offsets[lo + 1];
+    t.shift = lo * a.group_rows;
+  } else {
+    const int f = tile % a.tiles_f, g = f / a.tiles_per_group;
+    t.f0 = g * a.group_rows + (f % a.tiles_per_group) * GD_BM;
+    t.f_end = min(a.N, (g + 1) * a.group_rows);
+    t.m0 = (tile / a.tiles_f) * GD_BN;
+    t.m_end = a.M;
+    t.x0 = t.m0 + g * a.xplane;
+    t.shift = g * (a.group_rows - a.ygroup);
+  }
+  return t;
+}
 
 // ---- pre-pass: operands -> bf16 hi (and lo), K-major --------------------------------------------
 
@@ -116,19 +158,24 @@ __global__ void __launch_bounds__(256) xsplit_kernel(const float *__restrict__ x
 // shared-memory tile of the warp and comes back transposed: a lane then owns four consecutive features of
 // four rows and moves 16 bytes per instruction (bias, activation, residual and the optional split-bf16
 // output are applied on that side).
-template <int ACT>
-__device__ __forceinline__ void gd_store_block(const GdArgs &a, const float *stg, int lane, float4 bias4, int64_t o0, bool o_ok, int m_first) {
+template <int ACT, bool EXPERTS>
+__device__ __forceinline__ void gd_store_block(const GdArgs &a, const float *stg, int lane, float4 bias4, int64_t o0, bool o_ok, int m_first, int m_end) {
   const int fg = lane & 7, tr = lane >> 3;
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
     const int t = 4 * j + tr;
     const int64_t m = (int64_t)m_first + t;
-    if (!o_ok || m >= a.M) continue;
+    if (!o_ok || m >= m_end) continue;
     const float4 acc = *reinterpret_cast<const float4 *>(stg + t * 32 + 4 * fg);
     float v[4] = {acc.x + bias4.x, acc.y + bias4.y, acc.z + bias4.z, acc.w + bias4.w};
-    if (ACT == CATEN_B200_ACT_RELU_GLU) {  // two (gate, up) pairs -> two outputs
-      const float g0 = relu_glu(v[0], v[1]), g1 = relu_glu(v[2], v[3]);
-      const int64_t at2 = m * (a.N / 2) + o0 / 2;
+    if (EXPERTS && a.er.weight) {
+      const float wt = a.er.weight[m];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = v[e] * wt;
+    }
+    if (act_is_glu(ACT)) {  // two (gate, up) pairs -> two outputs
+      const float g0 = glu(ACT, v[0], v[1]), g1 = glu(ACT, v[2], v[3]);
+      const int64_t at2 = m * a.ldy + o0 / 2;
       if (a.yhi) {
         *reinterpret_cast<uint32_t *>(a.yhi + at2) = pack_bf16(g0, g1);
         if (a.ylo) *reinterpret_cast<uint32_t *>(a.ylo + at2) = pack_bf16(bf16_lo(g0), bf16_lo(g1));
@@ -137,7 +184,7 @@ __device__ __forceinline__ void gd_store_block(const GdArgs &a, const float *stg
       }
       continue;
     }
-    const int64_t at = m * a.N + o0;
+    const int64_t at = m * a.ldy + o0;
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       if (ACT == CATEN_B200_ACT_GELU) v[e] = gelu_ref(v[e]);
@@ -178,14 +225,17 @@ __device__ __forceinline__ uint64_t gd_desc(uint32_t saddr) {
   return d;
 }
 
-template <int NSPLIT>
+template <int NSPLIT, bool EXPERTS>
 __global__ void __launch_bounds__(GD_THREADS, 1)
 gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_constant__ CUtensorMap tw_lo,
                   const __grid_constant__ CUtensorMap tx_hi, const __grid_constant__ CUtensorMap tx_lo, const GdArgs a) {
   constexpr int BK = GdStage<NSPLIT>::BK;
   constexpr uint32_t ROW_BYTES = BK * 2u;
-  constexpr uint32_t W_BYTES = GD_BM * ROW_BYTES, X_BYTES = GD_BN * ROW_BYTES;
-  constexpr uint32_t STAGE_BYTES = (W_BYTES + X_BYTES) * (NSPLIT == 3 ? 2u : 1u);
+  constexpr bool WLO = NSPLIT == 3 && !EXPERTS;   // (experts' weights are bf16: no low part)
+  const int BN = EXPERTS ? a.bn : GD_BN;
+  constexpr uint32_t W_BYTES = GD_BM * ROW_BYTES;
+  const uint32_t X_BYTES = (uint32_t)BN * ROW_BYTES;
+  const uint32_t STAGE_BYTES = W_BYTES * (WLO ? 2u : 1u) + X_BYTES * (NSPLIT == 3 ? 2u : 1u);
   extern __shared__ uint8_t smem_raw[];
   uint8_t *smem = reinterpret_cast<uint8_t *>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   const int S = a.stages;
@@ -203,7 +253,7 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
   const uint32_t stage0 = smem_u32(smem);
   auto st_whi = [&](int s) { return stage0 + (uint32_t)s * STAGE_BYTES; };
   auto st_wlo = [&](int s) { return stage0 + (uint32_t)s * STAGE_BYTES + W_BYTES; };
-  auto st_xhi = [&](int s) { return stage0 + (uint32_t)s * STAGE_BYTES + (NSPLIT == 3 ? 2u : 1u) * W_BYTES; };
+  auto st_xhi = [&](int s) { return stage0 + (uint32_t)s * STAGE_BYTES + (WLO ? 2u : 1u) * W_BYTES; };
   auto st_xlo = [&](int s) { return st_xhi(s) + X_BYTES; };
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -235,12 +285,34 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
     tma_prefetch_map(&tw_hi);
     tma_prefetch_map(&tx_hi);
     if (NSPLIT == 3) {
-      tma_prefetch_map(&tw_lo);
+      if (WLO) tma_prefetch_map(&tw_lo);
       tma_prefetch_map(&tx_lo);
     }
   }
   // both operands and the residual were written by preceding kernels
   pdl_wait();
+  int tiles = a.tiles;
+  int *first = reinterpret_cast<int *>(smem + (size_t)S * STAGE_BYTES + GD_EPI_WARPS * 2048);   // EXPERTS: [experts + 1]
+  if (EXPERTS) {
+    if (warp == 0) {
+      int sum = 0;
+      for (int e0 = 0; e0 < a.er.experts; e0 += 32) {
+        const int e = e0 + lane;
+        const int mine = e < a.er.experts ? (a.er.offsets[e + 1] - a.er.offsets[e] + BN - 1) / BN * a.tiles_f : 0;
+        int inc = mine;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+          const int up = __shfl_up_sync(0xffffffffu, inc, o);
+          if (lane >= o) inc += up;
+        }
+        if (e < a.er.experts) first[e] = sum + inc - mine;
+        sum += __shfl_sync(0xffffffffu, inc, 31);
+      }
+      if (lane == 0) first[a.er.experts] = sum;
+    }
+    __syncthreads();
+    tiles = first[a.er.experts];
+  }
 
   if (warp == 0) {
     // ---------------- TMA producer ----------------
@@ -248,9 +320,8 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
       int issued = 0, s = 0;
       uint32_t ph = 0;
       bool ok = true;
-      for (int tile = blockIdx.x; tile < a.tiles && ok; tile += gridDim.x) {
-        const int f0 = (tile % a.tiles_f) * GD_BM, m0 = (tile / a.tiles_f) * GD_BN;
-        const int y0 = m0 + (f0 / a.group_rows) * a.xplane;
+      for (int tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x) {
+        const GdTile t = gd_tile<EXPERTS>(a, tile, first);
         for (int kc = 0; kc < num_k; ++kc) {
           if (!mbar_wait(empty(s), ph ^ 1u, abort_flag)) {
             if (!*abort_flag) { *abort_flag = 1; atomicCAS(a.status, 0, DEV_WAIT_TIMEOUT); a.status[1] = 11; a.status[2] = tile; }
@@ -258,10 +329,10 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
             break;
           }
           mbar_expect_tx(full(s), STAGE_BYTES);
-          tma_load_2d(st_whi(s), &tw_hi, full(s), kc * BK, f0);
-          if (NSPLIT == 3) tma_load_2d(st_wlo(s), &tw_lo, full(s), kc * BK, f0);
-          tma_load_2d(st_xhi(s), &tx_hi, full(s), kc * BK, y0);
-          if (NSPLIT == 3) tma_load_2d(st_xlo(s), &tx_lo, full(s), kc * BK, y0);
+          tma_load_2d(st_whi(s), &tw_hi, full(s), kc * BK, t.f0);
+          if (WLO) tma_load_2d(st_wlo(s), &tw_lo, full(s), kc * BK, t.f0);
+          tma_load_2d(st_xhi(s), &tx_hi, full(s), kc * BK, t.x0);
+          if (NSPLIT == 3) tma_load_2d(st_xlo(s), &tx_lo, full(s), kc * BK, t.x0);
           ++issued;
           if (++s == S) { s = 0; ph ^= 1u; }
         }
@@ -276,7 +347,7 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
     int s = 0, it = 0;
     uint32_t ph = 0;
     bool ok = true;
-    for (int tile = blockIdx.x; tile < a.tiles && ok; tile += gridDim.x, ++it) {
+    for (int tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++it) {
       const int b = it & 1;
       // the epilogue has drained this accumulator (first use of each passes at once)
       if (!mbar_wait(acc_empty(b), (((uint32_t)it >> 1) & 1u) ^ 1u, abort_flag)) {
@@ -301,7 +372,7 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
             const uint64_t adv = (uint64_t)(k4 * 2);  // 16 bf16 = 32 bytes = 2 descriptor units
             umma_bf16(acc, dwh + adv, dxh + adv, a.idesc, (kc > 0 || k4 > 0) ? 1u : 0u);
             if (NSPLIT == 3) {
-              umma_bf16(acc, dwl + adv, dxh + adv, a.idesc, 1u);
+              if (WLO) umma_bf16(acc, dwl + adv, dxh + adv, a.idesc, 1u);
               umma_bf16(acc, dwh + adv, dxl + adv, a.idesc, 1u);
             }
           }
@@ -320,9 +391,9 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
     float *stg = reinterpret_cast<float *>(smem + (size_t)S * STAGE_BYTES) + (warp - 2) * 512;  // 16 rows x 32 features
     int it = 0;
     bool ok = true;
-    for (int tile = blockIdx.x; tile < a.tiles && ok; tile += gridDim.x, ++it) {
+    for (int tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++it) {
       const int b = it & 1;
-      const int f0 = (tile % a.tiles_f) * GD_BM, m0 = (tile / a.tiles_f) * GD_BN;
+      const GdTile t = gd_tile<EXPERTS>(a, tile, first);
       int got = 0;
       if (lane == 0) {
         got = mbar_wait(acc_full(b), ((uint32_t)it >> 1) & 1u, abort_flag) ? 1 : 0;
@@ -332,12 +403,15 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
       if (!got) { ok = false; break; }
       tc_fence_after();
       // after the transpose a lane owns features o0 .. o0 + 3 (N % 4 == 0: all inside or all outside)
-      const int64_t o0 = (int64_t)f0 + quad * 32 + 4 * (lane & 7);
-      const bool o_ok = o0 < a.N;
+      const int64_t o0 = (int64_t)t.f0 + quad * 32 + 4 * (lane & 7);
+      const bool o_ok = o0 < t.f_end;
+      const int64_t oc = o0 - t.shift;   // output column
+      const int cols = EXPERTS ? (BN >= 32 ? BN / 2 : half == 0 ? 16 : 0) : GD_BN / 2;
       float4 bias4 = make_float4(0.f, 0.f, 0.f, 0.f);
       if (a.bias && o_ok) bias4 = *reinterpret_cast<const float4 *>(a.bias + o0);
-      const uint32_t trow = tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(b * GD_BN + half * (GD_BN / 2));
-      for (int c = 0; c < GD_BN / 2; c += 16) {
+      const uint32_t trow = tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(b * GD_BN + half * (BN / 2));
+      for (int c = 0; c < cols; c += 16) {
+        if (EXPERTS && t.m0 + half * (BN / 2) + c >= t.m_end) break;
         uint32_t r[16];
         tmem_ld16(trow + (uint32_t)c, r);
         tmem_ld_wait();
@@ -345,11 +419,12 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tw_hi, const __grid_consta
 #pragma unroll
         for (int i = 0; i < 16; ++i) stg[i * 32 + lane] = __uint_as_float(r[i]);
         __syncwarp();
-        const int m_first = m0 + half * (GD_BN / 2) + c;
-        if (a.act == CATEN_B200_ACT_GELU) gd_store_block<CATEN_B200_ACT_GELU>(a, stg, lane, bias4, o0, o_ok, m_first);
-        else if (a.act == CATEN_B200_ACT_RELU_GLU) gd_store_block<CATEN_B200_ACT_RELU_GLU>(a, stg, lane, bias4, o0, o_ok, m_first);
-        else if (a.act == CATEN_B200_ACT_RELU) gd_store_block<CATEN_B200_ACT_RELU>(a, stg, lane, bias4, o0, o_ok, m_first);
-        else gd_store_block<CATEN_B200_ACT_NONE>(a, stg, lane, bias4, o0, o_ok, m_first);
+        const int m_first = t.m0 + half * (BN / 2) + c;
+        if (a.act == CATEN_B200_ACT_SILU_GLU) gd_store_block<CATEN_B200_ACT_SILU_GLU, EXPERTS>(a, stg, lane, bias4, oc, o_ok, m_first, t.m_end);
+        else if (a.act == CATEN_B200_ACT_RELU_GLU) gd_store_block<CATEN_B200_ACT_RELU_GLU, EXPERTS>(a, stg, lane, bias4, oc, o_ok, m_first, t.m_end);
+        else if (!EXPERTS && a.act == CATEN_B200_ACT_GELU) gd_store_block<CATEN_B200_ACT_GELU, EXPERTS>(a, stg, lane, bias4, oc, o_ok, m_first, t.m_end);
+        else if (!EXPERTS && a.act == CATEN_B200_ACT_RELU) gd_store_block<CATEN_B200_ACT_RELU, EXPERTS>(a, stg, lane, bias4, oc, o_ok, m_first, t.m_end);
+        else gd_store_block<CATEN_B200_ACT_NONE, EXPERTS>(a, stg, lane, bias4, oc, o_ok, m_first, t.m_end);
       }
       tc_fence_before();
       __syncwarp();
@@ -455,8 +530,13 @@ int launch_gemm_dense(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *
   GdArgs a;
   a.bias = bias; a.res = res; a.y = y; a.yhi = ybf.hi; a.ylo = ybf.lo; a.status = ctx->d_status;
   a.act = act; a.M = (int)M; a.N = (int)N; a.K = (int)K;
-  a.tiles_f = (int)((N + GD_BM - 1) / GD_BM);
-  a.group_rows = grp.group_rows ? (int)grp.group_rows : a.tiles_f * GD_BM; a.xplane = (int)grp.xplane;
+  a.group_rows = grp.group_rows ? (int)grp.group_rows : (int)((N + GD_BM - 1) / GD_BM * GD_BM); a.xplane = (int)grp.xplane;
+  a.tiles_per_group = (a.group_rows + GD_BM - 1) / GD_BM;
+  a.tiles_f = (int)((N + a.group_rows - 1) / a.group_rows) * a.tiles_per_group;
+  a.ygroup = grp.ygroup ? (int)grp.ygroup : a.group_rows;
+  a.ldy = grp.ldy ? (int)grp.ldy : (int)(act_is_glu(act) ? N / 2 : N);
+  a.bn = GD_BN;
+  if (res && !grp.plain_output()) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemm_dense: a residual needs the plain output layout");
   const int64_t tiles = (int64_t)a.tiles_f * ((M + GD_BN - 1) / GD_BN);
   if (tiles > 0x7fffffff) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemm_dense: too many tiles");
   a.tiles = (int)tiles;
@@ -479,11 +559,54 @@ int launch_gemm_dense(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *
   cfg.attrs = at;
   cfg.numAttrs = take_pdl(ctx) ? 1 : 0;
   if (nsplit == 3) {
-    CB_CUDA(ctx, cudaFuncSetAttribute(gemm_dense_kernel<3>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    CB_CUDA(ctx, cudaLaunchKernelEx(&cfg, gemm_dense_kernel<3>, twh, twl, txh, txl, a));
+    CB_CUDA(ctx, cudaFuncSetAttribute(gemm_dense_kernel<3, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    CB_CUDA(ctx, cudaLaunchKernelEx(&cfg, gemm_dense_kernel<3, false>, twh, twl, txh, txl, a));
   } else {
-    CB_CUDA(ctx, cudaFuncSetAttribute(gemm_dense_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    CB_CUDA(ctx, cudaLaunchKernelEx(&cfg, gemm_dense_kernel<1>, twh, twl, txh, txl, a));
+    CB_CUDA(ctx, cudaFuncSetAttribute(gemm_dense_kernel<1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    CB_CUDA(ctx, cudaLaunchKernelEx(&cfg, gemm_dense_kernel<1, false>, twh, twl, txh, txl, a));
+  }
+  CB_LAUNCH_CHECK(ctx, "gemm_dense_kernel");
+  return 0;
+}
+
+int launch_gemm_experts(caten_b200_ctx *ctx, const caten_b200_weight *w, const ExpertRows &er, BfOut x, int act, float *y, BfOut ybf, int nsplit) {
+  if (er.pairs <= 0) return 0;
+  if (!ctx->encode_tiled) return fail(ctx, CATEN_B200_ECUDA, "gemm_experts: cuTensorMapEncodeTiled is not available");
+  const int64_t N = w->rows, K = w->cols;
+  if (w->type != CATEN_B200_BF16 || K % GD_BK || er.experts < 1 || er.experts > GD_MAX_EXPERTS || N % er.experts || N / er.experts % 4 || N > 0x7fffffff || er.pairs > 0x7fffffff ||
+      act == CATEN_B200_ACT_GELU || act == CATEN_B200_ACT_RELU || !x.hi || (nsplit == 3 && !x.lo))
+    return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemm_experts: %d experts, weight %lldx%lld", er.experts, (long long)N, (long long)K);
+  GdArgs a;
+  a.bias = a.res = nullptr; a.y = y; a.yhi = ybf.hi; a.ylo = ybf.lo; a.status = ctx->d_status;
+  a.act = act; a.M = (int)er.pairs; a.N = (int)N; a.K = (int)K;
+  a.group_rows = (int)(N / er.experts); a.xplane = 0; a.ygroup = a.group_rows;
+  a.tiles_f = a.tiles_per_group = (a.group_rows + GD_BM - 1) / GD_BM;
+  a.ldy = act_is_glu(act) ? a.group_rows / 2 : a.group_rows;
+  a.tiles = 0;
+  // twice the rows an expert has on average, so that most experts need one row tile
+  int bn = 16;
+  while (bn < GD_BN && (int64_t)bn * er.experts < 2 * er.pairs) bn *= 2;
+  a.bn = bn;
+  a.er = er;
+  const int bk = nsplit == 3 ? GdStage<3>::BK : GdStage<1>::BK;
+  CUtensorMap tw, txh, txl;
+  if (int rc = make_map(ctx, &tw, w->qs, N, K, GD_BM, bk)) return rc;
+  if (int rc = make_map(ctx, &txh, x.hi, er.pairs, K, bn, bk)) return rc;
+  if (int rc = make_map(ctx, &txl, nsplit == 3 ? x.lo : x.hi, er.pairs, K, bn, bk)) return rc;
+  const size_t stage = (size_t)bk * 2 * (GD_BM + (size_t)bn * (nsplit == 3 ? 2 : 1));
+  int stages = (int)((196 * 1024) / stage);
+  if (stages > 10) stages = 10;
+  a.stages = stages;
+  a.idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(bn >> 3) << 17) | ((uint32_t)(GD_BM >> 4) << 24);
+  const size_t smem = 2048 + stage * stages + (size_t)GD_EPI_WARPS * 2048 + (GD_MAX_EXPERTS + 1) * sizeof(int);
+  const int64_t most = (er.pairs / bn + (er.pairs < er.experts ? er.pairs : er.experts)) * a.tiles_f;
+  const int grid = most < ctx->sm_count ? (int)most : ctx->sm_count;
+  if (nsplit == 3) {
+    CB_CUDA(ctx, cudaFuncSetAttribute(gemm_dense_kernel<3, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    launch_k(ctx, gemm_dense_kernel<3, true>, dim3((unsigned)grid), dim3(GD_THREADS), smem, tw, tw, txh, txl, a);
+  } else {
+    CB_CUDA(ctx, cudaFuncSetAttribute(gemm_dense_kernel<1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    launch_k(ctx, gemm_dense_kernel<1, true>, dim3((unsigned)grid), dim3(GD_THREADS), smem, tw, tw, txh, txl, a);
   }
   CB_LAUNCH_CHECK(ctx, "gemm_dense_kernel");
   return 0;

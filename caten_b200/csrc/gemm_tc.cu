@@ -54,8 +54,9 @@ struct TcArgs {
   int splits, cps;
   int cluster;  // 1: the `splits` CTAs of a tile form a thread-block cluster and reduce through distributed shared memory
   float *part;
-  // output rows [g * group_rows, (g + 1) * group_rows) read input plane g, `xplane` rows after the one before it
-  int group_rows, xplane;
+  // output rows [g * group_rows, (g + 1) * group_rows) read input plane g, `xplane` rows after the one before it, and go to
+  // columns [g * ygroup, ..) of rows of ldy; a group has tiles_per_group tiles, the last one possibly partial
+  int group_rows, xplane, ygroup, ldy, tiles_per_group;
   // when yhi is set the epilogue writes the result as split bf16 (operand of the next GEMM), not y
   __nv_bfloat16 *yhi, *ylo;
 };
@@ -316,13 +317,13 @@ template <> struct WRow<WT_F32_T> {
 template <int WT> constexpr int tc_threads() { return (WRow<WT>::GROUPS * 4 + 2) * 32; }
 
 // Two (gate, up) pairs of row m, features o .. o + 3 (o a multiple of 4), summed and gated: outputs o / 2 and o / 2 + 1.
-__device__ __forceinline__ void store_glu4(const float *r, const float *bias, int64_t o, int64_t N, int64_t m, float *y, __nv_bfloat16 *yhi,
+__device__ __forceinline__ void store_glu4(int act, const float *r, const float *bias, int64_t o, int64_t N, int64_t row_at, float *y, __nv_bfloat16 *yhi,
                                            __nv_bfloat16 *ylo) {
 #pragma unroll
   for (int e = 0; e < 4; e += 2) {
     if (o + e < N) {
-      const float v = relu_glu(bias ? r[e] + bias[o + e] : r[e], bias ? r[e + 1] + bias[o + e + 1] : r[e + 1]);
-      const int64_t at = m * (N / 2) + (o + e) / 2;
+      const float v = glu(act, bias ? r[e] + bias[o + e] : r[e], bias ? r[e + 1] + bias[o + e + 1] : r[e + 1]);
+      const int64_t at = row_at + (o + e) / 2;
       if (yhi) {
         const __nv_bfloat16 h = __float2bfloat16_rn(v);
         yhi[at] = h;
@@ -334,11 +335,11 @@ __device__ __forceinline__ void store_glu4(const float *r, const float *bias, in
   }
 }
 
-// Epilogue of one 16-column group held in registers: y[m, o] = act(acc + bias) + res.
+// Epilogue of one 16-column group held in registers: y[m, o] = act(acc + bias) + res; `o` is the output column.
 template <int ACT>
 __device__ __forceinline__ void epi_store16(const TcArgs &a, const uint32_t *r, float bias, int64_t o, int m_first) {
-  float *yp = a.y + (int64_t)m_first * a.N + o;
-  const float *rp = a.res ? a.res + (int64_t)m_first * a.N + o : nullptr;
+  float *yp = a.y + (int64_t)m_first * a.ldy + o;
+  const float *rp = a.res ? a.res + (int64_t)m_first * a.ldy + o : nullptr;
   const int lim = a.M - m_first < 16 ? a.M - m_first : 16;
 #pragma unroll
   for (int i = 0; i < 16; ++i) {
@@ -346,14 +347,14 @@ __device__ __forceinline__ void epi_store16(const TcArgs &a, const uint32_t *r, 
       float v = __uint_as_float(r[i]) + bias;
       if (ACT == CATEN_B200_ACT_GELU) v = gelu_ref(v);
       if (ACT == CATEN_B200_ACT_RELU) v = v > 0.0f ? v : 0.0f;
-      if (rp) v = rp[(int64_t)i * a.N] + v;
+      if (rp) v = rp[(int64_t)i * a.ldy] + v;
       if (a.yhi) {
-        const int64_t at = ((int64_t)m_first + i) * a.N + o;
+        const int64_t at = ((int64_t)m_first + i) * a.ldy + o;
         const __nv_bfloat16 h = __float2bfloat16_rn(v);
         a.yhi[at] = h;
         if (a.ylo) a.ylo[at] = __float2bfloat16_rn(v - __bfloat162float(h));
       } else {
-        yp[(int64_t)i * a.N] = v;
+        yp[(int64_t)i * a.ldy] = v;
       }
     }
   }
@@ -362,14 +363,13 @@ __device__ __forceinline__ void epi_store16(const TcArgs &a, const uint32_t *r, 
 // Gated form: the lane pair (2j, 2j + 1) of the warp holds a (gate, up) feature pair; the whole warp calls it.
 __device__ __forceinline__ void epi_glu16(const TcArgs &a, const uint32_t *r, float bias, int64_t o, bool o_ok, int m_first) {
   const int lim = a.M - m_first < 16 ? a.M - m_first : 16;
-  const int64_t n2 = a.N / 2;
 #pragma unroll
   for (int i = 0; i < 16; ++i) {
     const float mine = __uint_as_float(r[i]) + bias;
     const float other = __shfl_xor_sync(0xffffffffu, mine, 1);
     if (i < lim && o_ok && !(o & 1)) {
-      const float v = relu_glu(mine, other);
-      const int64_t at = ((int64_t)m_first + i) * n2 + (o >> 1);
+      const float v = glu(a.act, mine, other);
+      const int64_t at = ((int64_t)m_first + i) * a.ldy + (o >> 1);
       if (a.yhi) {
         const __nv_bfloat16 h = __float2bfloat16_rn(v);
         a.yhi[at] = h;
@@ -411,7 +411,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_hi, const __grid_constant_
   auto stage_xlo = [&](int s) { return smem + (size_t)s * stage_bytes + xbytes; };
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int n0 = blockIdx.x * TC_BM, m0 = blockIdx.y * bnx;
+  const int group = blockIdx.x / a.tiles_per_group;
+  const int n0 = group * a.group_rows + (blockIdx.x % a.tiles_per_group) * TC_BM, n_end = min(a.N, (group + 1) * a.group_rows), m0 = blockIdx.y * bnx;
+  const int shift = group * (a.group_rows - a.ygroup);   // output column = row of W - shift
   const int kc0 = blockIdx.z * a.cps;
   const int num_k = min(a.K / TC_BK - kc0, a.cps);  // chunks of this CTA: [kc0, kc0 + num_k)
 
@@ -448,7 +450,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_hi, const __grid_constant_
     // earlier chunks run, so conversion, barrier latency and the MMAs overlap.
     const int g = warp >> 2, quad = warp & 3;
     const int64_t row = (int64_t)n0 + quad * 32 + lane;
-    const bool row_ok = row < a.N;
+    const bool row_ok = row < n_end;
     const uint32_t t_quad = tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)TC_WCOL0;
     // An mbarrier wait tells two consecutive phases apart and no more, so a group must not skip
     // a phase of a stage's `empty` barrier: with S stages at most S groups take chunks (then a
@@ -524,12 +526,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_hi, const __grid_constant_
           tmem_ld_wait();
         }
         if (a.splits == 1) {
-          if (a.act == CATEN_B200_ACT_RELU_GLU) {
-            if (m0 + c < a.M) epi_glu16(a, r, bias, o, o_ok, m0 + c);
+          if (act_is_glu(a.act)) {
+            if (m0 + c < a.M) epi_glu16(a, r, bias, o - shift, o_ok, m0 + c);
           } else if (o_ok && m0 + c < a.M) {
-            if (a.act == CATEN_B200_ACT_GELU) epi_store16<CATEN_B200_ACT_GELU>(a, r, bias, o, m0 + c);
-            else if (a.act == CATEN_B200_ACT_RELU) epi_store16<CATEN_B200_ACT_RELU>(a, r, bias, o, m0 + c);
-            else epi_store16<CATEN_B200_ACT_NONE>(a, r, bias, o, m0 + c);
+            if (a.act == CATEN_B200_ACT_GELU) epi_store16<CATEN_B200_ACT_GELU>(a, r, bias, o - shift, m0 + c);
+            else if (a.act == CATEN_B200_ACT_RELU) epi_store16<CATEN_B200_ACT_RELU>(a, r, bias, o - shift, m0 + c);
+            else epi_store16<CATEN_B200_ACT_NONE>(a, r, bias, o - shift, m0 + c);
           }
         } else if (a.cluster) {
           // partial tile -> this CTA's shared memory, [column][row]; the stage buffers are free now
@@ -556,7 +558,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_hi, const __grid_constant_
       pdl_wait();  // x is written by the preceding kernel
       int issued = 0, s = 0;
       uint32_t ph = 0;
-      const int y0 = m0 + (n0 / a.group_rows) * a.xplane;  // first row of the input plane this tile's output rows read
+      const int y0 = m0 + group * a.xplane;  // first row of the input plane this tile's output rows read
       for (int kc = 0; kc < num_k; ++kc) {
         if (!mbar_wait(empty(s), ph ^ 1u, abort_flag)) {
           if (!*abort_flag) { *abort_flag = 1; atomicCAS(a.status, 0, DEV_WAIT_TIMEOUT); a.status[1] = 3; a.status[2] = kc; }
@@ -649,24 +651,25 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_hi, const __grid_constant_
           v.x += p.x; v.y += p.y; v.z += p.z; v.w += p.w;
         }
         const float r[4] = {v.x, v.y, v.z, v.w};
-        if (a.act == CATEN_B200_ACT_RELU_GLU) {
-          store_glu4(r, a.bias, (int64_t)n0 + r4, a.N, m, a.y, a.yhi, a.ylo);
+        if (act_is_glu(a.act)) {
+          store_glu4(a.act, r, a.bias, (int64_t)n0 + r4, n_end, m * a.ldy - shift / 2, a.y, a.yhi, a.ylo);
           continue;
         }
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int64_t o = (int64_t)n0 + r4 + e;
-          if (o < a.N) {
+          if (o < n_end) {
+            const int64_t at = m * a.ldy + o - shift;
             float t = r[e];
             if (a.bias) t = t + a.bias[o];
             t = apply_act(t, a.act);
-            if (a.res) t = a.res[m * a.N + o] + t;
+            if (a.res) t = a.res[at] + t;
             if (a.yhi) {
               const __nv_bfloat16 h = __float2bfloat16_rn(t);
-              a.yhi[m * a.N + o] = h;
-              if (a.ylo) a.ylo[m * a.N + o] = __float2bfloat16_rn(t - __bfloat162float(h));
+              a.yhi[at] = h;
+              if (a.ylo) a.ylo[at] = __float2bfloat16_rn(t - __bfloat162float(h));
             } else {
-              a.y[m * a.N + o] = t;
+              a.y[at] = t;
             }
           }
         }
@@ -687,14 +690,17 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_hi, const __grid_constant_
 // coalesced and the loads of different splits overlap.
 __global__ void __launch_bounds__(256) splitk_reduce_kernel(const float *__restrict__ part, int splits, int tiles_x, int tiles,
                                                             int bnx, const float *__restrict__ bias, const float *res, float *y,
-                                                            __nv_bfloat16 *yhi, __nv_bfloat16 *ylo, int act, int M, int N) {
+                                                            __nv_bfloat16 *yhi, __nv_bfloat16 *ylo, int act, int M, int N, int group_rows,
+                                                            int tiles_per_group, int ygroup, int ldy) {
   pdl_enter();
   const int64_t idx = (int64_t)blockIdx.x * 256 + threadIdx.x;
   const int row = (int)(idx & 31) * 4;
   const int64_t rest = idx >> 5;
   const int col = (int)(rest % bnx), tile = (int)(rest / bnx);
   if (tile >= tiles) return;
-  const int64_t o = (int64_t)(tile % tiles_x) * TC_BM + row, m = (int64_t)(tile / tiles_x) * bnx + col;
+  const int group = tile % tiles_x / tiles_per_group, shift = group * (group_rows - ygroup);
+  N = min(N, (group + 1) * group_rows);
+  const int64_t o = (int64_t)group * group_rows + (int64_t)(tile % tiles_x % tiles_per_group) * TC_BM + row, m = (int64_t)(tile / tiles_x) * bnx + col;
   if (o >= N || m >= M) return;
   const size_t zstride = (size_t)tiles * bnx * TC_BM;
   const float *p = part + ((size_t)tile * bnx + col) * TC_BM + row;
@@ -715,23 +721,24 @@ __global__ void __launch_bounds__(256) splitk_reduce_kernel(const float *__restr
     v.x += a0.x; v.y += a0.y; v.z += a0.z; v.w += a0.w;
   }
   float r[4] = {v.x, v.y, v.z, v.w};
-  if (act == CATEN_B200_ACT_RELU_GLU) {
-    store_glu4(r, bias, o, N, m, y, yhi, ylo);
+  if (act_is_glu(act)) {
+    store_glu4(act, r, bias, o, N, m * ldy - shift / 2, y, yhi, ylo);
     return;
   }
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
     if (o + e < N) {
+      const int64_t at = m * ldy + o + e - shift;
       float t = r[e];
       if (bias) t = t + bias[o + e];
       t = apply_act(t, act);
-      if (res) t = res[m * N + o + e] + t;
+      if (res) t = res[at] + t;
       if (yhi) {
         const __nv_bfloat16 h = __float2bfloat16_rn(t);
-        yhi[m * N + o + e] = h;
-        if (ylo) ylo[m * N + o + e] = __float2bfloat16_rn(t - __bfloat162float(h));
+        yhi[at] = h;
+        if (ylo) ylo[at] = __float2bfloat16_rn(t - __bfloat162float(h));
       } else {
-        y[m * N + o + e] = t;
+        y[at] = t;
       }
     }
   }
@@ -819,7 +826,7 @@ struct TcPlan {
   size_t stage_bytes;
 };
 
-static int tc_plan(caten_b200_ctx *ctx, const char *who, int64_t M, int64_t N, int64_t K, int nsplit, int split_cap, TcPlan *p) {
+static int tc_plan(caten_b200_ctx *ctx, const char *who, int64_t M, int64_t N, int64_t K, int nsplit, int split_cap, TcPlan *p, int64_t group_rows = 0) {
   if (!ctx->encode_tiled) return fail(ctx, CATEN_B200_ECUDA, "%s: cuTensorMapEncodeTiled is not available", who);
   if (K % TC_BK) return fail(ctx, CATEN_B200_EUNSUPPORTED, "%s: inner dimension %lld is not a multiple of 64", who, (long long)K);
   if (M > 0x7fffffff || N > 0x7fffffff || K > 0x7fffffff) return fail(ctx, CATEN_B200_EUNSUPPORTED, "%s: dimension too large", who);
@@ -833,7 +840,7 @@ static int tc_plan(caten_b200_ctx *ctx, const char *who, int64_t M, int64_t N, i
   p->stage_bytes = (size_t)bnx * 128 * (nsplit == 3 ? 2 : 1);
   p->gy = (M + bnx - 1) / bnx;
   if (p->gy > 65535) return fail(ctx, CATEN_B200_EUNSUPPORTED, "%s: too many rows for one launch (%lld)", who, (long long)M);
-  p->gx = (N + TC_BM - 1) / TC_BM;
+  p->gx = group_rows ? (N + group_rows - 1) / group_rows * ((group_rows + TC_BM - 1) / TC_BM) : (N + TC_BM - 1) / TC_BM;
   p->tiles = p->gx * p->gy;
   // split-K when the output tiles alone cannot occupy the GPU (decode: few activation rows)
   const int num_k = (int)(K / TC_BK);
@@ -862,7 +869,7 @@ static int run_tc(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *x,
                   const __nv_bfloat16 *xhi_pre = nullptr, const __nv_bfloat16 *xlo_pre = nullptr, BfOut ybf = BfOut(),
                   PartIn *defer = nullptr, LinGroups grp = LinGroups()) {
   if (defer) *defer = PartIn();
-  if (grp.group_rows % TC_BM) return fail(ctx, CATEN_B200_EINVAL, "gemm_tc: input groups must be multiples of %d rows", TC_BM);
+  if (grp.group_rows % 4 || grp.ygroup % 4 || grp.ldy % 4 || (res && !grp.plain_output())) return fail(ctx, CATEN_B200_EINVAL, "gemm_tc: bad input groups or output layout");
   if (grp.group_rows && !xhi_pre) return fail(ctx, CATEN_B200_EINVAL, "gemm_tc: grouped inputs are given as bf16");
   if (M <= 0 || N <= 0) return 0;
   // thousands of rows (prefill): expand the weights once, both operands through TMA
@@ -871,9 +878,10 @@ static int run_tc(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *x,
   if (gemm_dense_applies(ctx, M, N, K) && !(align_bits & 15)) return launch_gemm_dense(ctx, wt, ws, x, xhi_pre, xlo_pre, bias, res, act, y, ybf, M, N, K, nsplit, grp);
   TcPlan p;
   // reduce inside a cluster: always (mode 1) or only when this launch needs its own epilogue (mode 2)
-  const bool own_epilogue = !(defer && act == CATEN_B200_ACT_NONE && !ybf.hi && N % 4 == 0);
+  const bool can_defer = defer && act == CATEN_B200_ACT_NONE && !ybf.hi && N % 4 == 0 && grp.plain_output() && grp.group_rows % TC_BM == 0;
+  const bool own_epilogue = !can_defer;
   const bool want_cluster = ctx->splitk_cluster == 1 || (ctx->splitk_cluster == 2 && own_epilogue);
-  if (int rc = tc_plan(ctx, "gemm_tc", M, N, K, nsplit, want_cluster ? 8 : 32, &p)) return rc;  // 8 = portable cluster size
+  if (int rc = tc_plan(ctx, "gemm_tc", M, N, K, nsplit, want_cluster ? 8 : 32, &p, grp.group_rows)) return rc;  // 8 = portable cluster size
   uint8_t *xhi, *xlo;
   if (xhi_pre) {
     // the producer of x already wrote the split bf16 operand
@@ -899,6 +907,9 @@ static int run_tc(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *x,
 
   TcArgs a;
   a.group_rows = grp.group_rows ? (int)grp.group_rows : (int)(p.gx * TC_BM); a.xplane = (int)grp.xplane;
+  a.ygroup = grp.ygroup ? (int)grp.ygroup : a.group_rows;
+  a.ldy = grp.ldy ? (int)grp.ldy : (int)(act_is_glu(act) ? N / 2 : N);
+  a.tiles_per_group = (a.group_rows + TC_BM - 1) / TC_BM;
   a.qs = ws.qs; a.d = ws.d; a.m = ws.m; a.qh = ws.qh; a.bias = bias; a.res = res; a.y = y; a.status = ctx->d_status; a.act = act;
   a.yhi = ybf.hi; a.ylo = ybf.lo;
   a.M = (int)M; a.N = (int)N; a.K = (int)K; a.nkb = (int)ws.nkb; a.bnx = p.bnx;
@@ -916,7 +927,7 @@ static int run_tc(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *x,
   const dim3 grid((unsigned)p.gx, (unsigned)p.gy, (unsigned)p.splits);
   const int rc = launch_tc(ctx, wt, nsplit, mh, ml, a, grid, smem);
   if (rc || p.splits == 1 || a.cluster) return rc;
-  if (defer && act == CATEN_B200_ACT_NONE && !a.yhi && N % 4 == 0) {
+  if (can_defer) {
     // the consumer of this linear sums the partial tiles itself (and adds bias / residual)
     defer->part = a.part; defer->bias = bias; defer->splits = p.splits; defer->tiles_x = (int)p.gx; defer->bnx = p.bnx;
     defer->zstride = (long long)p.tiles * p.bnx * TC_BM;
@@ -924,7 +935,7 @@ static int run_tc(caten_b200_ctx *ctx, int wt, const WSrc &ws, const float *x,
   }
   const int64_t total = p.tiles * p.bnx * (TC_BM / 4);
   launch_k(ctx, splitk_reduce_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, a.part, p.splits, (int)p.gx, (int)p.tiles, p.bnx, bias,
-                                                                              res, y, a.yhi, a.ylo, act, (int)M, (int)N);
+                                                                              res, y, a.yhi, a.ylo, act, (int)M, (int)N, a.group_rows, a.tiles_per_group, a.ygroup, a.ldy);
   CB_LAUNCH_CHECK(ctx, "splitk_reduce_kernel");
   return 0;
 }
@@ -983,7 +994,7 @@ int launch_gemm_tc_noalloc(caten_b200_ctx *ctx, const caten_b200_weight *w, cons
   if (int rc = make_x_map(ctx, &ml, nsplit == 3 ? xlo : xhi, M, K, p.bnx)) return rc;
 
   TcArgs a;
-  a.group_rows = (int)(p.gx * TC_BM); a.xplane = 0;
+  a.group_rows = a.ygroup = (int)(p.gx * TC_BM); a.xplane = 0; a.tiles_per_group = (int)p.gx; a.ldy = (int)(act_is_glu(act) ? N / 2 : N);
   a.qs = w->qs; a.d = w->d; a.m = w->m; a.qh = w->qh; a.bias = bias; a.res = res; a.y = y; a.status = ctx->d_status; a.act = act;
   a.yhi = nullptr; a.ylo = nullptr;
   a.M = (int)M; a.N = (int)N; a.K = (int)K; a.nkb = (int)w->nkb; a.bnx = p.bnx;
@@ -996,7 +1007,7 @@ int launch_gemm_tc_noalloc(caten_b200_ctx *ctx, const caten_b200_weight *w, cons
   if (rc || p.splits == 1) return rc;
   const int64_t total = p.tiles * p.bnx * (TC_BM / 4);
   launch_k(ctx, splitk_reduce_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, a.part, p.splits, (int)p.gx, (int)p.tiles, p.bnx, bias,
-                                                                              res, y, a.yhi, a.ylo, act, (int)M, (int)N);
+                                                                              res, y, a.yhi, a.ylo, act, (int)M, (int)N, a.group_rows, a.tiles_per_group, a.ygroup, a.ldy);
   CB_LAUNCH_CHECK(ctx, "splitk_reduce_kernel");
   return 0;
 }

@@ -152,24 +152,35 @@ template <> struct DenseLoad<__nv_bfloat16> {
   }
 };
 
-// blockIdx.y = group of `group_rows` output rows with an input plane of its own (one group: N rows)
-template <typename T, int RI>
+// blockIdx.y = group of `group_rows` output rows with an input plane of its own (one group: N rows).  EXPERTS: blockIdx.y
+// is a (token, expert) pair; expert[pair] says which group of rows it uses, its input is row pair / xplane, its products
+// are scaled by weight[pair].
+template <typename T, int RI, bool EXPERTS>
 __global__ void __launch_bounds__(256) gemv_dense_kernel(const T *__restrict__ W, const float *__restrict__ x,
                                                          const float *__restrict__ bias, const float *__restrict__ res,
-                                                         float *__restrict__ y, int act, int N, int K, int group_rows, int64_t xplane) {
+                                                         float *__restrict__ y, int act, int N, int K, int group_rows, int64_t xplane, int64_t ygroup,
+                                                         const int *__restrict__ expert, const float *__restrict__ weight) {
   extern __shared__ float xs[];
-  {
+  float wt = 1.0f;
+  if (EXPERTS) {
+    pdl_enter();   // which rows to read comes from the kernel before
+    W += (int64_t)expert[blockIdx.y] * group_rows * K;
+    x += (int64_t)(blockIdx.y / xplane) * K;
+    y += (int64_t)blockIdx.y * ygroup;
+    if (weight) wt = weight[blockIdx.y];
+    N = group_rows;
+  } else {
     const int64_t r0 = (int64_t)blockIdx.y * group_rows;
     W += r0 * K;
     x += (int64_t)blockIdx.y * xplane * K;
-    y += r0;
+    y += (int64_t)blockIdx.y * ygroup;
     if (bias) bias += r0;
     if (res) res += r0;
     N = N - r0 < group_rows ? (int)(N - r0) : group_rows;
   }
   // weights depend on no other kernel: the first tile of this warp's rows is loaded before the
   // wait for the producer of x
-  pdl_launch_dependents();
+  if (!EXPERTS) pdl_launch_dependents();
   constexpr int VEC = DenseLoad<T>::VEC;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int nvec = K / VEC;
@@ -183,7 +194,7 @@ __global__ void __launch_bounds__(256) gemv_dense_kernel(const T *__restrict__ W
       for (int j = 0; j < VEC; ++j) w0[i][j] = 0.0f;
     }
   }
-  pdl_wait();
+  if (!EXPERTS) pdl_wait();
   for (int i = threadIdx.x; i < K; i += blockDim.x) xs[i] = x[i];
   __syncthreads();
   for (int64_t base = first; base < N; base += (int64_t)gridDim.x * 8 * RI) {
@@ -227,11 +238,12 @@ __global__ void __launch_bounds__(256) gemv_dense_kernel(const T *__restrict__ W
         }
       }
     }
-    if (RI == 2 && act == CATEN_B200_ACT_RELU_GLU) {  // rows (base, base + 1) are a (gate, up) pair: base is even
+    if (RI == 2 && act_is_glu(act)) {  // rows (base, base + 1) are a (gate, up) pair: base is even
       float g = warp_sum(acc[0]), u = warp_sum(acc[RI - 1]);
       if (lane == 0 && base < N) {
         if (bias) { g = g + bias[base]; u = u + bias[base + 1]; }
-        y[base >> 1] = relu_glu(g, u);
+        if (EXPERTS) { g = g * wt; u = u * wt; }
+        y[base >> 1] = glu(act, g, u);
       }
       continue;
     }
@@ -241,6 +253,7 @@ __global__ void __launch_bounds__(256) gemv_dense_kernel(const T *__restrict__ W
       const int64_t row = base + i;
       if (lane == 0 && row < N) {
         if (bias) s = s + bias[row];
+        if (EXPERTS) s = s * wt;
         s = apply_act(s, act);
         if (res) s = res[row] + s;
         y[row] = s;
@@ -269,7 +282,7 @@ int launch_gemv(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x,
   if (w->rows > 0x7fffffff || w->cols > 0x7fffffff) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv: dimension too large");
   const int N = (int)w->rows, K = (int)w->cols;
   if (type_is_packed(w->type)) {
-    if (grp.group_rows || act == CATEN_B200_ACT_RELU_GLU) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv: input groups and the gated activation take dense weights");
+    if (grp.group_rows || act_is_glu(act)) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv: input groups and the gated activation take dense weights");
     GemvArgs a;
     a.qs = w->qs; a.d = w->d; a.m = w->m; a.qh = w->qh; a.x = x; a.bias = bias; a.res = res; a.y = y; a.act = act; a.N = N;
     a.nkb = (int)w->nkb;
@@ -290,7 +303,8 @@ int launch_gemv(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x,
   const int ng = grp.group_rows > 0 ? (int)((N + grp.group_rows - 1) / grp.group_rows) : 1;
   const int rows = grp.group_rows > 0 ? (int)grp.group_rows : N;  // per group
   // two rows per warp when that still gives every SM a CTA (or the rows are pairs), else one row per warp (more CTAs)
-  const bool two = act == CATEN_B200_ACT_RELU_GLU || ((int64_t)rows + 15) / 16 * ng >= ctx->sm_count;
+  const int64_t ygroup = grp.ygroup ? grp.ygroup : rows;
+  const bool two = act_is_glu(act) || ((int64_t)rows + 15) / 16 * ng >= ctx->sm_count;
   const int64_t groups = two ? ((int64_t)rows + 15) / 16 : ((int64_t)rows + 7) / 8;
   int64_t grid = ((int64_t)ctx->sm_count * 4 + ng - 1) / ng;
   if (grid > groups) grid = groups;
@@ -298,12 +312,12 @@ int launch_gemv(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x,
   do {                                                                                                                           \
     if (K % DenseLoad<CT>::VEC) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv " T ": cols %% %d != 0", DenseLoad<CT>::VEC);    \
     if (smem > 48 * 1024) {                                                                                                      \
-      cudaFuncSetAttribute(gemv_dense_kernel<CT, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                    \
-      cudaFuncSetAttribute(gemv_dense_kernel<CT, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                    \
+      cudaFuncSetAttribute(gemv_dense_kernel<CT, 2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);             \
+      cudaFuncSetAttribute(gemv_dense_kernel<CT, 1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);             \
     }                                                                                                                            \
     const dim3 g((unsigned)grid, (unsigned)ng);                                                                                  \
-    if (two) launch_k(ctx, gemv_dense_kernel<CT, 2>, g, dim3(256), smem, (const CT *)w->qs, x, bias, res, y, act, N, K, rows, grp.xplane); \
-    else launch_k(ctx, gemv_dense_kernel<CT, 1>, g, dim3(256), smem, (const CT *)w->qs, x, bias, res, y, act, N, K, rows, grp.xplane);     \
+    if (two) launch_k(ctx, gemv_dense_kernel<CT, 2, false>, g, dim3(256), smem, (const CT *)w->qs, x, bias, res, y, act, N, K, rows, grp.xplane, ygroup, nullptr, nullptr); \
+    else launch_k(ctx, gemv_dense_kernel<CT, 1, false>, g, dim3(256), smem, (const CT *)w->qs, x, bias, res, y, act, N, K, rows, grp.xplane, ygroup, nullptr, nullptr);     \
   } while (0)
   switch (w->type) {
     case CATEN_B200_F32: GEMV_DENSE("f32", float); break;
@@ -312,6 +326,27 @@ int launch_gemv(caten_b200_ctx *ctx, const caten_b200_weight *w, const float *x,
     default: return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv: weight type %d", w->type);
   }
 #undef GEMV_DENSE
+  CB_LAUNCH_CHECK(ctx, "gemv_dense_kernel");
+  return 0;
+}
+
+int launch_gemv_experts(caten_b200_ctx *ctx, const caten_b200_weight *w, int64_t rows, const float *x, const int *expert, const float *weight,
+                        int64_t pairs, int xdiv, int act, float *y) {
+  if (pairs <= 0) return 0;
+  const int64_t K = w->cols;
+  const size_t smem = (size_t)K * sizeof(float);
+  if (w->type != CATEN_B200_BF16 || K % 8 || rows % 2) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv: experts take BF16 weights");
+  if (smem > 160 * 1024 || pairs > 65535) return fail(ctx, CATEN_B200_EUNSUPPORTED, "gemv: cols=%lld or %lld pairs", (long long)K, (long long)pairs);
+  const bool two = act_is_glu(act) || (rows + 15) / 16 * pairs >= ctx->sm_count;
+  const int64_t groups = two ? (rows + 15) / 16 : (rows + 7) / 8;
+  int64_t grid = ((int64_t)ctx->sm_count * 4 + pairs - 1) / pairs;
+  if (grid > groups) grid = groups;
+  const dim3 g((unsigned)grid, (unsigned)pairs);
+  const float *none = nullptr;
+  const int64_t ld = act_is_glu(act) ? rows / 2 : rows;
+  auto kernel = two ? gemv_dense_kernel<__nv_bfloat16, 2, true> : gemv_dense_kernel<__nv_bfloat16, 1, true>;
+  if (smem > 48 * 1024) CB_CUDA(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  launch_k(ctx, kernel, g, dim3(256), smem, (const __nv_bfloat16 *)w->qs, x, none, none, y, act, (int)rows, (int)K, (int)rows, (int64_t)xdiv, ld, expert, weight);
   CB_LAUNCH_CHECK(ctx, "gemv_dense_kernel");
   return 0;
 }

@@ -1,0 +1,52 @@
+// Latent attention (latent.cu): queries, keys and values of all heads come from low-rank latents, and the cache
+// holds one normed latent and one rotated key part per token.  Arguments and launchers.
+#pragma once
+#include "common.cuh"
+
+namespace cb {
+
+struct LatentArgs {
+  int H = 0, D = 0, Dp = 0, P = 0, Pp = 0, E = 0, Ep = 0;   // heads; unrotated and rotated query/key dims, value dims, and their storage (p16)
+  int K = 0, Kp = 0, Kr = 0;        // latent size, its storage in the cache (p16) and as a linear's input (p64)
+  int Q = 0, Qr = 0;                // query latent size, and as a linear's input (p64)
+  const float *freq = nullptr;      // [P / 2]: rotated dims i and i + P / 2 turn by position * freq[i]
+  const float *q_norm = nullptr, *kv_norm = nullptr;   // [Qr], [Kp] gains of the latents (zero in the padding)
+  float eps = 0.0f, scale = 1.0f;   // score = (q . k) * scale
+  // cache [B, cap, Kp + Pp]: latent, rotated key part; bf16 or fp32
+  void *cache = nullptr;
+  bool cache_bf16 = false;
+  int64_t cap = 0;
+  int B = 0, s = 0, n = 0;          // s tokens per sequence at positions n ..
+  const int *d_n = nullptr;         // single-token steps: position on the device
+
+  int KC() const { return Kp + Pp; }
+  int Dq() const { return Dp + Pp; }
+};
+
+// Rows of the projection [query latent (Qr) | latent (Kp) | key part (Pp)] (y, or its split-K partial tiles): the normed query
+// latent [rows, Qr] as the next linear's input, the normed latent and the rotated key part into the cache.
+int launch_latent_prep(caten_b200_ctx *ctx, const LatentArgs &a, const float *y, PartIn pin, int64_t ld, float *cq, BfOut cq_bf);
+// Queries [rows, ld], head h at column h * Dq, for the expanded form: rotated and scaled in place.
+int launch_latent_q_expanded(caten_b200_ctx *ctx, const LatentArgs &a, float *q, int64_t ld);
+// Queries (or their partial tiles) for the absorbed form: unrotated parts as planes [H][plane][p64(D)] (input of the product with
+// W_uk^T), rotated parts into qcat [rows, H, Kp + Pp] from column Kp on.
+int launch_latent_q_absorbed(caten_b200_ctx *ctx, const LatentArgs &a, const float *q, PartIn pin, int64_t ld, int64_t plane, float *qn, BfOut qn_bf,
+                             float *qcat, BfOut qcat_bf);
+// Cached rows [0, t) of sequences b0 .. b0 + nb: latents [nb * t, Kr] as a linear's input, key parts [nb * t, Pp] in fp32.
+int launch_latent_gather(caten_b200_ctx *ctx, const LatentArgs &a, int b0, int nb, int t, float *c, BfOut c_bf, float *kr);
+
+struct LatentAbsorbed {
+  const float *qcat = nullptr;      // [rows, H, Kp + Pp] fp32, or
+  BfOut qcat_bf;                    // bf16
+  float *o = nullptr;               // planes [H][plane][Kr]: sum_j p_j c_j per head; fp32, or
+  BfOut o_bf;                       // bf16
+  int64_t plane = 0;
+  float *part = nullptr, *ml = nullptr;   // several splits: [splits, rows, H, Kr] and [splits, rows, H, 2]
+  int splits = 1;
+};
+// Key splits of a launch over `rows` rows that may see `keys` keys.
+int latent_splits(const caten_b200_ctx *ctx, const LatentArgs &a, int64_t rows, int64_t keys);
+// Softmax attention of every row (sequence, token) over its cached latents.
+int launch_latent_absorbed(caten_b200_ctx *ctx, const LatentArgs &a, const LatentAbsorbed &x);
+
+}  // namespace cb

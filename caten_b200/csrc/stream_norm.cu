@@ -5,9 +5,12 @@
 //           EMBED  a row of the token embedding (kept in x0 as well when a later stage needs it)
 //           COPY   the output y of a linear
 //           ADD    x + y * post / rms(y)          (norm of the sublayer's output, then the residual sum)
+//           SUM    x + y [+ the outputs of the row's experts]
 //           KEEP   x as it is
 //   out   what the next operation reads
 //           NORM   x * pre / rms(x)
+//           NORM2  x * w1 / rms(x) and x * w2 / rms(x), a gain per coordinate (mixer and feed-forward side by side);
+//                  before that the row may get the step vector of a loop pass and the embedding output
 //           SHIFT  NORM, then the five token-shift mixes h + (h_prev - h) * mu of a time-mixing layer
 //                  (single-token steps: h_prev comes from the carried state, which becomes h)
 //           CONCAT [x ; x0]
@@ -51,6 +54,9 @@ __device__ __forceinline__ float4 mix4(float4 h, float4 p, float4 mu) {
   return make_float4(fmaf(p.x - h.x, mu.x, h.x), fmaf(p.y - h.y, mu.y, h.y), fmaf(p.z - h.z, mu.z, h.z), fmaf(p.w - h.w, mu.w, h.w));
 }
 
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+__device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+
 template <int IN, int OUT, int MAXV>
 __global__ void __launch_bounds__(SN_THREADS) stream_norm_kernel(const StreamArgs a) {
   __shared__ float red[SN_THREADS / 32];
@@ -84,7 +90,7 @@ __global__ void __launch_bounds__(SN_THREADS) stream_norm_kernel(const StreamArg
     for (int i = 0; i < MAXV; ++i) {
       const int c = threadIdx.x + SN_THREADS * i;
       if (c < d4) {
-        if (IN == SN_ADD) xr[i] = reinterpret_cast<const float4 *>(a.x)[src * d4 + c];
+        if (IN == SN_ADD || IN == SN_SUM) xr[i] = reinterpret_cast<const float4 *>(a.x)[src * d4 + c];
         v[i] = a.pin.splits > 0 ? partin_load4(a.pin, src, 4 * c) : reinterpret_cast<const float4 *>(a.y)[src * d4 + c];
       }
     }
@@ -104,15 +110,42 @@ __global__ void __launch_bounds__(SN_THREADS) stream_norm_kernel(const StreamArg
         }
       }
     }
+    if (IN == SN_SUM) {
+      for (int k = 0; k < a.top; ++k) {
+        const int64_t p = a.pos ? a.pos[src * a.top + k] : src * a.top + k;
+#pragma unroll
+        for (int i = 0; i < MAXV; ++i) {
+          const int c = threadIdx.x + SN_THREADS * i;
+          if (c < d4) v[i] = add4(v[i], reinterpret_cast<const float4 *>(a.ye)[p * d4 + c]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < MAXV; ++i)
+        if (threadIdx.x + SN_THREADS * i < d4) v[i] = add4(xr[i], v[i]);
+    }
   }
-  if (IN != SN_KEEP && a.x_out) {
+  if (IN == SN_EMBED && a.x_out && a.x0) {
+#pragma unroll
+    for (int i = 0; i < MAXV; ++i) {
+      const int c = threadIdx.x + SN_THREADS * i;
+      if (c < d4) reinterpret_cast<float4 *>(a.x0)[src * d4 + c] = v[i];
+    }
+  }
+  if (OUT == SN_NORM2 && a.step) {
 #pragma unroll
     for (int i = 0; i < MAXV; ++i) {
       const int c = threadIdx.x + SN_THREADS * i;
       if (c < d4) {
-        reinterpret_cast<float4 *>(a.x_out)[src * d4 + c] = v[i];
-        if (IN == SN_EMBED && a.x0) reinterpret_cast<float4 *>(a.x0)[src * d4 + c] = v[i];
+        if (a.add_x0) v[i] = add4(v[i], reinterpret_cast<const float4 *>(a.x0)[src * d4 + c]);
+        v[i] = add4(v[i], reinterpret_cast<const float4 *>(a.step)[c]);
       }
+    }
+  }
+  if ((IN != SN_KEEP || (OUT == SN_NORM2 && a.step)) && a.x_out) {
+#pragma unroll
+    for (int i = 0; i < MAXV; ++i) {
+      const int c = threadIdx.x + SN_THREADS * i;
+      if (c < d4) reinterpret_cast<float4 *>(a.x_out)[src * d4 + c] = v[i];
     }
   }
   if (OUT == SN_NORM || OUT == SN_SHIFT) {
@@ -139,6 +172,22 @@ __global__ void __launch_bounds__(SN_THREADS) stream_norm_kernel(const StreamArg
             sn_store(a.h, a.hb, (j * a.plane + row) * d4 + c, mix4(h, p, mu));
           }
         }
+      }
+    }
+  }
+  if (OUT == SN_NORM2) {
+    float sq = 0.0f;
+#pragma unroll
+    for (int i = 0; i < MAXV; ++i)
+      if (threadIdx.x + SN_THREADS * i < d4) sq += sq4(v[i]);
+    const float rs = 1.0f / sqrtf(sn_block_sum(sq, red) * a.invd + a.eps);
+#pragma unroll
+    for (int i = 0; i < MAXV; ++i) {
+      const int c = threadIdx.x + SN_THREADS * i;
+      if (c < d4) {
+        const float4 u = make_float4(v[i].x * rs, v[i].y * rs, v[i].z * rs, v[i].w * rs);
+        sn_store(a.h, a.hb, row * d4 + c, mul4(u, reinterpret_cast<const float4 *>(a.w1)[c]));
+        if (a.w2) sn_store(a.h, a.hb, (a.plane + row) * d4 + c, mul4(u, reinterpret_cast<const float4 *>(a.w2)[c]));
       }
     }
   }
@@ -180,6 +229,13 @@ int launch_stream_norm(caten_b200_ctx *ctx, int in, int out, const StreamArgs &a
   if (rows <= 0) return 0;
   if (a.d4 < 1 || a.d4 > 8 * SN_THREADS) return fail(ctx, CATEN_B200_EUNSUPPORTED, "stream_norm: width %d (at most 8192)", 4 * a.d4);
   if (rows > 0x7fffffff) return fail(ctx, CATEN_B200_EUNSUPPORTED, "stream_norm: too many rows");
+  if (out == SN_NORM2 || in == SN_SUM) {   // the pairs a decoder with parallel sublayers uses
+    if (out == SN_NORM2 && in == SN_EMBED) return launch_sn<SN_EMBED, SN_NORM2>(ctx, a, rows);
+    if (out == SN_NORM2 && in == SN_KEEP) return launch_sn<SN_KEEP, SN_NORM2>(ctx, a, rows);
+    if (out == SN_NORM2 && in == SN_SUM) return launch_sn<SN_SUM, SN_NORM2>(ctx, a, rows);
+    if (out == SN_NONE && in == SN_SUM) return launch_sn<SN_SUM, SN_NONE>(ctx, a, rows);
+    return fail(ctx, CATEN_B200_EUNSUPPORTED, "stream_norm: stages %d, %d", in, out);
+  }
   switch (in) {
     case SN_EMBED: return launch_sn_in<SN_EMBED>(ctx, out, a, rows);
     case SN_COPY: return launch_sn_in<SN_COPY>(ctx, out, a, rows);

@@ -18,7 +18,6 @@ namespace cb {
 
 namespace {
 
-__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float decay(float d) { return expf(-expf(d)); }
 
 __device__ __forceinline__ void st_out(float *out, BfOut bf, int64_t at, float v) {
@@ -504,8 +503,8 @@ static int check_wkv(caten_b200_ctx *ctx, const WkvArgs &a) {
 static int launch_chunked(caten_b200_ctx *ctx, const WkvArgs &a) {
   const int chunks = (a.s + WC_T - 1) / WC_T;
   const size_t n = (size_t)a.B * a.H * chunks;
-  if (int rc = scratch_reserve(ctx, &ctx->wkv_chunks, n * (WC_D * WC_D + WC_D) * sizeof(float))) return rc;
-  float *U = (float *)ctx->wkv_chunks.ptr, *decays = U + n * (WC_D * WC_D);
+  if (int rc = scratch_reserve(ctx, &ctx->chunk_states, n * (WC_D * WC_D + WC_D) * sizeof(float))) return rc;
+  float *U = (float *)ctx->chunk_states.ptr, *decays = U + n * (WC_D * WC_D);
   const dim3 grid((unsigned)chunks, (unsigned)a.H, (unsigned)a.B);
   CB_CUDA(ctx, cudaFuncSetAttribute(wkv_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)WC_SMEM));
   launch_k(ctx, wkv_chunk_kernel, grid, dim3(WC_THREADS), WC_SMEM, a, U, decays);

@@ -21,7 +21,12 @@ def _binusun(path: str, runtime: Optional[B200Runtime], **kw) -> Model:
     return binusun.load(path, runtime, **kw)
 
 
-ARCHITECTURES = {"gpt2": _gpt2, "Binusun": _binusun}
+def _goselix(path: str, runtime: Optional[B200Runtime], **kw) -> Model:
+    from . import goselix
+    return goselix.load(path, runtime, **kw)
+
+
+ARCHITECTURES = {"gpt2": _gpt2, "Binusun": _binusun, "Goselix": _goselix}
 
 
 def architecture_of(path: str) -> str:

@@ -55,7 +55,9 @@ enum { CATEN_B200_ACT_NONE = 0, CATEN_B200_ACT_GELU = 1, CATEN_B200_ACT_RELU = 2
   /* gated: the weight's rows come in (gate, up) pairs, rows 2j and 2j + 1, and the linear has rows / 2
    * outputs y[m, j] = max(gate, 0) * up.  Dense weights (F32, F16, BF16), an even number of rows, no
    * residual. */
-  CATEN_B200_ACT_RELU_GLU = 3 };
+  CATEN_B200_ACT_RELU_GLU = 3,
+  /* the same with silu(gate) * up, silu(z) = z / (1 + exp(-z)) */
+  CATEN_B200_ACT_SILU_GLU = 4 };
 
 /* arithmetic of the Linear kernels when more than a few rows are multiplied at once:
  *   FP32    fp32 operands and accumulation on the CUDA cores (max-abs 1e-3 logit class)
@@ -320,9 +322,11 @@ int caten_b200_wkv(caten_b200_ctx *ctx, const caten_b200_wkv_desc *desc, const f
  * run several times with the same weights (every pass has its own cache or state).  RMS norms with one
  * scalar gain stand before and after every sublayer:
  *   x += rms(mixer(rms(x) * norm1)) * norm1b;   x += rms(ff(rms(x) * norm2)) * norm2b
+ * or, in a `parallel` layer, mixer and feed-forward read the same stream through norms with a gain per coordinate:
+ *   x += mixer(rms(x) * norm1_w) + ff(rms(x) * norm2_w)
  * Storage: heads are padded with zeros to a multiple of 16 (p16), rows of activations and the columns
  * of weights to a multiple of 64 (p64); padded weight entries are zero.  wp = p64(width). */
-enum { CATEN_B200_MIX_ATTENTION = 0, CATEN_B200_MIX_WKV = 1 };
+enum { CATEN_B200_MIX_ATTENTION = 0, CATEN_B200_MIX_WKV = 1, CATEN_B200_MIX_LATENT = 2, CATEN_B200_MIX_RETENTION = 3 };
 typedef struct {
   int32_t mixer;               /* CATEN_B200_MIX_* */
   int32_t heads, dim;          /* query heads / heads of the recurrence and their size (<= 256) */
@@ -347,6 +351,27 @@ typedef struct {
   const caten_b200_weight *w2;      /* time mixing, BF16: [p64(heads * p16(dim)), low_rank] */
   const caten_b200_weight *ff_in;   /* (gate, up) row pairs [2 * p64(ff), wp]; NULL: no feed-forward */
   const caten_b200_weight *ff_out;  /* [wp, p64(ff)] */
+  /* latent attention: per head dim unrotated and rot_dims rotated query/key dims (rotated dims i and i + rot_dims / 2 turn by
+   * position * rot_freq[i]), vdim value dims; queries from a normed latent of q_rank, keys and values from one of kv_rank, which
+   * is cached beside one rotated key part for all heads.  q_norm [p64(q_rank)], kv_norm [p16(kv_rank)] (zero padding).
+   *   in_w   rows: query latent (p64), latent (p16), key part (p16), padded to p64; cols wp
+   *   uq_w   [heads * (p16(dim) + p16(rot_dims)), p64(q_rank)]
+   *   uk_w   BF16, the key projection transposed per head: [heads * p16(kv_rank), p64(dim)]
+   *   kv_w   BF16 [heads * p16(dim) + heads * p16(vdim), p64(kv_rank)]: keys of all heads, then values
+   * retention: state S[key, value] per head, S = decay S + k v^T, o = S^T q, then o / rms(o) * silu(gate); q and k rotated as above
+   * (rot_dims of dim), k times dim^(-1/2); powers [heads, 65]: decay^0 .. decay^64.
+   *   in_w   rows: q, k [heads * p16(dim)], v, gate [heads * p16(vdim)], padded to p64; cols wp */
+  int32_t kv_rank, q_rank;
+  /* parallel layers: out_w reads the mixer's output beside the feed-forward's activations, [wp, p64(heads * p16(vdim)) + p64(ff)]
+   * with ff_out NULL; ff_act CATEN_B200_ACT_*_GLU (sequential layers: RELU_GLU) */
+  int32_t parallel, ff_act;
+  /* experts > 0 (parallel layers): the feed-forward is a mixture.  Every row uses the `top` experts with the largest sigmoid(router
+   * logit), an expert's input is scaled by it, the outputs are added.  router BF16 [p64(experts), wp]; ff_in BF16
+   * [experts * 2 * p64(ff), wp], ff_out BF16 [experts * wp, p64(ff)]: the experts' weights one after the other; out_w without ff */
+  int32_t experts, top;
+  const float *norm1_w, *norm2_w;   /* parallel: [wp], zero padding */
+  const float *q_norm, *kv_norm, *powers;
+  const caten_b200_weight *uq_w, *uk_w, *kv_w, *router;
 } caten_b200_layer_desc;
 typedef struct {
   int32_t n_layers, width, vocab, max_seq_len, batch, precision;
@@ -358,7 +383,10 @@ typedef struct {
   float final_gain;            /* gain of the norm before `head`, times the scale of the logits */
   const caten_b200_weight *embed;    /* BF16 [vocab, wp] */
   const caten_b200_weight *head;     /* [vocab, wp] */
-  const caten_b200_weight *loop_in;  /* x = loop_in . [x ; embedding output] before each pass: [wp, 2 wp]; NULL without a loop */
+  /* before each pass of the loop, either (parallel layers: the second form) */
+  const caten_b200_weight *loop_in;  /* x = loop_in . [x ; embedding output]: [wp, 2 wp], or NULL */
+  const float *loop_step;            /* device [loop_times, wp]: x += loop_step[t], and before all passes but the first x += embedding output */
+  const float *final_norm;           /* device [wp]: gain per coordinate of the norm before `head`; NULL: final_gain */
   const caten_b200_layer_desc *layers;
 } caten_b200_decoder_desc;
 typedef struct caten_b200_decoder caten_b200_decoder;
@@ -476,8 +504,8 @@ enum {
   CATEN_B200_K_EMBED = 0, CATEN_B200_K_LAYERNORM = 1, CATEN_B200_K_GEMV = 2, CATEN_B200_K_GEMM = 3,
   CATEN_B200_K_ATTN_DECODE = 4, CATEN_B200_K_ATTN_PREFILL = 5, CATEN_B200_K_ARGMAX = 6,
   CATEN_B200_K_DECODE_STEP = 7,   /* the whole single-token step of 1..4 sequences, which is one kernel */
-  CATEN_B200_K_WKV = 8,           /* recurrence of a time-mixing layer */
-  CATEN_B200_K_PREP = 9,          /* rotation, q/k norm and cache append; token-shift mixes */
+  CATEN_B200_K_WKV = 8,           /* recurrence of a time-mixing or retention layer */
+  CATEN_B200_K_PREP = 9,          /* rotation, q/k norm and cache append; token-shift mixes; expert routing */
   CATEN_B200_K_COUNT = 10
 };
 /* Starts timing the classes whose bit (1 << class) is set in class_mask. */
