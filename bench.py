@@ -3,7 +3,7 @@
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
                     [--workload xl-q4_0-b256|medium-q4_0-b64|small-q8_0-b1|small-f32-b1|xl-q4_0-b1]
                     [--precision bf16x3|bf16|fp32] [--scaling strong|weak]
-    python bench.py --compare binusun      # prefill and decode of Binusun layers beside GPT-2 at equal size
+    python bench.py --compare binusun      # prefill and decode of Binusun layers beside GPT-2 at equal size (goselix: beside Binusun)
 
 A "step" is one KV-cached greedy decode step of the whole batch (one new token per sequence).
 Default workload: GPT-2 XL, Q4_0 weights, ONE batch of 256 sequences, 512-token prompts, 256 decoded
@@ -201,58 +201,115 @@ def oracle_parity(model, params, fsd, nb: int, precision: str, threads: int, pro
             "ids_equal_where_decisive": f"{ids_equal}/{ids_checked}"}
 
 
-# ------------------------------------------------------------------ --compare binusun
-# Layers of the sizes a real model would have, random weights, one GPU; GPT-2 with the same width, vocabulary and weight
-# format (bf16) and about the same number of weights read per token.
-COMPARE_SIZES = {
-    # width: (layer order, ff, heads, kv_heads, head size, window, heads and head size of the time mixing, loop, GPT-2 layers)
+# ------------------------------------------------------------------ --compare
+# A design's layers at the sizes a real model would have, random weights, one GPU, beside the closest model the package had
+# before it, with the same width, vocabulary and weight format (bf16) and about the same number of weights: Binusun beside
+# GPT-2, Goselix beside Binusun.
+COMPARE_VOCAB = 32000
+COMPARE_BINUSUN = {
+    # width: (layer order, ff, heads, kv_heads, head size, window, heads and head size of the time mixing), GPT-2 layers
     1024: dict(order="wAAwAAAAAAAA", ff=2816, heads=8, kv_heads=4, dim=128, window=1024, wkv=(16, 64), gpt2_layers=10),
     2048: dict(order="wAAwAAAA", ff=5632, heads=16, kv_heads=4, dim=128, window=1024, wkv=(32, 64), gpt2_layers=6),
+}
+COMPARE_GOSELIX = {
+    # width: the Goselix layers, and the Binusun layer order beside them (its other sizes as above)
+    1024: (dict(order="ldlmrdlmrmldlmrd", ff=2816, heads=16, dim=48, rot_dim=16, vdim=64, q_rank=384, kv_rank=128, ret_heads=8, ret_dim=64, ret_vdim=128,
+                ret_rot=64, experts=8, top=2, expert_ff=704), "wAAwAAAAAAAA"),
+    2048: (dict(order="ldlmrdlmrmld", ff=5632, heads=16, dim=96, rot_dim=32, vdim=128, q_rank=768, kv_rank=256, ret_heads=8, ret_dim=128, ret_vdim=256,
+                ret_rot=128, experts=8, top=2, expert_ff=1408), "wAAwAAAAA"),
 }
 COMPARE_PREFILL = ((1, 2048), (8, 1024))     # (sequences, tokens)
 COMPARE_DECODE = (1, 16, 64, 256)            # sequences, at contexts of about 1 100 tokens
 
 
-def compare_rooflines(kind, model, mode, B, s, ctx, peaks):
+def compare_rooflines(kind, mode, B, s, ctx, peaks):
     """Algorithmic work of one step by kernel class -> seconds at the measured peaks.  ``kind``: dict of the sizes;
     ``mode``: "prefill" (s tokens per sequence from position 0) or "decode" (one token at context ``ctx``)."""
     hbm, tf = peaks
     w, rows = kind["width"], B * (s if mode == "prefill" else 1)
     t = {}
+    # keys each query sees, summed over the tokens of a sequence
+    pairs = lambda win: sum(min(i + 1, win) if win else i + 1 for i in range(s))
     if mode == "prefill":
         t["linears"] = max(2.0 * rows * kind["layer_weights"] / tf, 2.0 * kind["layer_weights"] / hbm)
-        # keys each query sees, summed over the tokens of a sequence
-        pairs = lambda win: sum(min(i + 1, win) if win else i + 1 for i in range(s))
-        t["attention"] = sum(4.0 * B * H * D * pairs(win) for H, G, D, win in kind["attn"]) / tf
-        t["norms"] = kind["norms"] * rows * w * kind["norm_bytes"][mode] / hbm
+        t["attention"] = (sum(4.0 * B * H * D * pairs(win) for H, G, D, win in kind.get("attn", ())) +
+                          sum(2.0 * B * H * (D + P + E) * pairs(0) for H, D, P, E, K in kind.get("latent", ()))) / tf
         # r, k, v, gate, decay in; out
-        t["wkv"] = sum(rows * H * D * (5 * 4 + 2) for H, D in kind["wkv"]) / hbm
+        t["wkv"] = (sum(rows * H * D * (5 * 4 + 2) for H, D in kind.get("wkv", ())) +
+                    sum(rows * H * (8 * D + 8 * E + 2 * E) for H, D, E in kind.get("retention", ()))) / hbm   # q, k, v, gate in; out
     else:
         t["linears"] = 2.0 * (kind["layer_weights"] + kind["head_weights"]) / hbm
-        t["attention"] = sum(8.0 * B * G * D * (min(ctx, win) if win else ctx) for H, G, D, win in kind["attn"]) / hbm
-        t["norms"] = kind["norms"] * rows * w * kind["norm_bytes"][mode] / hbm
-        t["wkv"] = sum(8.0 * B * H * D * D for H, D in kind["wkv"]) / hbm
+        t["attention"] = (sum(8.0 * B * G * D * (min(ctx, win) if win else ctx) for H, G, D, win in kind.get("attn", ())) / hbm +
+                          sum(max(2.0 * B * (K + P) * ctx / hbm, 2.0 * B * H * (2 * K + P) * ctx / tf) for H, D, P, E, K in kind.get("latent", ())))
+        t["wkv"] = sum(8.0 * B * H * D * E for H, D, E in [(H, D, D) for H, D in kind.get("wkv", ())] + list(kind.get("retention", ()))) / hbm
+    t["norms"] = kind["norms"] * rows * w * kind["norm_bytes"][mode] / hbm
+    # an expert's weights are read if any row uses it
+    t["experts"] = sum(max(2.0 * rows * top * n / tf, 2.0 * n * E * (1.0 - (1.0 - top / E) ** rows) / hbm) for E, top, n in kind.get("experts", ()))
     return {k: v for k, v in t.items() if v}
 
 
-COMPARE_CLASSES = {"linears": ("gemm", "gemv"), "attention": ("attn_prefill", "attn_decode"), "norms": ("layernorm",), "wkv": ("wkv",), "prep": ("prep",)}
+COMPARE_CLASSES = {"linears": ("gemm", "gemv"), "experts": ("experts",), "attention": ("attn_prefill", "attn_decode"), "norms": ("layernorm",), "wkv": ("wkv",),
+                   "prep": ("prep",)}
 
 
-def compare_binusun():
-    import torch
-    from caten_b200 import _lib as L_
+def compare_binusun_model(rt, width, z, order, V):
     from caten_b200 import synthetic as S
     from caten_b200.binusun import Binusun, parse_config
+    cfg = S.binusun_config(width, V, order, z["ff"], z["heads"], z["kv_heads"], z["dim"], z["dim"], z["window"], *z["wkv"], rot_dims=z["dim"] // 2)
+    tensors = S.synth_binusun(cfg, seed=0, low_rank=64)
+    n_layer = sum(v.size for k, v in tensors.items() if v.ndim == 2 and k[0] == "l")
+    kind = dict(width=width, layer_weights=n_layer, head_weights=V * width, norms=sum(4 if l["mlp"] else 2 for l in cfg["layers"]) / 2,
+                norm_bytes={"prefill": 14, "decode": 14},   # sublayer output and stream in, stream and bf16 operand out
+                attn=[(m["heads"], m["kv_heads"], m["dim"], m["mask"]["size"]) for m in (l["mixer"] for l in cfg["layers"] if l["type"] == "attention")],
+                wkv=[(m["heads"], m["dim"]) for m in (l["mixer"] for l in cfg["layers"] if l["type"] == "wkv")])
+    return "binusun", kind, lambda B, T: Binusun(rt, parse_config(cfg), tensors, max_seq_len=T, batch=B, precision="bf16")
+
+
+def compare_gpt2_model(rt, width, layers, V):
+    from caten_b200 import _lib as L_
+    from caten_b200 import synthetic as S
     from caten_b200.gpt2 import GPT2
-    from caten_b200.runtime import B200Runtime
     from caten_b200.safetensors import f32_to_bf16
+    gp = S.GPT2Params(layers, width // 64, width, V)
+    gsd = S.synth_state_dict(gp, "f32", seed=0, max_seq_len=2304)
+    for k, v in gsd.items():
+        if v.ndim == 2 and not k.startswith("w"):
+            gsd[k] = S.Packed(L_.BF16, v.shape[0], v.shape[1], f32_to_bf16(v).view(np.uint8).reshape(-1))
+    kind = dict(width=width, layer_weights=12 * width * width * gp.n_layers, head_weights=V * width, norms=2 * gp.n_layers,
+                norm_bytes={"prefill": 6, "decode": 14},    # prompts add the residual in the linear's epilogue
+                attn=[(gp.n_heads, gp.n_heads, 64, 0)] * gp.n_layers)
+    return "gpt2", kind, lambda B, T: GPT2(rt, gp, gsd, max_seq_len=T, batch=B, precision="bf16")
+
+
+def compare_goselix_model(rt, width, z, V):
+    from caten_b200 import synthetic as S
+    from caten_b200.goselix import Goselix, parse_config
+    cfg = S.goselix_config(width, V, **z)
+    tensors = S.synth_goselix(cfg, seed=0)
+    mats = {k: v.size for k, v in tensors.items() if v.ndim == 2 and k[0] == "l"}
+    n_expert = sum(n for k, n in mats.items() if ".mlp.e" in k)
+    lat = [l["mixer"] for l in cfg["layers"] if l["type"] == "latent_attention"]
+    ret = [l["mixer"] for l in cfg["layers"] if l["type"] == "retention"]
+    moe = [l["mlp"] for l in cfg["layers"] if l["mlp"] and l["mlp"]["kind"] == "moe"]
+    # per layer: stream, mixer output and (with experts) `top` expert outputs in, stream and two bf16 operands out
+    bytes_in_out = 16 + 4.0 * sum(m["router"]["top"] for m in moe) / len(cfg["layers"])
+    kind = dict(width=width, layer_weights=sum(mats.values()) - n_expert, expert_weights=n_expert, head_weights=V * width, norms=len(cfg["layers"]),
+                norm_bytes={"prefill": bytes_in_out, "decode": bytes_in_out},
+                latent=[(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]) for m in lat], retention=[(m["heads"], m["dim"], m["vdim"]) for m in ret],
+                experts=[(m["router"]["experts"], m["router"]["top"], 3 * width * m["expert"]["ff"]) for m in moe])
+    return "goselix", kind, lambda B, T: Goselix(rt, parse_config(cfg), tensors, max_seq_len=T, batch=B, precision="bf16")
+
+
+def compare(design):
+    import torch
+    from caten_b200.runtime import B200Runtime
     torch.cuda.set_device(0)
     hbm, src = load_peaks()
     burst, sustained = load_tensor_peak()
     peaks = (hbm * 1e9, burst * 1e12)
     rt = B200Runtime(0)
     ext = torch.cuda.ExternalStream(rt.stream, device=torch.device("cuda", 0))
-    V = 32000
+    V = COMPARE_VOCAB
 
     def ev():
         e = torch.cuda.Event(enable_timing=True)
@@ -262,28 +319,11 @@ def compare_binusun():
     rng = np.random.Generator(np.random.PCG64(0))
     results = []
     sampler = ClockSampler(0)
-    for width, z in COMPARE_SIZES.items():
-        cfg = S.binusun_config(width, V, z["order"], z["ff"], z["heads"], z["kv_heads"], z["dim"], z["dim"], z["window"], *z["wkv"], rot_dims=z["dim"] // 2)
-        tensors = S.synth_binusun(cfg, seed=0, low_rank=64)
-        attn = [l["mixer"] for l in cfg["layers"] if l["type"] == "attention"]
-        wkv = [l["mixer"] for l in cfg["layers"] if l["type"] == "wkv"]
-        n_layer = sum(v.size for k, v in tensors.items() if v.ndim == 2 and k[0] == "l")
-        bin_kind = dict(width=width, layer_weights=n_layer, head_weights=V * width, norms=sum(4 if l["mlp"] else 2 for l in cfg["layers"]) / 2,
-                        norm_bytes={"prefill": 14, "decode": 14},   # sublayer output and stream in, stream and bf16 operand out
-                        attn=[(m["heads"], m["kv_heads"], m["dim"], m["mask"]["size"]) for m in attn], wkv=[(m["heads"], m["dim"]) for m in wkv])
-        gp = S.GPT2Params(z["gpt2_layers"], width // 64, width, V)
-        gsd = S.synth_state_dict(gp, "f32", seed=0, max_seq_len=2304)
-        for k, v in gsd.items():
-            if v.ndim == 2 and not k.startswith("w"):
-                gsd[k] = S.Packed(L_.BF16, v.shape[0], v.shape[1], f32_to_bf16(v).view(np.uint8).reshape(-1))
-        gpt_kind = dict(width=width, layer_weights=12 * width * width * gp.n_layers, head_weights=V * width, norms=2 * gp.n_layers,
-                        norm_bytes={"prefill": 6, "decode": 14},    # prompts add the residual in the linear's epilogue
-                        attn=[(gp.n_heads, gp.n_heads, 64, 0)] * gp.n_layers, wkv=[])
-
-        def make(name, B, T):
-            if name == "binusun":
-                return Binusun(rt, parse_config(cfg), tensors, max_seq_len=T, batch=B, precision="bf16")
-            return GPT2(rt, gp, gsd, max_seq_len=T, batch=B, precision="bf16")
+    for width, z in (COMPARE_BINUSUN if design == "binusun" else COMPARE_GOSELIX).items():
+        if design == "binusun":
+            models = [compare_binusun_model(rt, width, z, z["order"], V), compare_gpt2_model(rt, width, z["gpt2_layers"], V)]
+        else:
+            models = [compare_goselix_model(rt, width, z[0], V), compare_binusun_model(rt, width, COMPARE_BINUSUN[width], z[1], V)]
 
         def classes(prof, steps, roof):
             out = {}
@@ -296,12 +336,12 @@ def compare_binusun():
         for mode, cases in (("prefill", COMPARE_PREFILL), ("decode", [(B, 1024) for B in COMPARE_DECODE])):
             for B, s in cases:
                 row = {"width": width, "mode": mode, "sequences": B, "tokens" if mode == "prefill" else "context": s if mode == "prefill" else 1104}
-                for name, kind in (("binusun", bin_kind), ("gpt2", gpt_kind)):
-                    m = make(name, B, s if mode == "prefill" else 1200)
+                for name, kind, make in models:
+                    m = make(B, s if mode == "prefill" else 1200)
                     ids = rt.transfer_from_array(rng.integers(0, V, (B, s), dtype=np.int64))
                     out = rt.open_buffer((B,), np.int64)
                     m.forward_device(ids, s, 0, out)
-                    roof = compare_rooflines(kind, m, mode, B, s, 1104, peaks)
+                    roof = compare_rooflines(kind, mode, B, s, 1104, peaks)
                     if mode == "prefill":
                         for _ in range(3):
                             m.forward_device(ids, s, 0, out)
@@ -328,13 +368,14 @@ def compare_binusun():
                         m.decode_device_buffers(out, 1128, 8, None)
                         prof = rt.profile_end()
                         steps = 8
-                    row[name] = {"ms": round(ms, 4), "tokens_per_s": round(toks / ms * 1e3), "weights_M": round((kind["layer_weights"] + kind["head_weights"]) / 1e6, 1),
+                    weights = kind["layer_weights"] + kind["head_weights"] + kind.get("expert_weights", 0)
+                    row[name] = {"ms": round(ms, 4), "tokens_per_s": round(toks / ms * 1e3), "weights_M": round(weights / 1e6, 1),
                                  "frac_of_roofline": round(sum(roof.values()) * 1e3 / ms, 4), "classes": classes(prof, steps, roof)}
                     m.close(); ids.close(); out.close()
                 results.append(row)
     clocks = sampler.stop()
     rt.close()
-    print(json.dumps({"metric": "binusun_and_gpt2_layers", "data": "synthetic", "dtype": "bf16 weights and GEMM operands, fp32 otherwise", "n_gpus": 1,
+    print(json.dumps({"metric": f"{models[0][0]}_and_{models[1][0]}_layers", "data": "synthetic", "dtype": "bf16 weights and GEMM operands, fp32 otherwise", "n_gpus": 1,
                       "peaks": {"hbm_gbs": hbm, "bf16_tflops": burst, "source": src},
                       "timing": "CUDA events; decode steps replayed from a CUDA graph; classes from a separate pass with events around every launch (a few us each)",
                       "l2": "weights and caches exceed L2 except where the batch is small", "clocks": clocks, "results": results}))
@@ -342,7 +383,7 @@ def compare_binusun():
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--compare", choices=["binusun"], default=None, help="prefill and decode throughput of a design's layers beside GPT-2 at equal size, instead of the benchmark")
+    ap.add_argument("--compare", choices=["binusun", "goselix"], default=None, help="prefill and decode throughput of a design's layers beside the closest other model at equal size, instead of the benchmark")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=None)
     ap.add_argument("--warmup", type=int, default=3)
@@ -363,7 +404,7 @@ def main():
     ap.add_argument("--no-extras", action="store_true", help="skip the prefill/GEMV/kernel-breakdown side measurements")
     args = ap.parse_args()
     if args.compare:
-        return compare_binusun()
+        return compare(args.compare)
 
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))

@@ -21,8 +21,8 @@ Q2_K, Q3_K, Q4_K, Q5_K, Q6_K = 10, 11, 12, 13, 14        # expanded to fp32 at u
 BLOCK_FORMATS = (Q4_0, Q8_0, Q4_1, Q5_0, Q5_1, Q2_K, Q3_K, Q4_K, Q5_K, Q6_K)
 ACT_NONE, ACT_GELU, ACT_RELU, ACT_RELU_GLU, ACT_SILU_GLU = 0, 1, 2, 3, 4
 PREC_FP32, PREC_BF16, PREC_BF16X3 = 0, 1, 2
-K_EMBED, K_LAYERNORM, K_GEMV, K_GEMM, K_ATTN_DECODE, K_ATTN_PREFILL, K_ARGMAX, K_COUNT = 0, 1, 2, 3, 4, 5, 6, 10
-KERNEL_CLASSES = ["embed", "layernorm", "gemv", "gemm", "attn_decode", "attn_prefill", "argmax", "decode_step", "wkv", "prep"]
+K_EMBED, K_LAYERNORM, K_GEMV, K_GEMM, K_ATTN_DECODE, K_ATTN_PREFILL, K_ARGMAX, K_COUNT = 0, 1, 2, 3, 4, 5, 6, 11
+KERNEL_CLASSES = ["embed", "layernorm", "gemv", "gemm", "attn_decode", "attn_prefill", "argmax", "decode_step", "wkv", "prep", "experts"]
 DIST_ID_BYTES = 128
 PRECISIONS = {"fp32": PREC_FP32, "bf16": PREC_BF16, "bf16x3": PREC_BF16X3}
 

@@ -532,7 +532,7 @@ class StepRunner {
     next->ye = m_->ye;
     next->top = c.top;
     next->pos = sorted ? m_->ex_pos : nullptr;
-    ProfScope prof(ctx_, sorted ? CATEN_B200_K_GEMM : CATEN_B200_K_GEMV);
+    ProfScope prof(ctx_, CATEN_B200_K_EXPERTS);
     if (!sorted) {
       if (int rc = launch_gemv_experts(ctx_, c.ff_in, rows_in, h2, m_->ex_id, m_->ex_w, pairs, c.top, c.ff_act, m_->ea)) return rc;
       return launch_gemv_experts(ctx_, c.ff_out, m_->wp, m_->ea, m_->ex_id, nullptr, pairs, 1, CATEN_B200_ACT_NONE, m_->ye);
@@ -573,6 +573,9 @@ class StepRunner {
       x.qcat = m_->qcat; x.qcat_bf = bf(m_->qcat_bf); x.o = m_->olat; x.o_bf = bf(m_->olat_bf); x.plane = m_->abs_rows; x.part = m_->part; x.ml = m_->ml;
       x.splits = latent_splits(ctx_, a, R_, p_.d_n ? a.cap : p_.n + p_.s);
       while (x.splits > 1 && x.splits * R_ * a.H * a.Kr > m_->part_floats) --x.splits;
+      // (the kernel in front is the product with W_uk^T; the one before it starts nothing until the kernels before it, the cache's
+      // append among them, are complete)
+      x.early = true;
       { ProfScope prof(ctx_, CATEN_B200_K_ATTN_DECODE); if (int rc = launch_latent_absorbed(ctx_, a, x)) return rc; }
       LinGroups down;
       down.group_rows = a.Ep; down.xplane = m_->abs_rows; down.ygroup = a.Ep; down.ldy = c.out_w->cols;

@@ -6,14 +6,17 @@
 //   expanded   keys and values of all heads are formed from the cached latents by one linear and go through the
 //              ordinary prompt attention (attention_tc.cu, attn_window.cu).  Longer portions.
 //
-// latent_attn_tc_kernel (bf16 models): tcgen05.  A CTA serves up to 64 heads of one row: the 128 lanes of tensor memory hold every
-// head twice, so that both halves find the same scores and probabilities, and the upper half stores the high, the lower half the
-// low bf16 part of p as the A operand of the second product: p keeps 16 bits and the two partial outputs are added at the end.
-//   warp 4      TMA: tiles of KT cached rows, all columns, as 64-column blocks with the 128-byte swizzle.  The same tile is the K-major B
-//               operand of S = Q.C^T and the MN-major B operand of O += P.C
-//   warp 5      tcgen05.mma: S of the next tile is issued before O of this one, so that it runs during the softmax
-//   warps 0..3  one score row per thread: lazily moved reference maximum (as in attention_tc.cu), p to tensor memory
-// Value columns go in blocks of 256 per CTA, keys may be split over CTAs; latent_combine_kernel then merges the parts.
+// latent_attn_tc_kernel (bf16 models): tcgen05.  A CTA serves NH = 16 or 32 heads of one row; keys go in tiles of 128, and both
+// products have the keys' or the latent's dims, not the heads, as the 128 lanes of tensor memory, so that few heads waste nothing:
+//   warp 4      TMA: a tile of 128 cached rows as 64-column blocks with the 128-byte swizzle, two blocks to a barrier.  The same
+//               blocks are the K-major A operand of S^T = C.Q^T and the MN-major A operand of O^T += C^T.P^T
+//   warps 5, 6  tcgen05.mma: one warp issues the scores of tile after tile, as soon as a tile has arrived and its score columns have
+//               been read, the other the outputs.  With few heads a product takes less time than issuing it, so the two streams
+//               of issues run side by side, and a tile is given back as soon as its output is formed
+//   warps 0..3  one key per thread, all its heads: a head's reference maximum moves lazily (as in attention_tc.cu: only when a score
+//               exceeds it by LA_TAU; one vote per tile finds out), p = hi + lo in bf16 goes to shared memory as the 2 NH rows of the
+//               second product's B operand (hi of all heads, then lo), so p keeps 16 bits; the two halves of O are added at the end
+// Keys may be split over CTAs; latent_combine_kernel then merges the parts.
 // Every mbarrier wait is bounded: when one runs out the CTA records it in the status word, leaves its loops, waits for its
 // copies in flight, frees tensor memory and writes no output.
 #include "latent.cuh"
@@ -313,7 +316,7 @@ __global__ void __launch_bounds__(LS_THREADS) latent_attn_simt_kernel(const Late
     }
     if (out.splits > 1 && tid == 0) {
       float *ml = out.ml + (((int64_t)split * out.rows + r) * a.H + h0 + h) * 2;
-      ml[0] = stat[LS_H + h];
+      ml[0] = stat[LS_H + h] * kLog2e;
       ml[1] = l;
     }
   }
@@ -330,12 +333,12 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentOut out
   float l = 0.0f;
   for (int z = 0; z < out.splits; ++z) {
     const float lz = out.ml[(z * step + at) * 2 + 1];
-    if (lz > 0.0f) l = fmaf(exp2f((out.ml[(z * step + at) * 2] - m) * kLog2e), lz, l);
+    if (lz > 0.0f) l = fmaf(exp2f(out.ml[(z * step + at) * 2] - m), lz, l);
   }
   for (int c = threadIdx.x; c < out.Kr; c += 128) {
     float o = 0.0f;
     for (int z = 0; z < out.splits; ++z)   // fixed order; a part without keys counts nothing
-      if (out.ml[(z * step + at) * 2 + 1] > 0.0f) o = fmaf(exp2f((out.ml[(z * step + at) * 2] - m) * kLog2e), out.part[(z * step + at) * out.Kr + c], o);
+      if (out.ml[(z * step + at) * 2 + 1] > 0.0f) o = fmaf(exp2f(out.ml[(z * step + at) * 2] - m), out.part[(z * step + at) * out.Kr + c], o);
     st1(out.o, out.o_bf, ((int64_t)h * out.plane + r) * out.Kr + c, o / l);
   }
 }
@@ -343,13 +346,12 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentOut out
 // ---------------------------------------------------------------------------------------------
 // Absorbed attention on the tensor cores
 // ---------------------------------------------------------------------------------------------
-constexpr int LA_H = 64;                // heads per CTA
-constexpr int LA_THREADS = 192;
-constexpr int LA_MAX_STAGES = 4, LA_MAX_BLOCKS = 9;   // 64-column blocks of a cached row: up to 576 columns
-constexpr int LA_VBLOCKS = 4;           // value blocks per CTA
-constexpr float LA_TAU = 8.0f;          // slack of the reference maximum, in units of the score
-constexpr uint32_t LA_COL_O = 0, LA_COL_S = 256, LA_COL_P = 384;   // two score tiles of 64 columns, two P tiles of 32
-constexpr int LA_OLD = 260;             // row pitch (floats) of the output exchange buffer
+constexpr int LA_KEYS = 128;              // cached rows per tile
+constexpr int LA_THREADS = 224;
+constexpr int LA_MAX_BLOCKS = 9;          // 64-column blocks of a cached row: up to 576 columns
+constexpr int LA_MAX_STAGES = 4, LA_MAX_PAIRS = 10, LA_BARS = 2 * LA_MAX_PAIRS + 6;   // full, empty of the ring's pairs; s, p, o (two each); then q
+constexpr uint32_t LA_BLOCK = LA_KEYS * 128;   // bytes
+constexpr float LA_TAU = 11.5f;           // slack of the reference maximum, in powers of two
 
 __device__ __forceinline__ uint32_t la_sw128(int row, int chunk) { return (uint32_t)((row >> 3) * 1024 + (row & 7) * 128 + ((chunk ^ (row & 7)) << 4)); }
 __device__ __forceinline__ float la_ex2(float x) {
@@ -357,40 +359,70 @@ __device__ __forceinline__ float la_ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));   // results below 2^-126 flush to zero
   return y;
 }
+__device__ __forceinline__ void la_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ bool la_any(bool x) {   // over the softmax threads
+  uint32_t r;
+  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.u32 p, %1, 0;\n\tbarrier.cta.red.or.pred q, 1, 128, p;\n\tselp.u32 %0, 1, 0, q;\n\t}" : "=r"(r) : "r"(x ? 1u : 0u) : "memory");
+  return r != 0;
+}
+// NH values per lane, reduced over the warp: each exchange halves the values a lane carries; afterwards red[h] holds head h's.
+template <int NH, bool MAX>
+__device__ __forceinline__ void la_reduce(const float *x, int lane, float *red) {
+  float v[NH];
+#pragma unroll
+  for (int h = 0; h < NH; ++h) v[h] = x[h];
+  int head = 0, step = 16;
+#pragma unroll
+  for (int n = NH; n > 1; n >>= 1, step >>= 1) {
+    const bool up = (lane & step) != 0;
+#pragma unroll
+    for (int i = 0; i < n / 2; ++i) {
+      const float give = up ? v[i] : v[i + n / 2], keep = up ? v[i + n / 2] : v[i];
+      const float got = __shfl_xor_sync(0xffffffffu, give, step);
+      v[i] = MAX ? fmaxf(keep, got) : keep + got;
+    }
+    head += up ? n / 2 : 0;
+  }
+#pragma unroll
+  for (int o = 16 / NH; o > 0; o >>= 1) {   // (NH = 16: one more exchange between the lanes that hold the same head)
+    const float got = __shfl_xor_sync(0xffffffffu, v[0], o);
+    v[0] = MAX ? fmaxf(v[0], got) : v[0] + got;
+  }
+  if ((lane & (32 / NH - 1)) == 0) red[head] = v[0];
+}
 
-// KT: cached rows per tile
-template <int KT>
+// MN-major operand, 128-byte swizzle: 64-element blocks LA_BLOCK bytes apart, groups of 8 along k 1024 bytes apart
+__device__ __forceinline__ uint64_t la_desc_mn(uint32_t saddr) { return umma_desc(saddr) - ((uint64_t)1 << 16) + ((uint64_t)(LA_BLOCK >> 4) << 16); }
+
+template <int NH>
 __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentArgs a, const float *__restrict__ qcat,
-                                                                       const __nv_bfloat16 *__restrict__ qcat_hi, const LatentOut out, const int stages,
-                                                                       const uint32_t idesc_s, const uint32_t idesc_pv, int *status) {
+                                                                       const __nv_bfloat16 *__restrict__ qcat_hi, const LatentOut out, const int stages, const int early,
+                                                                       const uint32_t tmem_cols, const uint32_t idesc_s, const uint32_t idesc_pv, int *status) {
   extern __shared__ unsigned char la_raw[];
   unsigned char *sm = reinterpret_cast<unsigned char *>((reinterpret_cast<uintptr_t>(la_raw) + 1023) & ~(uintptr_t)1023);
-  const int KC = a.Kp + a.Pp, nkc = (KC + 63) / 64, ksteps = KC / 16;
-  const uint32_t stage_bytes = (uint32_t)nkc * KT * 128;
-  unsigned char *qs = sm, *kv = sm + nkc * 16384;
-  // (the tiles become the output exchange buffer at the end)
-  uint64_t *bars = reinterpret_cast<uint64_t *>(sm + max((size_t)nkc * 16384 + (size_t)stages * stage_bytes, (size_t)LA_H * LA_OLD * 4));
+  constexpr uint32_t QB = NH * 128, PB = 2 * 2 * NH * 128;   // bytes of a Q block; of a P buffer (two blocks of 64 keys, 2 NH rows)
+  const int KC = a.Kp + a.Pp, nkc = (KC + 63) / 64, np = (nkc + 1) / 2, ksteps = KC / 16, npv = (out.Kr / 64 + 1) / 2;
+  unsigned char *kv = sm, *qs = kv + (size_t)stages * nkc * LA_BLOCK, *ps = qs + nkc * QB;
+  uint64_t *bars = reinterpret_cast<uint64_t *>(ps + 2 * PB);
+  float *red = reinterpret_cast<float *>(bars + LA_BARS + 1);   // [4][NH]
   const uint32_t bar0 = smem_u32(bars);
-  auto full = [&](int s) { return bar0 + 8u * s; };
-  auto empty = [&](int s) { return bar0 + 8u * (LA_MAX_STAGES + s); };
-  auto s_full = [&](int b) { return bar0 + 8u * (2 * LA_MAX_STAGES + b); };
-  auto p_full = [&](int b) { return bar0 + 8u * (2 * LA_MAX_STAGES + 2 + b); };
-  auto o_done = [&](int b) { return bar0 + 8u * (2 * LA_MAX_STAGES + 4 + b); };
-  const uint32_t q_full = bar0 + 8u * (2 * LA_MAX_STAGES + 6);
-  uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(bars + 2 * LA_MAX_STAGES + 7);
-  volatile int *abort_flag = reinterpret_cast<volatile int *>(tmem_slot + 1);   // [0] a wait ran out; [1] never set
-  float *lsum = reinterpret_cast<float *>(tmem_slot + 4);                       // [LA_H]
-
+  auto full = [&](int s, int p) { return bar0 + 8u * (s * np + p); };
+  auto empty = [&](int s, int p) { return bar0 + 8u * (LA_MAX_PAIRS + s * np + p); };
+  auto s_full = [&](int b) { return bar0 + 8u * (2 * LA_MAX_PAIRS + b); };
+  auto p_full = [&](int b) { return bar0 + 8u * (2 * LA_MAX_PAIRS + 2 + b); };
+  auto o_done = [&](int b) { return bar0 + 8u * (2 * LA_MAX_PAIRS + 4 + b); };
+  const uint32_t q_full = bar0 + 8u * LA_BARS;
+  __shared__ uint32_t tmem_slot;
+  __shared__ volatile int flags[2];   // [0] a wait ran out; [1] never set
+  volatile int *abort_flag = flags;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int vparts = (out.Kr / 64 + LA_VBLOCKS - 1) / LA_VBLOCKS;
-  const int h0 = blockIdx.x / vparts * LA_H, vb0 = blockIdx.x % vparts * LA_VBLOCKS, nvb = min(LA_VBLOCKS, out.Kr / 64 - vb0);
-  const int hn = min(LA_H, a.H - h0), split = blockIdx.z;
+  const int h0 = blockIdx.x * NH, hn = min(NH, a.H - h0), split = blockIdx.z;
   const int64_t r = blockIdx.y;
 
   if (tid == 0) {
-    for (int s = 0; s < stages; ++s) {
-      mbar_init(full(s), 1);
-      mbar_init(empty(s), 1);
+    for (int i = 0; i < stages * np; ++i) {
+      mbar_init(bar0 + 8u * i, 1);
+      mbar_init(bar0 + 8u * (LA_MAX_PAIRS + i), 1);
     }
     for (int b = 0; b < 2; ++b) {
       mbar_init(s_full(b), 1);
@@ -398,223 +430,256 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
       mbar_init(o_done(b), 1);
     }
     mbar_init(q_full, 4);
-    abort_flag[0] = abort_flag[1] = 0;
+    flags[0] = flags[1] = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   if (warp == 5) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)), "r"(512u) : "memory");
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(tmem_cols) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem_base = *tmem_slot;
+  const uint32_t tmem_base = tmem_slot, col_s = (uint32_t)npv * 2 * NH;   // O: npv x 2 NH columns, then two score tiles of NH
   if (warp == 4 && lane == 0) tma_prefetch_map(&map);
-  pdl_enter();
+  // `early`: the cache and the position were complete before the kernel in front of this one started; only Q comes from it
+  if (warp != 4 || !early) pdl_wait();
+  pdl_launch_dependents();
   const int t = (a.d_n ? *a.d_n : a.n) + (int)(r % a.s) + 1;   // keys this row sees
-  const int tiles = (t + KT - 1) / KT, per = (tiles + out.splits - 1) / out.splits;
+  const int tiles = (t + LA_KEYS - 1) / LA_KEYS, per = (tiles + out.splits - 1) / out.splits;
   const int tile0 = min(split * per, tiles), nt = min(tile0 + per, tiles) - tile0;
   auto give_up = [&](int where) {
     if (!*abort_flag) { *abort_flag = 1; atomicCAS(status, 0, DEV_WAIT_TIMEOUT); status[1] = where; }
   };
 
-  float m = -INFINITY, l = 0.0f;   // softmax threads
   bool ok = true;
   if (warp == 4) {
     if (lane == 0) {
       int issued = 0, s = 0;
       uint32_t ph = 1;
-      const int row0 = (int)(r / a.s * a.cap);
-      for (int i = 0; i < nt; ++i) {
-        if (!mbar_wait(empty(s), ph, abort_flag)) { give_up(30); break; }
-        mbar_expect_tx(full(s), stage_bytes);
-        for (int c = 0; c < nkc; ++c)
-          tma_load_2d(smem_u32(kv) + s * stage_bytes + (uint32_t)c * KT * 128, &map, full(s), c * 64, row0 + (tile0 + i) * KT);
-        issued = i + 1;
+      const int row0 = (int)(r / a.s * a.cap) + tile0 * LA_KEYS;
+      for (int i = 0; i < nt && ok; ++i) {
+        for (int p = 0; p < np; ++p) {
+          if (!mbar_wait(empty(s, p), ph, abort_flag)) { give_up(30); ok = false; break; }
+          const int blocks = min(2, nkc - 2 * p);
+          mbar_expect_tx(full(s, p), (uint32_t)blocks * LA_BLOCK);
+          for (int c = 0; c < blocks; ++c)
+            tma_load_2d(smem_u32(kv) + (uint32_t)(s * nkc + 2 * p + c) * LA_BLOCK, &map, full(s, p), (2 * p + c) * 64, row0 + i * LA_KEYS);
+          ++issued;
+        }
         if (++s == stages) { s = 0; ph ^= 1u; }
       }
       if (*abort_flag)   // copies in flight land before the CTA's shared memory is released
-        for (int i = issued > stages ? issued - stages : 0; i < issued; ++i) mbar_wait(full(i % stages), (uint32_t)(i / stages) & 1u, abort_flag + 1);
+        for (int i = issued > stages * np ? issued - stages * np : 0; i < issued; ++i)
+          mbar_wait(full(i / np % stages, i % np), (uint32_t)(i / np / stages) & 1u, abort_flag + 1);
     }
     __syncwarp();
   } else if (warp == 5) {
-    const uint64_t dq = umma_desc(smem_u32(qs)), dk0 = umma_desc(smem_u32(kv));
-    const uint32_t stage16 = stage_bytes >> 4;
+    const uint64_t dq = umma_desc(smem_u32(qs)), dk = umma_desc(smem_u32(kv));
     ok = nt == 0 || mbar_wait(q_full, 0, abort_flag);
     if (!ok && lane == 0) give_up(31);
-    tc_fence_after();
-    auto scores = [&](int i) {   // S(i) into its tile
-      if (!mbar_wait(full(i % stages), (uint32_t)(i / stages) & 1u, abort_flag)) {
-        if (lane == 0) give_up(32);
-        return false;
-      }
-      tc_fence_after();
-      if (elect_one()) {
-        const uint64_t dk = dk0 + (uint64_t)(i % stages) * stage16;
-        for (int k = 0; k < ksteps; ++k)   // 16 columns = 32 bytes = 2 descriptor units; a Q block has 1024 units, a tile's block KT * 8
-          umma_bf16(tmem_base + LA_COL_S + 64 * (i & 1), dq + (uint64_t)((k >> 2) * 1024 + 2 * (k & 3)), dk + (uint64_t)((k >> 2) * (KT * 8) + 2 * (k & 3)), idesc_s, k > 0 ? 1u : 0u);
-        umma_commit(s_full(i & 1));
-      }
-      __syncwarp();
-      return true;
-    };
-    if (ok && nt > 0) ok = scores(0);
+    int s = 0;
+    uint32_t ph = 0;
     for (int i = 0; i < nt && ok; ++i) {
-      // (tile i + 1's scores overwrite those of i - 1, which the softmax has read: its P(i - 1) was waited for)
-      if (i + 1 < nt && !(ok = scores(i + 1))) break;
-      if (!mbar_wait(p_full(i & 1), (uint32_t)(i >> 1) & 1u, abort_flag)) {
+      // the scores of tile i - 2 in these columns have been read
+      if (i >= 2 && !(ok = mbar_wait(p_full(i & 1), (uint32_t)((i - 2) >> 1) & 1u, abort_flag))) {
+        if (lane == 0) give_up(38);
+        break;
+      }
+      for (int p = 0; p < np && ok; ++p) {
+        if (!(ok = mbar_wait(full(s, p), ph, abort_flag))) {
+          if (lane == 0) give_up(32);
+          break;
+        }
+        tc_fence_after();
+        if (elect_one()) {
+          const uint64_t da = dk + (uint64_t)((s * nkc + 2 * p) * (int)(LA_BLOCK >> 4)), db = dq + (uint64_t)(2 * p * (int)(QB >> 4));
+          const int left = ksteps - 8 * p;
+#pragma unroll
+          for (int k = 0; k < 8; ++k)   // 16 columns = 32 bytes = 2 descriptor units
+            if (k < left)
+              umma_bf16(tmem_base + col_s + NH * (i & 1), da + (uint64_t)((k >> 2) * (LA_BLOCK >> 4) + 2 * (k & 3)), db + (uint64_t)((k >> 2) * (QB >> 4) + 2 * (k & 3)), idesc_s,
+                        p > 0 || k > 0 ? 1u : 0u);
+          if (p == np - 1) umma_commit(s_full(i & 1));
+        }
+        __syncwarp();
+      }
+      if (++s == stages) { s = 0; ph ^= 1u; }
+    }
+  } else if (warp == 6) {
+    const uint64_t dm = la_desc_mn(smem_u32(kv)), dp = umma_desc(smem_u32(ps));
+    int s = 0;
+    for (int i = 0; i < nt; ++i) {
+      if (!(ok = mbar_wait(p_full(i & 1), (uint32_t)(i >> 1) & 1u, abort_flag))) {
         if (lane == 0) give_up(33);
-        ok = false;
         break;
       }
       tc_fence_after();
       if (elect_one()) {
-        const uint64_t dv = dk0 + (uint64_t)(i % stages) * stage16 + (uint64_t)(vb0 * KT * 8);
-        for (int w = 0; w < nvb; ++w)
+        const uint64_t db = dp + (uint64_t)((i & 1) * (int)(PB >> 4));
+        for (int j = 0; j < npv; ++j) {
+          const uint64_t da = dm + (uint64_t)((s * nkc + 2 * j) * (int)(LA_BLOCK >> 4));
+          const uint32_t acc = tmem_base + (uint32_t)j * 2 * NH;
 #pragma unroll
-          for (int k4 = 0; k4 < KT / 16; ++k4)   // 16 keys = 16 rows of 128 bytes = 128 descriptor units
-            umma_bf16_ts(tmem_base + LA_COL_O + 64 * w, tmem_base + LA_COL_P + 32 * (i & 1) + 8 * k4, dv + (uint64_t)(w * KT * 8 + 128 * k4), idesc_pv, (i > 0 || k4 > 0) ? 1u : 0u);
+          for (int k = 0; k < LA_KEYS / 16; ++k)   // A: 16 keys = 16 rows of 128 bytes = 128 descriptor units
+            umma_bf16(acc, da + (uint64_t)(128 * k), db + (uint64_t)((k >> 2) * (PB >> 5) + 2 * (k & 3)), idesc_pv, (i > 0 || k > 0) ? 1u : 0u);
+          umma_commit(empty(s, j));
+        }
+        // (the tile's scores, which also read it, were complete before its probabilities were formed)
+        for (int p = npv; p < np; ++p) umma_commit(empty(s, p));
         umma_commit(o_done(i & 1));
-        umma_commit(empty(i % stages));
       }
       __syncwarp();
+      if (++s == stages) s = 0;
     }
   } else {
-    // ---- softmax: thread = lane of tensor memory; head h0 + (tid & 63), high part of p in lanes 0..63, low part in 64..127 ----
+    // ---- softmax: thread = lane of tensor memory = key of the tile ----
     const uint32_t tlane = tmem_base + ((uint32_t)(warp * 32) << 16);
     {
-      const int pieces = KC / 8;
-      for (int i = tid; i < 64 * nkc * 8; i += 128) {   // 16-byte pieces, both copies of the head's row
-        const int row = i / (nkc * 8), c = i % (nkc * 8);
-        uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (row < hn && c < pieces) {
-          const int64_t at = (r * a.H + h0 + row) * KC + 8 * c;
-          if (qcat_hi) {
-            v = *reinterpret_cast<const uint4 *>(qcat_hi + at);
-          } else {
-            const float4 x = *reinterpret_cast<const float4 *>(qcat + at), y = *reinterpret_cast<const float4 *>(qcat + at + 4);
-            v = make_uint4(pack_bf16(x.x, x.y), pack_bf16(x.z, x.w), pack_bf16(y.x, y.y), pack_bf16(y.z, y.w));
+      const int pieces = KC / 8, all = NH * nkc * 8;   // 16-byte pieces of the heads' rows, five per thread requested together
+      for (int i0 = tid; i0 < all; i0 += 5 * 128) {
+        uint4 v[5];
+#pragma unroll
+        for (int u = 0; u < 5; ++u) {
+          const int i = i0 + 128 * u, row = i / (nkc * 8), c = i % (nkc * 8);
+          v[u] = make_uint4(0u, 0u, 0u, 0u);
+          if (i < all && row < hn && c < pieces) {
+            const int64_t at = (r * a.H + h0 + row) * KC + 8 * c;
+            if (qcat_hi) {
+              v[u] = *reinterpret_cast<const uint4 *>(qcat_hi + at);
+            } else {
+              const float4 x = *reinterpret_cast<const float4 *>(qcat + at), y = *reinterpret_cast<const float4 *>(qcat + at + 4);
+              v[u] = make_uint4(pack_bf16(x.x, x.y), pack_bf16(x.z, x.w), pack_bf16(y.x, y.y), pack_bf16(y.z, y.w));
+            }
           }
         }
-        *reinterpret_cast<uint4 *>(qs + (c >> 3) * 16384 + la_sw128(row, c & 7)) = v;
-        *reinterpret_cast<uint4 *>(qs + (c >> 3) * 16384 + la_sw128(64 + row, c & 7)) = v;
+#pragma unroll
+        for (int u = 0; u < 5; ++u) {
+          const int i = i0 + 128 * u, row = i / (nkc * 8), c = i % (nkc * 8);
+          if (i < all) *reinterpret_cast<uint4 *>(qs + (c >> 3) * QB + la_sw128(row, c & 7)) = v[u];
+        }
       }
       fence_proxy_async();
       __syncwarp();
       if (lane == 0) mbar_arrive(q_full);
     }
-    const float f = a.scale;
-    for (int i = 0; i < nt; ++i) {
-      ok = __all_sync(0xffffffffu, mbar_wait(s_full(i & 1), (uint32_t)(i >> 1) & 1u, abort_flag));
-      if (!ok) { if (lane == 0) give_up(34); break; }
-      tc_fence_after();
-      uint32_t sc[KT];
+    const float f = a.scale * kLog2e;
+    float m[NH], l[NH];   // in powers of two, the same in every thread; this key's share of the sum
 #pragma unroll
-      for (int c = 0; c < KT; c += 16) tmem_ld16(tlane + LA_COL_S + 64 * (i & 1) + c, sc + c);
-      tmem_ld_wait();
-      const int lim = t - 1 - (tile0 + i) * KT;   // key e of the tile is visible iff e <= lim
-      float mx = -INFINITY;
-#pragma unroll
-      for (int e = 0; e < KT; ++e) {
-        const float v = e <= lim ? __uint_as_float(sc[e]) * f : -INFINITY;
-        sc[e] = __float_as_uint(v);
-        mx = fmaxf(mx, v);
-      }
-      const bool move = mx > m + LA_TAU;   // also at the first tile (m = -inf)
-      const float m_new = move ? mx : m;
-      if (i > 0 && __any_sync(0xffffffffu, move)) {
-        ok = __all_sync(0xffffffffu, mbar_wait(o_done((i - 1) & 1), (uint32_t)((i - 1) >> 1) & 1u, abort_flag));
-        if (!ok) { if (lane == 0) give_up(35); break; }
-        tc_fence_after();
-        const float g = move ? exp2f((m - m_new) * kLog2e) : 1.0f;
-        l *= g;
-        for (int c = 0; c < 64 * nvb; c += 16) {
-          uint32_t o[16];
-          tmem_ld16(tlane + LA_COL_O + c, o);
-          tmem_ld_wait();
-#pragma unroll
-          for (int e = 0; e < 16; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * g);
-          tmem_st16(tlane + LA_COL_O + c, o);
-        }
-      }
-      m = m_new;
-      if (i >= 2) {   // this P tile has been read
-        ok = __all_sync(0xffffffffu, mbar_wait(o_done(i & 1), (uint32_t)((i - 2) >> 1) & 1u, abort_flag));
-        if (!ok) { if (lane == 0) give_up(36); break; }
-        tc_fence_after();
-      }
-#pragma unroll
-      for (int c = 0; c < KT; c += 16) {
-        float p[16];
-        uint32_t w[8];
-#pragma unroll
-        for (int e = 0; e < 16; ++e) {
-          p[e] = la_ex2((__uint_as_float(sc[c + e]) - m) * kLog2e);   // (hidden keys: 2^-inf = 0)
-          l += p[e];
-        }
-#pragma unroll
-        for (int e = 0; e < 8; ++e) w[e] = warp < 2 ? pack_bf16(p[2 * e], p[2 * e + 1]) : pack_bf16(bf16_lo(p[2 * e]), bf16_lo(p[2 * e + 1]));
-        tmem_st8(tlane + LA_COL_P + 32 * (i & 1) + c / 2, w);
-      }
-      tmem_st_wait();
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(p_full(i & 1));
-    }
-    if (ok && nt > 0) {   // the last product (and so all of them) is complete
-      ok = __all_sync(0xffffffffu, mbar_wait(o_done((nt - 1) & 1), (uint32_t)((nt - 1) >> 1) & 1u, abort_flag));
-      if (!ok && lane == 0) give_up(37);
-      tc_fence_after();
-    }
-  }
-  ok = __syncthreads_and(ok ? 1 : 0) != 0 && !*abort_flag;   // nothing reads the tiles any more: they become the exchange buffer
-  float *ex = reinterpret_cast<float *>(sm);                 // [LA_H][LA_OLD]
-  if (ok && warp < 4) {
-    const uint32_t tlane = tmem_base + ((uint32_t)(warp * 32) << 16);
-    float *mine = ex + (tid & 63) * LA_OLD;
-    if (tid < LA_H) lsum[tid] = l;
-    auto part = [&](bool add) {
-      for (int c = 0; c < 64 * nvb; c += 16) {
-        uint32_t o[16];
-        if (nt > 0) {
-          tmem_ld16(tlane + LA_COL_O + c, o);
-          tmem_ld_wait();
-        } else {
-#pragma unroll
-          for (int e = 0; e < 16; ++e) o[e] = 0u;
-        }
-#pragma unroll
-        for (int e = 0; e < 16; e += 4) {
-          float4 v = make_float4(__uint_as_float(o[e]), __uint_as_float(o[e + 1]), __uint_as_float(o[e + 2]), __uint_as_float(o[e + 3]));
-          float4 *dst = reinterpret_cast<float4 *>(mine + c + e);
-          if (add) { const float4 x = *dst; v = make_float4(x.x + v.x, x.y + v.y, x.z + v.z, x.w + v.w); }
-          *dst = v;
-        }
-      }
+    for (int h = 0; h < NH; ++h) { m[h] = -INFINITY; l[h] = 0.0f; }
+    // (a warp that gives up stays in the loop, without waiting for anything, so that all warps reach the same block barriers)
+    auto wait = [&](uint32_t bar, uint32_t parity, int where) {
+      if (!ok) return;
+      ok = __all_sync(0xffffffffu, mbar_wait(bar, parity, abort_flag));
+      if (!ok && lane == 0) give_up(where);
     };
-    if (warp >= 2) part(false);
-    asm volatile("bar.sync 1, 128;" ::: "memory");
-    if (warp < 2) part(true);
-    if (out.splits > 1 && vb0 == 0 && tid < hn) {
-      float *ml = out.ml + (((int64_t)split * out.rows + r) * a.H + h0 + tid) * 2;
-      ml[0] = m;
-      ml[1] = l;
+    for (int i = 0; i < nt; ++i) {
+      wait(s_full(i & 1), (uint32_t)(i >> 1) & 1u, 34);
+      float v[NH];
+      bool above = false;
+      if (ok) {
+        tc_fence_after();
+        uint32_t raw[NH];
+#pragma unroll
+        for (int c = 0; c < NH; c += 16) tmem_ld16(tlane + col_s + NH * (i & 1) + c, raw + c);
+        tmem_ld_wait();
+        const bool visible = (tile0 + i) * LA_KEYS + tid < t;
+#pragma unroll
+        for (int h = 0; h < NH; ++h) {
+          v[h] = visible ? __uint_as_float(raw[h]) * f : -INFINITY;
+          above |= v[h] > m[h] + LA_TAU;   // (every score at the first visible key: m = -inf)
+        }
+      }
+      if (la_any(above || !ok)) {
+        if (ok) la_reduce<NH, true>(v, lane, red + warp * NH);
+        la_sync();
+        if (i > 0) wait(o_done((i - 1) & 1), (uint32_t)((i - 1) >> 1) & 1u, 35);
+        tc_fence_after();
+        float g[NH];
+#pragma unroll
+        for (int h = 0; h < NH; ++h) {
+          const float mx = fmaxf(fmaxf(red[h], red[NH + h]), fmaxf(red[2 * NH + h], red[3 * NH + h]));
+          const bool move = mx > m[h] + LA_TAU;
+          g[h] = move ? exp2f(m[h] - mx) : 1.0f;
+          if (move) m[h] = mx;
+          l[h] *= g[h];
+        }
+        if (ok && i > 0)
+          for (int c = 0; c < npv * 2 * NH; c += 16) {
+            uint32_t o[16];
+            tmem_ld16(tlane + c, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int e = 0; e < 16; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * (NH == 16 ? g[e] : (c & 16) ? g[(16 + e) % NH] : g[e]));
+            tmem_st16(tlane + c, o);
+          }
+        tmem_st_wait();
+      }
+      if (i >= 2) wait(o_done(i & 1), (uint32_t)((i - 2) >> 1) & 1u, 36);   // this P buffer has been read
+      unsigned char *pb = ps + (i & 1) * PB + (tid >> 6) * (PB / 2) + (tid & 7) * 2;
+      const int chunk = (tid & 63) >> 3;
+      if (ok) {
+#pragma unroll
+        for (int h = 0; h < NH; ++h) {
+          const float p = la_ex2(v[h] - m[h]);   // (a hidden key: 2^-inf = 0)
+          l[h] += p;
+          const __nv_bfloat16 hi = __float2bfloat16_rn(p);
+          *reinterpret_cast<__nv_bfloat16 *>(pb + la_sw128(h, chunk)) = hi;
+          *reinterpret_cast<__nv_bfloat16 *>(pb + la_sw128(NH + h, chunk)) = __float2bfloat16_rn(p - __bfloat162float(hi));
+        }
+        fence_proxy_async();
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(p_full(i & 1));
+      }
+    }
+    if (nt > 0) wait(o_done((nt - 1) & 1), (uint32_t)((nt - 1) >> 1) & 1u, 37);   // the last product (and so all of them) is complete
+    tc_fence_after();
+    la_sync();
+    la_reduce<NH, false>(l, lane, red + warp * NH);
+    la_sync();
+    if (__all_sync(0xffffffffu, ok && !*abort_flag)) {
+#pragma unroll
+      for (int h = 0; h < NH; ++h) l[h] = red[h] + red[NH + h] + red[2 * NH + h] + red[3 * NH + h];
+      float inv[NH];
+#pragma unroll
+      for (int h = 0; h < NH; ++h) inv[h] = out.splits == 1 ? 1.0f / l[h] : 1.0f;
+      // head h0's first value of this row, and from one head to the next
+      const int64_t first = out.splits == 1 ? ((int64_t)h0 * out.plane + r) * out.Kr : (((int64_t)split * out.rows + r) * a.H + h0) * out.Kr;
+      const int64_t step = out.splits == 1 ? out.plane * out.Kr : out.Kr;
+      float *of = out.splits == 1 ? out.o : out.part;
+      const BfOut ob = out.splits == 1 ? out.o_bf : BfOut();
+      for (int j = 0; j < npv; ++j) {
+        const int c = 128 * j + tid;   // this lane's column of the latent (columns past it belong to the key part)
+        uint32_t x[2 * NH];
+        if (nt > 0) {
+#pragma unroll
+          for (int q = 0; q < 2 * NH; q += 16) tmem_ld16(tlane + j * 2 * NH + q, x + q);
+          tmem_ld_wait();
+        }
+        const bool in = nt > 0 && c < a.Kp;
+        if (c < out.Kr) {
+          int64_t at = first + c;
+#pragma unroll
+          for (int h = 0; h < NH; ++h, at += step)
+            if (h < hn) st1(of, ob, at, in ? (__uint_as_float(x[h]) + __uint_as_float(x[NH + h])) * inv[h] : 0.0f);
+        }
+      }
+      if (out.splits > 1 && tid == 0)
+#pragma unroll
+        for (int h = 0; h < NH; ++h)
+          if (h < hn) {
+            float *ml = out.ml + (((int64_t)split * out.rows + r) * a.H + h0 + h) * 2;
+            ml[0] = m[h];
+            ml[1] = l[h];
+          }
     }
   }
   tc_fence_before();
   __syncthreads();
-  if (ok) {
-    const int cols = 64 * nvb, c0 = 64 * vb0;
-    for (int i = tid; i < hn * cols; i += LA_THREADS) {
-      const int h = i / cols, c = i % cols;
-      const float v = c0 + c < a.Kp ? ex[h * LA_OLD + c] : 0.0f;   // (columns past the latent belong to the key part)
-      if (out.splits == 1) st1(out.o, out.o_bf, ((int64_t)(h0 + h) * out.plane + r) * out.Kr + c0 + c, v / lsum[h]);
-      else out.part[(((int64_t)split * out.rows + r) * a.H + h0 + h) * out.Kr + c0 + c] = v;
-    }
-  }
   if (warp == 5) {
     tc_fence_after();
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(512u) : "memory");
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(tmem_cols) : "memory");
   }
 }
 
@@ -623,21 +688,21 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
 static bool latent_tc(const caten_b200_ctx *ctx, const LatentArgs &a) {
   return a.cache_bf16 && ctx->attn_tc && ctx->encode_tiled && a.KC() <= 64 * LA_MAX_BLOCKS;
 }
-static int latent_tile(const LatentArgs &a) { return a.KC() <= 320 ? 64 : 32; }   // a ring of at least two tiles beside Q
+static int latent_heads(const LatentArgs &a) { return a.H <= 16 ? 16 : 32; }   // per CTA
 static int64_t latent_ctas(const LatentArgs &a, bool tc, int64_t rows) {
-  if (!tc) return (a.H + LS_H - 1) / LS_H * rows;
-  return (int64_t)((a.H + LA_H - 1) / LA_H) * ((a.Kr / 64 + LA_VBLOCKS - 1) / LA_VBLOCKS) * rows;
+  const int per = tc ? latent_heads(a) : LS_H;
+  return (a.H + per - 1) / per * rows;
 }
 
 int latent_splits(const caten_b200_ctx *ctx, const LatentArgs &a, int64_t rows, int64_t keys) {
   const bool tc = latent_tc(ctx, a);
-  const int kt = tc ? latent_tile(a) : LS_KEYS;
+  const int kt = tc ? LA_KEYS : LS_KEYS, fixed = tc ? 2 : 6;   // what a CTA costs besides its tiles, in tiles
   const int64_t tiles = (keys + kt - 1) / kt, ctas = latent_ctas(a, tc, rows), slots = (int64_t)ctx->sm_count * (tc ? 1 : 4);
   int best = 1;
   int64_t cost = INT64_MAX;
-  for (int S = 1; S <= 32 && (S == 1 || tiles >= 2 * S); S = S < 4 ? S + 1 : S + S / 4) {
-    // waves x (tiles of a CTA + what a CTA costs besides), and merging the parts
-    const int64_t c = (ctas * S + slots - 1) / slots * ((tiles + S - 1) / S + 6) + (S > 1 ? 6 : 0);
+  for (int S = 1; S <= 32 && S <= tiles; S = S < 4 ? S + 1 : S + S / 4) {
+    // waves x (tiles of a CTA + its fixed part), and merging the parts
+    const int64_t c = (ctas * S + slots - 1) / slots * ((tiles + S - 1) / S + fixed) + (S > 1 ? 2 : 0);
     if (c < cost) { cost = c; best = S; }
   }
   return best;
@@ -646,25 +711,28 @@ int latent_splits(const caten_b200_ctx *ctx, const LatentArgs &a, int64_t rows, 
 typedef CUresult (*EncodeTiledFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *, const cuuint32_t *, const cuuint32_t *,
                                   CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-template <int KT>
+template <int NH>
 static int launch_tc(caten_b200_ctx *ctx, const LatentArgs &a, const LatentAbsorbed &x, const LatentOut &out, dim3 grid) {
-  const int KC = a.KC(), nkc = (KC + 63) / 64;
+  const int KC = a.KC(), nkc = (KC + 63) / 64, np = (nkc + 1) / 2, npv = (a.Kr / 64 + 1) / 2;
   const cuuint64_t dims[2] = {(cuuint64_t)KC, (cuuint64_t)(a.B * a.cap)}, strides[1] = {(cuuint64_t)KC * 2};
-  const cuuint32_t box[2] = {64, KT}, estr[2] = {1, 1};
+  const cuuint32_t box[2] = {64, LA_KEYS}, estr[2] = {1, 1};
   CUtensorMap map;
   const CUresult e = ((EncodeTiledFn)ctx->encode_tiled)(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.cache, dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                                                         CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   if (e != CUDA_SUCCESS) return fail(ctx, CATEN_B200_ECUDA, "cuTensorMapEncodeTiled failed (%d)", (int)e);
-  const size_t stage = (size_t)nkc * KT * 128, q = (size_t)nkc * 16384, tail = (2 * LA_MAX_STAGES + 7) * 8 + 16 + LA_H * 4;
-  int stages = (int)((224 * 1024 - q) / stage);
+  const size_t stage = (size_t)nkc * LA_BLOCK, rest = (size_t)nkc * NH * 128 + 2 * 4 * NH * 128 + (LA_BARS + 1) * 8 + 4 * NH * sizeof(float);
+  int stages = (int)((224 * 1024 - rest) / stage);
   if (stages > LA_MAX_STAGES) stages = LA_MAX_STAGES;
-  size_t tiles = q + stage * stages;
-  if (tiles < (size_t)LA_H * LA_OLD * 4) tiles = (size_t)LA_H * LA_OLD * 4;
-  const size_t smem = 1024 + tiles + tail;
+  while (stages * np > LA_MAX_PAIRS) --stages;
+  // (one stage: the last pair may be a single block beside which the second product's operand reaches into Q, harmlessly)
+  const size_t smem = 1024 + stage * stages + rest;
+  uint32_t cols = 32;
+  while (cols < (uint32_t)(npv * 2 * NH + 2 * NH)) cols *= 2;
   const uint32_t base = (1u << 4) | (1u << 7) | (1u << 10) | (8u << 24);   // fp32 accumulate, bf16 x bf16, M = 128
-  const uint32_t idesc_s = base | ((uint32_t)(KT >> 3) << 17), idesc_pv = base | ((uint32_t)(64 >> 3) << 17) | (1u << 16);
-  CB_CUDA(ctx, cudaFuncSetAttribute(latent_attn_tc_kernel<KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  launch_k(ctx, latent_attn_tc_kernel<KT>, grid, dim3(LA_THREADS), smem, map, a, x.qcat_bf.hi ? nullptr : x.qcat, x.qcat_bf.hi, out, stages, idesc_s, idesc_pv, ctx->d_status);
+  const uint32_t idesc_s = base | ((uint32_t)(NH >> 3) << 17), idesc_pv = base | ((uint32_t)(2 * NH >> 3) << 17) | (1u << 15);   // second product: A MN-major
+  CB_CUDA(ctx, cudaFuncSetAttribute(latent_attn_tc_kernel<NH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  launch_k(ctx, latent_attn_tc_kernel<NH>, grid, dim3(LA_THREADS), smem, map, a, x.qcat_bf.hi ? nullptr : x.qcat, x.qcat_bf.hi, out, stages, x.early ? 1 : 0, cols, idesc_s,
+           idesc_pv, ctx->d_status);
   CB_LAUNCH_CHECK(ctx, "latent_attn_tc_kernel");
   return 0;
 }
@@ -679,7 +747,7 @@ int launch_latent_absorbed(caten_b200_ctx *ctx, const LatentArgs &a, const Laten
   out.o = x.o; out.o_bf = x.o_bf; out.part = x.part; out.ml = x.ml; out.plane = x.plane; out.rows = rows; out.Kr = a.Kr; out.H = a.H; out.splits = x.splits;
   if (latent_tc(ctx, a)) {
     const dim3 grid((unsigned)(latent_ctas(a, true, 1)), (unsigned)rows, (unsigned)x.splits);
-    if (int rc = latent_tile(a) == 64 ? launch_tc<64>(ctx, a, x, out, grid) : launch_tc<32>(ctx, a, x, out, grid)) return rc;
+    if (int rc = latent_heads(a) == 16 ? launch_tc<16>(ctx, a, x, out, grid) : launch_tc<32>(ctx, a, x, out, grid)) return rc;
   } else {
     const size_t smem = (size_t)(LS_H * (a.KC() + LS_KEYS) + 3 * LS_H) * sizeof(float);
     launch_k(ctx, latent_attn_simt_kernel, dim3((unsigned)((a.H + LS_H - 1) / LS_H), (unsigned)rows, (unsigned)x.splits), dim3(LS_THREADS), smem, a, x.qcat, x.qcat_bf, out);

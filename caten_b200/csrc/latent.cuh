@@ -43,6 +43,7 @@ struct LatentAbsorbed {
   int64_t plane = 0;
   float *part = nullptr, *ml = nullptr;   // several splits: [splits, rows, H, Kr] and [splits, rows, H, 2]
   int splits = 1;
+  bool early = false;               // cache and position are complete before the kernel in front of this one starts
 };
 // Key splits of a launch over `rows` rows that may see `keys` keys.
 int latent_splits(const caten_b200_ctx *ctx, const LatentArgs &a, int64_t rows, int64_t keys);

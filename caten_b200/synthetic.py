@@ -210,6 +210,73 @@ def synth_binusun(cfg: dict, seed: int = 0, low_rank: int = 16) -> dict:
     return t
 
 
+def goselix_config(width: int, vocab: int, order: str, ff: int, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int, ret_heads: int,
+                   ret_dim: int, ret_vdim: int, ret_rot: int, experts: int = 4, top: int = 1, expert_ff: int = 32, rot_base: float = 10000.0,
+                   ret_base: float = 10000.0, scale: float | None = None, decay=None, loop: tuple | None = None, eps: float = 1e-5) -> dict:
+    """A Goselix configuration (the content of config.json).  ``order``: two letters per layer, "l" latent attention or
+    "r" retention, then "d" a dense feed-forward, "m" a mixture of experts or "-" none.  ``loop``: (start, stop, times)."""
+    lat = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank,
+           "scale": (dim + rot_dim) ** -0.5 if scale is None else scale, "rot": {"base": rot_base, "dims": rot_dim}}
+    ret = {"heads": ret_heads, "dim": ret_dim, "vdim": ret_vdim, "rot": {"base": ret_base, "dims": ret_rot},
+           "decay": list(decay) if decay is not None else [1.0 - 2.0 ** (-3 - h % 8) for h in range(ret_heads)]}
+    mlp = {"d": {"kind": "dense", "ff": ff}, "m": {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": expert_ff}}, "-": None}
+    layers = [{"type": "latent_attention" if a == "l" else "retention", "mixer": dict(lat) if a == "l" else dict(ret), "mlp": mlp[b]}
+              for a, b in zip(order[0::2], order[1::2])]
+    return {"architecture": "Goselix", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": eps},
+            "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]} if loop else None}
+
+
+def synth_goselix(cfg: dict, seed: int = 0) -> dict:
+    """Random weights of a Goselix configuration: tensor name -> bf16 bit patterns (uint16).  Matrices ~ N(0, 1 / in); norm
+    gains around 1; router rows large enough that scores spread over (0, 1) and choices are rarely close."""
+    from .safetensors import f32_to_bf16
+    rng = np.random.Generator(np.random.PCG64(seed))
+    width, vocab, t = cfg["width"], cfg["vocab"], {}
+
+    def mat(name, rows, cols, gain=1.0):
+        t[name] = f32_to_bf16(rng.standard_normal((rows, cols), dtype=np.float32) * np.float32(gain * cols ** -0.5))
+
+    def vec(name, shape, mean, std):
+        t[name] = f32_to_bf16(np.float32(mean) + rng.standard_normal(shape, dtype=np.float32) * np.float32(std))
+
+    def glu(pre, ff):
+        mat(pre + "gate", ff, width)
+        mat(pre + "up", ff, width)
+        mat(pre + "down", width, ff)
+
+    t["embed"] = f32_to_bf16(rng.standard_normal((vocab, width), dtype=np.float32))
+    if cfg.get("loop"):
+        vec("loop.step", (cfg["loop"]["times"], width), 0.0, 0.5)
+    for i, l in enumerate(cfg["layers"]):
+        pre, m, mlp = f"l{i}.", l["mixer"], l["mlp"]
+        mix = pre + "mix."
+        H, D, E = m["heads"], m["dim"], m["vdim"]
+        for n in ("norm1", "norm2")[:2 if mlp else 1]:
+            vec(pre + n, (width,), 1.0, 0.1)
+        if l["type"] == "latent_attention":
+            P, Q, K = m["rot_dim"], m["q_rank"], m["kv_rank"]
+            mat(mix + "dq", Q, width)
+            vec(mix + "dq.norm", (Q,), 1.0, 0.1)
+            mat(mix + "uq", H * (D + P), Q)
+            mat(mix + "dkv", K + P, width)
+            vec(mix + "dkv.norm", (K,), 1.0, 0.1)
+            mat(mix + "uk", H * D, K)
+            mat(mix + "uv", H * E, K)
+        else:
+            for c, n in (("q", D), ("k", D), ("v", E), ("g", E)):
+                mat(mix + c, H * n, width)
+        mat(mix + "o", width, H * E)
+        if mlp and mlp["kind"] == "dense":
+            glu(pre + "mlp.", mlp["ff"])
+        elif mlp:
+            mat(pre + "mlp.router", mlp["router"]["experts"], width, 2.0)
+            for e in range(mlp["router"]["experts"]):
+                glu(f"{pre}mlp.e{e}.", mlp["expert"]["ff"])
+    vec("final.norm", (width,), 1.0, 0.1)
+    mat("head", vocab, width)
+    return t
+
+
 def synth_prompts(batch: int, length: int, vocab: int, seed: int = 0) -> np.ndarray:
     """[batch, length] int64 token ids uniform in [0, vocab)."""
     rng = np.random.Generator(np.random.PCG64(seed))

@@ -506,7 +506,8 @@ enum {
   CATEN_B200_K_DECODE_STEP = 7,   /* the whole single-token step of 1..4 sequences, which is one kernel */
   CATEN_B200_K_WKV = 8,           /* recurrence of a time-mixing or retention layer */
   CATEN_B200_K_PREP = 9,          /* rotation, q/k norm and cache append; token-shift mixes; expert routing */
-  CATEN_B200_K_COUNT = 10
+  CATEN_B200_K_EXPERTS = 10,      /* linears of a mixture of experts */
+  CATEN_B200_K_COUNT = 11
 };
 /* Starts timing the classes whose bit (1 << class) is set in class_mask. */
 int caten_b200_profile_begin(caten_b200_ctx *ctx, unsigned class_mask);
