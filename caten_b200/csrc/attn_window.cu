@@ -292,9 +292,6 @@ int launch_attn_window_prefill(caten_b200_ctx *ctx, const AttnArgs &args, int te
 constexpr int AD_WORK = 256, AD_THREADS = AD_WORK + 32, AD_MIN_STAGES = 3, AD_MAX_STAGES = 8;
 
 __device__ __forceinline__ void work_sync() { asm volatile("bar.sync 1, %0;" ::"n"(AD_WORK) : "memory"); }
-__device__ __forceinline__ void bulk_load(uint32_t dst, const void *src, uint32_t bytes, uint32_t bar) {
-  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
-}
 __device__ __forceinline__ void bulk_hint(const void *src, uint32_t bytes) {
   asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(src), "r"(bytes) : "memory");
 }

@@ -34,7 +34,7 @@ struct Run {            // one execution of a layer in a step
   float *kc = nullptr, *vc = nullptr;        // attention: ring caches [B, G, cap, Dp / Ep]
   int64_t cap = 0;
   float *state = nullptr, *shift = nullptr;  // time mixing: [B, H, Dp, Dp] and [B, wp]; retention: [B, H, Dp, Ep]
-  uint8_t *latents = nullptr;                // latent attention: [B, cap, p16(kv_rank) + p16(rot_dims)], bf16 or fp32
+  uint8_t *latents = nullptr;                // latent attention: see LatentArgs::cache
 };
 
 }  // namespace
@@ -158,6 +158,8 @@ static LatentArgs latent_args(const Dec *m, const caten_b200_layer_desc &c) {
   a.K = c.kv_rank; a.Kp = (int)p16(c.kv_rank); a.Kr = (int)p64(c.kv_rank); a.Q = c.q_rank; a.Qr = (int)p64(c.q_rank);
   a.freq = c.rot_freq; a.q_norm = c.q_norm; a.kv_norm = c.kv_norm; a.eps = m->desc.eps; a.scale = c.scale;
   a.cache_bf16 = m->desc.precision == CATEN_B200_PREC_BF16;
+  a.tiled = a.cache_bf16 && a.KC() <= 576;
+  a.cap = (m->desc.max_seq_len + 127) / 128 * 128;
   return a;
 }
 
@@ -233,7 +235,7 @@ int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc
       most(&l_cq, p64(c.q_rank)); most(&l_q, H * (Dp + Pp)); most(&l_qn, H * p64(c.dim)); most(&l_cat, H * (Kp + Pp)); most(&l_o, H * Kr);
       most(&l_c, Kr); most(&l_kr, Pp > 0 ? Pp : 16); most(&l_kv, c.kv_w->rows);
       LatentArgs a = latent_args(m, c);
-      a.B = (int)B; a.cap = p64(T);
+      a.B = (int)B;
       most(&l_part, latent_splits(ctx, a, B, a.cap) * B * H * Kr);
       most(&l_part, 4 * B * H * Kr);
       caten_b200_weight &uv = m->uv[(size_t)(&c - m->layers.data())];
@@ -262,8 +264,8 @@ int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc
       if (!rc) rc = dec_floats(m, &r.vc, B * c.kv_heads * r.cap * Ep);
       bytes = B * c.kv_heads * r.cap * (Dp + Ep) * 4;
     } else if (c.mixer == CATEN_B200_MIX_LATENT) {
-      r.cap = p64(T);
-      bytes = B * r.cap * (p16(c.kv_rank) + p16(c.rot_dims)) * (dsc->precision == CATEN_B200_PREC_BF16 ? 2 : 4);
+      const LatentArgs a = latent_args(m, c);
+      bytes = B * a.seq_elems() * (a.cache_bf16 ? 2 : 4);
       rc = dec_alloc(m, (void **)&r.latents, (size_t)bytes);
     } else if (c.mixer == CATEN_B200_MIX_RETENTION) {
       bytes = B * c.heads * Dp * p16(c.vdim) * 4;
@@ -555,8 +557,7 @@ class StepRunner {
     LatentArgs a = latent_args(m_, c);
     PartIn pin;
     if (int rc = linear(c.in_w, m_->hp, m_->hp_bf, nullptr, m_->y, none_, defer_ ? &pin : nullptr)) return rc;
-    a.cap = r.cap;
-    a.cache = r.latents + p_.b0 * r.cap * a.KC() * (a.cache_bf16 ? 2 : 4);
+    a.cache = r.latents + p_.b0 * a.seq_elems() * (a.cache_bf16 ? 2 : 4);
     a.B = (int)p_.nb; a.s = (int)p_.s; a.n = (int)p_.n; a.d_n = p_.d_n;
     { ProfScope prof(ctx_, CATEN_B200_K_PREP); if (int rc = launch_latent_prep(ctx_, a, m_->y, pin, c.in_w->rows, m_->cq, bf(m_->cq_bf))) return rc; }
     const bool absorbed = p_.s <= LATENT_ABSORB;

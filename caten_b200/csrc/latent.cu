@@ -8,14 +8,16 @@
 //
 // latent_attn_tc_kernel (bf16 models): tcgen05.  A CTA serves NH = 16 or 32 heads of one row; keys go in tiles of 128, and both
 // products have the keys' or the latent's dims, not the heads, as the 128 lanes of tensor memory, so that few heads waste nothing:
-//   warp 4      TMA: a tile of 128 cached rows as 64-column blocks with the 128-byte swizzle, two blocks to a barrier.  The same
-//               blocks are the K-major A operand of S^T = C.Q^T and the MN-major A operand of O^T += C^T.P^T
-//   warps 5, 6  tcgen05.mma: one warp issues the scores of tile after tile, as soon as a tile has arrived and its score columns have
+//   warp 8      bulk copies: a tile of 128 cached rows, stored in device memory as the operand tiles it becomes (LatentArgs::cache), two
+//               64-column blocks to a barrier.  The same blocks are the K-major A operand of S^T = C.Q^T and the MN-major A operand
+//               of O^T += C^T.P^T
+//   warps 9, 10 tcgen05.mma: one warp issues the scores of tile after tile, as soon as a tile has arrived and its score columns have
 //               been read, the other the outputs.  With few heads a product takes less time than issuing it, so the two streams
 //               of issues run side by side, and a tile is given back as soon as its output is formed
-//   warps 0..3  one key per thread, all its heads: a head's reference maximum moves lazily (as in attention_tc.cu: only when a score
-//               exceeds it by LA_TAU; one vote per tile finds out), p = hi + lo in bf16 goes to shared memory as the 2 NH rows of the
-//               second product's B operand (hi of all heads, then lo), so p keeps 16 bits; the two halves of O are added at the end
+//   warps 0..7  one key and half of the heads per thread: a head's reference maximum moves lazily (as in attention_tc.cu: only when a
+//               score exceeds it by LA_TAU; one vote per tile finds out), p = hi + lo in bf16 goes to shared memory as the 2 NH rows
+//               of the second product's B operand (hi of all heads, then lo), so p keeps 16 bits; the two halves of O are added at
+//               the end
 // Keys may be split over CTAs; latent_combine_kernel then merges the parts.
 // Every mbarrier wait is bounded: when one runs out the CTA records it in the status word, leaves its loops, waits for its
 // copies in flight, frees tensor memory and writes no output.
@@ -78,9 +80,9 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(const LatentArg
   for (int w = 0; w < LP_THREADS / 32; ++w) { sq += red[0][w]; sc += red[1][w]; }
   const float rq = 1.0f / sqrtf(sq / (float)a.Q + a.eps), rc = 1.0f / sqrtf(sc / (float)a.K + a.eps);
   for (int c = tid; c < a.Qr; c += LP_THREADS) st1(cq, cq_bf, r * a.Qr + c, row[c] * rq * a.q_norm[c]);
-  const int64_t at = ((r / a.s) * a.cap + pos) * (a.Kp + a.Pp);
+  const int64_t seq = r / a.s;
   const float *lat = row + a.Qr, *key = lat + a.Kp;
-  for (int c = tid; c < a.Kp; c += LP_THREADS) st_cache(a.cache, a.cache_bf16, at + c, lat[c] * rc * a.kv_norm[c]);
+  for (int c = tid; c < a.Kp; c += LP_THREADS) st_cache(a.cache, a.cache_bf16, a.at(seq, pos, c), lat[c] * rc * a.kv_norm[c]);
   const int half = a.P / 2;
   for (int i = tid; i < a.Pp; i += LP_THREADS) {
     float v = 0.0f;
@@ -90,12 +92,13 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(const LatentArg
       sincosf((float)pos * a.freq[f], &sn, &cs);
       v = i < half ? key[i] * cs - key[i + half] * sn : key[i] * cs + key[f] * sn;
     }
-    st_cache(a.cache, a.cache_bf16, at + a.Kp + i, v);
+    st_cache(a.cache, a.cache_bf16, a.at(seq, pos, a.Kp + i), v);
   }
 }
 
 static int check_latent(caten_b200_ctx *ctx, const LatentArgs &a) {
-  if (a.H <= 0 || a.D <= 0 || a.E <= 0 || a.K <= 0 || a.Q <= 0 || a.P < 0 || a.P % 2 || a.Dp % 16 || a.Pp % 16 || a.Ep % 16 || a.Kp % 16 || a.Kr % 64 || a.Qr % 64 || a.n < 0 || a.cap <= 0)
+  if (a.H <= 0 || a.D <= 0 || a.E <= 0 || a.K <= 0 || a.Q <= 0 || a.P < 0 || a.P % 2 || a.Dp % 16 || a.Pp % 16 || a.Ep % 16 || a.Kp % 16 || a.Kr % 64 || a.Qr % 64 || a.n < 0 || a.cap <= 0 ||
+      (a.tiled && (!a.cache_bf16 || a.cap % 128)))
     return fail(ctx, CATEN_B200_EINVAL, "latent attention: bad shape");
   if (a.K > 1024 || a.P > 256 || a.Q > 8192 || a.H > 4096) return fail(ctx, CATEN_B200_EUNSUPPORTED, "latent attention: latent of %d or rotated part of %d", a.K, a.P);
   if (!a.d_n && (int64_t)a.n + a.s > a.cap) return fail(ctx, CATEN_B200_EINVAL, "latent attention: %lld tokens in a cache of %lld", (long long)a.n + a.s, (long long)a.cap);
@@ -194,13 +197,17 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const LatentArgs a, 
   pdl_enter();
   const int64_t r = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
   if (r >= rows) return;
-  const int lane = threadIdx.x & 31, KC = a.Kp + a.Pp;
-  const int64_t from = ((int64_t)(b0 + r / t) * a.cap + r % t) * KC;
-  for (int j = lane; j < a.Kr; j += 32) {
-    if (a.cache_bf16 && c_bf.hi) c_bf.hi[r * a.Kr + j] = j < a.Kp ? reinterpret_cast<const __nv_bfloat16 *>(a.cache)[from + j] : __float2bfloat16_rn(0.0f);
-    else st1(c, c_bf, r * a.Kr + j, j < a.Kp ? ld_cache(a.cache, a.cache_bf16, from + j) : 0.0f);
+  const int lane = threadIdx.x & 31;
+  const int64_t seq = b0 + r / t, row = r % t;
+  for (int j = 8 * lane; j < a.Kr; j += 256) {   // 8 columns a lane
+    const int64_t to = r * a.Kr + j, from = a.at(seq, row, j);
+    if (a.cache_bf16 && c_bf.hi) {
+      *reinterpret_cast<uint4 *>(c_bf.hi + to) = j < a.Kp ? *reinterpret_cast<const uint4 *>(reinterpret_cast<const __nv_bfloat16 *>(a.cache) + from) : make_uint4(0u, 0u, 0u, 0u);
+    } else {
+      for (int e = 0; e < 8; ++e) st1(c, c_bf, to + e, j < a.Kp ? ld_cache(a.cache, a.cache_bf16, from + e) : 0.0f);
+    }
   }
-  for (int j = lane; j < a.Pp; j += 32) kr[r * a.Pp + j] = ld_cache(a.cache, a.cache_bf16, from + a.Kp + j);
+  for (int j = lane; j < a.Pp; j += 32) kr[r * a.Pp + j] = ld_cache(a.cache, a.cache_bf16, a.at(seq, row, a.Kp + j));
 }
 
 int launch_latent_gather(caten_b200_ctx *ctx, const LatentArgs &a, int b0, int nb, int t, float *c, BfOut c_bf, float *kr) {
@@ -236,7 +243,7 @@ __global__ void __launch_bounds__(LS_THREADS) latent_attn_simt_kernel(const Late
   const int t = (a.d_n ? *a.d_n : a.n) + (int)(r % a.s) + 1;
   const int blocks = (t + LS_KEYS - 1) / LS_KEYS, per = (blocks + out.splits - 1) / out.splits;
   const int jb = split * per * LS_KEYS, je = min(t, (split + 1) * per * LS_KEYS);
-  const int64_t base = (r / a.s) * a.cap * KC;
+  const int64_t seq = r / a.s;
   for (int i = tid; i < LS_H * KC; i += LS_THREADS) {
     const int h = h0 + i / KC;
     const int64_t at = (r * a.H + h) * KC + i % KC;
@@ -258,7 +265,7 @@ __global__ void __launch_bounds__(LS_THREADS) latent_attn_simt_kernel(const Late
       for (int h = 0; h < LS_H; ++h) s[h] = 0.0f;
       if (j < je)
         for (int c = lane; c < KC; c += 32) {
-          const float x = ld_cache(a.cache, a.cache_bf16, base + (int64_t)j * KC + c);
+          const float x = ld_cache(a.cache, a.cache_bf16, a.at(seq, j, c));
 #pragma unroll
           for (int h = 0; h < LS_H; ++h) s[h] = fmaf(q[h * KC + c], x, s[h]);
         }
@@ -294,7 +301,7 @@ __global__ void __launch_bounds__(LS_THREADS) latent_attn_simt_kernel(const Late
       for (int i = 0; i < LS_COLS; ++i) {
         const int c = tid + LS_THREADS * i;
         if (c < a.Kp) {
-          const float x = ld_cache(a.cache, a.cache_bf16, base + (int64_t)(j0 + j) * KC + c);
+          const float x = ld_cache(a.cache, a.cache_bf16, a.at(seq, j0 + j, c));
 #pragma unroll
           for (int h = 0; h < LS_H; ++h) acc[h][i] = fmaf(p[h * LS_KEYS + j], x, acc[h][i]);
         }
@@ -347,7 +354,8 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentOut out
 // Absorbed attention on the tensor cores
 // ---------------------------------------------------------------------------------------------
 constexpr int LA_KEYS = 128;              // cached rows per tile
-constexpr int LA_THREADS = 224;
+constexpr int LA_SOFT = 256;              // softmax threads
+constexpr int LA_THREADS = LA_SOFT + 96;
 constexpr int LA_MAX_BLOCKS = 9;          // 64-column blocks of a cached row: up to 576 columns
 constexpr int LA_MAX_STAGES = 4, LA_MAX_PAIRS = 10, LA_BARS = 2 * LA_MAX_PAIRS + 6;   // full, empty of the ring's pairs; s, p, o (two each); then q
 constexpr uint32_t LA_BLOCK = LA_KEYS * 128;   // bytes
@@ -359,21 +367,22 @@ __device__ __forceinline__ float la_ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));   // results below 2^-126 flush to zero
   return y;
 }
-__device__ __forceinline__ void la_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ void la_sync() { asm volatile("bar.sync 1, %0;" ::"n"(LA_SOFT) : "memory"); }
 __device__ __forceinline__ bool la_any(bool x) {   // over the softmax threads
   uint32_t r;
-  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.u32 p, %1, 0;\n\tbarrier.cta.red.or.pred q, 1, 128, p;\n\tselp.u32 %0, 1, 0, q;\n\t}" : "=r"(r) : "r"(x ? 1u : 0u) : "memory");
+  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.u32 p, %1, 0;\n\tbarrier.cta.red.or.pred q, 1, %2, p;\n\tselp.u32 %0, 1, 0, q;\n\t}"
+               : "=r"(r) : "r"(x ? 1u : 0u), "n"(LA_SOFT) : "memory");
   return r != 0;
 }
-// NH values per lane, reduced over the warp: each exchange halves the values a lane carries; afterwards red[h] holds head h's.
-template <int NH, bool MAX>
+// N values per lane, reduced over the warp: each exchange halves the values a lane carries; afterwards red[i] holds value i's.
+template <int N, bool MAX>
 __device__ __forceinline__ void la_reduce(const float *x, int lane, float *red) {
-  float v[NH];
+  float v[N];
 #pragma unroll
-  for (int h = 0; h < NH; ++h) v[h] = x[h];
-  int head = 0, step = 16;
+  for (int i = 0; i < N; ++i) v[i] = x[i];
+  int which = 0, step = 16;
 #pragma unroll
-  for (int n = NH; n > 1; n >>= 1, step >>= 1) {
+  for (int n = N; n > 1; n >>= 1, step >>= 1) {
     const bool up = (lane & step) != 0;
 #pragma unroll
     for (int i = 0; i < n / 2; ++i) {
@@ -381,30 +390,44 @@ __device__ __forceinline__ void la_reduce(const float *x, int lane, float *red) 
       const float got = __shfl_xor_sync(0xffffffffu, give, step);
       v[i] = MAX ? fmaxf(keep, got) : keep + got;
     }
-    head += up ? n / 2 : 0;
+    which += up ? n / 2 : 0;
   }
 #pragma unroll
-  for (int o = 16 / NH; o > 0; o >>= 1) {   // (NH = 16: one more exchange between the lanes that hold the same head)
+  for (int o = 16 / N; o > 0; o >>= 1) {   // the lanes that hold the same value
     const float got = __shfl_xor_sync(0xffffffffu, v[0], o);
     v[0] = MAX ? fmaxf(v[0], got) : v[0] + got;
   }
-  if ((lane & (32 / NH - 1)) == 0) red[head] = v[0];
+  if ((lane & (32 / N - 1)) == 0) red[which] = v[0];
+}
+template <int N> __device__ __forceinline__ void la_ld(uint32_t taddr, uint32_t *r) {
+  if (N == 8) tmem_ld8(taddr, r);
+  else tmem_ld16(taddr, r);
+}
+template <int N> __device__ __forceinline__ void la_st(uint32_t taddr, const uint32_t *r) {
+  if (N == 8) tmem_st8(taddr, r);
+  else tmem_st16(taddr, r);
 }
 
 // MN-major operand, 128-byte swizzle: 64-element blocks LA_BLOCK bytes apart, groups of 8 along k 1024 bytes apart
 __device__ __forceinline__ uint64_t la_desc_mn(uint32_t saddr) { return umma_desc(saddr) - ((uint64_t)1 << 16) + ((uint64_t)(LA_BLOCK >> 4) << 16); }
+// K-major operand with rows of 64 bytes, 64-byte swizzle, 8-row groups 512 bytes apart
+__device__ __forceinline__ uint64_t la_desc_narrow(uint32_t saddr) {
+  return (uint64_t)((saddr >> 4) & 0x3FFF) | (uint64_t)1 << 16 | (uint64_t)(512 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)4 << 61;
+}
 
 template <int NH>
-__global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __grid_constant__ CUtensorMap map, const LatentArgs a, const float *__restrict__ qcat,
-                                                                       const __nv_bfloat16 *__restrict__ qcat_hi, const LatentOut out, const int stages, const int early,
-                                                                       const uint32_t tmem_cols, const uint32_t idesc_s, const uint32_t idesc_pv, int *status) {
+__global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const LatentArgs a, const float *__restrict__ qcat, const __nv_bfloat16 *__restrict__ qcat_hi,
+                                                                       const LatentOut out, const int stages, const int early, const uint32_t tmem_cols, const uint32_t idesc_s,
+                                                                       const uint32_t idesc_pv, int *status) {
   extern __shared__ unsigned char la_raw[];
   unsigned char *sm = reinterpret_cast<unsigned char *>((reinterpret_cast<uintptr_t>(la_raw) + 1023) & ~(uintptr_t)1023);
+  constexpr int HT = NH / 2;   // heads of a softmax thread
   constexpr uint32_t QB = NH * 128, PB = 2 * 2 * NH * 128;   // bytes of a Q block; of a P buffer (two blocks of 64 keys, 2 NH rows)
-  const int KC = a.Kp + a.Pp, nkc = (KC + 63) / 64, np = (nkc + 1) / 2, ksteps = KC / 16, npv = (out.Kr / 64 + 1) / 2;
-  unsigned char *kv = sm, *qs = kv + (size_t)stages * nkc * LA_BLOCK, *ps = qs + nkc * QB;
+  const int KC = a.KC(), nkc = a.blocks(), np = (nkc + 1) / 2, ksteps = KC / 16, npv = (out.Kr / 64 + 1) / 2;
+  const uint32_t tile_bytes = (uint32_t)a.tile_elems() * 2u;
+  unsigned char *kv = sm, *qs = kv + (size_t)stages * tile_bytes, *ps = qs + nkc * QB;
   uint64_t *bars = reinterpret_cast<uint64_t *>(ps + 2 * PB);
-  float *red = reinterpret_cast<float *>(bars + LA_BARS + 1);   // [4][NH]
+  float *red = reinterpret_cast<float *>(bars + LA_BARS + 1);   // [4][NH]: a row per quadrant of keys
   const uint32_t bar0 = smem_u32(bars);
   auto full = [&](int s, int p) { return bar0 + 8u * (s * np + p); };
   auto empty = [&](int s, int p) { return bar0 + 8u * (LA_MAX_PAIRS + s * np + p); };
@@ -426,14 +449,14 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
     }
     for (int b = 0; b < 2; ++b) {
       mbar_init(s_full(b), 1);
-      mbar_init(p_full(b), 4);
+      mbar_init(p_full(b), LA_SOFT / 32);
       mbar_init(o_done(b), 1);
     }
-    mbar_init(q_full, 4);
+    mbar_init(q_full, LA_SOFT / 32);
     flags[0] = flags[1] = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
-  if (warp == 5) {
+  if (warp == 9) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(tmem_cols) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
@@ -441,9 +464,8 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = tmem_slot, col_s = (uint32_t)npv * 2 * NH;   // O: npv x 2 NH columns, then two score tiles of NH
-  if (warp == 4 && lane == 0) tma_prefetch_map(&map);
   // `early`: the cache and the position were complete before the kernel in front of this one started; only Q comes from it
-  if (warp != 4 || !early) pdl_wait();
+  if (warp != 8 || !early) pdl_wait();
   pdl_launch_dependents();
   const int t = (a.d_n ? *a.d_n : a.n) + (int)(r % a.s) + 1;   // keys this row sees
   const int tiles = (t + LA_KEYS - 1) / LA_KEYS, per = (tiles + out.splits - 1) / out.splits;
@@ -453,18 +475,17 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
   };
 
   bool ok = true;
-  if (warp == 4) {
+  if (warp == 8) {
     if (lane == 0) {
       int issued = 0, s = 0;
       uint32_t ph = 1;
-      const int row0 = (int)(r / a.s * a.cap) + tile0 * LA_KEYS;
-      for (int i = 0; i < nt && ok; ++i) {
+      const unsigned char *src = reinterpret_cast<const unsigned char *>(a.cache) + (r / a.s) * a.seq_elems() * 2 + (int64_t)tile0 * tile_bytes;
+      for (int i = 0; i < nt && ok; ++i, src += tile_bytes) {
         for (int p = 0; p < np; ++p) {
           if (!mbar_wait(empty(s, p), ph, abort_flag)) { give_up(30); ok = false; break; }
-          const int blocks = min(2, nkc - 2 * p);
-          mbar_expect_tx(full(s, p), (uint32_t)blocks * LA_BLOCK);
-          for (int c = 0; c < blocks; ++c)
-            tma_load_2d(smem_u32(kv) + (uint32_t)(s * nkc + 2 * p + c) * LA_BLOCK, &map, full(s, p), (2 * p + c) * 64, row0 + i * LA_KEYS);
+          const uint32_t at = (uint32_t)p * 2 * LA_BLOCK, bytes = min(2 * LA_BLOCK, tile_bytes - at);
+          mbar_expect_tx(full(s, p), bytes);
+          bulk_load(smem_u32(kv) + s * tile_bytes + at, src + at, bytes, full(s, p));
           ++issued;
         }
         if (++s == stages) { s = 0; ph ^= 1u; }
@@ -474,8 +495,9 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
           mbar_wait(full(i / np % stages, i % np), (uint32_t)(i / np / stages) & 1u, abort_flag + 1);
     }
     __syncwarp();
-  } else if (warp == 5) {
-    const uint64_t dq = umma_desc(smem_u32(qs)), dk = umma_desc(smem_u32(kv));
+  } else if (warp == 9) {
+    const uint64_t dq = umma_desc(smem_u32(qs)), dk0 = umma_desc(smem_u32(kv)), dn0 = la_desc_narrow(smem_u32(kv));
+    const int narrow = a.narrow() ? nkc - 1 : -1;
     ok = nt == 0 || mbar_wait(q_full, 0, abort_flag);
     if (!ok && lane == 0) give_up(31);
     int s = 0;
@@ -493,20 +515,20 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
         }
         tc_fence_after();
         if (elect_one()) {
-          const uint64_t da = dk + (uint64_t)((s * nkc + 2 * p) * (int)(LA_BLOCK >> 4)), db = dq + (uint64_t)(2 * p * (int)(QB >> 4));
+          const uint64_t at = (uint64_t)((s * tile_bytes + (uint32_t)p * 2 * LA_BLOCK) >> 4), db = dq + (uint64_t)(2 * p * (int)(QB >> 4));
           const int left = ksteps - 8 * p;
 #pragma unroll
           for (int k = 0; k < 8; ++k)   // 16 columns = 32 bytes = 2 descriptor units
             if (k < left)
-              umma_bf16(tmem_base + col_s + NH * (i & 1), da + (uint64_t)((k >> 2) * (LA_BLOCK >> 4) + 2 * (k & 3)), db + (uint64_t)((k >> 2) * (QB >> 4) + 2 * (k & 3)), idesc_s,
-                        p > 0 || k > 0 ? 1u : 0u);
+              umma_bf16(tmem_base + col_s + NH * (i & 1), (2 * p + (k >> 2) == narrow ? dn0 : dk0) + at + (uint64_t)((k >> 2) * (LA_BLOCK >> 4) + 2 * (k & 3)),
+                        db + (uint64_t)((k >> 2) * (QB >> 4) + 2 * (k & 3)), idesc_s, p > 0 || k > 0 ? 1u : 0u);
           if (p == np - 1) umma_commit(s_full(i & 1));
         }
         __syncwarp();
       }
       if (++s == stages) { s = 0; ph ^= 1u; }
     }
-  } else if (warp == 6) {
+  } else if (warp == 10) {
     const uint64_t dm = la_desc_mn(smem_u32(kv)), dp = umma_desc(smem_u32(ps));
     int s = 0;
     for (int i = 0; i < nt; ++i) {
@@ -518,7 +540,7 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
       if (elect_one()) {
         const uint64_t db = dp + (uint64_t)((i & 1) * (int)(PB >> 4));
         for (int j = 0; j < npv; ++j) {
-          const uint64_t da = dm + (uint64_t)((s * nkc + 2 * j) * (int)(LA_BLOCK >> 4));
+          const uint64_t da = dm + (uint64_t)((s * tile_bytes + (uint32_t)j * 2 * LA_BLOCK) >> 4);
           const uint32_t acc = tmem_base + (uint32_t)j * 2 * NH;
 #pragma unroll
           for (int k = 0; k < LA_KEYS / 16; ++k)   // A: 16 keys = 16 rows of 128 bytes = 128 descriptor units
@@ -533,15 +555,16 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
       if (++s == stages) s = 0;
     }
   } else {
-    // ---- softmax: thread = lane of tensor memory = key of the tile ----
-    const uint32_t tlane = tmem_base + ((uint32_t)(warp * 32) << 16);
+    // ---- softmax: thread = (key of the tile = lane of tensor memory, half of the heads) ----
+    const int quad = warp & 3, hh = (warp >> 2) * HT, key = quad * 32 + lane;
+    const uint32_t tlane = tmem_base + ((uint32_t)(quad * 32) << 16);
     {
-      const int pieces = KC / 8, all = NH * nkc * 8;   // 16-byte pieces of the heads' rows, five per thread requested together
-      for (int i0 = tid; i0 < all; i0 += 5 * 128) {
-        uint4 v[5];
+      const int pieces = KC / 8, all = NH * nkc * 8;   // 16-byte pieces of the heads' rows, three per thread requested together
+      for (int i0 = tid; i0 < all; i0 += 3 * LA_SOFT) {
+        uint4 v[3];
 #pragma unroll
-        for (int u = 0; u < 5; ++u) {
-          const int i = i0 + 128 * u, row = i / (nkc * 8), c = i % (nkc * 8);
+        for (int u = 0; u < 3; ++u) {
+          const int i = i0 + LA_SOFT * u, row = i / (nkc * 8), c = i % (nkc * 8);
           v[u] = make_uint4(0u, 0u, 0u, 0u);
           if (i < all && row < hn && c < pieces) {
             const int64_t at = (r * a.H + h0 + row) * KC + 8 * c;
@@ -554,8 +577,8 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
           }
         }
 #pragma unroll
-        for (int u = 0; u < 5; ++u) {
-          const int i = i0 + 128 * u, row = i / (nkc * 8), c = i % (nkc * 8);
+        for (int u = 0; u < 3; ++u) {
+          const int i = i0 + LA_SOFT * u, row = i / (nkc * 8), c = i % (nkc * 8);
           if (i < all) *reinterpret_cast<uint4 *>(qs + (c >> 3) * QB + la_sw128(row, c & 7)) = v[u];
         }
       }
@@ -564,9 +587,9 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
       if (lane == 0) mbar_arrive(q_full);
     }
     const float f = a.scale * kLog2e;
-    float m[NH], l[NH];   // in powers of two, the same in every thread; this key's share of the sum
+    float m[HT], l[HT];   // in powers of two, the same for every key; this key's share of the sum
 #pragma unroll
-    for (int h = 0; h < NH; ++h) { m[h] = -INFINITY; l[h] = 0.0f; }
+    for (int h = 0; h < HT; ++h) { m[h] = -INFINITY; l[h] = 0.0f; }
     // (a warp that gives up stays in the loop, without waiting for anything, so that all warps reach the same block barriers)
     auto wait = [&](uint32_t bar, uint32_t parity, int where) {
       if (!ok) return;
@@ -575,57 +598,57 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
     };
     for (int i = 0; i < nt; ++i) {
       wait(s_full(i & 1), (uint32_t)(i >> 1) & 1u, 34);
-      float v[NH];
+      float v[HT];
       bool above = false;
       if (ok) {
         tc_fence_after();
-        uint32_t raw[NH];
-#pragma unroll
-        for (int c = 0; c < NH; c += 16) tmem_ld16(tlane + col_s + NH * (i & 1) + c, raw + c);
+        uint32_t raw[HT];
+        la_ld<HT>(tlane + col_s + NH * (i & 1) + hh, raw);
         tmem_ld_wait();
-        const bool visible = (tile0 + i) * LA_KEYS + tid < t;
+        const bool visible = (tile0 + i) * LA_KEYS + key < t;
 #pragma unroll
-        for (int h = 0; h < NH; ++h) {
+        for (int h = 0; h < HT; ++h) {
           v[h] = visible ? __uint_as_float(raw[h]) * f : -INFINITY;
           above |= v[h] > m[h] + LA_TAU;   // (every score at the first visible key: m = -inf)
         }
       }
       if (la_any(above || !ok)) {
-        if (ok) la_reduce<NH, true>(v, lane, red + warp * NH);
+        if (ok) la_reduce<HT, true>(v, lane, red + quad * NH + hh);
         la_sync();
         if (i > 0) wait(o_done((i - 1) & 1), (uint32_t)((i - 1) >> 1) & 1u, 35);
         tc_fence_after();
-        float g[NH];
+        float g[HT];
 #pragma unroll
-        for (int h = 0; h < NH; ++h) {
-          const float mx = fmaxf(fmaxf(red[h], red[NH + h]), fmaxf(red[2 * NH + h], red[3 * NH + h]));
+        for (int h = 0; h < HT; ++h) {
+          const float *x = red + hh + h;
+          const float mx = fmaxf(fmaxf(x[0], x[NH]), fmaxf(x[2 * NH], x[3 * NH]));
           const bool move = mx > m[h] + LA_TAU;
           g[h] = move ? exp2f(m[h] - mx) : 1.0f;
           if (move) m[h] = mx;
           l[h] *= g[h];
         }
         if (ok && i > 0)
-          for (int c = 0; c < npv * 2 * NH; c += 16) {
-            uint32_t o[16];
-            tmem_ld16(tlane + c, o);
+          for (int c = hh; c < npv * 2 * NH; c += NH) {   // this thread's heads in the hi and lo columns of every block
+            uint32_t o[HT];
+            la_ld<HT>(tlane + c, o);
             tmem_ld_wait();
 #pragma unroll
-            for (int e = 0; e < 16; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * (NH == 16 ? g[e] : (c & 16) ? g[(16 + e) % NH] : g[e]));
-            tmem_st16(tlane + c, o);
+            for (int e = 0; e < HT; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * g[e]);
+            la_st<HT>(tlane + c, o);
           }
         tmem_st_wait();
       }
       if (i >= 2) wait(o_done(i & 1), (uint32_t)((i - 2) >> 1) & 1u, 36);   // this P buffer has been read
-      unsigned char *pb = ps + (i & 1) * PB + (tid >> 6) * (PB / 2) + (tid & 7) * 2;
-      const int chunk = (tid & 63) >> 3;
+      unsigned char *pb = ps + (i & 1) * PB + (key >> 6) * (PB / 2) + (key & 7) * 2;
+      const int chunk = (key & 63) >> 3;
       if (ok) {
 #pragma unroll
-        for (int h = 0; h < NH; ++h) {
+        for (int h = 0; h < HT; ++h) {
           const float p = la_ex2(v[h] - m[h]);   // (a hidden key: 2^-inf = 0)
           l[h] += p;
           const __nv_bfloat16 hi = __float2bfloat16_rn(p);
-          *reinterpret_cast<__nv_bfloat16 *>(pb + la_sw128(h, chunk)) = hi;
-          *reinterpret_cast<__nv_bfloat16 *>(pb + la_sw128(NH + h, chunk)) = __float2bfloat16_rn(p - __bfloat162float(hi));
+          *reinterpret_cast<__nv_bfloat16 *>(pb + la_sw128(hh + h, chunk)) = hi;
+          *reinterpret_cast<__nv_bfloat16 *>(pb + la_sw128(NH + hh + h, chunk)) = __float2bfloat16_rn(p - __bfloat162float(hi));
         }
         fence_proxy_async();
         tc_fence_before();
@@ -636,40 +659,43 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
     if (nt > 0) wait(o_done((nt - 1) & 1), (uint32_t)((nt - 1) >> 1) & 1u, 37);   // the last product (and so all of them) is complete
     tc_fence_after();
     la_sync();
-    la_reduce<NH, false>(l, lane, red + warp * NH);
+    la_reduce<HT, false>(l, lane, red + quad * NH + hh);
     la_sync();
     if (__all_sync(0xffffffffu, ok && !*abort_flag)) {
+      float inv[HT];
 #pragma unroll
-      for (int h = 0; h < NH; ++h) l[h] = red[h] + red[NH + h] + red[2 * NH + h] + red[3 * NH + h];
-      float inv[NH];
-#pragma unroll
-      for (int h = 0; h < NH; ++h) inv[h] = out.splits == 1 ? 1.0f / l[h] : 1.0f;
-      // head h0's first value of this row, and from one head to the next
-      const int64_t first = out.splits == 1 ? ((int64_t)h0 * out.plane + r) * out.Kr : (((int64_t)split * out.rows + r) * a.H + h0) * out.Kr;
+      for (int h = 0; h < HT; ++h) {
+        const float *x = red + hh + h;
+        l[h] = x[0] + x[NH] + x[2 * NH] + x[3 * NH];
+        inv[h] = out.splits == 1 ? 1.0f / l[h] : 1.0f;
+      }
+      // this thread's first head in this row, and from one head to the next
+      const int hb = h0 + hh;
+      const int64_t first = out.splits == 1 ? ((int64_t)hb * out.plane + r) * out.Kr : (((int64_t)split * out.rows + r) * a.H + hb) * out.Kr;
       const int64_t step = out.splits == 1 ? out.plane * out.Kr : out.Kr;
       float *of = out.splits == 1 ? out.o : out.part;
       const BfOut ob = out.splits == 1 ? out.o_bf : BfOut();
       for (int j = 0; j < npv; ++j) {
-        const int c = 128 * j + tid;   // this lane's column of the latent (columns past it belong to the key part)
-        uint32_t x[2 * NH];
+        const int c = 128 * j + key;   // this lane's column of the latent (columns past it belong to the key part)
+        uint32_t hi[HT], lo[HT];
         if (nt > 0) {
-#pragma unroll
-          for (int q = 0; q < 2 * NH; q += 16) tmem_ld16(tlane + j * 2 * NH + q, x + q);
+          la_ld<HT>(tlane + j * 2 * NH + hh, hi);
+          la_ld<HT>(tlane + j * 2 * NH + NH + hh, lo);
           tmem_ld_wait();
         }
         const bool in = nt > 0 && c < a.Kp;
         if (c < out.Kr) {
           int64_t at = first + c;
 #pragma unroll
-          for (int h = 0; h < NH; ++h, at += step)
-            if (h < hn) st1(of, ob, at, in ? (__uint_as_float(x[h]) + __uint_as_float(x[NH + h])) * inv[h] : 0.0f);
+          for (int h = 0; h < HT; ++h, at += step)
+            if (hb + h < a.H) st1(of, ob, at, in ? (__uint_as_float(hi[h]) + __uint_as_float(lo[h])) * inv[h] : 0.0f);
         }
       }
-      if (out.splits > 1 && tid == 0)
+      if (out.splits > 1 && key == 0)
 #pragma unroll
-        for (int h = 0; h < NH; ++h)
-          if (h < hn) {
-            float *ml = out.ml + (((int64_t)split * out.rows + r) * a.H + h0 + h) * 2;
+        for (int h = 0; h < HT; ++h)
+          if (hb + h < a.H) {
+            float *ml = out.ml + (((int64_t)split * out.rows + r) * a.H + hb + h) * 2;
             ml[0] = m[h];
             ml[1] = l[h];
           }
@@ -677,7 +703,7 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 5) {
+  if (warp == 9) {
     tc_fence_after();
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(tmem_cols) : "memory");
   }
@@ -686,7 +712,7 @@ __global__ void __launch_bounds__(LA_THREADS, 1) latent_attn_tc_kernel(const __g
 // ---- host ---------------------------------------------------------------------------------------
 
 static bool latent_tc(const caten_b200_ctx *ctx, const LatentArgs &a) {
-  return a.cache_bf16 && ctx->attn_tc && ctx->encode_tiled && a.KC() <= 64 * LA_MAX_BLOCKS;
+  return a.tiled && ctx->attn_tc && a.KC() <= 64 * LA_MAX_BLOCKS;
 }
 static int latent_heads(const LatentArgs &a) { return a.H <= 16 ? 16 : 32; }   // per CTA
 static int64_t latent_ctas(const LatentArgs &a, bool tc, int64_t rows) {
@@ -708,30 +734,21 @@ int latent_splits(const caten_b200_ctx *ctx, const LatentArgs &a, int64_t rows, 
   return best;
 }
 
-typedef CUresult (*EncodeTiledFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *, const cuuint32_t *, const cuuint32_t *,
-                                  CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
 template <int NH>
 static int launch_tc(caten_b200_ctx *ctx, const LatentArgs &a, const LatentAbsorbed &x, const LatentOut &out, dim3 grid) {
-  const int KC = a.KC(), nkc = (KC + 63) / 64, np = (nkc + 1) / 2, npv = (a.Kr / 64 + 1) / 2;
-  const cuuint64_t dims[2] = {(cuuint64_t)KC, (cuuint64_t)(a.B * a.cap)}, strides[1] = {(cuuint64_t)KC * 2};
-  const cuuint32_t box[2] = {64, LA_KEYS}, estr[2] = {1, 1};
-  CUtensorMap map;
-  const CUresult e = ((EncodeTiledFn)ctx->encode_tiled)(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.cache, dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                                                        CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  if (e != CUDA_SUCCESS) return fail(ctx, CATEN_B200_ECUDA, "cuTensorMapEncodeTiled failed (%d)", (int)e);
-  const size_t stage = (size_t)nkc * LA_BLOCK, rest = (size_t)nkc * NH * 128 + 2 * 4 * NH * 128 + (LA_BARS + 1) * 8 + 4 * NH * sizeof(float);
+  const int nkc = a.blocks(), np = (nkc + 1) / 2, npv = (a.Kr / 64 + 1) / 2;
+  const size_t stage = (size_t)a.tile_elems() * 2, rest = (size_t)nkc * NH * 128 + 2 * 4 * NH * 128 + (LA_BARS + 1) * 8 + 4 * NH * sizeof(float);
   int stages = (int)((224 * 1024 - rest) / stage);
   if (stages > LA_MAX_STAGES) stages = LA_MAX_STAGES;
   while (stages * np > LA_MAX_PAIRS) --stages;
-  // (one stage: the last pair may be a single block beside which the second product's operand reaches into Q, harmlessly)
+  // (beside a pair of a single block the second product's operand reaches into what follows, at least 16 KB: rows of O nobody reads)
   const size_t smem = 1024 + stage * stages + rest;
   uint32_t cols = 32;
   while (cols < (uint32_t)(npv * 2 * NH + 2 * NH)) cols *= 2;
   const uint32_t base = (1u << 4) | (1u << 7) | (1u << 10) | (8u << 24);   // fp32 accumulate, bf16 x bf16, M = 128
   const uint32_t idesc_s = base | ((uint32_t)(NH >> 3) << 17), idesc_pv = base | ((uint32_t)(2 * NH >> 3) << 17) | (1u << 15);   // second product: A MN-major
   CB_CUDA(ctx, cudaFuncSetAttribute(latent_attn_tc_kernel<NH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  launch_k(ctx, latent_attn_tc_kernel<NH>, grid, dim3(LA_THREADS), smem, map, a, x.qcat_bf.hi ? nullptr : x.qcat, x.qcat_bf.hi, out, stages, x.early ? 1 : 0, cols, idesc_s,
+  launch_k(ctx, latent_attn_tc_kernel<NH>, grid, dim3(LA_THREADS), smem, a, x.qcat_bf.hi ? nullptr : x.qcat, x.qcat_bf.hi, out, stages, x.early ? 1 : 0, cols, idesc_s,
            idesc_pv, ctx->d_status);
   CB_LAUNCH_CHECK(ctx, "latent_attn_tc_kernel");
   return 0;

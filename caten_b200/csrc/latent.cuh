@@ -12,15 +12,30 @@ struct LatentArgs {
   const float *freq = nullptr;      // [P / 2]: rotated dims i and i + P / 2 turn by position * freq[i]
   const float *q_norm = nullptr, *kv_norm = nullptr;   // [Qr], [Kp] gains of the latents (zero in the padding)
   float eps = 0.0f, scale = 1.0f;   // score = (q . k) * scale
-  // cache [B, cap, Kp + Pp]: latent, rotated key part; bf16 or fp32
+  // cache of `cap` rows per sequence: latent (Kp), rotated key part (Pp).  fp32, or bf16, row after row; or (tiled, bf16, at most 576
+  // columns, cap a multiple of 128) tiles of 128 rows laid out as the shared-memory operand tiles of the decode kernel: blocks
+  // of 64 columns, rows of 128 bytes with the 128-byte swizzle; a last block that holds up to 32 columns of the key part alone has
+  // rows of 64 bytes with the 64-byte swizzle
   void *cache = nullptr;
-  bool cache_bf16 = false;
+  bool cache_bf16 = false, tiled = false;
   int64_t cap = 0;
   int B = 0, s = 0, n = 0;          // s tokens per sequence at positions n ..
   const int *d_n = nullptr;         // single-token steps: position on the device
 
-  int KC() const { return Kp + Pp; }
+  __host__ __device__ int KC() const { return Kp + Pp; }
   int Dq() const { return Dp + Pp; }
+  __host__ __device__ int blocks() const { return (KC() + 63) / 64; }
+  __host__ __device__ bool narrow() const { return KC() % 64 != 0 && KC() % 64 <= 32 && (KC() / 64) * 64 >= Kp; }
+  __host__ __device__ int tile_elems() const { return blocks() * 128 * 64 - (narrow() ? 128 * 32 : 0); }
+  __host__ __device__ int64_t seq_elems() const { return tiled ? cap / 128 * tile_elems() : cap * KC(); }
+  // where column c of a sequence's row is; 8 columns from a multiple of 8 on are contiguous
+  __host__ __device__ int64_t at(int64_t seq, int64_t row, int c) const {
+    if (!tiled) return (seq * cap + row) * KC() + c;
+    const int r = (int)(row & 127), b = c >> 6, chunk = (c & 63) >> 3;
+    const int64_t tile = seq * seq_elems() + (row >> 7) * tile_elems() + b * 8192 + (c & 7);
+    if (narrow() && b == blocks() - 1) return tile + r * 32 + ((chunk ^ ((r >> 1) & 3)) << 3);
+    return tile + r * 64 + ((chunk ^ (r & 7)) << 3);
+  }
 };
 
 // Rows of the projection [query latent (Qr) | latent (Kp) | key part (Pp)] (y, or its split-K partial tiles): the normed query

@@ -125,6 +125,7 @@ def test_cache_sizes(rt):
     """Latent layers hold kv_rank + rot_dim numbers a token, retention layers a state, whatever the heads are."""
     m = make(rt, "latent", "bf16", max_seq_len=100)
     assert m.cache_nbytes == 128 * (48 + 16) * 2
+    assert make(rt, "dense", "bf16", max_seq_len=129, batch=3).cache_nbytes == 3 * (256 * (64 + 32) * 2 + 2 * 32 * 64 * 4)   # rot_dim 16 stored as 32
     m.close()
     m = make(rt, "latent", "fp32", max_seq_len=100)
     assert m.cache_nbytes == 128 * (48 + 16) * 4
