@@ -135,6 +135,7 @@ int caten_b200_destroy(caten_b200_ctx *ctx) {
   for (auto e : ctx->prof_pool) cudaEventDestroy(e);
   if (ctx->xbf.ptr) cudaFree(ctx->xbf.ptr);
   if (ctx->wtmp.ptr) cudaFree(ctx->wtmp.ptr);
+  if (ctx->wtmp_side.ptr) cudaFree(ctx->wtmp_side.ptr);
   if (ctx->wbf.ptr) cudaFree(ctx->wbf.ptr);
   if (ctx->wkv_tmp.ptr) cudaFree(ctx->wkv_tmp.ptr);
   if (ctx->chunk_states.ptr) cudaFree(ctx->chunk_states.ptr);

@@ -115,6 +115,7 @@ struct caten_b200_ctx {
   int *h_status = nullptr;   // pinned mirror
   cb::Scratch xbf;           // bf16 copy (hi, lo) of the activation operand of the tensor-core GEMM
   cb::Scratch wtmp;          // split-K partial tiles of the tensor-core GEMM
+  cb::Scratch wtmp_side;     // the same for launches on a decoder's side stream
   cb::Scratch wbf;           // bf16 copy (hi, lo) of the weight operand of the many-row GEMM
   cb::Scratch chunk_states;    // per-chunk states of a recurrent layer's prompt
   cb::Scratch wkv_tmp;       // intermediates of a stand-alone time-mixing call

@@ -7,6 +7,7 @@
 #include <string.h>
 
 #include <new>
+#include <utility>
 #include <vector>
 
 #include "attn_window.cuh"
@@ -64,12 +65,16 @@ struct caten_b200_decoder {
   BfOut cq_bf, qn_bf, qcat_bf, olat_bf, lat_bf;
   float *ret_o = nullptr;                                   // retention: raw outputs of heads with values wider than 256
   // mixture of experts
+  float *ex_z = nullptr;                                    // router logits
   int *ex_id = nullptr, *ex_off = nullptr, *ex_src = nullptr, *ex_pos = nullptr;
   float *ex_w = nullptr, *ex_ws = nullptr, *ea = nullptr, *ye = nullptr;   // ea: experts' activations; ye: their outputs [pairs, wp]
   BfOut xs_bf, ea_bf;                                       // rows sorted by expert
   float *last = nullptr, *logits = nullptr;
   int *d_rows = nullptr;
   int64_t *ids = nullptr, *h_ids = nullptr, *h_out = nullptr;
+  // parallel layers with few rows: the feed-forward runs beside the mixer on a stream of its own
+  cudaStream_t side = nullptr;
+  cudaEvent_t fork = nullptr, join = nullptr;
   StepLoop loop;
   int64_t pos = 0;        // where the next step continues
   float *capture = nullptr;
@@ -244,7 +249,7 @@ int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc
       uv.qs = (uint16_t *)uv.qs + H * Dp * uv.cols;
     }
     if (c.mixer == CATEN_B200_MIX_RETENTION && p16(c.vdim) > 256) most(&ret_o, c.heads * p16(c.vdim));
-    if (c.experts) { most(&ny, c.router->rows); most(&experts, c.experts); most(&top, c.top); most(&ex_ff, c.ff_out->cols); }
+    if (c.experts) { most(&experts, c.experts); most(&top, c.top); most(&ex_ff, c.ff_out->cols); }
   }
   m->planes = m->any_wkv ? 5 : loops || any_par ? 2 : 1;
   const bool exact = dsc->precision == CATEN_B200_PREC_FP32;
@@ -314,7 +319,8 @@ int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc
   if (!rc && ret_o) rc = dec_floats(m, &m->ret_o, R * ret_o);
   if (!rc && experts) {
     const int64_t P = R * top;
-    rc = dec_alloc(m, (void **)&m->ex_id, (size_t)P * sizeof(int));
+    rc = dec_floats(m, &m->ex_z, R * p64(experts));
+    if (!rc) rc = dec_alloc(m, (void **)&m->ex_id, (size_t)P * sizeof(int));
     if (!rc) rc = dec_alloc(m, (void **)&m->ex_off, (size_t)(experts + 1) * sizeof(int));
     if (!rc) rc = dec_alloc(m, (void **)&m->ex_src, (size_t)P * sizeof(int));
     if (!rc) rc = dec_alloc(m, (void **)&m->ex_pos, (size_t)P * sizeof(int));
@@ -333,6 +339,13 @@ int caten_b200_decoder_create(caten_b200_ctx *ctx, const caten_b200_decoder_desc
   if (!rc) rc = step_loop_alloc(ctx, &m->loop, B, T);
   if (!rc && cudaMallocHost(&m->h_ids, (size_t)B * T * sizeof(int64_t)) != cudaSuccess) rc = fail(ctx, CATEN_B200_ECUDA, "cudaMallocHost(ids)");
   if (!rc && cudaMallocHost(&m->h_out, (size_t)B * sizeof(int64_t)) != cudaSuccess) rc = fail(ctx, CATEN_B200_ECUDA, "cudaMallocHost(out ids)");
+  if (!rc && any_par) {
+    const char *e = getenv("CATEN_B200_SIDE_STREAM");   // 0: one kernel after the other
+    if (!e || atoi(e) != 0)
+      if (cudaStreamCreateWithFlags(&m->side, cudaStreamNonBlocking) != cudaSuccess || cudaEventCreateWithFlags(&m->fork, cudaEventDisableTiming) != cudaSuccess ||
+          cudaEventCreateWithFlags(&m->join, cudaEventDisableTiming) != cudaSuccess)
+        rc = fail(ctx, CATEN_B200_ECUDA, "decoder_create: side stream");
+  }
   if (rc) { caten_b200_decoder_destroy(m); return rc; }
   m->launches0 = ctx->launches;
   *out = m;
@@ -344,6 +357,9 @@ int caten_b200_decoder_destroy(caten_b200_decoder *m) {
   cudaSetDevice(m->ctx->device);
   cudaStreamSynchronize(m->ctx->stream);
   step_loop_free(&m->loop);
+  if (m->side) { cudaStreamSynchronize(m->side); cudaStreamDestroy(m->side); }
+  if (m->fork) cudaEventDestroy(m->fork);
+  if (m->join) cudaEventDestroy(m->join);
   for (void *p : m->owned) cudaFree(p);
   if (m->h_ids) cudaFreeHost(m->h_ids);
   if (m->h_out) cudaFreeHost(m->h_out);
@@ -470,8 +486,10 @@ class StepRunner {
 
   int layer(const Run &r, size_t finished_runs) {
     const caten_b200_layer_desc &c = m_->layers[r.layer];
+    if (c.parallel) return parallel_layer(r, c, finished_runs);
+    if (c.mixer != CATEN_B200_MIX_WKV)
+      if (int rc = boundary(SN_NORM, c.norm1, finished_runs)) return rc;
     if (int rc = mixer(r, c, finished_runs)) return rc;
-    if (c.parallel) return finish_parallel(c);
     if (int rc = linear(c.out_w, m_->act, m_->act_bf, nullptr, m_->y2, none_, defer_ ? &pend_.pin : nullptr)) return rc;
     pend_.in = SN_ADD;
     pend_.post = c.norm1b;
@@ -486,44 +504,71 @@ class StepRunner {
 
   int mixer(const Run &r, const caten_b200_layer_desc &c, size_t finished_runs) {
     switch (c.mixer) {
-      case CATEN_B200_MIX_ATTENTION: return attention(r, c, finished_runs);
-      case CATEN_B200_MIX_LATENT: return latent(r, c, finished_runs);
-      case CATEN_B200_MIX_RETENTION: return retention(r, c, finished_runs);
-      default: return wkv(r, c, finished_runs);
+      case CATEN_B200_MIX_ATTENTION: return attention(r, c);
+      case CATEN_B200_MIX_LATENT: return latent(r, c);
+      case CATEN_B200_MIX_RETENTION: return retention(r, c);
+      default: return wkv(r, c, finished_runs);   // (its norm is part of the token shift)
     }
   }
 
-  // The norm before a mixer; a parallel layer's feed-forward gets its own beside it (plane 1).
-  int enter(const Run &r, const caten_b200_layer_desc &c, size_t finished_runs) {
-    if (!c.parallel) return boundary(SN_NORM, c.norm1, finished_runs);
-    return boundary(SN_NORM2, 0.0f, finished_runs, nullptr, nullptr, nullptr, &c, r.pass_start && !m_->desc.loop_in ? &r : nullptr);
-  }
-
-  // The feed-forward beside the mixer, and one linear over both outputs.
-  int finish_parallel(const caten_b200_layer_desc &c) {
-    const float *h2 = m_->hp + plane_ * m_->wp;
-    const BfOut h2_bf = offset(m_->hp_bf, plane_ * m_->wp);
+  // Mixer and feed-forward of the same stream, and one linear over both outputs.  With few rows both are chains of short kernels,
+  // and run side by side on two streams.
+  int parallel_layer(const Run &r, const caten_b200_layer_desc &c, size_t finished_runs) {
+    if (int rc = boundary(SN_NORM2, 0.0f, finished_runs, nullptr, nullptr, nullptr, &c, r.pass_start && !m_->desc.loop_in ? &r : nullptr)) return rc;
     Pending next;
     next.in = SN_SUM;
-    if (c.experts) {
-      if (int rc = experts(c, h2, h2_bf, &next)) return rc;
+    const bool beside = m_->side && c.ff_in && R_ <= 256 && ctx_->prof_mask == 0;
+    if (beside) {
+      CB_CUDA(ctx_, cudaEventRecord(m_->fork, ctx_->stream));
+      CB_CUDA(ctx_, cudaStreamWaitEvent(m_->side, m_->fork, 0));
+      if (int rc = on_side([&] { return feed_forward(c, &next); })) return rc;
+      CB_CUDA(ctx_, cudaEventRecord(m_->join, m_->side));
+    }
+    if (int rc = mixer(r, c, finished_runs)) return rc;
+    if (beside) {
+      CB_CUDA(ctx_, cudaStreamWaitEvent(ctx_->stream, m_->join, 0));
+      full_edge();
     } else if (c.ff_in) {
-      LinGroups to;
-      to.ldy = c.out_w->cols;
-      const int64_t col = mixer_cols(c);
-      if (int rc = linear(c.ff_in, h2, h2_bf, nullptr, m_->act + col, offset(bf(m_->act_bf), col), nullptr, c.ff_act, to)) return rc;
+      if (int rc = feed_forward(c, &next)) return rc;
     }
     if (int rc = linear(c.out_w, m_->act, m_->act_bf, nullptr, m_->y2, none_, defer_ ? &next.pin : nullptr)) return rc;
     pend_ = next;
     return 0;
   }
 
+  // The next launch waits for everything before it to complete (a programmatic dependent launch has one predecessor only).
+  void full_edge() { ctx_->weights_pending = true; }
+
+  // Launches of f go to the side stream, with scratch of their own.
+  template <class F>
+  int on_side(F f) {
+    cudaStream_t main = ctx_->stream;
+    std::swap(ctx_->wtmp, ctx_->wtmp_side);
+    ctx_->stream = m_->side;
+    full_edge();
+    const int rc = f();
+    ctx_->stream = main;
+    std::swap(ctx_->wtmp, ctx_->wtmp_side);
+    return rc;
+  }
+
+  // Feed-forward of the second norm's rows: dense, its activations beside the mixer's output; experts, their outputs into ye.
+  int feed_forward(const caten_b200_layer_desc &c, Pending *next) {
+    const float *h2 = m_->hp + plane_ * m_->wp;
+    const BfOut h2_bf = offset(m_->hp_bf, plane_ * m_->wp);
+    if (c.experts) return experts(c, h2, h2_bf, next);
+    LinGroups to;
+    to.ldy = c.out_w->cols;
+    const int64_t col = mixer_cols(c);
+    return linear(c.ff_in, h2, h2_bf, nullptr, m_->act + col, offset(bf(m_->act_bf), col), nullptr, c.ff_act, to);
+  }
+
   int experts(const caten_b200_layer_desc &c, const float *h2, BfOut h2_bf, Pending *next) {
     RouteArgs a;
-    if (int rc = linear(c.router, h2, h2_bf, nullptr, m_->y, none_, defer_ ? &a.pin : nullptr)) return rc;
+    if (int rc = linear(c.router, h2, h2_bf, nullptr, m_->ex_z, none_, defer_ ? &a.pin : nullptr)) return rc;
     const bool sorted = R_ > 4;
     const int64_t rows_in = c.ff_in->rows / c.experts, pairs = R_ * c.top;
-    a.z = m_->y; a.ld = c.router->rows; a.rows = (int)R_; a.experts = c.experts; a.top = c.top;
+    a.z = m_->ex_z; a.ld = c.router->rows; a.rows = (int)R_; a.experts = c.experts; a.top = c.top;
     a.expert = m_->ex_id; a.weight = m_->ex_w; a.offsets = m_->ex_off; a.src = m_->ex_src; a.sorted_weight = m_->ex_ws; a.pos = m_->ex_pos;
     {
       ProfScope prof(ctx_, CATEN_B200_K_PREP);
@@ -552,8 +597,7 @@ class StepRunner {
     return launch_gemm_experts(ctx_, c.ff_out, er, m_->ea_bf, CATEN_B200_ACT_NONE, m_->ye, none_, nsplit);
   }
 
-  int latent(const Run &r, const caten_b200_layer_desc &c, size_t finished_runs) {
-    if (int rc = enter(r, c, finished_runs)) return rc;
+  int latent(const Run &r, const caten_b200_layer_desc &c) {
     LatentArgs a = latent_args(m_, c);
     PartIn pin;
     if (int rc = linear(c.in_w, m_->hp, m_->hp_bf, nullptr, m_->y, none_, defer_ ? &pin : nullptr)) return rc;
@@ -608,8 +652,7 @@ class StepRunner {
     return 0;
   }
 
-  int retention(const Run &r, const caten_b200_layer_desc &c, size_t finished_runs) {
-    if (int rc = enter(r, c, finished_runs)) return rc;
+  int retention(const Run &r, const caten_b200_layer_desc &c) {
     RetentionArgs a;
     if (int rc = linear(c.in_w, m_->hp, m_->hp_bf, nullptr, m_->y, none_, defer_ && p_.s == 1 ? &a.pin : nullptr)) return rc;
     a.H = c.heads; a.D = c.dim; a.Dp = (int)p16(c.dim); a.E = c.vdim; a.Ep = (int)p16(c.vdim);
@@ -629,8 +672,7 @@ class StepRunner {
     return launch_retention_chunks(ctx_, a);
   }
 
-  int attention(const Run &r, const caten_b200_layer_desc &c, size_t finished_runs) {
-    if (int rc = enter(r, c, finished_runs)) return rc;
+  int attention(const Run &r, const caten_b200_layer_desc &c) {
     AttnArgs a;
     if (int rc = linear(c.in_w, m_->hp, m_->hp_bf, nullptr, m_->y, none_, defer_ && p_.s == 1 ? &a.pin : nullptr)) return rc;
     a.H = c.heads; a.G = c.kv_heads;

@@ -11,7 +11,7 @@ struct StepLoop {
   int64_t *hist = nullptr;      // [T, B] row n = ids produced by the step that started at position n
   int *d_pos = nullptr;         // position of the next step
   cudaGraphExec_t graph = nullptr;
-  void *graph_xbf = nullptr, *graph_wtmp = nullptr;  // scratch pointers baked into the graph
+  void *graph_xbf = nullptr, *graph_wtmp = nullptr, *graph_side = nullptr;  // scratch pointers baked into the graph
   int64_t launches_per_step = 0;
 };
 
@@ -36,7 +36,7 @@ inline void step_loop_free(StepLoop *l) {
 template <class Step>
 int step_loop_run(caten_b200_ctx *ctx, StepLoop *l, int64_t n, int64_t steps, int64_t T, bool use_graph, Step step) {
   int64_t done = 0;
-  if (use_graph && l->graph && (l->graph_xbf != ctx->xbf.ptr || l->graph_wtmp != ctx->wtmp.ptr)) {
+  if (use_graph && l->graph && (l->graph_xbf != ctx->xbf.ptr || l->graph_wtmp != ctx->wtmp.ptr || l->graph_side != ctx->wtmp_side.ptr)) {
     cudaGraphExecDestroy(l->graph);  // scratch was re-allocated since the capture: its pointers are stale
     l->graph = nullptr;
   }
@@ -59,6 +59,7 @@ int step_loop_run(caten_b200_ctx *ctx, StepLoop *l, int64_t n, int64_t steps, in
     if (e2 != cudaSuccess) { l->graph = nullptr; return cuda_fail(ctx, e2, "cudaGraphInstantiate"); }
     l->graph_xbf = ctx->xbf.ptr;
     l->graph_wtmp = ctx->wtmp.ptr;
+    l->graph_side = ctx->wtmp_side.ptr;
   }
   for (; done < steps; ++done) {
     if (use_graph && l->graph) {
