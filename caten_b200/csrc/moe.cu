@@ -8,7 +8,7 @@ namespace cb {
 
 namespace {
 
-constexpr int MR_THREADS = 1024, MR_WARPS = MR_THREADS / 32, MR_MAX_EXPERTS = 1024, MR_FUSED_ROWS = 256;
+constexpr int MR_THREADS = 1024, MR_WARPS = MR_THREADS / 32, MR_MAX_EXPERTS = 1024, MR_FUSED_ROWS = 256, MR_U = 4;
 
 // One warp, one row: lane holds experts lane, lane + 32, ...
 template <int VPL>
@@ -71,11 +71,16 @@ __global__ void __launch_bounds__(MR_THREADS) moe_sort_kernel(const RouteArgs a,
   const int share = (pairs + MR_WARPS * 32 - 1) / (MR_WARPS * 32) * 32;
   const int p0 = min(warp * share, pairs), p1 = min(p0 + share, pairs);
   int *mine = counts + warp * E;
-  for (int p = p0; p < p1; p += 32) {
-    const int e = p + lane < p1 ? a.expert[p + lane] : -1 - lane;
-    const unsigned same = __match_any_sync(0xffffffffu, e);
-    if (e >= 0 && lane == __ffs(same) - 1) mine[e] += __popc(same);
-    __syncwarp();
+  for (int q = p0; q < p1; q += 32 * MR_U) {
+    int e[MR_U];   // requested together
+#pragma unroll
+    for (int u = 0; u < MR_U; ++u) e[u] = q + 32 * u + lane < p1 ? a.expert[q + 32 * u + lane] : -1 - lane;
+#pragma unroll
+    for (int u = 0; u < MR_U; ++u) {
+      const unsigned same = __match_any_sync(0xffffffffu, e[u]);
+      if (e[u] >= 0 && lane == __ffs(same) - 1) mine[e[u]] += __popc(same);
+      __syncwarp();
+    }
   }
   __syncthreads();
   int total = 0;
@@ -101,19 +106,30 @@ __global__ void __launch_bounds__(MR_THREADS) moe_sort_kernel(const RouteArgs a,
     for (int w = 0; w < MR_WARPS; ++w) counts[w * E + tid] += before;
   }
   __syncthreads();
-  for (int p = p0; p < p1; p += 32) {
-    const int e = p + lane < p1 ? a.expert[p + lane] : -1 - lane;
-    const unsigned same = __match_any_sync(0xffffffffu, e);
-    int at = 0;
-    if (e >= 0) at = mine[e] + __popc(same & ((1u << lane) - 1u));
-    __syncwarp();
-    if (e >= 0) {
-      a.pos[p + lane] = at;
-      a.src[at] = (p + lane) / a.top;
-      a.sorted_weight[at] = a.weight[p + lane];
-      if (lane == __ffs(same) - 1) mine[e] += __popc(same);
+  for (int q = p0; q < p1; q += 32 * MR_U) {
+    int e[MR_U];
+    float w[MR_U];
+#pragma unroll
+    for (int u = 0; u < MR_U; ++u) {
+      const int p = q + 32 * u + lane;
+      e[u] = p < p1 ? a.expert[p] : -1 - lane;
+      w[u] = p < p1 ? a.weight[p] : 0.0f;
     }
-    __syncwarp();
+#pragma unroll
+    for (int u = 0; u < MR_U; ++u) {
+      const int p = q + 32 * u + lane;
+      const unsigned same = __match_any_sync(0xffffffffu, e[u]);
+      int at = 0;
+      if (e[u] >= 0) at = mine[e[u]] + __popc(same & ((1u << lane) - 1u));
+      __syncwarp();
+      if (e[u] >= 0) {
+        a.pos[p] = at;
+        a.src[at] = p / a.top;
+        a.sorted_weight[at] = w[u];
+        if (lane == __ffs(same) - 1) mine[e[u]] += __popc(same);
+      }
+      __syncwarp();
+    }
   }
 }
 

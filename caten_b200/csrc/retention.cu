@@ -54,14 +54,22 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prep_kernel(const Retent
   for (int i = tid; i < a.H * rest; i += RT_THREADS) row[a.k_off + (int64_t)(i / rest) * a.Dp + 2 * np + i % rest] *= a.kscale;
 }
 
-// rows [r0, r0 + 64) x columns [c0, c0 + 4 * W4) of a matrix into shared memory, zeros outside [0, rows) x [0, cols)
+// Rows [r0, r0 + 64) x columns [c0, c0 + 4 * W4) of a matrix into shared memory, zeros outside [0, rows) x [0, cols); asynchronous.
 template <int W4>
 __device__ __forceinline__ void load_tile(float *dst, int ld, const float *src, int64_t src_ld, int r0, int rows, int c0, int cols, int tid) {
 #pragma unroll 4
   for (int e = tid; e < 64 * W4; e += RT_THREADS) {
     const int r = e / W4, c = (e % W4) * 4;
-    *reinterpret_cast<float4 *>(dst + r * ld + c) = r0 + r < rows && c0 + c < cols ? *reinterpret_cast<const float4 *>(src + (int64_t)(r0 + r) * src_ld + c0 + c) : zero4();
+    const bool in = r0 + r < rows && c0 + c < cols;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst + r * ld + c)),
+                 "l"(src + (in ? (int64_t)(r0 + r) * src_ld + c0 + c : 0)), "r"(in ? 16 : 0) : "memory");
   }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+}
+// all tiles but the `N` last ones have arrived
+template <int N> __device__ __forceinline__ void tiles_ready() {
+  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
+  __syncthreads();
 }
 
 // U of one chunk: a tile of 64 keys x 64 NEB values per CTA; grid (chunk, head x key tiles x value tiles, sequence)
@@ -79,7 +87,7 @@ __global__ void __launch_bounds__(RT_THREADS) retention_state_kernel(const Reten
   pdl_enter();
   load_tile<16>(ks, RT_LD, a.y + row0 * a.ld + a.k_off + (int64_t)h * a.Dp, a.ld, 0, tn, d0, a.Dp, tid);
   load_tile<16 * NEB>(vs, VLD, a.y + row0 * a.ld + a.v_off + (int64_t)h * a.Ep, a.ld, 0, tn, e0, a.Ep, tid);
-  __syncthreads();
+  tiles_ready<0>();
   float4 acc[4][NEB];
 #pragma unroll
   for (int j = 0; j < 4; ++j)
@@ -137,7 +145,7 @@ __global__ void __launch_bounds__(256) retention_scan_kernel(const RetentionArgs
 // grid (chunk, head x value tiles, sequence): 64 tokens x 64 NEB value columns.  Thread (ty, tx) owns tokens ty + 16 j and
 // columns 4 tx + 64 nb; of the token pairs (ty + 16 j, tx + 16 i).
 template <int NEB>
-__global__ void __launch_bounds__(RT_THREADS, NEB == 4 ? 1 : 2) retention_out_kernel(const RetentionArgs a, const float *__restrict__ U) {
+__global__ void __launch_bounds__(RT_THREADS, 2) retention_out_kernel(const RetentionArgs a, const float *__restrict__ U) {
   extern __shared__ __align__(16) float sm[];
   constexpr int VLD = 64 * NEB + 4;
   __shared__ float pw[RET_T + 1];
@@ -151,32 +159,60 @@ __global__ void __launch_bounds__(RT_THREADS, NEB == 4 ? 1 : 2) retention_out_ke
   if (tid <= RET_T) pw[tid] = a.powers[(int64_t)h * (RET_T + 1) + tid];
   const float *qg = a.y + row0 * a.ld + a.q_off + (int64_t)h * a.Dp, *kg = a.y + row0 * a.ld + a.k_off + (int64_t)h * a.Dp;
   const float *S = U + (((int64_t)b * a.H + h) * gridDim.x + c) * a.Dp * a.Ep;
-  float A[4][4];
+  float *as = ks;   // [token][earlier token], once the products are formed
+  {
+    float A[4][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) A[j][i] = 0.0f;
+    for (int d0 = 0; d0 < a.Dp; d0 += 64) {
+      __syncthreads();
+      load_tile<16>(qs, RT_LD, qg, a.ld, 0, tn, d0, a.Dp, tid);
+      load_tile<16>(ks, RT_LD, kg, a.ld, 0, tn, d0, a.Dp, tid);
+      if (d0 == 0) {   // the first block of the state arrives during the products
+        load_tile<16 * NEB>(vs, VLD, S, a.Ep, 0, a.Dp, e0, a.Ep, tid);
+        tiles_ready<1>();
+      } else {
+        tiles_ready<0>();
+      }
+      const int dn = min(64, a.Dp - d0);
+      for (int d = 0; d < dn; d += 4) {
+        float4 q[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) q[j] = *reinterpret_cast<const float4 *>(qs + (ty + 16 * j) * RT_LD + d);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float4 k = *reinterpret_cast<const float4 *>(ks + (tx + 16 * i) * RT_LD + d);
+#pragma unroll
+          for (int j = i; j < 4; ++j) A[j][i] = dot4(q[j], k, A[j][i]);   // (pairs with i > j are never used)
+        }
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int t = ty + 16 * j, s = tx + 16 * i;
+        as[t * RT_LD + s] = s <= t ? A[j][i] * pw[t - s] : 0.0f;
+      }
+  }
   float4 o[4][NEB];
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
-#pragma unroll
-    for (int i = 0; i < 4; ++i) A[j][i] = 0.0f;
+  for (int j = 0; j < 4; ++j)
 #pragma unroll
     for (int nb = 0; nb < NEB; ++nb) o[j][nb] = zero4();
-  }
   for (int d0 = 0; d0 < a.Dp; d0 += 64) {
     __syncthreads();
-    load_tile<16>(qs, RT_LD, qg, a.ld, 0, tn, d0, a.Dp, tid);
-    load_tile<16>(ks, RT_LD, kg, a.ld, 0, tn, d0, a.Dp, tid);
-    load_tile<16 * NEB>(vs, VLD, S, a.Ep, d0, a.Dp, e0, a.Ep, tid);
-    __syncthreads();
+    if (a.Dp > 64) load_tile<16>(qs, RT_LD, qg, a.ld, 0, tn, d0, a.Dp, tid);   // (a single block is still there)
+    if (d0 > 0) load_tile<16 * NEB>(vs, VLD, S, a.Ep, d0, a.Dp, e0, a.Ep, tid);
+    tiles_ready<0>();
     const int dn = min(64, a.Dp - d0);
     for (int d = 0; d < dn; d += 4) {
       float4 q[4];
 #pragma unroll
       for (int j = 0; j < 4; ++j) q[j] = *reinterpret_cast<const float4 *>(qs + (ty + 16 * j) * RT_LD + d);
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const float4 k = *reinterpret_cast<const float4 *>(ks + (tx + 16 * i) * RT_LD + d);
-#pragma unroll
-        for (int j = i; j < 4; ++j) A[j][i] = dot4(q[j], k, A[j][i]);   // (pairs with i > j are never used)
-      }
 #pragma unroll
       for (int nb = 0; nb < NEB; ++nb) {
         float4 v[4];
@@ -188,21 +224,14 @@ __global__ void __launch_bounds__(RT_THREADS, NEB == 4 ? 1 : 2) retention_out_ke
     }
   }
   __syncthreads();
-  float *as = ks;   // [token][earlier token]
+  load_tile<16 * NEB>(vs, VLD, a.y + row0 * a.ld + a.v_off + (int64_t)h * a.Ep, a.ld, 0, tn, e0, a.Ep, tid);
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
-    const int t = ty + 16 * j;
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int s = tx + 16 * i;
-      as[t * RT_LD + s] = s <= t ? A[j][i] * pw[t - s] : 0.0f;
-    }
-    const float f = pw[t + 1];
+    const float f = pw[ty + 16 * j + 1];
 #pragma unroll
     for (int nb = 0; nb < NEB; ++nb) o[j][nb] = make_float4(o[j][nb].x * f, o[j][nb].y * f, o[j][nb].z * f, o[j][nb].w * f);
   }
-  load_tile<16 * NEB>(vs, VLD, a.y + row0 * a.ld + a.v_off + (int64_t)h * a.Ep, a.ld, 0, tn, e0, a.Ep, tid);
-  __syncthreads();
+  tiles_ready<0>();
 #pragma unroll
   for (int sb = 0; sb < 4; ++sb) {
 #pragma unroll 2
