@@ -536,6 +536,8 @@ class StepRunner {
     return 0;
   }
 
+  size_t c_index(const caten_b200_layer_desc &c) const { return (size_t)(&c - m_->layers.data()); }
+
   // The next launch waits for everything before it to complete (a programmatic dependent launch has one predecessor only).
   void full_edge() { ctx_->weights_pending = true; }
 
@@ -609,22 +611,29 @@ class StepRunner {
     if (int rc = linear(c.uq_w, m_->cq, m_->cq_bf, nullptr, m_->q, none_, defer_ && absorbed ? &pin : nullptr)) return rc;
     const int64_t ldq = c.uq_w->rows;
     if (absorbed) {
+      LatentAbsorbed x;
+      x.qcat = m_->qcat; x.qcat_bf = bf(m_->qcat_bf); x.o = m_->olat; x.plane = m_->abs_rows; x.part = m_->part; x.ml = m_->ml;
+      x.splits = latent_splits(ctx_, a, R_, p_.d_n ? a.cap : p_.n + p_.s);
+      while (x.splits > 1 && x.splits * R_ * a.H * a.Kr > m_->part_floats) --x.splits;
+      // (the queries' kernel starts nothing before the kernels in front of it, the cache's append among them, are complete)
+      x.early = true;
+      if (latent_fused(a, R_)) {
+        { ProfScope prof(ctx_, CATEN_B200_K_PREP); if (int rc = launch_latent_up(ctx_, a, c.uk_w, m_->q, pin, ldq, m_->qcat, bf(m_->qcat_bf))) return rc; }
+        x.combine = false;
+        { ProfScope prof(ctx_, CATEN_B200_K_ATTN_DECODE); if (int rc = launch_latent_absorbed(ctx_, a, x)) return rc; }
+        ProfScope prof(ctx_, CATEN_B200_K_PREP);
+        return launch_latent_down(ctx_, a, x, &m_->uv[c_index(c)], m_->act, bf(m_->act_bf), c.out_w->cols);
+      }
       { ProfScope prof(ctx_, CATEN_B200_K_PREP);
         if (int rc = launch_latent_q_absorbed(ctx_, a, m_->q, pin, ldq, m_->abs_rows, m_->qn, bf(m_->qn_bf), m_->qcat, bf(m_->qcat_bf))) return rc; }
       LinGroups up;
       up.group_rows = a.Kp; up.xplane = m_->abs_rows; up.ygroup = a.KC(); up.ldy = (int64_t)a.H * a.KC();
       if (int rc = linear(c.uk_w, m_->qn, m_->qn_bf, nullptr, m_->qcat, bf(m_->qcat_bf), nullptr, CATEN_B200_ACT_NONE, up)) return rc;
-      LatentAbsorbed x;
-      x.qcat = m_->qcat; x.qcat_bf = bf(m_->qcat_bf); x.o = m_->olat; x.o_bf = bf(m_->olat_bf); x.plane = m_->abs_rows; x.part = m_->part; x.ml = m_->ml;
-      x.splits = latent_splits(ctx_, a, R_, p_.d_n ? a.cap : p_.n + p_.s);
-      while (x.splits > 1 && x.splits * R_ * a.H * a.Kr > m_->part_floats) --x.splits;
-      // (the kernel in front is the product with W_uk^T; the one before it starts nothing until the kernels before it, the cache's
-      // append among them, are complete)
-      x.early = true;
+      x.o_bf = bf(m_->olat_bf);
       { ProfScope prof(ctx_, CATEN_B200_K_ATTN_DECODE); if (int rc = launch_latent_absorbed(ctx_, a, x)) return rc; }
       LinGroups down;
       down.group_rows = a.Ep; down.xplane = m_->abs_rows; down.ygroup = a.Ep; down.ldy = c.out_w->cols;
-      return linear(&m_->uv[r.layer], m_->olat, m_->olat_bf, nullptr, m_->act, bf(m_->act_bf), nullptr, CATEN_B200_ACT_NONE, down);
+      return linear(&m_->uv[c_index(c)], m_->olat, m_->olat_bf, nullptr, m_->act, bf(m_->act_bf), nullptr, CATEN_B200_ACT_NONE, down);
     }
     { ProfScope prof(ctx_, CATEN_B200_K_PREP); if (int rc = launch_latent_q_expanded(ctx_, a, m_->q, ldq)) return rc; }
     // keys and values of every cached token, for as many sequences at a time as the buffer takes

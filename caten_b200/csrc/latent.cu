@@ -192,6 +192,98 @@ int launch_latent_q_absorbed(caten_b200_ctx *ctx, const LatentArgs &a, const flo
   return 0;
 }
 
+// grid (head, 16 rows, 64 latent dims): the head's queries, rotated, and their product with W_uk^T.  Four neighbouring threads
+// share a latent dim and take its row of weights in turn, 16 bytes each; the rows' queries are in shared memory.
+constexpr int LU_ROWS = 16, LU_DIMS = 64, LU_AHEAD = 4;
+
+__global__ void __launch_bounds__(256) latent_up_kernel(const LatentArgs a, const __nv_bfloat16 *__restrict__ uk, const float *__restrict__ q, const PartIn pin, int64_t ld,
+                                                        int64_t rows, float *__restrict__ qcat, BfOut qcat_bf) {
+  extern __shared__ __align__(16) float qs[];   // [LU_ROWS][Dp]
+  const int h = blockIdx.x, tid = threadIdx.x, half = a.P / 2, Dq = a.Dp + a.Pp, KC = a.KC(), Dr = (a.Dp + 63) / 64 * 64;
+  const int64_t r0 = (int64_t)blockIdx.y * LU_ROWS;
+  const int rn = (int)(rows - r0 < LU_ROWS ? rows - r0 : LU_ROWS);
+  const int k = blockIdx.z * LU_DIMS + (tid >> 2), part = tid & 3, nv = a.Dp / 8;
+  const bool on = k < a.Kp;
+  const uint4 *w = reinterpret_cast<const uint4 *>(uk + ((int64_t)h * a.Kp + (on ? k : 0)) * Dr);
+  uint4 x[LU_AHEAD];   // the first weights depend on no other kernel
+#pragma unroll
+  for (int u = 0; u < LU_AHEAD; ++u) x[u] = on && part + 4 * u < nv ? w[part + 4 * u] : make_uint4(0u, 0u, 0u, 0u);
+  pdl_enter();
+  const int d4 = a.Dp / 4;
+  for (int i = tid; i < LU_ROWS * d4; i += 256) {
+    const int r = i / d4, c = i % d4 * 4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (r < rn) v = pin.splits > 0 ? partin_load4(pin, r0 + r, h * Dq + c) : *reinterpret_cast<const float4 *>(q + (r0 + r) * ld + (int64_t)h * Dq + c);
+    *reinterpret_cast<float4 *>(qs + r * a.Dp + c) = v;
+  }
+  if (blockIdx.z == 0) {
+    const int n = a.d_n ? *a.d_n : a.n;
+    for (int i = tid; i < rn * a.Pp; i += 256) {
+      const int r = i / a.Pp, j = i % a.Pp;
+      float v = 0.0f;
+      if (j < a.P) {
+        const int f = j < half ? j : j - half;
+        auto at = [&](int d) { const int c = h * Dq + a.Dp + d; return pin.splits > 0 ? partin_load1(pin, r0 + r, c) : q[(r0 + r) * ld + c]; };
+        const float u = at(f), y = at(f + half);
+        float sn, cs;
+        sincosf((float)(n + (int)((r0 + r) % a.s)) * a.freq[f], &sn, &cs);
+        v = j < half ? u * cs - y * sn : y * cs + u * sn;
+      }
+      st1(qcat, qcat_bf, ((r0 + r) * a.H + h) * KC + a.Kp + j, v);
+    }
+  }
+  __syncthreads();
+  float acc[LU_ROWS];
+#pragma unroll
+  for (int r = 0; r < LU_ROWS; ++r) acc[r] = 0.0f;
+  for (int i0 = part; i0 < nv; i0 += 4 * LU_AHEAD) {
+#pragma unroll
+    for (int u = 0; u < LU_AHEAD; ++u) {
+      const int d = 8 * (i0 + 4 * u);
+      if (d >= a.Dp) continue;
+      const uint32_t b[4] = {x[u].x, x[u].y, x[u].z, x[u].w};
+      float f[8];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { f[2 * e] = __uint_as_float(b[e] << 16); f[2 * e + 1] = __uint_as_float(b[e] & 0xFFFF0000u); }
+#pragma unroll
+      for (int r = 0; r < LU_ROWS; ++r) {
+        if (r < rn) {
+          const float4 x0 = *reinterpret_cast<const float4 *>(qs + r * a.Dp + d), x1 = *reinterpret_cast<const float4 *>(qs + r * a.Dp + d + 4);
+          acc[r] = fmaf(f[0], x0.x, fmaf(f[1], x0.y, fmaf(f[2], x0.z, fmaf(f[3], x0.w, acc[r]))));
+          acc[r] = fmaf(f[4], x1.x, fmaf(f[5], x1.y, fmaf(f[6], x1.z, fmaf(f[7], x1.w, acc[r]))));
+        }
+      }
+    }
+    if (i0 + 4 * LU_AHEAD < nv) {
+#pragma unroll
+      for (int u = 0; u < LU_AHEAD; ++u) x[u] = on && i0 + 4 * (LU_AHEAD + u) < nv ? w[i0 + 4 * (LU_AHEAD + u)] : make_uint4(0u, 0u, 0u, 0u);
+    }
+  }
+  // the four threads' sums: each exchange halves the rows a thread carries
+  const bool hi2 = (tid & 2) != 0, hi1 = (tid & 1) != 0;
+#pragma unroll
+  for (int r = 0; r < 8; ++r) acc[r] = (hi2 ? acc[r + 8] : acc[r]) + __shfl_xor_sync(0xffffffffu, hi2 ? acc[r] : acc[r + 8], 2);
+#pragma unroll
+  for (int r = 0; r < 4; ++r) acc[r] = (hi1 ? acc[r + 4] : acc[r]) + __shfl_xor_sync(0xffffffffu, hi1 ? acc[r] : acc[r + 4], 1);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int r = (hi2 ? 8 : 0) + (hi1 ? 4 : 0) + i;
+    if (on && r < rn) st1(qcat, qcat_bf, ((r0 + r) * a.H + h) * KC + k, acc[i]);
+  }
+}
+
+int launch_latent_up(caten_b200_ctx *ctx, const LatentArgs &a, const caten_b200_weight *uk, const float *q, PartIn pin, int64_t ld, float *qcat, BfOut qcat_bf) {
+  if (int rc = check_latent(ctx, a)) return rc;
+  const int64_t rows = (int64_t)a.B * a.s;
+  if (rows <= 0) return 0;
+  if (uk->type != CATEN_B200_BF16) return fail(ctx, CATEN_B200_EUNSUPPORTED, "latent attention: W_uk must be BF16");
+  const size_t smem = (size_t)LU_ROWS * a.Dp * sizeof(float);
+  launch_k(ctx, latent_up_kernel, dim3((unsigned)a.H, (unsigned)((rows + LU_ROWS - 1) / LU_ROWS), (unsigned)((a.Kp + LU_DIMS - 1) / LU_DIMS)), dim3(256), smem, a,
+           (const __nv_bfloat16 *)uk->qs, q, pin, ld, rows, qcat, qcat_bf);
+  CB_LAUNCH_CHECK(ctx, "latent_up_kernel");
+  return 0;
+}
+
 // one warp per cached row
 __global__ void __launch_bounds__(256) latent_gather_kernel(const LatentArgs a, int b0, int t, int64_t rows, float *__restrict__ c, BfOut c_bf, float *__restrict__ kr) {
   pdl_enter();
@@ -347,6 +439,98 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentOut out
     for (int z = 0; z < out.splits; ++z)   // fixed order; a part without keys counts nothing
       if (out.ml[(z * step + at) * 2 + 1] > 0.0f) o = fmaf(exp2f(out.ml[(z * step + at) * 2] - m), out.part[(z * step + at) * out.Kr + c], o);
     st1(out.o, out.o_bf, ((int64_t)h * out.plane + r) * out.Kr + c, o / l);
+  }
+}
+
+// grid (head, 8 rows, part of the outputs): the rows' sums over the latents (merged from the key splits' parts), then W_uv.  `lanes` neighbouring
+// threads share an output and take its row of weights in turn, 16 bytes each.
+constexpr int LD_ROWS = 8, LD_MAX_SPLITS = 32;
+
+__global__ void __launch_bounds__(256) latent_down_kernel(const LatentArgs a, const LatentOut in, const __nv_bfloat16 *__restrict__ uv, int lanes, int per, float *__restrict__ out, BfOut bf,
+                                                          int64_t ld) {
+  extern __shared__ __align__(16) float os[];   // [LD_ROWS][Kr]
+  __shared__ float part_f[LD_ROWS][LD_MAX_SPLITS];
+  const int h = blockIdx.x, tid = threadIdx.x, Kr = in.Kr, S = in.splits;
+  const int64_t r0 = (int64_t)blockIdx.y * LD_ROWS;
+  const int rn = (int)(in.rows - r0 < LD_ROWS ? in.rows - r0 : LD_ROWS);
+  const int e0 = blockIdx.z * per + tid / lanes, e1 = min(a.Ep, (int)(blockIdx.z + 1) * per), es = 256 / lanes, ks = tid % lanes, nv = Kr / 8;
+  // the first weights depend on no other kernel
+  uint4 ahead[4];
+#pragma unroll
+  for (int u = 0; u < 4; ++u)
+    ahead[u] = e0 < e1 && ks + lanes * u < nv ? reinterpret_cast<const uint4 *>(uv + ((int64_t)h * a.Ep + e0) * Kr)[ks + lanes * u] : make_uint4(0u, 0u, 0u, 0u);
+  pdl_enter();
+  const int64_t step = in.rows * in.H;
+  if (S > 1) {   // one warp per row, one lane per part
+    const int r = tid >> 5, z = tid & 31;
+    float2 ml = make_float2(-INFINITY, 0.0f);
+    if (r < rn && z < S) ml = *reinterpret_cast<const float2 *>(in.ml + (z * step + (r0 + r) * in.H + h) * 2);
+    float m = ml.y > 0.0f ? ml.x : -INFINITY;   // (a part without keys counts nothing)
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+    const float f = ml.y > 0.0f ? exp2f(ml.x - m) : 0.0f, l = warp_sum(f * ml.y);
+    part_f[r][z] = f / l;
+    __syncthreads();
+  }
+  const int k4 = Kr / 4;
+  for (int i = tid; i < LD_ROWS * k4; i += 256) {
+    const int r = i / k4, c = i % k4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (r < rn) {
+      if (S == 1) {
+        v = reinterpret_cast<const float4 *>(in.o + ((int64_t)h * in.plane + r0 + r) * Kr)[c];
+      } else {
+        const float4 *p = reinterpret_cast<const float4 *>(in.part + ((r0 + r) * in.H + h) * Kr) + c;
+        for (int z0 = 0; z0 < S; z0 += 4) {   // fixed order, four parts requested together
+          float4 x[4];
+#pragma unroll
+          for (int u = 0; u < 4; ++u)
+            if (z0 + u < S) x[u] = p[(z0 + u) * step * k4];
+#pragma unroll
+          for (int u = 0; u < 4; ++u)
+            if (z0 + u < S) {
+              const float f = part_f[r][z0 + u];
+              v = make_float4(fmaf(f, x[u].x, v.x), fmaf(f, x[u].y, v.y), fmaf(f, x[u].z, v.z), fmaf(f, x[u].w, v.w));
+            }
+        }
+      }
+    }
+    *reinterpret_cast<float4 *>(os + r * Kr + 4 * c) = v;
+  }
+  __syncthreads();
+  for (int e = e0; e - tid / lanes < e1; e += es) {   // (whole warps: the lanes of an output exchange their sums)
+    const bool on = e < e1;
+    const uint4 *w = reinterpret_cast<const uint4 *>(uv + ((int64_t)h * a.Ep + (on ? e : 0)) * Kr);
+    float acc[LD_ROWS];
+#pragma unroll
+    for (int r = 0; r < LD_ROWS; ++r) acc[r] = 0.0f;
+    for (int i = ks; i < nv; i += 4 * lanes) {
+      uint4 x[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) x[u] = e == e0 && i == ks ? ahead[u] : on && i + lanes * u < nv ? w[i + lanes * u] : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int k = 8 * (i + lanes * u);
+        if (k >= Kr) continue;
+        const uint32_t b[4] = {x[u].x, x[u].y, x[u].z, x[u].w};
+        float f[8];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) { f[2 * j] = __uint_as_float(b[j] << 16); f[2 * j + 1] = __uint_as_float(b[j] & 0xFFFF0000u); }
+#pragma unroll
+        for (int r = 0; r < LD_ROWS; ++r) {
+          if (r < rn) {
+            const float4 x0 = *reinterpret_cast<const float4 *>(os + r * Kr + k), x1 = *reinterpret_cast<const float4 *>(os + r * Kr + k + 4);
+            acc[r] = fmaf(f[0], x0.x, fmaf(f[1], x0.y, fmaf(f[2], x0.z, fmaf(f[3], x0.w, acc[r]))));
+            acc[r] = fmaf(f[4], x1.x, fmaf(f[5], x1.y, fmaf(f[6], x1.z, fmaf(f[7], x1.w, acc[r]))));
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < LD_ROWS; ++r) {
+      for (int m = lanes >> 1; m > 0; m >>= 1) acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], m);
+      if (on && ks == 0 && r < rn) st1(out, bf, (r0 + r) * ld + (int64_t)h * a.Ep + e, acc[r]);
+    }
   }
 }
 
@@ -754,14 +938,37 @@ static int launch_tc(caten_b200_ctx *ctx, const LatentArgs &a, const LatentAbsor
   return 0;
 }
 
+static LatentOut latent_out(const LatentArgs &a, const LatentAbsorbed &x) {
+  LatentOut out;
+  out.o = x.o; out.o_bf = x.o_bf; out.part = x.part; out.ml = x.ml; out.plane = x.plane; out.rows = (int64_t)a.B * a.s; out.Kr = a.Kr; out.H = a.H; out.splits = x.splits;
+  return out;
+}
+
+int launch_latent_down(caten_b200_ctx *ctx, const LatentArgs &a, const LatentAbsorbed &x, const caten_b200_weight *uv, float *out, BfOut bf, int64_t ld) {
+  if (int rc = check_latent(ctx, a)) return rc;
+  const LatentOut in = latent_out(a, x);
+  if (in.rows <= 0) return 0;
+  if (uv->type != CATEN_B200_BF16 || x.splits > LD_MAX_SPLITS || (x.splits == 1 && x.o_bf.hi)) return fail(ctx, CATEN_B200_EINVAL, "latent attention: W_uv takes fp32 sums and BF16 weights");
+  // few rows: a head's outputs are split over CTAs (each merges the parts again)
+  const int64_t ctas = (in.rows + LD_ROWS - 1) / LD_ROWS * a.H;
+  int pieces = 1;
+  while (pieces < 4 && 2 * pieces * ctas <= ctx->sm_count && a.Ep / (2 * pieces) >= 16) pieces *= 2;
+  const int per = (a.Ep + pieces - 1) / pieces;
+  int lanes = 1;   // threads per output
+  while (lanes < 32 && 2 * lanes * per <= 256) lanes *= 2;
+  launch_k(ctx, latent_down_kernel, dim3((unsigned)a.H, (unsigned)((in.rows + LD_ROWS - 1) / LD_ROWS), (unsigned)pieces), dim3(256), (size_t)LD_ROWS * a.Kr * sizeof(float), a, in,
+           (const __nv_bfloat16 *)uv->qs, lanes, per, out, bf, ld);
+  CB_LAUNCH_CHECK(ctx, "latent_down_kernel");
+  return 0;
+}
+
 int launch_latent_absorbed(caten_b200_ctx *ctx, const LatentArgs &a, const LatentAbsorbed &x) {
   const int64_t rows = (int64_t)a.B * a.s;
   if (rows <= 0) return 0;
   if (int rc = check_latent(ctx, a)) return rc;
   if (rows > 65535) return fail(ctx, CATEN_B200_EUNSUPPORTED, "latent attention: %lld rows", (long long)rows);
   if (x.splits > 1 && (!x.part || !x.ml)) return fail(ctx, CATEN_B200_EINVAL, "latent attention: key splits need their buffers");
-  LatentOut out;
-  out.o = x.o; out.o_bf = x.o_bf; out.part = x.part; out.ml = x.ml; out.plane = x.plane; out.rows = rows; out.Kr = a.Kr; out.H = a.H; out.splits = x.splits;
+  const LatentOut out = latent_out(a, x);
   if (latent_tc(ctx, a)) {
     const dim3 grid((unsigned)(latent_ctas(a, true, 1)), (unsigned)rows, (unsigned)x.splits);
     if (int rc = latent_heads(a) == 16 ? launch_tc<16>(ctx, a, x, out, grid) : launch_tc<32>(ctx, a, x, out, grid)) return rc;
@@ -770,7 +977,7 @@ int launch_latent_absorbed(caten_b200_ctx *ctx, const LatentArgs &a, const Laten
     launch_k(ctx, latent_attn_simt_kernel, dim3((unsigned)((a.H + LS_H - 1) / LS_H), (unsigned)rows, (unsigned)x.splits), dim3(LS_THREADS), smem, a, x.qcat, x.qcat_bf, out);
     CB_LAUNCH_CHECK(ctx, "latent_attn_simt_kernel");
   }
-  if (x.splits > 1) {
+  if (x.splits > 1 && x.combine) {
     launch_k(ctx, latent_combine_kernel, dim3((unsigned)a.H, (unsigned)rows), dim3(128), 0, out);
     CB_LAUNCH_CHECK(ctx, "latent_combine_kernel");
   }

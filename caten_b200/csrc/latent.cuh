@@ -47,6 +47,10 @@ int launch_latent_q_expanded(caten_b200_ctx *ctx, const LatentArgs &a, float *q,
 // W_uk^T), rotated parts into qcat [rows, H, Kp + Pp] from column Kp on.
 int launch_latent_q_absorbed(caten_b200_ctx *ctx, const LatentArgs &a, const float *q, PartIn pin, int64_t ld, int64_t plane, float *qn, BfOut qn_bf,
                              float *qcat, BfOut qcat_bf);
+// The same and the product with W_uk^T (BF16 [H * Kp, p64(D)]) in one kernel, into all of qcat; with launch_latent_down for
+// the rows of latent_fused, above which the per-head products are better off on the tensor cores.
+inline bool latent_fused(const LatentArgs &a, int64_t rows) { return rows <= (a.Kr <= 128 ? 256 : 32); }
+int launch_latent_up(caten_b200_ctx *ctx, const LatentArgs &a, const caten_b200_weight *uk, const float *q, PartIn pin, int64_t ld, float *qcat, BfOut qcat_bf);
 // Cached rows [0, t) of sequences b0 .. b0 + nb: latents [nb * t, Kr] as a linear's input, key parts [nb * t, Pp] in fp32.
 int launch_latent_gather(caten_b200_ctx *ctx, const LatentArgs &a, int b0, int nb, int t, float *c, BfOut c_bf, float *kr);
 
@@ -58,11 +62,14 @@ struct LatentAbsorbed {
   int64_t plane = 0;
   float *part = nullptr, *ml = nullptr;   // several splits: [splits, rows, H, Kr] and [splits, rows, H, 2]
   int splits = 1;
+  bool combine = true;              // several splits: merge the parts into the planes (otherwise launch_latent_down does)
   bool early = false;               // cache and position are complete before the kernel in front of this one starts
 };
 // Key splits of a launch over `rows` rows that may see `keys` keys.
 int latent_splits(const caten_b200_ctx *ctx, const LatentArgs &a, int64_t rows, int64_t keys);
 // Softmax attention of every row (sequence, token) over its cached latents.
 int launch_latent_absorbed(caten_b200_ctx *ctx, const LatentArgs &a, const LatentAbsorbed &x);
+// Its result, in fp32 planes or still in parts, times W_uv (BF16 [H * Ep, Kr]) per head: out [rows, ld], head h at column h * Ep.
+int launch_latent_down(caten_b200_ctx *ctx, const LatentArgs &a, const LatentAbsorbed &x, const caten_b200_weight *uv, float *out, BfOut bf, int64_t ld);
 
 }  // namespace cb

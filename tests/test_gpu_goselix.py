@@ -231,15 +231,15 @@ def test_expert_mixtures(rt, experts, top, ff, precision):
 
 
 # ---- batches --------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("B", [5, 40, 300])
-def test_decoding_batches(rt, B):
-    """Row tiles, key splits and expert tiles change with the batch; a sequence's result does not."""
-    cfg, _, W = K.case("mixed")
+@pytest.mark.parametrize("name,B", [("mixed", 5), ("mixed", 40), ("mixed", 300), ("loop_once", 5), ("loop_once", 40)])
+def test_decoding_batches(rt, name, B):
+    """Row tiles, key splits, expert tiles and the form of the per-head products change with the batch; a sequence's result does not."""
+    cfg, _, W = K.case(name)
     T = 24
-    toks = np.stack([K.tokens("mixed", T, seed=s) for s in range(B)])
+    toks = np.stack([K.tokens(name, T, seed=s) for s in range(B)])
     want = [R.forward(cfg, W, toks[b]) for b in range(0, B, max(1, B // 4))]
     for precision in ("fp32", "bf16x3"):
-        m = make(rt, "mixed", precision, max_seq_len=T, batch=B)
+        m = make(rt, name, precision, max_seq_len=T, batch=B)
         got = np.concatenate([m.step(toks[:, :9], 0, range(9))[0]] + [m.step(toks[:, i:i + 1], i, [0])[0] for i in range(9, 20)] + [m.step(toks[:, 20:], 20, range(4))[0]], axis=1)
         for i, b in enumerate(range(0, B, max(1, B // 4))):
             check(got[b], want[i], precision, None, b)
